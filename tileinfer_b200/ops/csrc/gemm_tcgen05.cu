@@ -71,7 +71,6 @@ struct GemmParams {
   unsigned* tile_count;            // [tiles_n * tiles_m] arrival counters, zero between launches
   int M, N, K, ldo, epi;
   int kb_per_split;                // 128-byte k stages per gridDim.z slice
-  int ablate;                      // timing experiments only (TI_GEMM_ABLATE): 1 no MMA, 2 no activation copies, 4 no weight copies, 8 no epilogue, 16 no main loop, 32 no split-k reduction, 64 no fence before the split-k count
 };
 
 // kind::i8 instruction descriptor: D = s32, A = int8 (K-major), B = int8 / uint8 (K-major), M = 128, N = BN
@@ -188,7 +187,7 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
   // hits) and the limb planes of all tokens stay in L2
   const int tile_m = blockIdx.x, tile_n = blockIdx.y, split = blockIdx.z, S = gridDim.z;
   const int KB = (p.K + kBK * kKS - 1) / (kBK * kKS);               // stages of 128 bytes of k (a last half stage reads zeros)
-  const int kb0 = split * p.kb_per_split, kb1 = (p.ablate & 16) ? kb0 : min(KB, kb0 + p.kb_per_split);
+  const int kb0 = split * p.kb_per_split, kb1 = min(KB, kb0 + p.kb_per_split);
   constexpr uint32_t kCols = BMH * kAcc * BN < 32 ? 32 : BMH * kAcc * BN;   // TMEM allocation: a power of two >= 32
 
   if (threadIdx.x == 0) {
@@ -217,11 +216,11 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
     // (written by that kernel) after it.
     const int first = warp == 0 ? 0 : 1;
     const int n_it = kb1 - kb0, n_pre = min(kStages, n_it);
-    const uint32_t stage_tx = ((p.ablate & 4) ? 0 : BMH * kStageA) + ((p.ablate & 2) ? 0 : (BF16 ? 1 : 2) * kStageB) + ((p.ablate & 6) == 6 ? 0 : 0);
+    constexpr uint32_t stage_tx = kStageBytes;
     if (elect_one()) {
       for (int it = first; it < n_pre; it += 2) {
         mbar_expect_tx(full0 + 8 * it, stage_tx);
-        if (!(p.ablate & 4)) tma_load_4d(stage0 + it * kStageBytes, &p.map_w, 0, 0, (kb0 + it) * kKS, tile_n * (BMH * kBM / 8), full0 + 8 * it);
+        tma_load_4d(stage0 + it * kStageBytes, &p.map_w, 0, 0, (kb0 + it) * kKS, tile_n * (BMH * kBM / 8), full0 + 8 * it);
       }
     }
     __syncwarp();
@@ -229,7 +228,6 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
     if (elect_one()) {
       for (int it = first; it < n_pre; it += 2) {
         const uint32_t dst = stage0 + it * kStageBytes;
-        if (p.ablate & 2) continue;
         tma_load_2d(dst + BMH * kStageA, &p.map_xh, (kb0 + it) * kBK * kKS, tile_m * BN, full0 + 8 * it);
         if (!BF16) tma_load_2d(dst + BMH * kStageA + kStageB, &p.map_xl, (kb0 + it) * kBK * kKS, tile_m * BN, full0 + 8 * it);
       }
@@ -240,8 +238,7 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
         if (!mbar_wait(empty0 + 8 * s, par, kGemmWaitNs, p.status)) break;
         const uint32_t dst = stage0 + s * kStageBytes;
         mbar_expect_tx(full0 + 8 * s, stage_tx);
-        if (!(p.ablate & 4)) tma_load_4d(dst, &p.map_w, 0, 0, kb * kKS, tile_n * (BMH * kBM / 8), full0 + 8 * s);   // box: 2 slabs x BMH * 16 row tiles
-        if (p.ablate & 2) continue;
+        tma_load_4d(dst, &p.map_w, 0, 0, kb * kKS, tile_n * (BMH * kBM / 8), full0 + 8 * s);   // box: 2 slabs x BMH * 16 row tiles
         tma_load_2d(dst + BMH * kStageA, &p.map_xh, kb * kBK * kKS, tile_m * BN, full0 + 8 * s);
         if (!BF16) tma_load_2d(dst + BMH * kStageA + kStageB, &p.map_xl, kb * kBK * kKS, tile_m * BN, full0 + 8 * s);
       }
@@ -259,7 +256,6 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
         const uint32_t a = stage0 + s * kStageBytes, bh = a + BMH * kStageA, bl = bh + kStageB;
 #pragma unroll
         for (int j = 0; j < 2 * kKS; ++j) {                       // four 32-byte k steps inside the 128 bytes of the stage
-          if (p.ablate & 1) break;
           const uint32_t acc = (it > 0 || j > 0) ? 1u : 0u;
           // activations: rows of 128 bytes (128-byte swizzle); weights: per row tile the 8 x 64-byte rows of slab 0,
           // then those of slab 1 (64-byte swizzle, 8-row groups 1024 bytes apart)
@@ -297,7 +293,6 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
       const float ws = (ok && n < p.N) ? (BF16 ? 1.f : __bfloat162float(p.wscale[n])) : 0.f;
       const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(h * kAcc * BN);
       for (int c0 = 0; c0 < BN; c0 += 32) {
-        if (p.ablate & 8) break;
         if (tile_m * BN + c0 >= p.M) break;
         uint32_t hi[32], lo[32];
         tmem_ld32(taddr + c0, hi);
@@ -330,7 +325,7 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
   }
   if (S > 1) {
     // ---- split-k: the last CTA of this output tile to arrive adds the partials in split order
-    if (!(p.ablate & 64)) __threadfence();
+    __threadfence();
     __syncthreads();
     if (threadIdx.x == 0) {
       const unsigned prev = atomicAdd(p.tile_count + tile_n * gridDim.x + tile_m, 1u);
@@ -339,7 +334,7 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
       __threadfence();
     }
     __syncthreads();
-    if (s_last && warp >= 2 && warp < 6 && !(p.ablate & 32)) {
+    if (s_last && warp >= 2 && warp < 6) {
       // lane -> four adjacent output features, warp -> every fourth token.  The partial sums of four tokens and four
       // slices (and the residual rows) are requested together before the first is used: with the loads inside a
       // loop of run-time length each one waited for the one before it (12 memory round trips per four tokens; the
@@ -683,10 +678,6 @@ int ti_gemm_w8a16(const void* w, const void* wscale, int n_tiles, int N, int K, 
   p.resid = (const __nv_bfloat16*)resid;
   p.out = out;
   p.status = (unsigned*)status;
-  {
-    static const int ablate = [] { const char* e = getenv("TI_GEMM_ABLATE"); return e == nullptr ? 0 : atoi(e); }();
-    p.ablate = ablate;
-  }
   p.M = M;
   p.N = N;
   p.K = K;
