@@ -41,6 +41,8 @@ class Batch:
     state_slots: list                # [S] DeltaNet state slot per sequence
     # absolute token counts at which a DeltaNet state snapshot must be taken: [S] list[int]
     snapshot_at: list = field(default_factory=list)
+    # flat rows whose hidden states the step returns; None: the last token of every sequence
+    out_rows: list | None = None
 
     @property
     def num_seqs(self) -> int:
@@ -318,7 +320,9 @@ class TorchHybridModel:
             x = rmsnorm(h, lw["post_norm"], c.rms_eps).to(self.dtype)
             h = h + self.all_reduce(self._mlp(lw, x))
         self.snapshots = snaps
-        last = [batch.cu_seqlens[s + 1] - 1 for s in range(batch.num_seqs)]
+        last = batch.out_rows
+        if last is None:
+            last = [batch.cu_seqlens[s + 1] - 1 for s in range(batch.num_seqs)]
         return rmsnorm(h[last], self.final_norm, c.rms_eps).to(self.dtype)
 
     @torch.no_grad()

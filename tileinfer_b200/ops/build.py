@@ -1,7 +1,7 @@
-"""Ahead-of-time build of the sm_100a kernels into one in-tree shared library.
+"""Ahead-of-time build of the sm_100a kernels into in-tree shared libraries.
 
-`nvcc` compiles every `csrc/*.cu` for compute_100a/sm_100a only and links `libtileinfer_b200.so`
-next to this file; a stamp with the hash of the sources and flags makes rebuilds a no-op.  There is
+`nvcc` compiles the `csrc/*.cu` for compute_100a/sm_100a only and links one `libtileinfer_b200*.so` per group of
+sources next to this file; a stamp with the hash of the sources and flags makes rebuilds a no-op.  There is
 no JIT cache: the library is loaded with ctypes and its `extern "C"` launchers take raw device
 pointers and a stream, so they can be captured into CUDA graphs.
 """
@@ -16,8 +16,22 @@ import sys
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 BUILD = os.path.join(HERE, "build")
-LIB = os.path.join(HERE, "libtileinfer_b200.so")
-STAMP = os.path.join(BUILD, "stamp.txt")
+
+# One shared library per group of sources, so that a model is served after compiling only what it needs: "base" (products,
+# sampling, pointwise ops) is used by every model family, the others by the family that has the mechanism.
+GROUPS = {
+    "base": ("gemm_tcgen05.cu", "lm_head.cu", "pointwise.cu", "sampling.cu", "symm.cu"),
+    "hybrid": ("attn_paged.cu", "attn_prefill.cu", "fused_ar.cu", "gdn.cu", "gdn_chunk.cu", "gemv_w8a16.cu"),
+    "latent": ("latent_ops.cu", "latent_attn.cu"),
+}
+
+
+def lib_path(group: str = "base", debug: bool = False) -> str:
+    tail = ("" if group == "base" else "_" + group) + ("_dbg" if debug else "")
+    return os.path.join(HERE, f"libtileinfer_b200{tail}.so")
+
+
+LIB = lib_path()
 
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",
@@ -34,25 +48,38 @@ def _nvcc() -> str:
     return "nvcc"
 
 
-def sources() -> list:
-    return sorted(f for f in os.listdir(CSRC) if f.endswith(".cu"))
+def sources(group: str = None) -> list:
+    return [f for g, files in GROUPS.items() if group in (None, g) for f in files]
 
 
-def _hash() -> str:
-    h = hashlib.sha256(" ".join(NVCC_FLAGS).encode())
-    for f in sorted(os.listdir(CSRC)):
-        if f.endswith((".cu", ".cuh", ".h")):
-            with open(os.path.join(CSRC, f), "rb") as fh:
-                h.update(f.encode())
-                h.update(fh.read())
+def _flags(debug: bool) -> list:
+    return NVCC_FLAGS + (DEBUG_FLAGS if debug else [])
+
+
+def _hash(group: str, debug: bool = False) -> str:
+    """Hash of the flags, the group's sources and the headers."""
+    h = hashlib.sha256(" ".join(_flags(debug)).encode())
+    heads = [f for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
+    for f in sorted(heads + sources(group)):
+        with open(os.path.join(CSRC, f), "rb") as fh:
+            h.update(f.encode())
+            h.update(fh.read())
     return h.hexdigest()
 
 
-def is_current() -> bool:
-    if not (os.path.exists(LIB) and os.path.exists(STAMP)):
+def _build_dir(debug: bool) -> str:
+    return BUILD_DEBUG if debug else BUILD
+
+
+def _stamp(group: str, debug: bool) -> str:
+    return os.path.join(_build_dir(debug), f"stamp_{group}.txt")
+
+
+def is_current(group: str = "base", debug: bool = False) -> bool:
+    if not (os.path.exists(lib_path(group, debug)) and os.path.exists(_stamp(group, debug))):
         return False
-    with open(STAMP) as f:
-        return f.read().strip() == _hash()
+    with open(_stamp(group, debug)) as f:
+        return f.read().strip() == _hash(group, debug)
 
 
 # The checked variant: every peer-buffer / KV-page / workspace index that comes from run-time data goes through
@@ -60,34 +87,23 @@ def is_current() -> bool:
 # TI_JITTER adds random __nanosleep delays before packet sends and collects (stress of the flag protocols).
 # Selected at run time with TI_DEBUG_LIB=1 (see lib.py).
 DEBUG_FLAGS = ["-DTI_BOUNDS_CHECK", "-DTI_JITTER"]
-LIB_DEBUG = os.path.join(HERE, "libtileinfer_b200_dbg.so")
 BUILD_DEBUG = os.path.join(HERE, "build_dbg")
 
 
-def build_debug(force: bool = False) -> str:
-    """Compile the bounds-checked, jittered variant of the library (same sources, DEBUG_FLAGS)."""
-    global LIB, BUILD, STAMP, NVCC_FLAGS
-    keep = (LIB, BUILD, STAMP, NVCC_FLAGS)
-    LIB, BUILD, STAMP = LIB_DEBUG, BUILD_DEBUG, os.path.join(BUILD_DEBUG, "stamp.txt")
-    NVCC_FLAGS = keep[3] + DEBUG_FLAGS
-    try:
-        return build(force)
-    finally:
-        LIB, BUILD, STAMP, NVCC_FLAGS = keep
-
-
-def build(force: bool = False, verbose: bool = False) -> str:
-    """Compile (if needed) and return the path of the shared library."""
-    if not force and is_current():
-        return LIB
-    os.makedirs(BUILD, exist_ok=True)
+def build(force: bool = False, verbose: bool = False, groups=None, debug: bool = False) -> str:
+    """Compile (if needed) the given groups of sources (default: all) and return the path of the base library."""
+    todo = [g for g in (groups or GROUPS) if force or not is_current(g, debug)]
+    if not todo:
+        return lib_path("base", debug)
+    build_dir = _build_dir(debug)
+    os.makedirs(build_dir, exist_ok=True)
     nvcc = _nvcc()
     extra = ["-Xptxas", "-v"] if verbose else []
-    build_dir, lib_path, stamp_path = BUILD, LIB, STAMP
+    hashes = {g: _hash(g, debug) for g in todo}
 
     def one(src):
         obj = os.path.join(build_dir, src[:-3] + ".o")
-        cmd = [nvcc, *NVCC_FLAGS, *extra, "-I", CSRC, "-c", os.path.join(CSRC, src), "-o", obj]
+        cmd = [nvcc, *_flags(debug), *extra, "-I", CSRC, "-c", os.path.join(CSRC, src), "-o", obj]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"nvcc failed for {src}:\n{r.stdout}\n{r.stderr}")
@@ -96,14 +112,23 @@ def build(force: bool = False, verbose: bool = False) -> str:
         return obj
 
     with concurrent.futures.ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 2)) as ex:
-        objs = list(ex.map(one, sources()))
-    cmd = [nvcc, "-shared", "-o", lib_path, *objs, "-lcudart"]
-    r = subprocess.run(cmd, capture_output=True, text=True)
-    if r.returncode != 0:
-        raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
-    with open(stamp_path, "w") as f:
-        f.write(_hash())
-    return lib_path
+        jobs = {g: [ex.submit(one, s) for s in sources(g)] for g in todo}
+        for g in todo:
+            objs = [j.result() for j in jobs[g]]
+            # linked under a temporary name and moved: a process that starts meanwhile never loads half a file
+            tmp = f"{lib_path(g, debug)}.tmp{os.getpid()}"
+            r = subprocess.run([nvcc, "-shared", "-o", tmp, *objs, "-lcudart"], capture_output=True, text=True)
+            if r.returncode != 0:
+                raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+            os.replace(tmp, lib_path(g, debug))
+            with open(_stamp(g, debug), "w") as f:
+                f.write(hashes[g])
+    return lib_path("base", debug)
+
+
+def build_debug(force: bool = False) -> str:
+    """Compile the bounds-checked, jittered variant of every library (same sources, DEBUG_FLAGS)."""
+    return build(force, debug=True)
 
 
 if __name__ == "__main__":

@@ -58,6 +58,15 @@ template <int BN, bool BF16, int BMH = 1> struct GemmGeom {
 };
 constexpr unsigned long long kGemmWaitNs = 2000000000ull;
 
+// Operands of the epilogues for designs with an fp32 residual stream, a clamped gated unit or scaled logits.
+struct GemmEpilogue {
+  const float* resid32;            // RESID32: [M, ldo] fp32
+  __nv_bfloat16* out2;             // SPLIT_GLU: [M, ldo2], column (n - n_split) / 2 of the (gate, up) row pairs
+  int ldo2, n_split;               // SPLIT_GLU: rows below n_split are stored as they are, the others are pairs
+  float scale;                     // F32: factor of the stored values
+  float glu_limit, glu_alpha, glu_bias;   // g = min(g, limit), u = clamp(u, +-limit): g sigmoid(alpha g) (u + bias)
+};
+
 struct GemmParams {
   alignas(64) CUtensorMap map_w;   // uint8 [n_tiles][KB][8][64], box {64, 8, 2, 16 or 32}, 64B swizzle
   alignas(64) CUtensorMap map_xh;  // uint8 [M][K], box {128, BN}, 128B swizzle (bf16 mode: the activations, [M][2K] bytes)
@@ -70,6 +79,7 @@ struct GemmParams {
   float* part;                     // split-k partials [S][M][N] fp32
   unsigned* tile_count;            // [tiles_n * tiles_m] arrival counters, zero between launches
   int M, N, K, ldo, epi;
+  GemmEpilogue ex;
   int kb_per_split;                // 128-byte k stages per gridDim.z slice
 };
 
@@ -83,10 +93,28 @@ template <int BN> TI_DEVICE constexpr uint32_t idesc_bf16() {
   return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(kBM >> 4) << 24);
 }
 
-enum { GEPI_STORE = 0, GEPI_SWIGLU = 1, GEPI_ROWPAR = 2, GEPI_F32 = 3 };
+// RESID32: fp32 out = fp32 residual + product.  SPLIT_GLU: the first n_split rows are stored (bf16), the interleaved
+// (gate, up) rows after them go through the clamped gated unit into a second output.
+enum { GEPI_STORE = 0, GEPI_SWIGLU = 1, GEPI_ROWPAR = 2, GEPI_F32 = 3, GEPI_RESID32 = 4, GEPI_SPLIT_GLU = 5 };
+
+TI_DEVICE float clamped_glu(const GemmEpilogue& e, float g, float u) {
+  g = fminf(g, e.glu_limit);
+  u = fminf(fmaxf(u, -e.glu_limit), e.glu_limit);
+  return g * sigmoid_f(e.glu_alpha * g) * (u + e.glu_bias);
+}
 
 // fused epilogue for four adjacent weight rows n..n+3 of one token (N is a multiple of 4 here): split-k reduction
-TI_DEVICE void gemm_epilogue4(const GemmParams& p, int m, int n, float4 v, uint2 r) {
+TI_DEVICE void gemm_epilogue4(const GemmParams& p, int m, int n, float4 v, uint2 r, float4 r32) {
+  if (p.epi == GEPI_RESID32) {
+    *reinterpret_cast<float4*>(static_cast<float*>(p.out) + (size_t)m * p.ldo + n) =
+        make_float4(v.x + r32.x, v.y + r32.y, v.z + r32.z, v.w + r32.w);
+    return;
+  }
+  if (p.epi == GEPI_SPLIT_GLU && n >= p.ex.n_split) {
+    *reinterpret_cast<uint32_t*>(p.ex.out2 + (size_t)m * p.ex.ldo2 + ((n - p.ex.n_split) >> 1)) =
+        pack_bf16(clamped_glu(p.ex, v.x, v.y), clamped_glu(p.ex, v.z, v.w));
+    return;
+  }
   if (p.epi == GEPI_SWIGLU) {
     const float g0 = round_bf16(v.x), u0 = round_bf16(v.y), g1 = round_bf16(v.z), u1 = round_bf16(v.w);
     *reinterpret_cast<uint32_t*>(static_cast<__nv_bfloat16*>(p.out) + (size_t)m * p.ldo + (n >> 1)) =
@@ -94,7 +122,8 @@ TI_DEVICE void gemm_epilogue4(const GemmParams& p, int m, int n, float4 v, uint2
     return;
   }
   if (p.epi == GEPI_F32) {
-    *reinterpret_cast<float4*>(static_cast<float*>(p.out) + (size_t)m * p.ldo + n) = v;
+    const float sc = p.ex.scale;
+    *reinterpret_cast<float4*>(static_cast<float*>(p.out) + (size_t)m * p.ldo + n) = make_float4(v.x * sc, v.y * sc, v.z * sc, v.w * sc);
     return;
   }
   if (p.epi == GEPI_ROWPAR) {                      // r: the residual row's four values, loaded by the caller
@@ -136,12 +165,27 @@ TI_DEVICE void gemm_store8(const GemmParams& p, int m, int n, const float4 a, co
   }
   if (p.epi == GEPI_F32) {
     float* dst = static_cast<float*>(p.out) + (size_t)m * p.ldo + n;
+    const float sc = p.ex.scale;
     if (full && (p.ldo & 3) == 0 && (reinterpret_cast<uintptr_t>(p.out) & 15) == 0) {
-      *reinterpret_cast<float4*>(dst) = a;
-      *reinterpret_cast<float4*>(dst + 4) = b;
+      *reinterpret_cast<float4*>(dst) = make_float4(a.x * sc, a.y * sc, a.z * sc, a.w * sc);
+      *reinterpret_cast<float4*>(dst + 4) = make_float4(b.x * sc, b.y * sc, b.z * sc, b.w * sc);
     } else {
-      for (int i = 0; i < 8 && n + i < p.N; ++i) dst[i] = v[i];
+      for (int i = 0; i < 8 && n + i < p.N; ++i) dst[i] = v[i] * sc;
     }
+    return;
+  }
+  if (p.epi == GEPI_RESID32) {                     // N and ldo are multiples of 8 (checked by the launcher)
+    const size_t at = (size_t)m * p.ldo + n;
+    const float4 ra = *reinterpret_cast<const float4*>(p.ex.resid32 + at), rb = *reinterpret_cast<const float4*>(p.ex.resid32 + at + 4);
+    float* dst = static_cast<float*>(p.out) + at;
+    *reinterpret_cast<float4*>(dst) = make_float4(a.x + ra.x, a.y + ra.y, a.z + ra.z, a.w + ra.w);
+    *reinterpret_cast<float4*>(dst + 4) = make_float4(b.x + rb.x, b.y + rb.y, b.z + rb.z, b.w + rb.w);
+    return;
+  }
+  if (p.epi == GEPI_SPLIT_GLU && n >= p.ex.n_split) {   // N and n_split are multiples of 8
+    *reinterpret_cast<uint2*>(p.ex.out2 + (size_t)m * p.ex.ldo2 + ((n - p.ex.n_split) >> 1)) =
+        make_uint2(pack_bf16(clamped_glu(p.ex, v[0], v[1]), clamped_glu(p.ex, v[2], v[3])),
+                   pack_bf16(clamped_glu(p.ex, v[4], v[5]), clamped_glu(p.ex, v[6], v[7])));
     return;
   }
   float r[8];
@@ -346,12 +390,15 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
       for (int m0 = tile_m * BN + (warp - 2); m0 < m_end; m0 += 16) {
         float4 acc[4];
         uint2 rs[4];
+        float4 rs32[4];
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
+          rs32[u] = make_float4(0.f, 0.f, 0.f, 0.f);
           acc[u] = make_float4(0.f, 0.f, 0.f, 0.f);
           rs[u] = make_uint2(0u, 0u);
           const int m = m0 + 4 * u;
           if (m < m_end && p.epi == GEPI_ROWPAR) rs[u] = __ldcg(reinterpret_cast<const uint2*>(p.resid + (size_t)m * p.N + n4));
+          if (m < m_end && p.epi == GEPI_RESID32) rs32[u] = __ldcg(reinterpret_cast<const float4*>(p.ex.resid32 + (size_t)m * p.ldo + n4));
         }
         for (int z0 = 0; z0 < S; z0 += 4) {
           float4 v[4][4];
@@ -376,7 +423,7 @@ __global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) 
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
           const int m = m0 + 4 * u;
-          if (m < m_end) gemm_epilogue4(p, m, n4, acc[u], rs[u]);
+          if (m < m_end) gemm_epilogue4(p, m, n4, acc[u], rs[u], rs32[u]);
         }
       }
       }
@@ -636,9 +683,20 @@ static int plan_split(GemmParams& p, int KB, int tiles, int M, int N, int ldo, v
   return (KB + p.kb_per_split - 1) / p.kb_per_split;           // no empty slice
 }
 
+// Fills in the extended epilogue and refuses layouts whose vector accesses it could not make.
+static int set_epilogue(GemmParams& p, const GemmEpilogue* ex) {
+  p.ex.scale = 1.f;
+  if (ex != nullptr) p.ex = *ex;
+  if (p.epi == GEPI_RESID32 && (p.ex.resid32 == nullptr || p.N % 8 || p.ldo % 8 || ((uintptr_t)p.out | (uintptr_t)p.ex.resid32) % 16)) return -2;
+  if (p.epi == GEPI_SPLIT_GLU && (p.ex.out2 == nullptr || p.N % 8 || p.ex.n_split % 8 || p.ex.ldo2 % 4 || (uintptr_t)p.ex.out2 % 8)) return -2;
+  return 0;
+}
+
 }  // namespace ti
 
 extern "C" {
+
+int ti_gemm_epilogue_size() { return (int)sizeof(ti::GemmEpilogue); }
 
 // xh/xl/xscale <- limbs of x (optionally RMS-normalised with (1+norm_w)); one launch, M blocks.
 int ti_quant_rows(const void* x, int ldx, const void* norm_w, float eps, int M, int K, void* xh, void* xl, void* xscale,
@@ -660,9 +718,9 @@ int ti_quant_rows(const void* x, int ldx, const void* norm_w, float eps, int M, 
 // `part_bytes` / `n_count` are their capacities.  The token tile (32 / 64 / 128) and the k split follow from M, N.
 int ti_gemm_w8a16(const void* w, const void* wscale, int n_tiles, int N, int K, const void* xh, const void* xl,
                   const void* xscale, int M, const void* resid, void* out, int ldo, int epi, void* status, void* part,
-                  size_t part_bytes, void* tile_count, int n_count, void* stream) {
+                  size_t part_bytes, void* tile_count, int n_count, const ti::GemmEpilogue* ex, void* stream) {
   if (M <= 0) return 0;
-  if (K % 64 || N < 1 || epi < 0 || epi > 2) return -2;
+  if (K % 64 || N < 1 || epi < 0 || epi > 5) return -2;
   ti::GemmParams p = {};
   const int KB = K / 64, KS = (KB + ti::kKS - 1) / ti::kKS;      // 64-byte slabs of the weight layout; 128-byte stages
   const int BN = M <= 32 ? 32 : (M <= 64 ? 64 : 128);
@@ -683,6 +741,8 @@ int ti_gemm_w8a16(const void* w, const void* wscale, int n_tiles, int N, int K, 
   p.K = K;
   p.ldo = ldo;
   p.epi = epi;
+  rc = ti::set_epilogue(p, ex);
+  if (rc) return rc;
   const int rows = ti::kBM * BMH;
   const int tiles_n = (n_tiles * 8 + rows - 1) / rows, tiles_m = (M + BN - 1) / BN;
   const int S = ti::plan_split(p, KS, tiles_n * tiles_m, M, N, ldo, part, part_bytes, tile_count, n_count);
@@ -699,9 +759,10 @@ int ti_gemm_w8a16(const void* w, const void* wscale, int n_tiles, int N, int K, 
 // The same for bf16 weights tiled [n_tiles][K/32][8][32] (lm_head, unquantised mode) and bf16 activations x [M][K]
 // (contiguous rows): tcgen05.mma kind::f16, fp32 accumulation.  epi 3 stores fp32 (logits).
 int ti_gemm_bf16(const void* w, int n_tiles, int N, int K, const void* x, int M, const void* resid, void* out, int ldo,
-                 int epi, void* status, void* part, size_t part_bytes, void* tile_count, int n_count, void* stream) {
+                 int epi, void* status, void* part, size_t part_bytes, void* tile_count, int n_count, const ti::GemmEpilogue* ex,
+                 void* stream) {
   if (M <= 0) return 0;
-  if (K % 32 || N < 1 || epi < 0 || epi > 3) return -2;
+  if (K % 32 || N < 1 || epi < 0 || epi > 5) return -2;
   ti::GemmParams p = {};
   const int KB = K / 32, KS = (KB + ti::kKS - 1) / ti::kKS;    // 64-byte slabs; 128-byte stages
   const int BN = M <= 32 ? 32 : (M <= 64 ? 64 : 128);
@@ -718,6 +779,8 @@ int ti_gemm_bf16(const void* w, int n_tiles, int N, int K, const void* x, int M,
   p.K = 2 * K;                                                 // bytes of k: the kernel counts 64-byte slabs
   p.ldo = ldo;
   p.epi = epi;
+  rc = ti::set_epilogue(p, ex);
+  if (rc) return rc;
   const int rows = ti::kBM * BMH;
   const int tiles_n = (n_tiles * 8 + rows - 1) / rows, tiles_m = (M + BN - 1) / BN;
   const int S = ti::plan_split(p, KS, tiles_n * tiles_m, M, N, ldo, part, part_bytes, tile_count, n_count);

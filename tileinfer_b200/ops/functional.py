@@ -14,7 +14,7 @@ import torch
 from . import lib as _l
 from .lib import ChainParams, GemvParams, MAX_CHAIN, MAX_RANKS, check, ptr, stream
 
-_I, _P, _F = ctypes.c_int, ctypes.c_void_p, ctypes.c_float
+_I, _P, _F, _LL = ctypes.c_int, ctypes.c_void_p, ctypes.c_float, ctypes.c_longlong
 
 XGLOBAL, XNORM = 0, 1
 EPI_STORE, EPI_SWIGLU, EPI_ROWPAR, EPI_F32, EPI_ARGMAX = 0, 1, 2, 3, 4
@@ -67,6 +67,18 @@ class AttnParams(ctypes.Structure):
                 ("ld", _I), ("num_qg", _I), ("scale_log2e", _F), ("num_blocks", _I), ("status", _P)]
 
 
+class LatentAttnParams(ctypes.Structure):
+    _fields_ = [("q", _P), ("cache", _P), ("block_tables", _P), ("positions", _P), ("qg_seq", _P), ("qg_tok0", _P),
+                ("qg_ntok", _P), ("sink", _P), ("o_part", _P), ("ml_part", _P), ("out", _P), ("status", _P),
+                ("H", _I), ("R", _I), ("Rp", _I), ("max_blocks", _I), ("nsplit", _I), ("num_qg", _I), ("window", _I),
+                ("num_blocks", _I), ("scale", _F)]
+
+
+class GemmEpilogue(ctypes.Structure):
+    _fields_ = [("resid32", _P), ("out2", _P), ("ldo2", _I), ("n_split", _I), ("scale", _F), ("glu_limit", _F),
+                ("glu_alpha", _F), ("glu_bias", _F)]
+
+
 class TopkParams(ctypes.Structure):
     _fields_ = [("logits", _P), ("ws_val", _P), ("ws_idx", _P), ("out_val", _P), ("out_idx", _P),
                 ("step_ptr", _P), ("status", _P), ("peer_buf", ctypes.c_uint64 * MAX_RANKS),
@@ -93,8 +105,8 @@ class SampleParams(ctypes.Structure):
                 ("out_tok", _P), ("status_src", _P), ("M", _I), ("n_cand", _I)]
 
 
-_l.register("ti_ar_rows_params_size", _I, [])
-_l.register("ti_ar_rows", _I, [ctypes.POINTER(ArRowsParams), _P])
+_l.register("ti_ar_rows_params_size", _I, [], "hybrid")
+_l.register("ti_ar_rows", _I, [ctypes.POINTER(ArRowsParams), _P], "hybrid")
 _l.register("ti_edit_params_size", _I, [])
 _l.register("ti_sample_params_size", _I, [])
 _l.register("ti_logits_edit", _I, [ctypes.POINTER(EditParams), _P])
@@ -103,16 +115,16 @@ _l.register("ti_embed", _I, [_P, _P, _P, _I, _I, _I, _P, _P])
 _l.register("ti_rmsnorm", _I, [_P, _P, _P, _P, _P, _I, _I, _F, _I, _P])
 _l.register("ti_act_mul", _I, [_P, _P, _P, _I, _I, _I, _I, _I, _I, _P])
 _l.register("ti_swiglu_interleaved", _I, [_P, _P, _I, _I, _I, _I, _P])
-_l.register("ti_gdn_params_size", _I, [])
-_l.register("ti_gdn_step", _I, [ctypes.POINTER(GdnParams), _I, _I, _I, _I, _I, _P])
-_l.register("ti_gdn_chunk_params_size", _I, [])
-_l.register("ti_gdn_chunk_ws_bytes", _I, [_I, _I, _I])
-_l.register("ti_gdn_chunked", _I, [ctypes.POINTER(GdnChunkParams), _I, _I, _I, _I, _I, _P])
-_l.register("ti_qkv_prep_params_size", _I, [])
-_l.register("ti_attn_params_size", _I, [])
-_l.register("ti_qkv_prep", _I, [ctypes.POINTER(QkvPrepParams), _I, _I, _P])
-_l.register("ti_attn_paged", _I, [ctypes.POINTER(AttnParams), _I, _P])
-_l.register("ti_attn_prefill", _I, [_P, _I, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P])
+_l.register("ti_gdn_params_size", _I, [], "hybrid")
+_l.register("ti_gdn_step", _I, [ctypes.POINTER(GdnParams), _I, _I, _I, _I, _I, _P], "hybrid")
+_l.register("ti_gdn_chunk_params_size", _I, [], "hybrid")
+_l.register("ti_gdn_chunk_ws_bytes", _I, [_I, _I, _I], "hybrid")
+_l.register("ti_gdn_chunked", _I, [ctypes.POINTER(GdnChunkParams), _I, _I, _I, _I, _I, _P], "hybrid")
+_l.register("ti_qkv_prep_params_size", _I, [], "hybrid")
+_l.register("ti_attn_params_size", _I, [], "hybrid")
+_l.register("ti_qkv_prep", _I, [ctypes.POINTER(QkvPrepParams), _I, _I, _P], "hybrid")
+_l.register("ti_attn_paged", _I, [ctypes.POINTER(AttnParams), _I, _P], "hybrid")
+_l.register("ti_attn_prefill", _I, [_P, _I, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P], "hybrid")
 _l.register("ti_topk_params_size", _I, [])
 _l.register("ti_topk", _I, [ctypes.POINTER(TopkParams), _P])
 _l.register("ti_topk_merge", _I, [ctypes.POINTER(TopkParams), _P])
@@ -126,23 +138,41 @@ _l.register("ti_memset_async", _I, [_P, _I, ctypes.c_size_t, _P])
 _l.register("ti_wait_flag_probe", _I, [_P, ctypes.c_uint, ctypes.c_ulonglong, _P, _P, _P])
 
 _l.register("ti_quant_rows", _I, [_P, _I, _P, _F, _I, _I, _P, _P, _P, _P])
-_l.register("ti_gemm_bf16", _I, [_P, _I, _I, _I, _P, _I, _P, _P, _I, _I, _P, _P, ctypes.c_size_t, _P, _I, _P])
-_l.register("ti_gemm_w8a16", _I, [_P, _P, _I, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _P, _P, ctypes.c_size_t, _P, _I, _P])
+_l.register("ti_gemm_epilogue_size", _I, [])
+_l.register("ti_gemm_bf16", _I, [_P, _I, _I, _I, _P, _I, _P, _P, _I, _I, _P, _P, ctypes.c_size_t, _P, _I, _P, _P])
+_l.register("ti_gemm_w8a16", _I, [_P, _P, _I, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _P, _P, ctypes.c_size_t, _P, _I, _P, _P])
+_l.register("ti_latent_attn_params_size", _I, [], "latent")
+_l.register("ti_latent_attn_max_split_rank", _I, [], "latent")
+_l.register("ti_latent_attn", _I, [ctypes.POINTER(LatentAttnParams), _I, _P], "latent")
+_l.register("ti_embed_pos", _I, [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P, _I, _P], "latent")
+_l.register("ti_rmsnorm_f32", _I, [_P, _P, _P, _I, _I, _I, _F, _I, _P], "latent")
+_l.register("ti_latent_store", _I, [_P, _I, _I, _P, _P, _P, _LL, _I, _I, _I, _F, _I, _P], "latent")
+_l.register("ti_latent_gather", _I, [_P, _P, _LL, _P, _I, _I, _I, _P], "latent")
+_l.register("ti_head_product", _I, [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P], "latent")
+_l.register("ti_gemm_f32", _I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P], "latent")
 
-_checked = False
+_PARAM_SIZES = {"base": (("ti_topk_params_size", TopkParams), ("ti_edit_params_size", EditParams),
+                         ("ti_sample_params_size", SampleParams), ("ti_gemm_epilogue_size", GemmEpilogue)),
+                "latent": (("ti_latent_attn_params_size", LatentAttnParams),),
+                "hybrid": (("ti_gdn_params_size", GdnParams), ("ti_gdn_chunk_params_size", GdnChunkParams),
+                           ("ti_qkv_prep_params_size", QkvPrepParams), ("ti_attn_params_size", AttnParams),
+                           ("ti_ar_rows_params_size", ArRowsParams), ("ti_gemv_params_size", GemvParams),
+                           ("ti_chain_params_size", ChainParams))}
+_checked = set()
 
 
-def L():
-    global _checked
+def L(*groups: str):
+    """The kernel libraries; the named groups (default: "base" and "hybrid") are loaded now, with their parameter
+    blocks checked against the Python structures."""
     lib = _l.lib()
-    if not _checked:
-        for fn, st in (("ti_gdn_params_size", GdnParams), ("ti_gdn_chunk_params_size", GdnChunkParams), ("ti_qkv_prep_params_size", QkvPrepParams),
-                       ("ti_attn_params_size", AttnParams), ("ti_topk_params_size", TopkParams),
-                       ("ti_edit_params_size", EditParams), ("ti_sample_params_size", SampleParams),
-                       ("ti_ar_rows_params_size", ArRowsParams)):
-            if getattr(lib, fn)() != ctypes.sizeof(st):
-                raise RuntimeError(f"{st.__name__} layout mismatch between Python and CUDA")
-        _checked = True
+    groups = groups or ("base", "hybrid")
+    if not _checked.issuperset(groups):
+        _l.build_groups(*groups)
+        for g in groups:
+            for fn, st in _PARAM_SIZES.get(g, ()):
+                if getattr(lib, fn)() != ctypes.sizeof(st):
+                    raise RuntimeError(f"{st.__name__} layout mismatch between Python and CUDA")
+            _checked.add(g)
     return lib
 
 
@@ -359,7 +389,7 @@ def make_chain(params: list) -> ChainParams:
 
 def gemv_chain_launch(params: list, wt: int, ncta: int = NUM_SMS):
     c = make_chain(params)
-    check(L().ti_gemv_chain(ctypes.byref(c), wt, ncta, stream()), "ti_gemv_chain")
+    check(_l.lib().ti_gemv_chain(ctypes.byref(c), wt, ncta, stream()), "ti_gemv_chain")
 
 
 def gemv_launch(p: GemvParams, wt: int, xmode: int = None, epi: int = None, ncta: int = NUM_SMS):
@@ -391,14 +421,14 @@ def gemv(W: LinearW, x: torch.Tensor, *, out=None, xmode=XGLOBAL, epi=EPI_STORE,
 # ------------------------------------------------------------------------------------ pointwise
 def embed(ids, table, out, step_ptr=0):
     M, H = out.shape
-    check(L().ti_embed(ptr(ids), ptr(table), ptr(out), M, H, table.shape[0], step_ptr, stream()), "ti_embed")
+    check(_l.lib().ti_embed(ptr(ids), ptr(table), ptr(out), M, H, table.shape[0], step_ptr, stream()), "ti_embed")
 
 
 def rmsnorm(x, w, eps, *, add=None, out=None, r_out=None, one_plus=True):
     M, H = x.shape
     if out is None:
         out = torch.empty_like(x)
-    check(L().ti_rmsnorm(ptr(x), ptr(add), ptr(w), ptr(out), ptr(r_out), M, H, eps, int(one_plus), stream()), "ti_rmsnorm")
+    check(_l.lib().ti_rmsnorm(ptr(x), ptr(add), ptr(w), ptr(out), ptr(r_out), M, H, eps, int(one_plus), stream()), "ti_rmsnorm")
     return out
 
 
@@ -406,7 +436,7 @@ def act_mul(a, b, out=None, mode=0):
     M, n = a.shape
     if out is None:
         out = torch.empty(M, n, dtype=torch.bfloat16, device=a.device)
-    check(L().ti_act_mul(ptr(a), ptr(b), ptr(out), M, n, a.stride(0), b.stride(0), out.stride(0), mode, stream()), "ti_act_mul")
+    check(_l.lib().ti_act_mul(ptr(a), ptr(b), ptr(out), M, n, a.stride(0), b.stride(0), out.stride(0), mode, stream()), "ti_act_mul")
     return out
 
 
@@ -414,7 +444,7 @@ def swiglu_interleaved(gu, out=None):
     M, n2 = gu.shape
     if out is None:
         out = torch.empty(M, n2 // 2, dtype=torch.bfloat16, device=gu.device)
-    check(L().ti_swiglu_interleaved(ptr(gu), ptr(out), M, n2 // 2, gu.stride(0), out.stride(0), stream()), "ti_swiglu")
+    check(_l.lib().ti_swiglu_interleaved(ptr(gu), ptr(out), M, n2 // 2, gu.stride(0), out.stride(0), stream()), "ti_swiglu")
     return out
 
 
@@ -428,7 +458,7 @@ def gdn_step(p: GdnParams, num_seqs: int, dk: int, dv: int, state_bf16: bool, sp
     mode = (3 if staged else 2) if single else int(split)
     if not p.status:
         p.status = status_ptr()
-    check(L().ti_gdn_step(ctypes.byref(p), num_seqs, dk, dv, int(state_bf16), mode, stream()), "ti_gdn_step")
+    check(_l.lib().ti_gdn_step(ctypes.byref(p), num_seqs, dk, dv, int(state_bf16), mode, stream()), "ti_gdn_step")
 
 
 GDN_CHUNK = 64
@@ -468,7 +498,7 @@ class GdnChunkWorkspace:
 
     def get(self, n_items: int, dk: int, dv: int):
         if n_items > self.cap or self.bufs is None or self.key != (dk, dv):
-            lib = L()
+            lib = _l.lib()
             sizes = [lib.ti_gdn_chunk_ws_bytes(dk, dv, i) for i in range(6)]
             cap = max(n_items, 2 * self.cap)
             self.bufs = [torch.empty(cap * sz, dtype=torch.uint8, device=self.device) for sz in sizes]
@@ -477,19 +507,19 @@ class GdnChunkWorkspace:
 
 
 def gdn_chunked(p: GdnChunkParams, num_seqs: int, T: int, dk: int, dv: int, state_bf16: bool):
-    check(L().ti_gdn_chunked(ctypes.byref(p), num_seqs, T, dk, dv, int(state_bf16), stream()), "ti_gdn_chunked")
+    check(_l.lib().ti_gdn_chunked(ctypes.byref(p), num_seqs, T, dk, dv, int(state_bf16), stream()), "ti_gdn_chunked")
 
 
 def qkv_prep(p: QkvPrepParams, T: int, D: int):
     if not p.status:
         p.status = status_ptr()
-    check(L().ti_qkv_prep(ctypes.byref(p), T, D, stream()), "ti_qkv_prep")
+    check(_l.lib().ti_qkv_prep(ctypes.byref(p), T, D, stream()), "ti_qkv_prep")
 
 
 def attn_paged(p: AttnParams, D: int):
     if not p.status:
         p.status = status_ptr()
-    check(L().ti_attn_paged(ctypes.byref(p), D, stream()), "ti_attn_paged")
+    check(_l.lib().ti_attn_paged(ctypes.byref(p), D, stream()), "ti_attn_paged")
 
 
 def attn_prefill(q, kcache, vcache, num_blocks, block_tables, positions, tiles, gate_src, out, *, hq, hkv, D,
@@ -498,7 +528,7 @@ def attn_prefill(q, kcache, vcache, num_blocks, block_tables, positions, tiles, 
     `tiles`: int32 [3, n] = (sequence, first flat token, tokens <= 128) per tile, longest KV first."""
     n = tiles.shape[1]
     scale = D ** -0.5 * 1.4426950408889634
-    check(L().ti_attn_prefill(ptr(q), q.shape[0], ptr(kcache), ptr(vcache), num_blocks, ptr(block_tables), ptr(positions),
+    check(_l.lib().ti_attn_prefill(ptr(q), q.shape[0], ptr(kcache), ptr(vcache), num_blocks, ptr(block_tables), ptr(positions),
                               ptr(tiles[0]), ptr(tiles[1]), ptr(tiles[2]), n, ptr(gate_src), ptr(out), hq, hkv,
                               max_blocks, ld, scale, D, status_ptr(), stream()), "ti_attn_prefill")
 
@@ -527,29 +557,35 @@ def ar_rows(comm, parity: int, M: int, N: int, resid, h_out, *, order: int, mode
     p.M, p.N, p.tp, p.rank, p.order, p.mode, p.eps = M, N, comm.tp, comm.rank, order, mode, eps
     p.rows_cap = int(getattr(comm, "ar_rows", 0) or 0)
     p.two_shot = int(two_shot)
-    check(L().ti_ar_rows(ctypes.byref(p), stream()), "ti_ar_rows")
+    check(_l.lib().ti_ar_rows(ctypes.byref(p), stream()), "ti_ar_rows")
 
 
 def logits_edit(p: EditParams):
-    check(L().ti_logits_edit(ctypes.byref(p), stream()), "ti_logits_edit")
+    check(_l.lib().ti_logits_edit(ctypes.byref(p), stream()), "ti_logits_edit")
 
 
 def sample(p: SampleParams):
-    check(L().ti_sample(ctypes.byref(p), stream()), "ti_sample")
+    check(_l.lib().ti_sample(ctypes.byref(p), stream()), "ti_sample")
 
 
 def topk(p: TopkParams):
-    check(L().ti_topk(ctypes.byref(p), stream()), "ti_topk")
+    check(_l.lib().ti_topk(ctypes.byref(p), stream()), "ti_topk")
 
 
 def topk_merge(p: TopkParams):
     """Second stage only: merges the per-chunk candidates already in ws_val / ws_idx (written, for instance, by the
     arg-max epilogue of the lm_head GEMV: one candidate per row and CTA) and exchanges the winners between ranks."""
-    check(L().ti_topk_merge(ctypes.byref(p), stream()), "ti_topk_merge")
+    check(_l.lib().ti_topk_merge(ctypes.byref(p), stream()), "ti_topk_merge")
 
 
 # ------------------------------------------------------------------------------------ prefill GEMM (tcgen05)
-GEPI_STORE, GEPI_SWIGLU, GEPI_ROWPAR, GEPI_F32 = 0, 1, 2, 3
+GEPI_STORE, GEPI_SWIGLU, GEPI_ROWPAR, GEPI_F32, GEPI_RESID32, GEPI_SPLIT_GLU = 0, 1, 2, 3, 4, 5
+
+
+def gemm_epilogue(*, resid32=None, out2=None, n_split=0, scale=1.0, glu=(math.inf, 1.0, 0.0)) -> GemmEpilogue:
+    """Operands of the extended epilogues: an fp32 residual (GEPI_RESID32), the second output and the constants
+    (limit, alpha, bias) of the clamped gated unit (GEPI_SPLIT_GLU), a factor of the stored fp32 values (GEPI_F32)."""
+    return GemmEpilogue(ptr(resid32), ptr(out2), 0 if out2 is None else out2.stride(0), n_split, scale, *glu)
 
 
 class Limbs:
@@ -562,30 +598,34 @@ class Limbs:
         self.scale = torch.empty(M, dtype=torch.float32, device=device)
 
 
+def _ref(struct):
+    return None if struct is None else ctypes.addressof(struct)
+
+
 def quant_rows(x: torch.Tensor, norm_w=None, eps: float = 1e-6, out: Limbs = None) -> Limbs:
     """Limb planes of x [M, K] (bf16, row stride x.stride(0)); RMSNorm(1+w) fused when norm_w is given."""
     M, K = x.shape
     if out is None:
         out = Limbs(M, K, x.device)
-    check(L().ti_quant_rows(ptr(x), x.stride(0), ptr(norm_w), eps, M, K, ptr(out.hi), ptr(out.lo), ptr(out.scale),
+    check(_l.lib().ti_quant_rows(ptr(x), x.stride(0), ptr(norm_w), eps, M, K, ptr(out.hi), ptr(out.lo), ptr(out.scale),
                             stream()), "ti_quant_rows")
     return out
 
 
-def gemm_w8a16(W: "LinearW", limbs: Limbs, *, out=None, epi=GEPI_STORE, resid=None) -> torch.Tensor:
+def gemm_w8a16(W: "LinearW", limbs: Limbs, *, out=None, epi=GEPI_STORE, resid=None, ex=None) -> torch.Tensor:
     """y = x W^T on the tcgen05 tensor cores for int8-tiled W and the limb planes of x (any M)."""
     assert W.wt == W_INT8 and limbs.K == W.K
     M = limbs.M
     if out is None:
         out = torch.empty(M, W.N // 2 if epi == GEPI_SWIGLU else W.N, dtype=torch.bfloat16, device=limbs.hi.device)
     part, count = _gemm_workspace(limbs.hi.device)
-    check(L().ti_gemm_w8a16(ptr(W.tiles), ptr(W.scale), W.n_tiles, W.N, W.K, ptr(limbs.hi), ptr(limbs.lo),
+    check(_l.lib().ti_gemm_w8a16(ptr(W.tiles), ptr(W.scale), W.n_tiles, W.N, W.K, ptr(limbs.hi), ptr(limbs.lo),
                             ptr(limbs.scale), M, ptr(resid), ptr(out), out.stride(0), epi, status_ptr(), ptr(part),
-                            part.numel() * 4, ptr(count), count.numel(), stream()), "ti_gemm_w8a16")
+                            part.numel() * 4, ptr(count), count.numel(), _ref(ex), stream()), "ti_gemm_w8a16")
     return out
 
 
-def gemm_bf16(W: "LinearW", x: torch.Tensor, *, out=None, epi=GEPI_STORE, resid=None) -> torch.Tensor:
+def gemm_bf16(W: "LinearW", x: torch.Tensor, *, out=None, epi=GEPI_STORE, resid=None, ex=None) -> torch.Tensor:
     """y = x W^T on the tcgen05 tensor cores (kind::f16) for bf16-tiled W and bf16 x [M, K] with contiguous rows.
     epi GEPI_F32 stores fp32 (logits)."""
     assert W.wt == W_BF16 and x.shape[1] == W.K and x.stride(1) == 1 and x.stride(0) == W.K and x.dtype == torch.bfloat16
@@ -594,8 +634,8 @@ def gemm_bf16(W: "LinearW", x: torch.Tensor, *, out=None, epi=GEPI_STORE, resid=
         cols = W.N // 2 if epi == GEPI_SWIGLU else W.N
         out = torch.empty(M, cols, dtype=torch.float32 if epi == GEPI_F32 else torch.bfloat16, device=x.device)
     part, count = _gemm_workspace(x.device)
-    check(L().ti_gemm_bf16(ptr(W.tiles), W.n_tiles, W.N, W.K, ptr(x), M, ptr(resid), ptr(out), out.stride(0), epi,
-                           status_ptr(), ptr(part), part.numel() * 4, ptr(count), count.numel(), stream()), "ti_gemm_bf16")
+    check(_l.lib().ti_gemm_bf16(ptr(W.tiles), W.n_tiles, W.N, W.K, ptr(x), M, ptr(resid), ptr(out), out.stride(0), epi,
+                           status_ptr(), ptr(part), part.numel() * 4, ptr(count), count.numel(), _ref(ex), stream()), "ti_gemm_bf16")
     return out
 
 
@@ -610,3 +650,58 @@ def _gemm_workspace(device):
         _GEMM_WS[key] = (torch.empty(8 << 20, dtype=torch.float32, device=device),
                          torch.zeros(256, dtype=torch.int32, device=device))
     return _GEMM_WS[key]
+
+
+# ------------------------------------------------------------------------------------ latent attention, fp32 residual
+def _f32(t) -> int:
+    assert t.dtype in (torch.float32, torch.bfloat16), t.dtype
+    return int(t.dtype == torch.float32)
+
+
+def embed_pos(ids, positions, embed, pos, norm_w, x, W, eps, step_ptr=0):
+    """x[m] (fp32) = rmsnorm(embed[ids[m]] + pos[positions[m]]) * norm_w; `pos` and `norm_w` may be None."""
+    check(_l.lib().ti_embed_pos(ptr(ids), ptr(positions), ptr(embed), ptr(pos), ptr(norm_w), ptr(x), x.shape[0], W, x.stride(0),
+                                embed.shape[0], 0 if pos is None else pos.shape[0], eps, step_ptr, _f32(embed), stream()), "ti_embed_pos")
+
+
+def rmsnorm_f32(x, norm_w, y, W, eps):
+    """y = rmsnorm(x) * norm_w for fp32 rows x [M, pitch] of true width W; y bf16 or fp32 of the same pitch."""
+    assert x.stride(0) == y.stride(0) and norm_w.numel() == x.stride(0)
+    check(_l.lib().ti_rmsnorm_f32(ptr(x), ptr(norm_w), ptr(y), x.shape[0], W, x.stride(0), eps, _f32(y), stream()), "ti_rmsnorm_f32")
+
+
+def latent_store(proj, col0, norm_w, slots, cache, R, eps):
+    """Normalised latents proj[:, col0 : col0 + R] into their slots of `cache` [blocks, 16, Rp]."""
+    Rp = cache.shape[-1]
+    assert norm_w.numel() == Rp and cache.dtype == proj.dtype
+    check(_l.lib().ti_latent_store(ptr(proj), proj.stride(0), col0, ptr(norm_w), ptr(slots), ptr(cache), cache.numel() // Rp,
+                                   proj.shape[0], R, Rp, eps, _f32(proj), stream()), "ti_latent_store")
+
+
+def latent_gather(cache, slots, out):
+    """Rows of the listed slots (int64) of `cache` [blocks, 16, Rp] -> out [n, Rp]."""
+    Rp = cache.shape[-1]
+    check(_l.lib().ti_latent_gather(ptr(cache), ptr(slots), cache.numel() // Rp, ptr(out), slots.numel(), Rp, _f32(cache), stream()),
+          "ti_latent_gather")
+
+
+def head_product(x, w, out, gate=None, gcol=0):
+    """out[t, h] = w[h] x[t, h] per head (w [H, N, K]), times sigmoid(gate[t, gcol + h]) when a gate is given.  x and out
+    are row views whose heads lie side by side."""
+    H, N, K = w.shape
+    check(_l.lib().ti_head_product(ptr(x), ptr(w), ptr(gate), ptr(out), x.shape[0], H, N, K, x.stride(0), out.stride(0),
+                                   0 if gate is None else gate.stride(0), gcol, _f32(w), stream()), "ti_head_product")
+
+
+def latent_attn(p: LatentAttnParams, f32: bool):
+    if not p.status:
+        p.status = status_ptr()
+    check(_l.lib().ti_latent_attn(ctypes.byref(p), int(f32), stream()), "ti_latent_attn")
+
+
+def gemm_f32(w, x, *, out, epi=GEPI_F32, ex=None):
+    """y = x W^T in fp32 FMAs (w [N, K] row-major) with the GEPI_F32 / GEPI_RESID32 / GEPI_SPLIT_GLU epilogues."""
+    e = ex if ex is not None else gemm_epilogue()
+    N, K = w.shape
+    check(_l.lib().ti_gemm_f32(ptr(w), ptr(x), e.resid32, ptr(out), e.out2, x.shape[0], N, K, x.stride(0), out.stride(0), e.ldo2,
+                               e.n_split, epi, e.scale, e.glu_limit, e.glu_alpha, e.glu_bias, stream()), "ti_gemm_f32")

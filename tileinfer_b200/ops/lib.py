@@ -37,41 +37,65 @@ class ChainParams(ctypes.Structure):
     _fields_ = [("n_ops", ctypes.c_int), ("x_bytes", ctypes.c_int), ("op", GemvParams * MAX_CHAIN)]
 
 
-def lib() -> ctypes.CDLL:
+class _Library:
+    """The kernel libraries behind one object: a launcher's library is loaded (and built, if it is not current) the
+    first time one of its symbols is used."""
+
+    def __init__(self, debug: bool):
+        self._debug, self._dlls = debug, {}
+
+    def _dll(self, group: str) -> ctypes.CDLL:
+        dll = self._dlls.get(group)
+        if dll is None:
+            if not _build.is_current(group, self._debug):
+                _build.build(groups=(group,), debug=self._debug)
+            dll = self._dlls[group] = ctypes.CDLL(_build.lib_path(group, self._debug))
+        return dll
+
+    @property
+    def _name(self) -> str:
+        return _build.lib_path("base", self._debug)
+
+    def __getattr__(self, name: str):
+        if not name.startswith("ti_") or not hasattr(_Sigs, name):
+            raise AttributeError(name)
+        restype, argtypes, group = getattr(_Sigs, name)
+        fn = getattr(self._dll(group), name, None)
+        if fn is None:
+            raise RuntimeError(f"{_build.lib_path(group, self._debug)} lacks symbol {name}; "
+                               "rebuild with python -m tileinfer_b200.ops.build --force")
+        fn.restype, fn.argtypes = restype, argtypes
+        setattr(self, name, fn)
+        return fn
+
+
+def lib() -> _Library:
     global _LIB
     if _LIB is None:
-        if os.environ.get("TI_DEBUG_LIB", "0") == "1":
-            path = _build.build_debug()          # bounds-checked + jittered variant (tests, debugging)
-        else:
-            path = _build.LIB
-            if not _build.is_current():
-                path = _build.build()
-        _LIB = ctypes.CDLL(path)
-        for name in dir(_Sigs):
-            if name.startswith("ti_"):
-                fn = getattr(_LIB, name, None)
-                if fn is None:
-                    raise RuntimeError(f"{path} lacks symbol {name}; rebuild with python -m tileinfer_b200.ops.build --force")
-                fn.restype, fn.argtypes = getattr(_Sigs, name)
-        if _LIB.ti_gemv_params_size() != ctypes.sizeof(GemvParams) or \
-                _LIB.ti_chain_params_size() != ctypes.sizeof(ChainParams):
-            raise RuntimeError("GemvParams / ChainParams layout mismatch between Python and CUDA")
+        # TI_DEBUG_LIB=1: bounds-checked + jittered variant (tests, debugging)
+        _LIB = _Library(os.environ.get("TI_DEBUG_LIB", "0") == "1")
     return _LIB
+
+
+def build_groups(*groups: str):
+    """Build several groups together (their sources compile in parallel) before the first of their symbols is used."""
+    _build.build(groups=groups, debug=lib()._debug)
 
 
 _I, _P, _F, _U64 = ctypes.c_int, ctypes.c_void_p, ctypes.c_float, ctypes.c_uint64
 
 
 class _Sigs:
-    ti_gemv_chain = (_I, [ctypes.POINTER(ChainParams), _I, _I, _P])
-    ti_gemv_chain_prepare = (_I, [ctypes.POINTER(ChainParams), _I, _I])
-    ti_gemv_ranks = (_I, [ctypes.POINTER(ChainParams), _P, _I, _I, _P])
-    ti_gemv_params_size = (_I, [])
-    ti_chain_params_size = (_I, [])
+    ti_gemv_chain = (_I, [ctypes.POINTER(ChainParams), _I, _I, _P], "hybrid")
+    ti_gemv_chain_prepare = (_I, [ctypes.POINTER(ChainParams), _I, _I], "hybrid")
+    ti_gemv_ranks = (_I, [ctypes.POINTER(ChainParams), _P, _I, _I, _P], "hybrid")
+    ti_gemv_params_size = (_I, [], "hybrid")
+    ti_chain_params_size = (_I, [], "hybrid")
 
 
-def register(name: str, restype, argtypes):
-    setattr(_Sigs, name, (restype, argtypes))
+def register(name: str, restype, argtypes, group: str = "base"):
+    """Declare a launcher exported by the library of `group` (build.py)."""
+    setattr(_Sigs, name, (restype, argtypes, group))
 
 
 def ptr(t) -> int:
