@@ -1,8 +1,8 @@
 """Engine configuration.
 
 Field names and defaults follow the reference's Config dataclass (engine/config.py:11-41).
-`model` may be a preset ("preset:tiny-hybrid", "preset:qwen3.6-27b") or a local HuggingFace
-directory; presets need neither a checkpoint nor a tokenizer on disk.  Additional fields are new
+`model` may be a preset ("preset:tiny-hybrid", "preset:qwen3.6-27b", "preset:tiny-kabadra") or a local
+model directory (HuggingFace, or a config.json that names its architecture); presets need neither a checkpoint nor a tokenizer on disk.  Additional fields are new
 and all have defaults.
 """
 from __future__ import annotations
@@ -10,7 +10,7 @@ from __future__ import annotations
 import os
 from dataclasses import dataclass
 
-from ..models.config import ModelConfig, from_hf_config, get_preset, PRESETS
+from ..models import registry
 
 
 @dataclass
@@ -28,7 +28,6 @@ class Config:
     # execution
     enforce_eager: bool = False
     cuda_graph_max_batch_size: int = 256
-    hf_config: object = None
     eos: list = None
     max_prefill_chunk_tokens: int = 4096
     enable_prefix_caching: bool = True
@@ -38,7 +37,7 @@ class Config:
     nccl_timeout: float = 600.0
     # ---- additions -------------------------------------------------------
     weights: str = "random:0"          # "random:<seed>" or "hf"
-    quantization: str = "w8a16"        # "w8a16" or "bf16"
+    quantization: str = "w8a16"        # "w8a16" or "bf16"; "fp32" (everything in 32 bits) where the family has it
     device: str = "auto"               # "auto" | "cuda" | "cpu"
     prefix_state_stride: int = 256     # DeltaNet state snapshots at stride * 2^j prompt tokens
     gdn_state_dtype: str = "fp32"      # recurrent-state pool dtype on the GPU: "fp32" | "bf16"
@@ -47,23 +46,21 @@ class Config:
     heartbeat_interval: float = 0.0    # seconds between peer heartbeats under tensor parallelism (0: watchdog off)
     heartbeat_timeout: float = 10.0    # a peer silent for this long is reported lost before the next step
     weight_cache_dir: str = None       # on-disk cache of per-rank quantised shards
-    model_config: ModelConfig = None
-    tokenizer: str = "auto"            # "auto" | "byte" | local path
+    model_config: object = None        # ModelConfig, KabadraConfig, ... (models/registry.py)
+    tokenizer: str = "auto"            # "auto" | "byte" | "ids" | local path
 
     def __post_init__(self):
         if self.model_config is None:
             name = self.model
-            if name.startswith("preset:") or name in PRESETS:
-                self.model_config = get_preset(name)
+            if registry.is_preset(name):
+                self.model_config = registry.get_preset(name)
             elif os.path.isdir(name):
-                from transformers import AutoConfig
-                self.hf_config = AutoConfig.from_pretrained(name, trust_remote_code=False)
-                self.model_config = from_hf_config(self.hf_config)
+                self.model_config = registry.config_from_dir(name)
                 if self.weights.startswith("random") and os.path.exists(os.path.join(name, "config.json")) \
                         and any(f.endswith(".safetensors") for f in os.listdir(name)):
                     self.weights = "hf"
             else:
-                raise ValueError(f"model {name!r} is neither a preset ({sorted(PRESETS)}) nor a local directory")
+                raise ValueError(f"model {name!r} is neither a preset ({sorted(registry.all_presets())}) nor a local directory")
         mc = self.model_config
         self.max_model_len = min(self.max_model_len, mc.max_position_embeddings)
         if self.eos is None:
@@ -77,6 +74,7 @@ class Config:
             raise ValueError("max_prefill_chunk_tokens must be a multiple of kvcache_block_size")
         if self.prefix_state_stride % self.kvcache_block_size:
             raise ValueError("prefix_state_stride must be a multiple of kvcache_block_size")
-        if self.quantization not in ("w8a16", "bf16"):
-            raise ValueError(f"quantization must be w8a16 or bf16, got {self.quantization}")
+        quants = registry.family(mc.family).quantizations
+        if self.quantization not in quants:
+            raise ValueError(f"quantization must be one of {', '.join(quants)} for {mc.name}, got {self.quantization}")
         mc.validate_tp(self.tp_size)

@@ -7,8 +7,8 @@ snapshots (host copies, LRU of max_prefix_states), batch building, sampling, and
 drops the last sequence of the batch (engine/model_runner.py:726-750).
 
 What is different:
-* the model is an explicit executor object (`TorchHybridModel` on CPU, `B200HybridModel` on the GPU)
-  instead of monkey-patched HuggingFace layers;
+* the model is an explicit executor object (`TorchHybridModel` on CPU, `B200HybridModel` on the GPU, or
+  what another family registers in models/registry.py) instead of monkey-patched HuggingFace layers;
 * one step may mix prefill chunks of several sequences with decode tokens (variable-length batch);
 * swap-out / swap-in of KV blocks plus DeltaNet state to host memory is implemented;
 * DeltaNet snapshots are taken at the prompt positions the scheduler asks for, also inside a chunk.
@@ -20,8 +20,8 @@ from collections import OrderedDict, deque
 
 import torch
 
-from ..models.reference_cpu import Batch, TorchHybridModel
-from ..models.weights import make_weight_source
+from ..models import registry
+from ..models.reference_cpu import Batch
 from .config import Config
 from .sampler import Sampler
 from .sequence import Sequence
@@ -60,15 +60,15 @@ class ModelRunner:
     # ---- model / cache ----------------------------------------------------
     def load_model(self):
         cfg = self.config
+        fam = registry.family(self.mc.family)
+        executor = fam.executor(cfg.device)
+        src = fam.make_weights(self.mc, cfg.weights, cfg.model, device=cfg.device)
         if cfg.device == "cuda":
-            from ..models.hybrid_b200 import B200HybridModel
-            src = make_weight_source(self.mc, cfg.weights, cfg.model, device="cuda")
-            self.model = B200HybridModel(self.mc, src, quant=cfg.quantization, tp=self.tp_size,
-                                         rank=self.tp_rank, comm=self.comm, config=cfg)
+            self.model = executor(self.mc, src, quant=cfg.quantization, tp=self.tp_size,
+                                  rank=self.tp_rank, comm=self.comm, config=cfg)
         else:
-            src = make_weight_source(self.mc, cfg.weights, cfg.model, device="cpu")
-            self.model = TorchHybridModel(self.mc, src, quant=cfg.quantization if cfg.quantization == "w8a16" else "none",
-                                          tp=self.tp_size, rank=self.tp_rank, comm=self.comm)
+            self.model = executor(self.mc, src, quant=cfg.quantization if cfg.quantization == "w8a16" else "none",
+                                  tp=self.tp_size, rank=self.tp_rank, comm=self.comm)
         self.sampler = Sampler(self.comm, self.model.vocab_start, cfg.eos, seed=0,
                                full_vocab_gather=cfg.baseline_full_vocab_gather)
         self.sampler._v_local = getattr(self.model, "v_local", self.mc.vocab_size // self.tp_size)
@@ -142,6 +142,8 @@ class ModelRunner:
         return True
 
     def has_prefix_state(self, seq: Sequence, node_id: int, num_tokens: int) -> bool:
+        if not self.mc.recurrent:
+            return True                      # the cached blocks are the whole state
         if node_id in self.prefix_state_cache:
             self.prefix_state_cache.move_to_end(node_id)
             self.pinned_prefix_states[seq.seq_id] = node_id
@@ -190,6 +192,19 @@ class ModelRunner:
                     torch.cuda.empty_cache()
                 self.oom_preempted.append(seqs.pop())
                 dropped += 1
+
+    def run_logits(self, seqs: list, out_rows: list) -> torch.Tensor:
+        """Execute one step without sampling; fp32 logits [len(out_rows), vocab] (this rank's shard) at the flat rows
+        asked for, on the host."""
+        self.steps += 1
+        batch = self.build_batch(seqs)
+        batch.out_rows = list(out_rows)
+        self.last_batch_tokens = batch.cu_seqlens[-1]
+        if hasattr(self.model, "step_logits"):
+            out = self.model.step_logits(batch).cpu()
+            self.model.check_status(self.model.peer_status())
+            return out
+        return self.model.logits(self.model.forward(batch)).float()
 
     def build_batch(self, seqs: list) -> Batch:
         bs = self.block_size

@@ -7,7 +7,7 @@ whole prefix and RoPE positions stay valid; engine/prefix_cache.py:1-8, 51-100).
   produced it and is released only by LRU eviction (`evict`).
 * Only blocks that have actually been prefilled are inserted.
 * A prefix is reusable only up to the deepest node that also has a recurrent-state snapshot; the
-  hybrid model cannot resume from KV blocks alone.
+  hybrid model cannot resume from KV blocks alone.  (`needs_state=False`: models without such state.)
 """
 from __future__ import annotations
 
@@ -27,7 +27,8 @@ class PrefixNode:
 
 
 class PrefixCache:
-    def __init__(self, block_size: int, block_manager=None):
+    def __init__(self, block_size: int, block_manager=None, needs_state: bool = True):
+        self.needs_state = needs_state
         self.block_size = block_size
         self.bm = block_manager
         self.root = PrefixNode(None, None, -1, 0)
@@ -63,7 +64,7 @@ class PrefixCache:
         if max_tokens is None:
             max_tokens = len(token_ids) - 1
         chain = self.match(token_ids, max_tokens)
-        while chain and not chain[-1].has_state:
+        while self.needs_state and chain and not chain[-1].has_state:
             chain.pop()
         if not chain:
             return [], 0

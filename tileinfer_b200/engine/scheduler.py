@@ -45,7 +45,9 @@ class Scheduler:
         self.tokenizer = tokenizer
         self.max_preempt_count = max(1, config.max_num_seqs // 4)
         self.enable_prefix_caching = config.enable_prefix_caching
-        self.prefix_cache = PrefixCache(self.block_size, self.block_manager)
+        # models without recurrent state resume from cached blocks alone
+        self.recurrent = getattr(config.model_config, "recurrent", True)
+        self.prefix_cache = PrefixCache(self.block_size, self.block_manager, needs_state=self.recurrent)
         if self.enable_prefix_caching:
             self.block_manager.evictor = self.prefix_cache.evict
             self.block_manager.evictable = self.prefix_cache.num_evictable
@@ -164,7 +166,7 @@ class Scheduler:
     def _snapshot_points(self, seq: Sequence, lo: int, hi: int) -> list:
         """Prompt positions in (lo, hi] at which the DeltaNet state is captured for prefix reuse:
         stride * 2^j, block-aligned chunk ends, and the last block boundary below the prompt end."""
-        if not self.enable_prefix_caching or seq.num_completion_tokens > 0:
+        if not self.enable_prefix_caching or not self.recurrent or seq.num_completion_tokens > 0:
             return []
         bs, pts = self.block_size, set()
         p = self.state_stride
@@ -191,13 +193,33 @@ class Scheduler:
                                            or self.on_prefix_hit(seq, chain[-1].node_id, n)):
                     bm.allocate_extra(seq)
                     seq.num_cached_tokens = n
-                    seq.prefix_restore_key = chain[-1].node_id
+                    seq.prefix_restore_key = chain[-1].node_id if self.recurrent else None
                     return True
                 bm.deallocate(seq)          # give the references back; the cache still holds its own
         if bm.can_allocate(seq):
             bm.allocate(seq)
             return True
         return False
+
+    # ---- replay: the caller decides which tokens of which sequences run ----------
+    def schedule_given(self, seq: Sequence):
+        """Schedule exactly the tokens of `seq` that are not cached yet, reserving their blocks (a new sequence is
+        admitted).  There is no preemption: too few blocks or too many sequences are the caller's error."""
+        if seq.seq_id not in self.running:
+            if len(self.running) >= self.max_num_seqs:
+                raise RuntimeError(f"more than {self.max_num_seqs} live sequences")
+            seq.status = SequenceStatus.RUNNING
+            self.running[seq.seq_id] = seq
+        if not self.block_manager.can_append(seq):
+            raise RuntimeError(f"out of KV blocks: a sequence of {seq.num_tokens} tokens does not fit")
+        self.block_manager.allocate_extra(seq)
+        seq.num_scheduled_tokens = seq.num_tokens - seq.num_cached_tokens
+        seq.is_prefill = seq.num_scheduled_tokens > 1
+
+    def finish_given(self, seq: Sequence):
+        """The scheduled tokens of `seq` have run."""
+        seq.num_cached_tokens += seq.num_scheduled_tokens
+        seq.num_scheduled_tokens = 0
 
     def advance_decode(self, seqs: list) -> list:
         """Between the sub-steps of multi-step decode: reserve the next KV slot of each sequence.

@@ -92,6 +92,12 @@ class Sequence:
         self.last_token = token_id
         self.num_tokens += 1
 
+    def extend(self, token_ids: list):
+        """Further tokens that arrive from outside (replayed requests)."""
+        self.token_ids.extend(token_ids)
+        self.last_token = token_ids[-1]
+        self.num_tokens = len(self.token_ids)
+
     _STATE = ("seq_id", "status", "num_tokens", "num_prompt_tokens", "num_cached_tokens",
               "num_scheduled_tokens", "block_table", "token_ids", "last_token", "is_prefill",
               "temperature", "max_tokens", "ignore_eos", "top_p", "top_k", "deltanet_state_slot",

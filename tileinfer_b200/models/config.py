@@ -36,6 +36,9 @@ class ModelConfig:
     eos_token_ids: tuple = ()
     max_position_embeddings: int = 262144
 
+    family = "hybrid"           # entry of models/registry.py
+    recurrent = True            # a prefix is reusable only where the recurrent state was captured
+
     # ---- derived sizes -------------------------------------------------
     @property
     def gdn_key_dim(self) -> int:

@@ -331,7 +331,7 @@ class DeviceRuntime:
         sp = SampleParams()
         sp.cand_val, sp.cand_idx = ptr(topk_state.out_val), ptr(topk_state.out_idx)
         sp.temperature, sp.top_p, sp.u, sp.top_k = ptr(t.fpar[0]), ptr(t.fpar[1]), ptr(t.fpar[2]), ptr(t.ipar[0])
-        sp.out_tok, sp.status_src = ptr(t.tok), self.ctrl.data_ptr() + 4
+        sp.out_tok, sp.status_src = ptr(t.tok), self._status_ptr()
         sp.M, sp.n_cand = n, topk_state.out_val.shape[1]
         t.sample = sp
         return t
@@ -369,21 +369,12 @@ class DeviceRuntime:
         """The step's only device -> host copy: n token ids and the communicator's status word."""
         t.h_tok.copy_(t.tok, non_blocking=True)
         torch.cuda.current_stream().synchronize()
-        status = int(t.h_tok[t.tok.shape[0] - 1])
-        if status != 0:
-            # a bounded device wait ran out (a peer's flag or packet, an mbarrier) or a checked index was out of range:
-            # whatever the kernels computed after that is not to be trusted, on one GPU as on eight
-            from ..parallel.watchdog import PeerLostError
-            err = PeerLostError([])
-            err.args = (f"device status word {status:#x}: a bounded wait ran out"
-                        f"{' on a tensor-parallel peer' if self.peer is not None else ''} or an index check failed; "
-                        "the tokens of this step are discarded",)
-            raise err
+        self.check_status(int(t.h_tok[t.tok.shape[0] - 1]))
         return t.h_tok[:n].tolist()
 
-    def _decode_graph_step(self, batch, k: int, spec=None):
+    def _decode_graph_step(self, batch, k: int, spec=None, keep_logits: bool = False):
         n = batch.num_seqs
-        g = self.decode_graph(n, k, edits=bool(spec and spec.get("edits")))
+        g = self.decode_graph(n, k, edits=keep_logits or bool(spec and spec.get("edits")))
         self._last_graph = g
         h, x = g.host, g.x
         h["ids"][:n] = batch.input_ids
@@ -414,6 +405,37 @@ class DeviceRuntime:
         self.host_steps += 1
         return g.topk.out_val[:n], g.topk.out_idx[:n]
 
+    def _graph_serves(self, batch) -> bool:
+        """One token per sequence, and a captured bucket holds the step."""
+        return bool(batch.cu_seqlens[-1] == batch.num_seqs and self.graphs and batch.num_seqs <= self.buckets[-1]
+                    and max(len(b) for b in batch.block_tables) <= self.graph_max_blocks)
+
+    @torch.no_grad()
+    def step_logits(self, batch) -> torch.Tensor:
+        """Runs the step the way generation does (captured graph for decode-only steps) and returns the fp32 logits
+        of this rank's vocabulary shard at `batch.out_rows` (default: the last token of every sequence)."""
+        rows = batch.out_rows if batch.out_rows is not None else [e - 1 for e in batch.cu_seqlens[1:]]
+        if self._graph_serves(batch):
+            self._decode_graph_step(batch, 1, keep_logits=True)
+            return self._last_graph.logits[rows]
+        hidden = self.forward(batch)
+        return self.logits(hidden) if rows else torch.empty(0, self.v_local, device=self.dev)
+
+    def _status_ptr(self) -> int:
+        """Device word the kernels of this executor OR their error bits into."""
+        return self.ctrl.data_ptr() + 4
+
+    def check_status(self, status: int):
+        """Raises when the device status word of a step is set: a bounded device wait ran out (a peer's flag or packet,
+        an mbarrier) or a checked index was out of range, and whatever was computed after that is not to be trusted."""
+        if status != 0:
+            from ..parallel.watchdog import PeerLostError
+            err = PeerLostError([])
+            err.args = (f"device status word {status:#x}: a bounded wait ran out"
+                        f"{' on a tensor-parallel peer' if self.peer is not None else ''} or an index check failed; "
+                        "the tokens of this step are discarded",)
+            raise err
+
     def _default_spec(self, n):
         return {"temperature": [0.0] * n, "top_k": [1] * n, "top_p": [1.0] * n, "u": [0.0] * n, "edits": []}
 
@@ -429,9 +451,7 @@ class DeviceRuntime:
         if spec is None:
             spec = self._default_spec(n)
         fused = self.tp == 1 or self.peer is not None        # candidates of all ranks are on this device after top-k
-        decode_only = batch.cu_seqlens[-1] == batch.num_seqs and n == batch.num_seqs
-        if decode_only and self.graphs and batch.num_seqs <= self.buckets[-1] \
-                and max(len(b) for b in batch.block_tables) <= self.graph_max_blocks:
+        if n == batch.num_seqs and self._graph_serves(batch):
             vals, idx = self._decode_graph_step(batch, k, spec)
             if fused:
                 return self._read_tokens(self._last_graph.samp, n)

@@ -209,7 +209,7 @@ def add_engine_args(ap: argparse.ArgumentParser):
     ap.add_argument("--tp-size", type=int, default=1)
     ap.add_argument("--num-scheduler-steps", type=int, default=1)
     ap.add_argument("--no-prefix-caching", action="store_true")
-    ap.add_argument("--quantization", default="w8a16", choices=["w8a16", "bf16"])
+    ap.add_argument("--quantization", default="w8a16", choices=["w8a16", "bf16", "fp32"])
     ap.add_argument("--swap-space-gb", type=float, default=0.0)
     ap.add_argument("--device", default="auto")
     ap.add_argument("--heartbeat-interval", type=float, default=0.0,

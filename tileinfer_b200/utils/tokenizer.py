@@ -72,17 +72,61 @@ class ByteTokenizer:
         return self.encode(text) if tokenize else text
 
 
+class IdTokenizer:
+    """Text is a list of token ids ("5 17 3"): for vocabularies too small for bytes and for runs that bring their own
+    ids.  There is no EOS."""
+    eos_token_id = None
+    eos_token = ""
+    pad_token_id = 0
+    all_special_ids: list = []
+
+    def __init__(self, vocab_size: int):
+        self.vocab_size = vocab_size
+
+    def __len__(self):
+        return self.vocab_size
+
+    def encode(self, text: str, add_special_tokens: bool = True) -> list:
+        ids = [int(w) for w in text.split()]
+        if any(not 0 <= i < self.vocab_size for i in ids):
+            raise ValueError(f"token id outside [0, {self.vocab_size})")
+        return ids
+
+    def __call__(self, text, **kw):
+        return {"input_ids": self.encode(text)}
+
+    def decode(self, ids, skip_special_tokens: bool = True) -> str:
+        return str(int(ids)) if isinstance(ids, int) else " ".join(str(int(i)) for i in ids)
+
+    def convert_ids_to_tokens(self, ids):
+        return [str(int(i)) for i in ids]
+
+    def apply_chat_template(self, messages, tokenize: bool = False, add_generation_prompt: bool = True, **kw):
+        text = " ".join(str(m.get("content", "")) for m in messages)
+        return self.encode(text) if tokenize else text
+
+
+def _builtin_tokenizer(vocab_size: int):
+    return ByteTokenizer(vocab_size) if vocab_size >= 258 else IdTokenizer(vocab_size)
+
+
 def load_tokenizer(config):
-    """Tokenizer for a Config: byte-level for presets, AutoTokenizer for a local model directory."""
+    """Tokenizer for a Config: byte-level for presets and for folders without tokenizer files (ids as text when the
+    vocabulary is too small for bytes), AutoTokenizer for other local model directories."""
     import os
     spec = config.tokenizer
-    if spec == "byte" or (spec == "auto" and not os.path.isdir(config.model)):
+    if spec == "ids":
+        return IdTokenizer(config.model_config.vocab_size)
+    if spec == "byte":
         return ByteTokenizer(config.model_config.vocab_size)
+    if spec == "auto" and (not os.path.isdir(config.model)
+                           or not any("token" in f or f.startswith("vocab") for f in os.listdir(config.model))):
+        return _builtin_tokenizer(config.model_config.vocab_size)
     from transformers import AutoTokenizer
     path = config.model if spec == "auto" else spec
     try:
         return AutoTokenizer.from_pretrained(path, trust_remote_code=False)
     except Exception:
         if spec == "auto":
-            return ByteTokenizer(config.model_config.vocab_size)
+            return _builtin_tokenizer(config.model_config.vocab_size)
         raise
