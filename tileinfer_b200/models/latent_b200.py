@@ -81,6 +81,9 @@ class B200LatentModel(DeviceRuntime):
         self.block_size, self.cache = PAGE, {}
         self.graphs, self.snapshots, self.host_steps = {}, {}, 0
         self.launches_per_decode_step = self._launches = 0
+        # sequences with at least this many tokens in a step expand keys and values (tcgen05 tiles)
+        tiled = not self.f32 and all(L.dp <= 256 and L.vp <= 256 for L in self.layers)
+        self.PREFILL_ATTN_MIN_TOKENS = 32 if tiled else 1 << 30
         self.status = F.status_ptr()
 
     # ------------------------------------------------------------------ weights
@@ -125,11 +128,14 @@ class B200LatentModel(DeviceRuntime):
             uv = pad_to(get(p + "mix.uv").view(H, m.vdim, -1), H, L.vp, L.Rp)
             L.uk_t = uk.transpose(1, 2).to(self.dtype).contiguous()          # [H, Rp, dp]
             L.uv = uv.to(self.dtype).contiguous()                            # [H, vp, Rp]
+            if not self.f32:                                                 # rows [K of all heads | V of all heads]
+                L.w_ukv = LinearW(torch.cat([uk.reshape(H * L.dp, L.Rp), uv.reshape(H * L.vp, L.Rp)]), False, dev)
             L.sink = get(p + "mix.sink").float().contiguous()
             self.layers.append(L)
         self.head = Product(pad_to(get("head"), c.vocab_size, Wp), "fp32" if self.f32 else "bf16", dev)
 
     def weight_bytes(self) -> int:
+        """Bytes of weights a decode step streams."""
         n = self.head.nbytes()
         for L in self.layers:
             n += L.w_in.nbytes() + L.w_out.nbytes() + (L.uk_t.numel() + L.uv.numel()) * L.uv.element_size()
@@ -206,6 +212,7 @@ class B200LatentModel(DeviceRuntime):
                 x.o_part = torch.empty(part, dtype=torch.float32, device=dev)
                 x.ml_part = torch.empty(part // 64 * 2, dtype=torch.float32, device=dev)
         x.short = (0, T)                    # rows [a, b) that hold every token of the split attention
+        x.reach = {}                        # window -> (cache slots in reach, query tiles) of the long portions
         return x
 
     def _attn_short(self, L, x: StepCtx, proj, cat):
@@ -227,6 +234,45 @@ class B200LatentModel(DeviceRuntime):
         F.head_product(o_lat[a:b], L.uv, cat[a:b], gate=proj[a:b], gcol=L.g_col)
         self._launches += 3 + (p.nsplit > 1)
 
+    def _prepare_step(self, x: StepCtx, batch):
+        """Which rows the split attention covers, and per window the cached rows in reach of the long portions of the step
+        with their query tiles (see `latent_prefill`)."""
+        bs, short, longs = self.block_size, [], []
+        for s in range(batch.num_seqs):
+            t0, t1 = batch.cu_seqlens[s], batch.cu_seqlens[s + 1]
+            (longs if t1 - t0 >= self.PREFILL_ATTN_MIN_TOKENS else short).append((s, t0, t1))
+        x.short = (short[0][1], short[-1][2]) if short else (0, 0)
+        x.reach, x.latents = {}, {}
+        for window in {L.window for L in self.layers} if longs else ():
+            slots, tiles, base = [], [], 0
+            for s, t0, t1 in longs:
+                end = batch.context_lens[s]
+                start = end - (t1 - t0)
+                lo = max(0, start - window + 1)
+                pos = torch.arange(lo, end)
+                slots.append(torch.tensor(batch.block_tables[s], dtype=torch.long)[pos // bs] * bs + pos % bs)
+                for a in range(t0, t1, 128):
+                    p0, n = start + a - t0, min(128, t1 - a)
+                    tiles.append((p0 + n - max(0, p0 - window + 1), a, n, p0, base, lo))
+                base += end - lo
+            tiles.sort(key=lambda t: -t[0])                    # most keys first
+            x.reach[window] = (torch.cat(slots).to(self.dev, non_blocking=True),
+                               torch.tensor([t[1:] for t in tiles], dtype=torch.int32).t().contiguous().to(self.dev, non_blocking=True))
+
+    def _attn_long(self, L, x: StepCtx, proj, cat):
+        """Long portions of prompts: keys and values of every cached latent in reach, then windowed query tiles."""
+        slots, tiles = x.reach[L.window]
+        n, key = slots.numel(), (L.owner, L.window)
+        if key not in x.latents:                               # layers that share latents share the gathered rows
+            x.latents[key] = torch.empty(n, L.Rp, dtype=self.dtype, device=self.dev)
+            F.latent_gather(self.cache[L.owner], slots, x.latents[key])
+            self._launches += 1
+        kv = torch.empty(n, L.w_ukv.N, dtype=self.dtype, device=self.dev)
+        F.gemm_bf16(L.w_ukv, x.latents[key], out=kv)
+        F.latent_prefill(proj, kv, tiles, cat, H=L.heads, dp=L.dp, vp=L.vp, window=L.window, scale=L.scale, sink=L.sink,
+                         gate=proj, gcol=L.g_col, status=self.status)
+        self._launches += 2
+
     def _run_layers(self, x: StepCtx):
         c, T = self.cfg, x.T
         F.embed_pos(x.ids, x.positions, self.embed, self.pos, self.embed_norm, x.x, self.W, c.rms_eps)
@@ -246,6 +292,8 @@ class B200LatentModel(DeviceRuntime):
                 n += 1
             if x.num_qg:
                 self._attn_short(L, x, proj, cat)
+            if x.reach:
+                self._attn_long(L, x, proj, cat)               # after the split attention, whose row range may span these
             n += L.w_out(cat, x.x, F.GEPI_RESID32, F.gemm_epilogue(resid32=x.x))
             self._launches += n + 1
         nvtx_end()
@@ -255,8 +303,6 @@ class B200LatentModel(DeviceRuntime):
         h = torch.empty(n, self.Wp, dtype=self.dtype, device=self.dev)
         F.rmsnorm_f32(hidden, self.final_norm, h, self.W, self.cfg.rms_eps)
         self._launches += 1 + self.head(h, logits, F.GEPI_F32, F.gemm_epilogue(scale=self.cfg.logit_scale))
-
-    PREFILL_ATTN_MIN_TOKENS = 1 << 30
 
     def _status_ptr(self) -> int:
         return self.status

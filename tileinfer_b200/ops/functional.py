@@ -144,6 +144,7 @@ _l.register("ti_gemm_w8a16", _I, [_P, _P, _I, _I, _I, _P, _P, _P, _I, _P, _P, _I
 _l.register("ti_latent_attn_params_size", _I, [], "latent")
 _l.register("ti_latent_attn_max_split_rank", _I, [], "latent")
 _l.register("ti_latent_attn", _I, [ctypes.POINTER(LatentAttnParams), _I, _P], "latent")
+_l.register("ti_latent_prefill", _I, [_P, _I, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P], "latent")
 _l.register("ti_embed_pos", _I, [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P, _I, _P], "latent")
 _l.register("ti_rmsnorm_f32", _I, [_P, _P, _P, _I, _I, _I, _F, _I, _P], "latent")
 _l.register("ti_latent_store", _I, [_P, _I, _I, _P, _P, _P, _LL, _I, _I, _I, _F, _I, _P], "latent")
@@ -697,6 +698,14 @@ def latent_attn(p: LatentAttnParams, f32: bool):
     if not p.status:
         p.status = status_ptr()
     check(_l.lib().ti_latent_attn(ctypes.byref(p), int(f32), stream()), "ti_latent_attn")
+
+
+def latent_prefill(q, kv, tiles, out, *, H, dp, vp, window, scale, sink=None, gate=None, gcol=0, status=0):
+    """Windowed attention of prefill query tiles over expanded rows kv [Nk, H * dp keys | H * vp values] (bf16).
+    `tiles`: int32 [5, n] = first flat token, tokens, its position, a row of kv, the position that row holds."""
+    check(_l.lib().ti_latent_prefill(ptr(q), q.shape[0], q.stride(0), ptr(kv), kv.shape[0], kv.stride(0), ptr(tiles), tiles.shape[1],
+                                     ptr(sink), ptr(gate), 0 if gate is None else gate.stride(0), gcol, ptr(out), out.stride(0),
+                                     H, dp, vp, H * dp, window, scale, status or status_ptr(), stream()), "ti_latent_prefill")
 
 
 def gemm_f32(w, x, *, out, epi=GEPI_F32, ex=None):
