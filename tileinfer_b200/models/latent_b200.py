@@ -76,8 +76,7 @@ class B200LatentModel(DeviceRuntime):
         self.vocab_start, self.v_local = 0, cfg.vocab_size
         self._build(src)
         torch.cuda.empty_cache()
-        # work items of the split attention per query token: groups of up to 32 heads
-        self.hkv = max(-(-L.heads // L.rows) for L in self.layers)
+        self.hkv = max(-(-L.heads // F.latent_rows(L.heads)) for L in self.layers)   # head groups per query token
         self.block_size, self.cache = PAGE, {}
         self.graphs, self.snapshots, self.host_steps = {}, {}, 0
         self.launches_per_decode_step = self._launches = 0
@@ -103,7 +102,6 @@ class B200LatentModel(DeviceRuntime):
             L.dp, L.vp, L.Rp = pad64(m.dim), pad64(m.vdim), pad64(m.kv_rank)
             L.window, L.scale = m.window, m.scale
             L.owner, L.stores = c.latent_layer(i), m.kv_from is None
-            L.rows = 32 if m.heads > 16 else 16                  # heads per block of the split attention
             L.norm1 = self._norm(get(p + "norm1"), Wp)
             H = m.heads
             q = pad_to(get(p + "mix.q").view(H, m.dim, -1), H, L.dp, Wp).reshape(H * L.dp, Wp)
@@ -189,11 +187,7 @@ class B200LatentModel(DeviceRuntime):
 
     # ------------------------------------------------------------------ step
     def _nsplit(self, L, num_qg: int) -> int:
-        """Splits of the key range: fill the SMs once, at least a tile of 64 keys each."""
-        if self.f32 or L.Rp > 512:
-            return 1
-        groups = -(-L.heads // L.rows)
-        return max(1, min(32, F.NUM_SMS // max(1, num_qg * groups), (L.window + PAGE - 2) // 64 + 1))
+        return 1 if self.f32 or L.Rp > 512 else F.latent_nsplit(num_qg, L.heads, L.Rp, L.window)
 
     def _alloc_ctx(self, T: int, S: int, max_blocks: int, num_qg: int, nsplit: int) -> StepCtx:
         x, dev, dt = self._alloc_inputs(T, S, max_blocks, num_qg, nsplit), self.dev, self.dtype
@@ -206,8 +200,8 @@ class B200LatentModel(DeviceRuntime):
         if num_qg:
             x.q_abs = new(T * max(L.heads * L.Rp for L in self.layers), dtype=dt, device=dev)
             x.o_lat = new(T * max(L.heads * L.Rp for L in self.layers), dtype=dt, device=dev)
-            part = max((num_qg * -(-L.heads // L.rows) * ns * L.rows * L.Rp
-                        for L in self.layers if (ns := self._nsplit(L, num_qg)) > 1), default=0)
+            part = max((F.latent_part_floats(num_qg, L.heads, L.Rp, ns) for L in self.layers if (ns := self._nsplit(L, num_qg)) > 1),
+                       default=0)
             if part:
                 x.o_part = torch.empty(part, dtype=torch.float32, device=dev)
                 x.ml_part = torch.empty(part // 64 * 2, dtype=torch.float32, device=dev)

@@ -694,6 +694,23 @@ def head_product(x, w, out, gate=None, gcol=0):
                                    0 if gate is None else gate.stride(0), gcol, _f32(w), stream()), "ti_head_product")
 
 
+def latent_rows(H: int) -> int:
+    """Heads a block of the split latent attention takes."""
+    return 32 if H > 16 else 16
+
+
+def latent_nsplit(num_qg: int, H: int, Rp: int, window: int) -> int:
+    """Splits of the key range (bf16, Rp <= 512): fill the SMs once, at least a tile of 64 keys each."""
+    groups = -(-H // latent_rows(H))
+    tiles = (window + 14) // 64 + 1 if window else 1 << 20
+    return max(1, min(32, NUM_SMS // max(1, num_qg * groups), tiles))
+
+
+def latent_part_floats(num_qg: int, H: int, Rp: int, nsplit: int) -> int:
+    """Size of the partial-output buffer; the (max, sum) buffer has two floats per row of Rp."""
+    return num_qg * -(-H // latent_rows(H)) * nsplit * latent_rows(H) * Rp
+
+
 def latent_attn(p: LatentAttnParams, f32: bool):
     if not p.status:
         p.status = status_ptr()
