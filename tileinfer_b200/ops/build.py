@@ -22,7 +22,7 @@ BUILD = os.path.join(HERE, "build")
 GROUPS = {
     "base": ("gemm_tcgen05.cu", "lm_head.cu", "pointwise.cu", "sampling.cu", "symm.cu"),
     "hybrid": ("attn_paged.cu", "attn_prefill.cu", "fused_ar.cu", "gdn.cu", "gdn_chunk.cu", "gemv_w8a16.cu"),
-    "latent": ("latent_ops.cu", "latent_attn.cu", "latent_prefill.cu"),
+    "latent": ("latent_ops.cu", "latent_attn.cu", "latent_decode.cu", "latent_prefill.cu"),
 }
 
 

@@ -8,52 +8,17 @@
 // A layer's mask is a parameter (window = 0: all earlier tokens; otherwise itself and the window - 1 tokens before it),
 // and so is the sink: one number per head that joins the denominator without key, value or scale (null: none).
 //
-// latent_decode_kernel (bf16, R up to 512): per (query token, head group, split) tiles of 64 keys, two tiles in flight by
+// latent_decode.cu (bf16, padded R of 256, 384, 512): the tcgen05 form for the sizes of large models.
+// latent_decode_kernel (bf16, other R up to 448): per (query token, head group, split) tiles of 64 keys, two tiles in flight by
 // cp.async; S = q~ c^T by mma.sync with the eight warps over (head tile, keys), softmax state in registers of the row's
 // threads, O += P c with the eight warps over column slices, the value fragments read from the SAME shared-memory tile
 // through ldmatrix.trans.  Splits meet in latent_merge_kernel, which also adds the sink.
 // latent_any_kernel (float for 32-bit mode, or bf16 with R above 512): one block per (query token, head).
-#include "common.cuh"
+#include "latent_attn.cuh"
 
 namespace ti {
 
-typedef __nv_bfloat16 bf16;
-
-struct LatentAttnParams {
-  const void* q;                 // [T][H][Rp] absorbed queries
-  const void* cache;             // [num_blocks][16][Rp]
-  const int* block_tables;       // [S, max_blocks]
-  const int* positions;          // [T]
-  const int* qg_seq;             // [num_qg] sequence of the query token
-  const int* qg_tok0;            // [num_qg] flat token
-  const int* qg_ntok;            // [num_qg] 1, or 0: padding
-  const float* sink;             // [H] or null
-  float* o_part;                 // [num_qg * head groups * nsplit][rows][Rp]
-  float* ml_part;                // [num_qg * head groups * nsplit][rows][2]
-  void* out;                     // [T][H][Rp]
-  unsigned* status;
-  int H, R, Rp, max_blocks, nsplit, num_qg, window, num_blocks;
-  float scale;
-};
-
-constexpr float kNeg = -1e30f;
-constexpr float kLog2e = 1.4426950408889634f;
 constexpr int kKeyTile = 64;
-constexpr int kMaxLatentSplit = 64;
-
-struct KeyRange { int pos, lo, page0, npages, ntiles, tps; };
-
-// keys of one query token: lo .. pos, walked in tiles of 64 from the start of lo's page; tps tiles per split
-TI_DEVICE KeyRange key_range(const LatentAttnParams& p, int tok) {
-  KeyRange r;
-  r.pos = p.positions[tok];
-  r.lo = p.window > 0 ? max(0, r.pos - p.window + 1) : 0;
-  r.page0 = r.lo >> 4;
-  r.npages = (r.pos >> 4) + 1;
-  r.ntiles = (r.pos - r.page0 * 16) / kKeyTile + 1;
-  r.tps = (r.ntiles + p.nsplit - 1) / p.nsplit;
-  return r;
-}
 
 TI_DEVICE void cpa16(uint32_t dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst), "l"(src) : "memory");
@@ -99,7 +64,7 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const __grid_constan
   pdl_wait();
   if (p.qg_ntok[qg] == 0) return;
   const int tok = p.qg_tok0[qg], seq = p.qg_seq[qg];
-  const KeyRange kr = key_range(p, tok);
+  const KeyRange kr = key_range(p, tok, kKeyTile);
   const int t0 = sp * kr.tps, t1 = min(kr.ntiles, t0 + kr.tps);
   if (t0 >= t1) return;                                           // inactive split: the merge never reads it
   const int* bt = p.block_tables + (size_t)seq * p.max_blocks;
@@ -278,14 +243,14 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const __grid_constan
 }
 
 // Combines the splits of one (query token, head) and adds the sink to the denominator.
-__global__ void __launch_bounds__(128) latent_merge_kernel(const __grid_constant__ LatentAttnParams p, int rows) {
+__global__ void __launch_bounds__(128) latent_merge_kernel(const __grid_constant__ LatentAttnParams p, int rows, int tile) {
   __shared__ float w_s[kMaxLatentSplit];
   const int qg = blockIdx.x, head = blockIdx.y, tid = threadIdx.x;
   pdl_trigger();
   pdl_wait();
   if (p.qg_ntok[qg] == 0) return;
   const int tok = p.qg_tok0[qg];
-  const KeyRange kr = key_range(p, tok);
+  const KeyRange kr = key_range(p, tok, tile);
   const int nact = (kr.ntiles + kr.tps - 1) / kr.tps;
   const int groups = (p.H + rows - 1) / rows, hg = head / rows, r = head - hg * rows;
   const size_t item0 = ((size_t)qg * groups + hg) * p.nsplit;
@@ -386,6 +351,10 @@ __global__ void __launch_bounds__(128) latent_any_kernel(const __grid_constant__
     if (tid + 128 * e < p.Rp) put(dst + tid + 128 * e, o[e] / l);
 }
 
+void launch_latent_merge(const LatentAttnParams& p, int rows, int tile, cudaStream_t st) {
+  launch_kernel(latent_merge_kernel, dim3(p.num_qg, p.H), dim3(128), 0, st, true, p, rows, tile);
+}
+
 template <int RT, int MT>
 static int launch_latent_decode(const LatentAttnParams& p, cudaStream_t st) {
   using G = LatentGeom<RT, MT>;
@@ -397,7 +366,7 @@ static int launch_latent_decode(const LatentAttnParams& p, cudaStream_t st) {
   }
   const int groups = (p.H + G::kRows - 1) / G::kRows;
   launch_kernel(k, dim3(p.num_qg, groups, p.nsplit), dim3(256), G::kSmem, st, true, p);
-  if (p.nsplit > 1) launch_kernel(latent_merge_kernel, dim3(p.num_qg, p.H), dim3(128), 0, st, true, p, (int)G::kRows);
+  if (p.nsplit > 1) launch_latent_merge(p, G::kRows, kKeyTile, st);
   return (int)cudaGetLastError();
 }
 
@@ -426,11 +395,9 @@ int ti_latent_attn(const ti::LatentAttnParams* pp, int f32, void* stream) {
     case 1: return two ? ti::launch_latent_decode<1, 2>(p, st) : ti::launch_latent_decode<1, 1>(p, st);
     case 2: return two ? ti::launch_latent_decode<2, 2>(p, st) : ti::launch_latent_decode<2, 1>(p, st);
     case 3: return two ? ti::launch_latent_decode<3, 2>(p, st) : ti::launch_latent_decode<3, 1>(p, st);
-    case 4: return two ? ti::launch_latent_decode<4, 2>(p, st) : ti::launch_latent_decode<4, 1>(p, st);
     case 5: return two ? ti::launch_latent_decode<5, 2>(p, st) : ti::launch_latent_decode<5, 1>(p, st);
-    case 6: return two ? ti::launch_latent_decode<6, 2>(p, st) : ti::launch_latent_decode<6, 1>(p, st);
     case 7: return two ? ti::launch_latent_decode<7, 2>(p, st) : ti::launch_latent_decode<7, 1>(p, st);
-    default: return two ? ti::launch_latent_decode<8, 2>(p, st) : ti::launch_latent_decode<8, 1>(p, st);
+    default: return ti::launch_latent_decode_tc(p, st);
   }
 }
 
