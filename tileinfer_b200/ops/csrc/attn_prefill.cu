@@ -308,33 +308,6 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
   }
 }
 
-// K cache [rows = blocks*hkv*16][D] seen as [groups of 8 rows][D/64 slabs][8 rows][64 columns]: one copy brings a
-// 16-key page as two 8-key groups with their column slabs side by side (the layout the QK^T descriptors walk).
-static int bf16_map_kpage(CUtensorMap* dst, const void* base, int D, long long rows) {
-  static std::map<AMapKey, CUtensorMap> cache;
-  static std::mutex mu;
-  std::lock_guard<std::mutex> lock(mu);
-  const AMapKey key{base, D, rows, 64, 8, -1};
-  auto it = cache.find(key);
-  if (it == cache.end()) {
-    EncodeTiledFn enc = encode_tiled_fn();
-    if (enc == nullptr) return 999;
-    CUtensorMap m;
-    const cuuint64_t dims[4] = {64, 8, (cuuint64_t)(D / 64), (cuuint64_t)(rows / 8)};
-    const cuuint64_t strides[3] = {(cuuint64_t)D * 2, 128, (cuuint64_t)D * 16};
-    const cuuint32_t box[4] = {64, 8, (cuuint32_t)(D / 64), 2};
-    const cuuint32_t elem[4] = {1, 1, 1, 1};
-    const CUresult r = enc(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, elem,
-                           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    if (r != CUDA_SUCCESS) return 1000 + (int)r;
-    if (cache.size() > 4096) cache.clear();
-    it = cache.emplace(key, m).first;
-  }
-  *dst = it->second;
-  return 0;
-}
-
 template <int D>
 static int launch_attn_prefill(const AttnPrefillParams& p, int num_tiles, cudaStream_t st) {
   static bool configured = false;
@@ -366,7 +339,7 @@ int ti_attn_prefill(const void* q, int T, const void* kcache, const void* vcache
   ti::AttnPrefillParams p = {};
   int rc = ti::bf16_map_2d(&p.map_q, q, (long long)hq * D, T, 64, 128, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
-  rc = ti::bf16_map_kpage(&p.map_k, kcache, D, (long long)num_blocks * hkv * 16);
+  rc = ti::bf16_map_groups(&p.map_k, kcache, D, (long long)num_blocks * hkv * 16, D / 64, 2);
   if (rc) return rc;
   rc = ti::bf16_map_2d(&p.map_v, vcache, 16, (long long)num_blocks * hkv * D, 16, D, CU_TENSOR_MAP_SWIZZLE_32B);
   if (rc) return rc;

@@ -127,18 +127,19 @@ TI_DEVICE uint64_t smem_desc_sw32(uint32_t saddr) {
 TI_DEVICE constexpr uint32_t idesc_f16_bf16(int M, int N) {
   return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(M >> 4) << 24);
 }
-// MN-major B operand (the contraction index counts rows): rows of 64 N-elements (128 bytes), 128-byte swizzle, 8-row
-// groups 1024 bytes apart; the next 64 N-elements start `lbo` bytes further.
-TI_DEVICE uint64_t smem_desc_mn128(uint32_t saddr, uint32_t lbo) {
+// MN-major operand (the contraction index counts rows): rows of 64 M- or N-elements (128 bytes), 128-byte swizzle, 8-row
+// groups `sbo` bytes apart; the next 64 M- or N-elements start `lbo` bytes further.
+TI_DEVICE uint64_t smem_desc_mn128(uint32_t saddr, uint32_t lbo, uint32_t sbo = 1024) {
   uint64_t d = 0;
   d |= (uint64_t)((saddr & 0x3FFFF) >> 4);
   d |= (uint64_t)(lbo >> 4) << 16;
-  d |= (uint64_t)(1024 >> 4) << 32;
+  d |= (uint64_t)(sbo >> 4) << 32;
   d |= (uint64_t)1 << 46;
   d |= (uint64_t)2 << 61;
   return d;
 }
-// the kind::f16 instruction descriptor with B in MN-major order
+// the kind::f16 instruction descriptor with A or B in MN-major order
+TI_DEVICE constexpr uint32_t idesc_f16_bf16_amn(int M, int N) { return idesc_f16_bf16(M, N) | (1u << 15); }
 TI_DEVICE constexpr uint32_t idesc_f16_bf16_bmn(int M, int N) { return idesc_f16_bf16(M, N) | (1u << 16); }
 TI_DEVICE void tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
   asm volatile(

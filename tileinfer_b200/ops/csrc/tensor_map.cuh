@@ -44,4 +44,31 @@ inline int bf16_map_2d(CUtensorMap* dst, const void* base, long long d0, long lo
   return 0;
 }
 
+// Rows of D columns seen as [groups of 8 rows][D/64 slabs][8 rows][64 columns], box `groups` x `slabs`: one copy brings
+// whole 8-row groups with some of their column slabs side by side (for instance a 16-key cache page).
+inline int bf16_map_groups(CUtensorMap* dst, const void* base, int D, long long rows, int slabs, int groups) {
+  static std::map<AMapKey, CUtensorMap> cache;
+  static std::mutex mu;
+  std::lock_guard<std::mutex> lock(mu);
+  const AMapKey key{base, D, rows, slabs, groups, -1};
+  auto it = cache.find(key);
+  if (it == cache.end()) {
+    EncodeTiledFn enc = encode_tiled_fn();
+    if (enc == nullptr) return 999;
+    CUtensorMap m;
+    const cuuint64_t dims[4] = {64, 8, (cuuint64_t)(D / 64), (cuuint64_t)(rows / 8)};
+    const cuuint64_t strides[3] = {(cuuint64_t)D * 2, 128, (cuuint64_t)D * 16};
+    const cuuint32_t box[4] = {64, 8, (cuuint32_t)slabs, (cuuint32_t)groups};
+    const cuuint32_t elem[4] = {1, 1, 1, 1};
+    const CUresult r = enc(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, elem,
+                           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) return 1000 + (int)r;
+    if (cache.size() > 4096) cache.clear();
+    it = cache.emplace(key, m).first;
+  }
+  *dst = it->second;
+  return 0;
+}
+
 }  // namespace ti
