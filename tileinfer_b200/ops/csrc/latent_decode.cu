@@ -1,40 +1,41 @@
 // Latent attention of decode tokens on the 5th-generation tensor cores (bf16, padded latent size 256, 384 or 512).
 //
 // All heads of a token attend to the same latents, so the latents are the wide operand and the heads the narrow one:
-// per tile of 128 keys   S^T [keys x heads] = C q~^T   and   O^T [R x heads] += C^T P^T,   where C [128 x R] is ONE copy
+// per tile of 64 keys   S^T [keys x heads] = C q~^T   and   O^T [R x heads] += C^T P^T,   where C [64 x R] is ONE copy
 // of the latents in shared memory: the K-major A operand of the first product, the MN-major A operand of the second.
 // N = 16 or 32 heads per block; tensor-core time follows the bytes of C, not the heads that a 128-row tile would waste.
 //
-//   warp 0     TMA producer: slots of 128 keys x 128 columns (32 KB), one 4-D copy per 16-key page, through the block table
-//   warp 1     MMA issuer: S^T of a tile as its slots land, then O^T slot by slot, each released as soon as it was read
+//   warp 0     TMA producer: slots of 64 keys x 256 columns (384 at R = 384), one 4-D copy per 16-key page, through the
+//              block table
+//   warp 1     MMA issuer: S^T of the next tile (two buffers) while the softmax works on this one, then O^T slot by slot,
+//              each slot released as soon as it was read
 //   warps 2-5  softmax over the keys of a tile (lanes = keys in TMEM; the scores change hands through shared memory so that
 //              a thread owns one head and a share of the keys), lazy rescaling of O^T, P^T written as the bf16 B operand
 //
-// The ring holds one tile and at least one slot more at R = 512 and more tiles below, so that the copies keep running
-// while the softmax works.  Every wait is bounded; on expiry the status word is set, the roles leave and TMEM is freed.
+// The ring holds two and a half tiles at R = 512 and more below.  Every wait is bounded; on expiry the status word is set, the roles leave and TMEM is freed.
 #include "latent_attn.cuh"
 #include "tensor_map.cuh"
 
 namespace ti {
 
-constexpr int kDkTile = 128;                     // keys per tile
-constexpr int kDkSlot = 128 * 128 * 2;           // bytes of a slot: 128 keys x 128 columns
+constexpr int kDkTile = 64;                      // keys per tile
 constexpr int kDkThreads = 192;
 constexpr int kDkMaxSlots = 7;
 constexpr unsigned long long kDkWaitNs = 500000000ull;
 constexpr float kDkGap = 8.f;                    // log2 units the running maximum may lag behind before O is rescaled
 
 struct LatentDecodeTcParams {
-  alignas(64) CUtensorMap map_c;                 // cache rows as [groups of 8][R/64 slabs][8][64], box {64, 8, 2, 2}
+  alignas(64) CUtensorMap map_c;                 // cache rows as [groups of 8][R/64 slabs][8][64], box {64, 8, slabs, 2}
   LatentAttnParams a;
-  int slots;
+  int slots, slabs;                              // of the ring; 64-column slabs per slot
 };
 
 template <int N> struct DkGeom {                 // N heads per block
   static constexpr int kPitch = N + 1;           // floats per key of the score exchange
   static constexpr int kParts = 128 / N;         // threads per head
+  static constexpr int kShare = kDkTile / kParts;        // keys per thread in the softmax
   static constexpr size_t fixed(int Rp) {        // everything but the ring
-    return (size_t)N * Rp * 2 + 2 * N * 128 + 128 * kPitch * 4 + (size_t)(kParts + 2) * N * 4 + 256 + 1024;
+    return (size_t)N * Rp * 2 + N * 128 + kDkTile * kPitch * 4 + (size_t)(kParts + 2) * N * 4 + 256 + 1024;
   }
 };
 
@@ -85,16 +86,18 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
   const LatentAttnParams& p = pp.a;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-  const int Rp = p.Rp, np = Rp >> 7, ns = pp.slots;              // column pairs (slots) of a tile, slots of the ring
-  const uint32_t ring = smem_u32(smem), q_s = ring + ns * kDkSlot, p_s = q_s + N * Rp * 2;
-  uint8_t* tail = smem + ns * kDkSlot + N * Rp * 2 + 2 * N * 128;
-  float* s_x = reinterpret_cast<float*>(tail);                   // [128 keys][N + 1]
-  float* mx_x = s_x + 128 * G::kPitch;                           // [parts][N]; at the end the sums
+  const int Rp = p.Rp, np = Rp >> 7, ns = pp.slots;              // 128-row blocks of O^T, slots of the ring
+  const int sc = pp.slabs, spt = (Rp >> 6) / sc;                 // slabs of a slot, slots of a tile
+  const uint32_t grp = sc * 1024, slot_bytes = 8 * grp;          // an 8-key group, 64 keys
+  const uint32_t ring = smem_u32(smem), q_s = ring + ns * slot_bytes, p_s = q_s + N * Rp * 2;
+  uint8_t* tail = smem + ns * slot_bytes + N * Rp * 2 + N * 128;
+  float* s_x = reinterpret_cast<float*>(tail);                   // [64 keys][N + 1]
+  float* mx_x = s_x + kDkTile * G::kPitch;                           // [parts][N]; at the end the sums
   float* alpha_x = mx_x + G::kParts * N;                         // [N]
   float* ml_x = alpha_x + N;                                     // [N]: factor of O
   const uint32_t bars = smem_u32(ml_x + N);
-  const uint32_t full = bars, empty = bars + 8 * kDkMaxSlots, s_full = bars + 16 * kDkMaxSlots, p_full = s_full + 8, o_full = s_full + 16,
-                 tmem_slot = s_full + 24;
+  const uint32_t full = bars, empty = bars + 8 * kDkMaxSlots, s_full = bars + 16 * kDkMaxSlots, p_empty = s_full + 16,
+                 p_full = s_full + 24, o_full = s_full + 32, tmem_slot = s_full + 40;
   uint32_t* tmem_slot_ptr = reinterpret_cast<uint32_t*>(smem + (tmem_slot - ring));
   volatile int* abort_flag = reinterpret_cast<int*>(tmem_slot_ptr + 1);
 
@@ -110,7 +113,7 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
 
   if (tid == 0) {
     *abort_flag = 0;
-    for (int i = 0; i < 2 * kDkMaxSlots + 1; ++i) mbar_init(bars + 8 * i, 1);
+    for (int i = 0; i < 2 * kDkMaxSlots + 3; ++i) mbar_init(bars + 8 * i, 1);
     mbar_init(p_full, 128);
     mbar_init(o_full, 1);
     fence_mbar_init();
@@ -133,7 +136,7 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = *tmem_slot_ptr, o_col = 32;              // S^T at column 0, O^T of pair b at 32 + b * N
+  const uint32_t tmem = *tmem_slot_ptr, o_col = 64;              // S^T at columns 0 and 32, O^T block b at 64 + b * N
 
   if (warp == 0) {
     // ------------------------------------------------------------ TMA producer
@@ -142,21 +145,21 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
       int it = 0;
       bool ok = true;
       for (int j = t0; j < t1 && ok; ++j) {
-        int blk[8];
+        int blk[4];
 #pragma unroll
-        for (int g = 0; g < 8; ++g) {
+        for (int g = 0; g < 4; ++g) {
           blk[g] = bt[min(kr.page0 + j * (kDkTile / 16) + g, kr.npages - 1)];           // past the end: masked
           if (!TI_CHECK(blk[g], p.num_blocks, p.status)) blk[g] = 0;
         }
-        for (int b = 0; b < np; ++b, ++it) {
+        for (int b = 0; b < spt; ++b, ++it) {
           const int s = it % ns;
           if (*abort_flag || (it >= ns && !mbar_wait(empty + 8 * s, (uint32_t)((it / ns - 1) & 1), kDkWaitNs, p.status))) {
             ok = false;
             break;
           }
-          mbar_expect_tx(full + 8 * s, kDkSlot);
+          mbar_expect_tx(full + 8 * s, slot_bytes);
 #pragma unroll
-          for (int g = 0; g < 8; ++g) tma_load_4d(ring + s * kDkSlot + g * 4096, &pp.map_c, 0, 0, 2 * b, blk[g] * 2, full + 8 * s);
+          for (int g = 0; g < 4; ++g) tma_load_4d(ring + s * slot_bytes + g * 2 * grp, &pp.map_c, 0, 0, sc * b, blk[g] * 2, full + 8 * s);
         }
       }
       if (!ok) *abort_flag = 1;
@@ -164,60 +167,68 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
   } else if (warp == 1) {
     // ------------------------------------------------------------ MMA issuer
     if (elect_one()) {
-      constexpr uint32_t idesc_s = idesc_f16_bf16(128, N), idesc_o = idesc_f16_bf16_amn(128, N);
-      bool ok = true;
-      for (int j = 0; j < t1 - t0 && ok; ++j) {
-        for (int b = 0; b < np && ok; ++b) {
-          const int it = j * np + b, s = it % ns;
-          ok = !*abort_flag && mbar_wait(full + 8 * s, (uint32_t)((it / ns) & 1), kDkWaitNs, p.status);
-          if (!ok) break;
+      constexpr uint32_t idesc_s = idesc_f16_bf16(64, N), idesc_o = idesc_f16_bf16_amn(128, N);
+      const int nt = t1 - t0;
+      auto scores = [&](int j) {                                 // S^T of tile j as its slots land
+        for (int b = 0; b < spt; ++b) {
+          const int it = j * spt + b, s = it % ns;
+          if (*abort_flag || !mbar_wait(full + 8 * s, (uint32_t)((it / ns) & 1), kDkWaitNs, p.status)) return false;
           tc_fence_after();
+          for (int c = 0; c < sc; ++c)
 #pragma unroll
-          for (int k = 0; k < 8; ++k)                            // two slabs of four 16-column steps
-            umma_bf16(tmem, smem_desc_sw128_sbo(ring + s * kDkSlot + (k >> 2) * 1024 + (k & 3) * 32, 2048),
-                      smem_desc_sw128(q_s + (2 * b + (k >> 2)) * (N * 128) + (k & 3) * 32), idesc_s, (b | k) ? 1u : 0u);
+            for (int k = 0; k < 4; ++k)
+              umma_bf16(tmem + (j & 1) * 32, smem_desc_sw128_sbo(ring + s * slot_bytes + c * 1024 + k * 32, grp),
+                        smem_desc_sw128(q_s + (b * sc + c) * (N * 128) + k * 32), idesc_s, (b | c | k) ? 1u : 0u);
         }
-        if (!ok) break;
-        umma_commit(s_full);
-        ok = mbar_wait(p_full, (uint32_t)(j & 1), kDkWaitNs, p.status);
+        umma_commit(s_full + 8 * (j & 1));
+        return true;
+      };
+      bool ok = scores(0);
+      for (int j = 0; j < nt && ok; ++j) {
+        if (j + 1 < nt) ok = scores(j + 1);
+        ok = ok && mbar_wait(p_full, (uint32_t)(j & 1), kDkWaitNs, p.status);
         if (!ok) break;
         tc_fence_after();
         for (int b = 0; b < np; ++b) {
-          const int s = (j * np + b) % ns;
+          const int slot = 2 * b / sc, s = (j * spt + slot) % ns;
+          const uint32_t a = ring + s * slot_bytes + (2 * b - slot * sc) * 1024;
 #pragma unroll
-          for (int g = 0; g < 8; ++g)                            // 16 keys each
-            umma_bf16(tmem + o_col + b * N, smem_desc_mn128(ring + s * kDkSlot + g * 4096, 1024, 2048),
-                      smem_desc_sw128(p_s + (g >> 2) * (N * 128) + (g & 3) * 32), idesc_o, (j | g) ? 1u : 0u);
-          umma_commit(empty + 8 * s);
+          for (int g = 0; g < kDkTile / 16; ++g)
+            umma_bf16(tmem + o_col + b * N, smem_desc_mn128(a + g * 2 * grp, 1024, grp), smem_desc_sw128(p_s + g * 32), idesc_o,
+                      (j | g) ? 1u : 0u);
+          if ((2 * b + 2) % sc == 0) umma_commit(empty + 8 * s);  // the slot's last block
         }
+        umma_commit(p_empty);
       }
       umma_commit(o_full);                                       // O^T complete (or the loop gave up)
       if (!ok) *abort_flag = 1;
     }
   } else {
     // ------------------------------------------------------------ softmax: in TMEM a thread is a key, then a share of a head
-    const int quarter = warp & 3, key_l = quarter * 32 + lane;   // key of the tile whose scores this thread reads from TMEM
-    const int u = tid - 64, head = u % N, part = u / N;          // head and share of N keys
+    const int quarter = warp & 3, key_l = quarter * 16 + (lane & 15);   // M = 64: 16 keys in each lane quarter
+    const int u = tid - 64, head = u % N, part = u / N;          // head and share of the keys
     const uint32_t lane_base = tmem + ((uint32_t)(quarter * 32) << 16);
     const float sc = p.scale * kLog2e;
     float m_used = kNeg, l = 0.f;
     bool ok = true;
     for (int j = 0; j < t1 - t0; ++j) {
-      ok = !*abort_flag && mbar_wait(s_full, (uint32_t)(j & 1), kDkWaitNs, p.status);   // also: O^T of the last tile is done
+      ok = !*abort_flag && mbar_wait(s_full + 8 * (j & 1), (uint32_t)((j >> 1) & 1), kDkWaitNs, p.status);
       if (!ok) *abort_flag = 1;
       __syncwarp();
       tc_fence_after();
       float v[N];
-      tmem_ld_n<N>(lane_base, v);
+      tmem_ld_n<N>(lane_base + (j & 1) * 32, v);
       const int key = kr.page0 * 16 + (t0 + j) * kDkTile + key_l;
       const bool seen = ok && key >= kr.lo && key <= kr.pos;
+      if (lane < 16) {
 #pragma unroll
-      for (int i = 0; i < N; ++i) s_x[key_l * G::kPitch + i] = seen ? v[i] * sc : kNeg;
+        for (int i = 0; i < N; ++i) s_x[key_l * G::kPitch + i] = seen ? v[i] * sc : kNeg;
+      }
       softmax_bar();
       float mx = kNeg;
 #pragma unroll
-      for (int i = 0; i < N; ++i) {
-        v[i] = s_x[(part * N + i) * G::kPitch + head];
+      for (int i = 0; i < G::kShare; ++i) {
+        v[i] = s_x[(part * G::kShare + i) * G::kPitch + head];
         mx = fmaxf(mx, v[i]);
       }
       mx_x[part * N + head] = mx;
@@ -232,8 +243,14 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
         m_used = m_new;
       }
       if (part == 0) alpha_x[head] = al;
+      if (j > 0) {                                               // P^T free, O^T quiescent: the last tile's product is done
+        ok = !*abort_flag && mbar_wait(p_empty, (uint32_t)((j - 1) & 1), kDkWaitNs, p.status);
+        if (!ok) *abort_flag = 1;
+        __syncwarp();
+        tc_fence_after();
+      }
 #pragma unroll
-      for (int i = 0; i < N; i += 8) {
+      for (int i = 0; i < G::kShare; i += 8) {
         uint32_t pk[4];
 #pragma unroll
         for (int e = 0; e < 8; e += 2) {
@@ -242,8 +259,8 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
           l += a + b;
           pk[e >> 1] = pack_bf16(a, b);
         }
-        const int k8 = part * N + i;                             // first of eight keys: chunk (k8 / 8) % 8 of slab k8 / 64
-        *reinterpret_cast<uint4*>(smem + (p_s - ring) + (k8 >> 6) * (N * 128) + head * 128 + ((((k8 >> 3) & 7) ^ (head & 7)) << 4)) =
+        const int chunk = (part * G::kShare + i) >> 3;           // eight keys
+        *reinterpret_cast<uint4*>(smem + (p_s - ring) + head * 128 + ((chunk ^ (head & 7)) << 4)) =
             make_uint4(pk[0], pk[1], pk[2], pk[3]);
       }
       softmax_bar();
@@ -317,25 +334,27 @@ template <int N>
 static int launch_dk(LatentDecodeTcParams& p, cudaStream_t st) {
   constexpr size_t kMax = 227 * 1024;
   const size_t fixed = DkGeom<N>::fixed(p.a.Rp);
-  p.slots = (int)((kMax - fixed) / kDkSlot);
+  const size_t slot = (size_t)p.slabs * 8192;
+  p.slots = (int)((kMax - fixed) / slot);
   if (p.slots > kDkMaxSlots) p.slots = kDkMaxSlots;
-  if (p.slots < p.a.Rp / 128) return -2;                          // the ring must hold a whole tile
+  if (p.slots < 2 * (p.a.Rp / 64 / p.slabs)) return -2;           // S^T runs one tile ahead of O^T
   auto k = latent_decode_tc_kernel<N>;
   static bool configured = false;
   if (!configured) {
     cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMax);
     configured = true;
   }
-  launch_kernel(k, dim3(p.a.num_qg, (p.a.H + N - 1) / N, p.a.nsplit), dim3(kDkThreads), fixed + (size_t)p.slots * kDkSlot, st, true, p);
+  launch_kernel(k, dim3(p.a.num_qg, (p.a.H + N - 1) / N, p.a.nsplit), dim3(kDkThreads), fixed + (size_t)p.slots * slot, st, true, p);
   if (p.a.nsplit > 1) launch_latent_merge(p.a, N, kDkTile, st);
   return (int)cudaGetLastError();
 }
 
 int launch_latent_decode_tc(const LatentAttnParams& a, cudaStream_t st) {
-  if (a.Rp % 128 || a.Rp > 512 || a.num_blocks < 1) return -2;
+  if ((a.Rp != 256 && a.Rp != 384 && a.Rp != 512) || a.num_blocks < 1) return -2;
   LatentDecodeTcParams p = {};
   p.a = a;
-  const int rc = bf16_map_groups(&p.map_c, a.cache, a.Rp, (long long)a.num_blocks * 16, 2, 2);
+  p.slabs = a.Rp % 256 == 0 ? 4 : 6;
+  const int rc = bf16_map_groups(&p.map_c, a.cache, a.Rp, (long long)a.num_blocks * 16, p.slabs, 2);
   if (rc) return rc;
   return a.H > 16 ? launch_dk<32>(p, st) : launch_dk<16>(p, st);
 }
