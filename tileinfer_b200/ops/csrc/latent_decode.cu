@@ -9,7 +9,7 @@
 //              block table
 //   warp 1     MMA issuer: S^T of the next tile (two buffers) while the softmax works on this one, then O^T slot by slot,
 //              each slot released as soon as it was read
-//   warps 2-5  softmax over the keys of a tile (lanes = keys in TMEM; the scores change hands through shared memory so that
+//   warps 2-9  softmax over the keys of a tile (lanes = keys in TMEM; the scores change hands through shared memory so that
 //              a thread owns one head and a share of the keys), lazy rescaling of O^T, P^T written as the bf16 B operand
 //
 // The ring holds two and a half tiles at R = 512 and more below.  Every wait is bounded; on expiry the status word is set, the roles leave and TMEM is freed.
@@ -19,7 +19,8 @@
 namespace ti {
 
 constexpr int kDkTile = 64;                      // keys per tile
-constexpr int kDkThreads = 192;
+constexpr int kDkSoftmax = 256;                  // threads of the softmax warps
+constexpr int kDkThreads = 64 + kDkSoftmax;
 constexpr int kDkMaxSlots = 7;
 constexpr unsigned long long kDkWaitNs = 500000000ull;
 constexpr float kDkGap = 8.f;                    // log2 units the running maximum may lag behind before O is rescaled
@@ -27,12 +28,12 @@ constexpr float kDkGap = 8.f;                    // log2 units the running maxim
 struct LatentDecodeTcParams {
   alignas(64) CUtensorMap map_c;                 // cache rows as [groups of 8][R/64 slabs][8][64], box {64, 8, slabs, 2}
   LatentAttnParams a;
-  int slots, slabs;                              // of the ring; 64-column slabs per slot
+  int slots;                                     // of the ring
 };
 
 template <int N> struct DkGeom {                 // N heads per block
   static constexpr int kPitch = N + 1;           // floats per key of the score exchange
-  static constexpr int kParts = 128 / N;         // threads per head
+  static constexpr int kParts = kDkSoftmax / N;         // threads per head
   static constexpr int kShare = kDkTile / kParts;        // keys per thread in the softmax
   static constexpr size_t fixed(int Rp) {        // everything but the ring
     return (size_t)N * Rp * 2 + N * 128 + kDkTile * kPitch * 4 + (size_t)(kParts + 2) * N * 4 + 256 + 1024;
@@ -44,7 +45,7 @@ TI_DEVICE float dk_ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
-TI_DEVICE void softmax_bar() { asm volatile("bar.sync 1, 128;\n" ::: "memory"); }
+TI_DEVICE void softmax_bar() { asm volatile("bar.sync 1, 256;\n" ::: "memory"); }
 template <int N> TI_DEVICE void tmem_ld_n(uint32_t taddr, float (&v)[N]);
 template <> TI_DEVICE void tmem_ld_n<32>(uint32_t taddr, float (&v)[32]) {
   uint32_t r[32];
@@ -65,6 +66,16 @@ template <> TI_DEVICE void tmem_ld_n<16>(uint32_t taddr, float (&v)[16]) {
 #pragma unroll
   for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
 }
+template <> TI_DEVICE void tmem_ld_n<8>(uint32_t taddr, float (&v)[8]) {
+  uint32_t r[8];
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0,%1,%2,%3,%4,%5,%6,%7}, [%8];\n"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+               : "r"(taddr)
+               : "memory");
+  tmem_ld_wait();
+#pragma unroll
+  for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(r[i]);
+}
 template <int N> TI_DEVICE void tmem_st_n(uint32_t taddr, const float (&v)[N]);
 template <> TI_DEVICE void tmem_st_n<32>(uint32_t taddr, const float (&v)[32]) {
   uint32_t r[32];
@@ -80,15 +91,16 @@ template <> TI_DEVICE void tmem_st_n<16>(uint32_t taddr, const float (&v)[16]) {
       : "memory");
 }
 
-template <int N>
+// SC: 64-column slabs of a ring slot
+template <int N, int SC>
 __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const __grid_constant__ LatentDecodeTcParams pp) {
   using G = DkGeom<N>;
   const LatentAttnParams& p = pp.a;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   const int Rp = p.Rp, np = Rp >> 7, ns = pp.slots;              // 128-row blocks of O^T, slots of the ring
-  const int sc = pp.slabs, spt = (Rp >> 6) / sc;                 // slabs of a slot, slots of a tile
-  const uint32_t grp = sc * 1024, slot_bytes = 8 * grp;          // an 8-key group, 64 keys
+  const int spt = (Rp >> 6) / SC;                                // slots of a tile
+  constexpr uint32_t grp = SC * 1024, slot_bytes = 8 * grp;      // an 8-key group, 64 keys
   const uint32_t ring = smem_u32(smem), q_s = ring + ns * slot_bytes, p_s = q_s + N * Rp * 2;
   uint8_t* tail = smem + ns * slot_bytes + N * Rp * 2 + N * 128;
   float* s_x = reinterpret_cast<float*>(tail);                   // [64 keys][N + 1]
@@ -114,7 +126,7 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
   if (tid == 0) {
     *abort_flag = 0;
     for (int i = 0; i < 2 * kDkMaxSlots + 3; ++i) mbar_init(bars + 8 * i, 1);
-    mbar_init(p_full, 128);
+    mbar_init(p_full, kDkSoftmax);
     mbar_init(o_full, 1);
     fence_mbar_init();
   }
@@ -159,7 +171,7 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
           }
           mbar_expect_tx(full + 8 * s, slot_bytes);
 #pragma unroll
-          for (int g = 0; g < 4; ++g) tma_load_4d(ring + s * slot_bytes + g * 2 * grp, &pp.map_c, 0, 0, sc * b, blk[g] * 2, full + 8 * s);
+          for (int g = 0; g < 4; ++g) tma_load_4d(ring + s * slot_bytes + g * 2 * grp, &pp.map_c, 0, 0, SC * b, blk[g] * 2, full + 8 * s);
         }
       }
       if (!ok) *abort_flag = 1;
@@ -174,11 +186,14 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
           const int it = j * spt + b, s = it % ns;
           if (*abort_flag || !mbar_wait(full + 8 * s, (uint32_t)((it / ns) & 1), kDkWaitNs, p.status)) return false;
           tc_fence_after();
-          for (int c = 0; c < sc; ++c)
+          // descriptors of one operand differ in the address field alone (units of 16 bytes)
+          const uint64_t da = smem_desc_sw128_sbo(ring + s * slot_bytes, grp), db = smem_desc_sw128(q_s + b * SC * (N * 128));
+          const uint32_t d = tmem + (j & 1) * 32;
+#pragma unroll
+          for (int c = 0; c < SC; ++c)
 #pragma unroll
             for (int k = 0; k < 4; ++k)
-              umma_bf16(tmem + (j & 1) * 32, smem_desc_sw128_sbo(ring + s * slot_bytes + c * 1024 + k * 32, grp),
-                        smem_desc_sw128(q_s + (b * sc + c) * (N * 128) + k * 32), idesc_s, (b | c | k) ? 1u : 0u);
+              umma_bf16(d, da + ((c * 1024 + k * 32) >> 4), db + ((c * N * 128 + k * 32) >> 4), idesc_s, (c | k) ? 1u : (b ? 1u : 0u));
         }
         umma_commit(s_full + 8 * (j & 1));
         return true;
@@ -189,14 +204,17 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
         ok = ok && mbar_wait(p_full, (uint32_t)(j & 1), kDkWaitNs, p.status);
         if (!ok) break;
         tc_fence_after();
-        for (int b = 0; b < np; ++b) {
-          const int slot = 2 * b / sc, s = (j * spt + slot) % ns;
-          const uint32_t a = ring + s * slot_bytes + (2 * b - slot * sc) * 1024;
+        const uint64_t db = smem_desc_sw128(p_s);
+        for (int t = 0; t < spt; ++t) {
+          const int s = (j * spt + t) % ns;
+          const uint64_t da = smem_desc_mn128(ring + s * slot_bytes, 1024, grp);
+          const uint32_t d = tmem + o_col + t * (SC / 2) * N;
 #pragma unroll
-          for (int g = 0; g < kDkTile / 16; ++g)
-            umma_bf16(tmem + o_col + b * N, smem_desc_mn128(a + g * 2 * grp, 1024, grp), smem_desc_sw128(p_s + g * 32), idesc_o,
-                      (j | g) ? 1u : 0u);
-          if ((2 * b + 2) % sc == 0) umma_commit(empty + 8 * s);  // the slot's last block
+          for (int c = 0; c < SC / 2; ++c)                       // 128 columns of C = 128 rows of O^T
+#pragma unroll
+            for (int g = 0; g < kDkTile / 16; ++g)
+              umma_bf16(d + c * N, da + ((c * 2048 + g * 2 * grp) >> 4), db + ((g * 32) >> 4), idesc_o, g ? 1u : (j ? 1u : 0u));
+          umma_commit(empty + 8 * s);
         }
         umma_commit(p_empty);
       }
@@ -205,7 +223,8 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
     }
   } else {
     // ------------------------------------------------------------ softmax: in TMEM a thread is a key, then a share of a head
-    const int quarter = warp & 3, key_l = quarter * 16 + (lane & 15);   // M = 64: 16 keys in each lane quarter
+    constexpr int NH = N / 2;                                    // two warps per lane quarter share the heads
+    const int quarter = warp & 3, half = (warp - 2) >> 2, key_l = quarter * 16 + (lane & 15);   // M = 64: 16 keys in each lane quarter
     const int u = tid - 64, head = u % N, part = u / N;          // head and share of the keys
     const uint32_t lane_base = tmem + ((uint32_t)(quarter * 32) << 16);
     const float sc = p.scale * kLog2e;
@@ -216,13 +235,18 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
       if (!ok) *abort_flag = 1;
       __syncwarp();
       tc_fence_after();
-      float v[N];
-      tmem_ld_n<N>(lane_base + (j & 1) * 32, v);
+      float v[NH > G::kShare ? NH : G::kShare];
+      {
+        float w[NH];
+        tmem_ld_n<NH>(lane_base + (j & 1) * 32 + half * NH, w);
+#pragma unroll
+        for (int i = 0; i < NH; ++i) v[i] = w[i];
+      }
       const int key = kr.page0 * 16 + (t0 + j) * kDkTile + key_l;
       const bool seen = ok && key >= kr.lo && key <= kr.pos;
       if (lane < 16) {
 #pragma unroll
-        for (int i = 0; i < N; ++i) s_x[key_l * G::kPitch + i] = seen ? v[i] * sc : kNeg;
+        for (int i = 0; i < NH; ++i) s_x[key_l * G::kPitch + half * NH + i] = seen ? v[i] * sc : kNeg;
       }
       softmax_bar();
       float mx = kNeg;
@@ -249,24 +273,23 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
         __syncwarp();
         tc_fence_after();
       }
+      uint32_t pk[G::kShare / 2];
 #pragma unroll
-      for (int i = 0; i < G::kShare; i += 8) {
-        uint32_t pk[4];
-#pragma unroll
-        for (int e = 0; e < 8; e += 2) {
-          const float a = v[i + e] > 0.5f * kNeg ? dk_ex2(v[i + e] - m_used) : 0.f;
-          const float b = v[i + e + 1] > 0.5f * kNeg ? dk_ex2(v[i + e + 1] - m_used) : 0.f;
-          l += a + b;
-          pk[e >> 1] = pack_bf16(a, b);
-        }
-        const int chunk = (part * G::kShare + i) >> 3;           // eight keys
-        *reinterpret_cast<uint4*>(smem + (p_s - ring) + head * 128 + ((chunk ^ (head & 7)) << 4)) =
-            make_uint4(pk[0], pk[1], pk[2], pk[3]);
+      for (int i = 0; i < G::kShare; i += 2) {                   // masked scores: exp2 of a huge negative number is 0
+        const float e0 = dk_ex2(v[i] - m_used), e1 = dk_ex2(v[i + 1] - m_used);
+        l += e0 + e1;
+        pk[i >> 1] = pack_bf16(e0, e1);
+      }
+      {
+        const int k0 = part * G::kShare;                         // 16-byte chunks of eight keys, swizzled by the row
+        uint8_t* dst = smem + (p_s - ring) + head * 128 + (((k0 >> 3) ^ (head & 7)) << 4) + (k0 & 7) * 2;
+        if constexpr (G::kShare == 8) *reinterpret_cast<uint4*>(dst) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+        else *reinterpret_cast<uint2*>(dst) = make_uint2(pk[0], pk[1]);
       }
       softmax_bar();
       if (j > 0 && __any_sync(0xffffffffu, alpha_x[lane % N] != 1.f)) {
 #pragma unroll 1
-        for (int b = 0; b < np; ++b) {
+        for (int b = half; b < np; b += 2) {
           float o[N];
           tmem_ld_n<N>(lane_base + o_col + b * N, o);
 #pragma unroll
@@ -304,7 +327,7 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
     if (__all_sync(0xffffffffu, ok)) {
       const int nh = min(N, p.H - hg * N);
 #pragma unroll 1
-      for (int b = 0; b < np; ++b) {
+      for (int b = half; b < np; b += 2) {
         float o[N];
         tmem_ld_n<N>(lane_base + o_col + b * N, o);
         const int r = b * 128 + quarter * 32 + lane;
@@ -330,15 +353,15 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
   }
 }
 
-template <int N>
+template <int N, int SC>
 static int launch_dk(LatentDecodeTcParams& p, cudaStream_t st) {
   constexpr size_t kMax = 227 * 1024;
   const size_t fixed = DkGeom<N>::fixed(p.a.Rp);
-  const size_t slot = (size_t)p.slabs * 8192;
+  const size_t slot = (size_t)SC * 8192;
   p.slots = (int)((kMax - fixed) / slot);
   if (p.slots > kDkMaxSlots) p.slots = kDkMaxSlots;
-  if (p.slots < 2 * (p.a.Rp / 64 / p.slabs)) return -2;           // S^T runs one tile ahead of O^T
-  auto k = latent_decode_tc_kernel<N>;
+  if (p.slots < 2 * (p.a.Rp / 64 / SC)) return -2;           // S^T runs one tile ahead of O^T
+  auto k = latent_decode_tc_kernel<N, SC>;
   static bool configured = false;
   if (!configured) {
     cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMax);
@@ -353,10 +376,11 @@ int launch_latent_decode_tc(const LatentAttnParams& a, cudaStream_t st) {
   if ((a.Rp != 256 && a.Rp != 384 && a.Rp != 512) || a.num_blocks < 1) return -2;
   LatentDecodeTcParams p = {};
   p.a = a;
-  p.slabs = a.Rp % 256 == 0 ? 4 : 6;
-  const int rc = bf16_map_groups(&p.map_c, a.cache, a.Rp, (long long)a.num_blocks * 16, p.slabs, 2);
+  const int slabs = a.Rp % 256 == 0 ? 4 : 6;
+  const int rc = bf16_map_groups(&p.map_c, a.cache, a.Rp, (long long)a.num_blocks * 16, slabs, 2);
   if (rc) return rc;
-  return a.H > 16 ? launch_dk<32>(p, st) : launch_dk<16>(p, st);
+  if (slabs == 4) return a.H > 16 ? launch_dk<32, 4>(p, st) : launch_dk<16, 4>(p, st);
+  return a.H > 16 ? launch_dk<32, 6>(p, st) : launch_dk<16, 6>(p, st);
 }
 
 }  // namespace ti
