@@ -36,7 +36,9 @@ ONE = config([layer(2, 32, 24, 40, 23, scale=0.4, ff=64, limit=1.5)], width=96, 
 # latents of the sizes that the widest kernels serve
 DEEP_RANK = config([layer(4, 64, 64, 512, 130, ff=128, limit=2.0), layer(33, 16, 16, 512, 70, kv_from=0),
                     layer(2, 64, 128, 640, 90, ff=64, limit=1.0)], width=256, vocab=300)
-CASES = {"mixed": MIXED, "wide": WIDE, "one": ONE, "deep_rank": DEEP_RANK}
+# heads wider than the tiled prefill kernel takes: every token goes through the split attention
+WIDE_HEADS = config([layer(2, 264, 280, 24, 40, ff=32), layer(1, 16, 300, 24, 90, kv_from=0)], width=48, vocab=140)
+CASES = {"wide_heads": WIDE_HEADS, "mixed": MIXED, "wide": WIDE, "one": ONE, "deep_rank": DEEP_RANK}
 
 
 def tokens(cfg, n, seed=0):

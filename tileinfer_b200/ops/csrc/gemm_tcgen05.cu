@@ -46,14 +46,15 @@ constexpr int kGemmProducerB = 6;
 #endif
 // bytes of operand ring per CTA.  96 lets two CTAs share an SM (TMEM: 2 x 256 columns), so that the epilogue of
 // one overlaps the main loop of the other.
-constexpr int kGemmRingBytes = TI_GEMM_RING_KB * 1024;
+constexpr int kGemmShortRingKb = 96;       // the ring of products with a short k (see short_k)
 // BN = tokens per CTA (TMEM columns per accumulator); BF16: bf16 weights and activations (one plane, one accumulator)
 // BMH = weight-row halves per CTA: 1 -> a 128-row tile; 2 -> a 256-row tile as two 128-row MMAs that share ONE
 // activation tile in shared memory (the bytes a CTA pulls through L2 per multiply-add drop by a third).
-template <int BN, bool BF16, int BMH = 1> struct GemmGeom {
+template <int BN, bool BF16, int BMH = 1, int RK = TI_GEMM_RING_KB> struct GemmGeom {
+  static constexpr int kRing = RK * 1024;
   static constexpr int kStageB = BN * kBK * kKS;                   // one limb plane / the bf16 activation tile (128-byte rows)
   static constexpr int kStageBytes = BMH * kStageA + (BF16 ? 1 : 2) * kStageB;
-  static constexpr int kStages = kGemmRingBytes / kStageBytes < 24 ? kGemmRingBytes / kStageBytes : 24;
+  static constexpr int kStages = kRing / kStageBytes < 24 ? kRing / kStageBytes : 24;
   static constexpr size_t kSmem = (size_t)kStages * kStageBytes + 16 * kStages + 64 + 1024;
 };
 constexpr unsigned long long kGemmWaitNs = 2000000000ull;
@@ -212,9 +213,9 @@ TI_DEVICE void gemm_store8(const GemmParams& p, int m, int n, const float4 a, co
   }
 }
 
-template <int BN, bool BF16, int BMH>
-__global__ void __launch_bounds__(kGemmThreads, TI_GEMM_RING_KB <= 100 ? 2 : 1) gemm_w8a16_kernel(const __grid_constant__ GemmParams p) {
-  using G = GemmGeom<BN, BF16, BMH>;
+template <int BN, bool BF16, int BMH, int RK>
+__global__ void __launch_bounds__(kGemmThreads, RK <= 100 ? 2 : 1) gemm_w8a16_kernel(const __grid_constant__ GemmParams p) {
+  using G = GemmGeom<BN, BF16, BMH, RK>;
   constexpr int kAcc = BF16 ? 1 : 2;                               // accumulators (limbs) per row half
   constexpr int kStages = G::kStages, kStageBytes = G::kStageBytes, kStageB = G::kStageB;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
@@ -628,16 +629,25 @@ static int cached_map(CUtensorMap* dst, const void* base, int d0, int d1, int bo
   return 0;
 }
 
-template <int BN, bool BF16, int BMH = 1>
+template <int BN, bool BF16, int BMH = 1, int RK = TI_GEMM_RING_KB>
 static int launch_gemm(const GemmParams& p, dim3 grid, cudaStream_t st) {
   static bool configured = false;
-  auto k = gemm_w8a16_kernel<BN, BF16, BMH>;
+  auto k = gemm_w8a16_kernel<BN, BF16, BMH, RK>;
   if (!configured) {
-    cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GemmGeom<BN, BF16, BMH>::kSmem);
+    cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GemmGeom<BN, BF16, BMH, RK>::kSmem);
     configured = true;
   }
-  const cudaError_t e = launch_kernel(k, grid, dim3(kGemmThreads), GemmGeom<BN, BF16, BMH>::kSmem, st, true, p);
+  const cudaError_t e = launch_kernel(k, grid, dim3(kGemmThreads), GemmGeom<BN, BF16, BMH, RK>::kSmem, st, true, p);
   return e != cudaSuccess ? (int)e : (int)cudaGetLastError();
+}
+
+// bf16 products with many tokens and a short or medium k (at most 160 stages of 128 bytes) run two CTAs per SM with half
+// the ring each (TMEM: 2 x 256 columns), so that the epilogue of one overlaps the main loop of the other.  Measured at
+// 8192 tokens (us, one CTA -> two): k 512 213 -> 131, 2048 631 -> 516, 4096 2240 -> 2073, 10240 406 -> 348; 14336 and
+// more lose 6-10 %.
+static bool short_k(int KS, int BN, long long tiles) {
+  static const int limit = [] { const char* e = getenv("TI_GEMM_SHORT_K"); return e == nullptr ? 160 : atoi(e); }();
+  return BN == 128 && KS <= limit && tiles >= 2 * 148;
 }
 
 // 256-row tiles when the token tile is full-size and there are enough tiles to fill the GPU several times over
@@ -786,6 +796,8 @@ int ti_gemm_bf16(const void* w, int n_tiles, int N, int K, const void* x, int M,
   const int S = ti::plan_split(p, KS, tiles_n * tiles_m, M, N, ldo, part, part_bytes, tile_count, n_count);
   dim3 grid(tiles_m, tiles_n, S);
   cudaStream_t st = (cudaStream_t)stream;
+  if (S == 1 && ti::short_k(KS, BN, (long long)tiles_n * tiles_m))
+    return BMH == 2 ? ti::launch_gemm<128, true, 2, ti::kGemmShortRingKb>(p, grid, st) : ti::launch_gemm<128, true, 1, ti::kGemmShortRingKb>(p, grid, st);
   if (BMH == 2 && BN == 32) return ti::launch_gemm<32, true, 2>(p, grid, st);
   if (BMH == 2 && BN == 64) return ti::launch_gemm<64, true, 2>(p, grid, st);
   if (BMH == 2) return ti::launch_gemm<128, true, 2>(p, grid, st);

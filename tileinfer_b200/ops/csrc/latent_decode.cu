@@ -36,7 +36,7 @@ template <int N> struct DkGeom {                 // N heads per block
   static constexpr int kParts = kDkSoftmax / N;         // threads per head
   static constexpr int kShare = kDkTile / kParts;        // keys per thread in the softmax
   static constexpr size_t fixed(int Rp) {        // everything but the ring
-    return (size_t)N * Rp * 2 + N * 128 + kDkTile * kPitch * 4 + (size_t)(kParts + 2) * N * 4 + 256 + 1024;
+    return (size_t)N * Rp * 2 + 2 * N * 128 + kDkTile * kPitch * 4 + (size_t)(kParts + 2) * N * 4 + 256 + 1024;
   }
 };
 
@@ -102,14 +102,14 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
   const int spt = (Rp >> 6) / SC;                                // slots of a tile
   constexpr uint32_t grp = SC * 1024, slot_bytes = 8 * grp;      // an 8-key group, 64 keys
   const uint32_t ring = smem_u32(smem), q_s = ring + ns * slot_bytes, p_s = q_s + N * Rp * 2;
-  uint8_t* tail = smem + ns * slot_bytes + N * Rp * 2 + N * 128;
+  uint8_t* tail = smem + ns * slot_bytes + N * Rp * 2 + 2 * N * 128;   // two P^T buffers
   float* s_x = reinterpret_cast<float*>(tail);                   // [64 keys][N + 1]
   float* mx_x = s_x + kDkTile * G::kPitch;                           // [parts][N]; at the end the sums
   float* alpha_x = mx_x + G::kParts * N;                         // [N]
   float* ml_x = alpha_x + N;                                     // [N]: factor of O
   const uint32_t bars = smem_u32(ml_x + N);
   const uint32_t full = bars, empty = bars + 8 * kDkMaxSlots, s_full = bars + 16 * kDkMaxSlots, p_empty = s_full + 16,
-                 p_full = s_full + 24, o_full = s_full + 32, tmem_slot = s_full + 40;
+                 p_full = s_full + 32, q_full = s_full + 48, o_full = s_full + 56, tmem_slot = s_full + 64;
   uint32_t* tmem_slot_ptr = reinterpret_cast<uint32_t*>(smem + (tmem_slot - ring));
   volatile int* abort_flag = reinterpret_cast<int*>(tmem_slot_ptr + 1);
 
@@ -125,8 +125,8 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
 
   if (tid == 0) {
     *abort_flag = 0;
-    for (int i = 0; i < 2 * kDkMaxSlots + 3; ++i) mbar_init(bars + 8 * i, 1);
-    mbar_init(p_full, kDkSoftmax);
+    for (int i = 0; i < 2 * kDkMaxSlots + 4; ++i) mbar_init(bars + 8 * i, 1);
+    for (int i = 0; i < 3; ++i) mbar_init(p_full + 8 * i, kDkSoftmax);   // P^T (two buffers), q~
     mbar_init(o_full, 1);
     fence_mbar_init();
   }
@@ -134,48 +134,34 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
     tmem_alloc(tmem_slot, 256);
     tmem_relinquish();
   }
-  // q~ as the B operand of S^T: per 64-column slab N rows of 128 bytes, 128-byte swizzle; missing heads are zero
-  {
-    const bf16* q = static_cast<const bf16*>(p.q) + ((size_t)tok * p.H + hg * N) * Rp;
-    const int cpr = Rp >> 3, nrow = min(N, p.H - hg * N);
-    for (int i = tid; i < N * cpr; i += kDkThreads) {
-      const int row = i / cpr, c = i - row * cpr, slab = c >> 3;
-      const uint4 v = row < nrow ? *reinterpret_cast<const uint4*>(q + (size_t)row * Rp + c * 8) : make_uint4(0, 0, 0, 0);
-      *reinterpret_cast<uint4*>(smem + (q_s - ring) + slab * (N * 128) + row * 128 + (((c & 7) ^ (row & 7)) << 4)) = v;
-    }
-    fence_proxy_async();
-  }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_slot_ptr, o_col = 64;              // S^T at columns 0 and 32, O^T block b at 64 + b * N
 
   if (warp == 0) {
-    // ------------------------------------------------------------ TMA producer
-    if (elect_one()) {
-      const int* bt = p.block_tables + (size_t)seq * p.max_blocks;
-      int it = 0;
-      bool ok = true;
-      for (int j = t0; j < t1 && ok; ++j) {
-        int blk[4];
-#pragma unroll
-        for (int g = 0; g < 4; ++g) {
-          blk[g] = bt[min(kr.page0 + j * (kDkTile / 16) + g, kr.npages - 1)];           // past the end: masked
-          if (!TI_CHECK(blk[g], p.num_blocks, p.status)) blk[g] = 0;
-        }
-        for (int b = 0; b < spt; ++b, ++it) {
-          const int s = it % ns;
-          if (*abort_flag || (it >= ns && !mbar_wait(empty + 8 * s, (uint32_t)((it / ns - 1) & 1), kDkWaitNs, p.status))) {
-            ok = false;
-            break;
-          }
-          mbar_expect_tx(full + 8 * s, slot_bytes);
-#pragma unroll
-          for (int g = 0; g < 4; ++g) tma_load_4d(ring + s * slot_bytes + g * 2 * grp, &pp.map_c, 0, 0, SC * b, blk[g] * 2, full + 8 * s);
-        }
+    // ------------------------------------------------------------ TMA producer: lane g of four copies page g of a tile
+    const int* bt = p.block_tables + (size_t)seq * p.max_blocks;
+    auto page = [&](int j) {                                     // pages past the end repeat the last one (masked)
+      const int blk = bt[min(kr.page0 + j * (kDkTile / 16) + (lane & 3), kr.npages - 1)];
+      return TI_CHECK(blk, p.num_blocks, p.status) ? blk : 0;
+    };
+    int it = 0, blk = page(t0);
+    bool ok = true;
+    for (int j = t0; j < t1 && ok; ++j) {
+      const int next = page(min(j + 1, t1 - 1));
+      for (int b = 0; b < spt; ++b, ++it) {
+        const int s = it % ns;
+        ok = !*abort_flag && (it < ns || mbar_wait(empty + 8 * s, (uint32_t)((it / ns - 1) & 1), kDkWaitNs, p.status));
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        if (lane == 0) mbar_expect_tx(full + 8 * s, slot_bytes);
+        __syncwarp();
+        if (lane < 4) tma_load_4d(ring + s * slot_bytes + lane * 2 * grp, &pp.map_c, 0, 0, SC * b, blk * 2, full + 8 * s);
       }
-      if (!ok) *abort_flag = 1;
+      blk = next;
     }
+    if (!ok) *abort_flag = 1;
   } else if (warp == 1) {
     // ------------------------------------------------------------ MMA issuer
     if (elect_one()) {
@@ -198,13 +184,13 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
         umma_commit(s_full + 8 * (j & 1));
         return true;
       };
-      bool ok = scores(0);
+      bool ok = mbar_wait(q_full, 0, kDkWaitNs, p.status) && scores(0);
       for (int j = 0; j < nt && ok; ++j) {
         if (j + 1 < nt) ok = scores(j + 1);
-        ok = ok && mbar_wait(p_full, (uint32_t)(j & 1), kDkWaitNs, p.status);
+        ok = ok && mbar_wait(p_full + 8 * (j & 1), (uint32_t)((j >> 1) & 1), kDkWaitNs, p.status);
         if (!ok) break;
         tc_fence_after();
-        const uint64_t db = smem_desc_sw128(p_s);
+        const uint64_t db = smem_desc_sw128(p_s + (j & 1) * (N * 128));
         for (int t = 0; t < spt; ++t) {
           const int s = (j * spt + t) % ns;
           const uint64_t da = smem_desc_mn128(ring + s * slot_bytes, 1024, grp);
@@ -216,7 +202,7 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
               umma_bf16(d + c * N, da + ((c * 2048 + g * 2 * grp) >> 4), db + ((g * 32) >> 4), idesc_o, g ? 1u : (j ? 1u : 0u));
           umma_commit(empty + 8 * s);
         }
-        umma_commit(p_empty);
+        umma_commit(p_empty + 8 * (j & 1));
       }
       umma_commit(o_full);                                       // O^T complete (or the loop gave up)
       if (!ok) *abort_flag = 1;
@@ -228,6 +214,19 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
     const int u = tid - 64, head = u % N, part = u / N;          // head and share of the keys
     const uint32_t lane_base = tmem + ((uint32_t)(quarter * 32) << 16);
     const float sc = p.scale * kLog2e;
+    // q~ as the B operand of S^T: per 64-column slab N rows of 128 bytes, 128-byte swizzle; missing heads are zero
+    {
+      const bf16* q = static_cast<const bf16*>(p.q) + ((size_t)tok * p.H + hg * N) * Rp;
+      const int cpr = Rp >> 3, nrow = min(N, p.H - hg * N);
+#pragma unroll 4
+      for (int i = u; i < N * cpr; i += kDkSoftmax) {
+        const int row = i / cpr, c = i - row * cpr;
+        const uint4 v = row < nrow ? *reinterpret_cast<const uint4*>(q + (size_t)row * Rp + c * 8) : make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(smem + (q_s - ring) + (c >> 3) * (N * 128) + row * 128 + (((c & 7) ^ (row & 7)) << 4)) = v;
+      }
+      fence_proxy_async();
+      asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(q_full) : "memory");
+    }
     float m_used = kNeg, l = 0.f;
     bool ok = true;
     for (int j = 0; j < t1 - t0; ++j) {
@@ -267,8 +266,8 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
         m_used = m_new;
       }
       if (part == 0) alpha_x[head] = al;
-      if (j > 0) {                                               // P^T free, O^T quiescent: the last tile's product is done
-        ok = !*abort_flag && mbar_wait(p_empty, (uint32_t)((j - 1) & 1), kDkWaitNs, p.status);
+      if (j > 1) {                                               // this P^T buffer is free: the product of tile j - 2 is done
+        ok = !*abort_flag && mbar_wait(p_empty + 8 * (j & 1), (uint32_t)(((j >> 1) - 1) & 1), kDkWaitNs, p.status);
         if (!ok) *abort_flag = 1;
         __syncwarp();
         tc_fence_after();
@@ -282,12 +281,17 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
       }
       {
         const int k0 = part * G::kShare;                         // 16-byte chunks of eight keys, swizzled by the row
-        uint8_t* dst = smem + (p_s - ring) + head * 128 + (((k0 >> 3) ^ (head & 7)) << 4) + (k0 & 7) * 2;
+        uint8_t* dst = smem + (p_s - ring) + (j & 1) * (N * 128) + head * 128 + (((k0 >> 3) ^ (head & 7)) << 4) + (k0 & 7) * 2;
         if constexpr (G::kShare == 8) *reinterpret_cast<uint4*>(dst) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
         else *reinterpret_cast<uint2*>(dst) = make_uint2(pk[0], pk[1]);
       }
       softmax_bar();
       if (j > 0 && __any_sync(0xffffffffu, alpha_x[lane % N] != 1.f)) {
+        // O^T quiescent: the product of the last tile is done
+        ok = !*abort_flag && mbar_wait(p_empty + 8 * ((j - 1) & 1), (uint32_t)(((j - 1) >> 1) & 1), kDkWaitNs, p.status);
+        if (!ok) *abort_flag = 1;
+        __syncwarp();
+        tc_fence_after();
 #pragma unroll 1
         for (int b = half; b < np; b += 2) {
           float o[N];
@@ -300,7 +304,7 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
       }
       tc_fence_before();
       fence_proxy_async();
-      asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(p_full) : "memory");
+      asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(p_full + 8 * (j & 1)) : "memory");
     }
     // ---- sums of the parts, then O^T
     mx_x[part * N + head] = l;

@@ -194,38 +194,50 @@ struct HeadProductParams {
   int M, H, N, K, ldx, ldo, ldg, gcol;
 };
 
-// 16 tokens x 64 outputs of one head per block; each warp 16 outputs.  The contraction index is permuted alike in both
-// operands (a lane's 16-byte load feeds two k steps), so fragments come straight from global memory.
+// 16 tokens x 64 outputs of one head per block.  The four warps take k steps of 32 in turn (a long contraction is then a
+// short chain of loads per warp) and their partial sums meet in shared memory.  The contraction index is permuted alike
+// in both operands (a lane's 16-byte load feeds two k steps), so fragments come straight from global memory.
 __global__ void __launch_bounds__(128) head_product_bf16_kernel(const __grid_constant__ HeadProductParams p) {
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-  const int h = blockIdx.y, n0 = blockIdx.x * 64 + warp * 16, m0 = blockIdx.z * 16;
+  __shared__ float part[4][16][68];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int h = blockIdx.y, n0 = blockIdx.x * 64, m0 = blockIdx.z * 16;
   const bf16* w = static_cast<const bf16*>(p.w) + ((size_t)h * p.N + n0) * p.K;
   const bf16* x = static_cast<const bf16*>(p.x) + (size_t)h * p.K;
-  const int ra = m0 + g, rb = m0 + g + 8;
-  const bf16* xa = x + (size_t)min(ra, p.M - 1) * p.ldx;
-  const bf16* xb = x + (size_t)min(rb, p.M - 1) * p.ldx;
+  const bf16* xa = x + (size_t)min(m0 + g, p.M - 1) * p.ldx;
+  const bf16* xb = x + (size_t)min(m0 + g + 8, p.M - 1) * p.ldx;
   pdl_trigger();
   pdl_wait();
-  float d0[4] = {0.f, 0.f, 0.f, 0.f}, d1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 4
-  for (int k = 8 * t; k < p.K; k += 32) {
+  float d[8][4] = {};
+#pragma unroll 2
+  for (int k = 32 * warp + 8 * t; k < p.K; k += 128) {
     const uint4 a = *reinterpret_cast<const uint4*>(xa + k), b = *reinterpret_cast<const uint4*>(xb + k);
-    const uint4 u = ldg_cached16(w + (size_t)g * p.K + k), v = ldg_cached16(w + (size_t)(g + 8) * p.K + k);
-    mma_bf16_16816(d0, a.x, b.x, a.y, b.y, u.x, u.y);
-    mma_bf16_16816(d0, a.z, b.z, a.w, b.w, u.z, u.w);
-    mma_bf16_16816(d1, a.x, b.x, a.y, b.y, v.x, v.y);
-    mma_bf16_16816(d1, a.z, b.z, a.w, b.w, v.z, v.w);
-  }
-  const bf16* gate = static_cast<const bf16*>(p.gate);
-  bf16* out = static_cast<bf16*>(p.out) + (size_t)h * p.N + n0 + 2 * t;
+    uint4 u[8];
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int r = i == 0 ? ra : rb;
-    if (r >= p.M) continue;
-    const float s = gate == nullptr ? 1.f : sigmoid_f(__bfloat162float(gate[(size_t)r * p.ldg + p.gcol + h]));
-    *reinterpret_cast<uint32_t*>(out + (size_t)r * p.ldo) = pack_bf16(d0[2 * i] * s, d0[2 * i + 1] * s);
-    *reinterpret_cast<uint32_t*>(out + (size_t)r * p.ldo + 8) = pack_bf16(d1[2 * i] * s, d1[2 * i + 1] * s);
+    for (int n = 0; n < 8; ++n) u[n] = ldg_cached16(w + (size_t)(n * 8 + g) * p.K + k);
+#pragma unroll
+    for (int n = 0; n < 8; ++n) {
+      mma_bf16_16816(d[n], a.x, b.x, a.y, b.y, u[n].x, u[n].y);
+      mma_bf16_16816(d[n], a.z, b.z, a.w, b.w, u[n].z, u[n].w);
+    }
   }
+#pragma unroll
+  for (int n = 0; n < 8; ++n) {
+    *reinterpret_cast<float2*>(&part[warp][g][n * 8 + 2 * t]) = make_float2(d[n][0], d[n][1]);
+    *reinterpret_cast<float2*>(&part[warp][g + 8][n * 8 + 2 * t]) = make_float2(d[n][2], d[n][3]);
+  }
+  __syncthreads();
+  const int r = tid >> 3, c = (tid & 7) * 8;
+  if (m0 + r >= p.M) return;
+  float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] += part[i][r][c + e];
+  const bf16* gate = static_cast<const bf16*>(p.gate);
+  const float s = gate == nullptr ? 1.f : sigmoid_f(__bfloat162float(gate[(size_t)(m0 + r) * p.ldg + p.gcol + h]));
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] *= s;
+  store8(static_cast<bf16*>(p.out) + (size_t)(m0 + r) * p.ldo + (size_t)h * p.N + n0 + c, v);
 }
 
 __global__ void __launch_bounds__(128) head_product_f32_kernel(const __grid_constant__ HeadProductParams p) {
@@ -377,7 +389,7 @@ int ti_latent_gather(const void* cache, const void* slots, long long num_slots, 
 int ti_head_product(const void* x, const void* w, const void* gate, void* out, int M, int H, int N, int K, int ldx, int ldo,
                     int ldg, int gcol, int f32, void* stream) {
   if (M <= 0) return 0;
-  if (K % 32 || N % 64 || ldx % 8 || ldo % 8) return -2;
+  if (K % 32 || N % 64 || ldx % 8 || ldo % 8 || (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15)) return -2;
   ti::HeadProductParams p = {x, w, gate, out, M, H, N, K, ldx, ldo, ldg, gcol};
   const dim3 grid(N / 64, H, (M + 15) / 16);
   ti::launch_kernel(f32 ? ti::head_product_f32_kernel : ti::head_product_bf16_kernel, grid, dim3(128), 0, (cudaStream_t)stream, true, p);
