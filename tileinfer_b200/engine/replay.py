@@ -66,8 +66,9 @@ class ReplaySession:
 
 def make_engine(model: str, dtype: str, max_tokens: int, device: str = "cuda", max_live: int = 4) -> LLMEngine:
     """An engine whose cache holds `max_tokens` tokens (each request rounded up to a whole block) and `max_live` requests."""
+    blocks = max(1, -(-max_tokens // 16))
     return LLMEngine(model, quantization={"bfloat16": "bf16", "float32": "fp32"}[dtype], device=device, tokenizer="ids",
-                     num_kvcache_blocks=max(1, -(-max_tokens // 16)), max_num_seqs=max_live, max_model_len=1 << 30,
+                     num_kvcache_blocks=blocks, max_num_seqs=max_live, max_model_len=16 * blocks,
                      max_num_batched_tokens=max(16, max_tokens), enable_prefix_caching=False)
 
 

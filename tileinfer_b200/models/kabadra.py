@@ -12,12 +12,11 @@ l<i>.mlp.{gate, up, down}; matrices are [out, in].
 """
 from __future__ import annotations
 
-import hashlib
 import json
 import os
 from dataclasses import dataclass
 
-import torch
+from .checkpoint import CheckpointWeights, make_source
 
 ARCHITECTURE = "Kabadra"
 MIXERS = ("latent_attention",)
@@ -175,61 +174,16 @@ def load_config(model_dir: str, d: dict) -> KabadraConfig:
 
 
 # --------------------------------------------------------------------------- weight sources
-class KabadraWeights:
-    """Reads a checkpoint folder tensor by tensor (model.safetensors, or shards with an index)."""
-
-    def __init__(self, cfg: KabadraConfig, model_dir: str, device="cpu"):
-        from safetensors import safe_open
-        self.cfg, self.device = cfg, torch.device(device)
-        self._files, self._where = {}, {}
-        for fn in sorted(f for f in os.listdir(model_dir) if f.endswith(".safetensors")):
-            h = self._files[fn] = safe_open(os.path.join(model_dir, fn), "pt")
-            for k in h.keys():
-                self._where[k] = fn
-        for name, shape in cfg.tensor_shapes().items():
-            if name not in self._where:
-                raise ValueError(f"{model_dir}: no tensor {name}")
-            have = tuple(self._files[self._where[name]].get_slice(name).get_shape())
-            if have != tuple(shape):
-                raise ValueError(f"{model_dir}: {name} has shape {have}, the configuration says {tuple(shape)}")
-
-    def get(self, name: str) -> torch.Tensor:
-        """Full tensor in fp32 on `self.device`."""
-        return self._files[self._where[name]].get_tensor(name).to(self.device).float()
+KabadraWeights = CheckpointWeights
 
 
-class KabadraRandomWeights:
-    """Deterministic weights of the architecture: every tensor has its own generator stream; matrices are scaled by
-    their input size and rounded to bf16, norm weights are 1, sinks are N(0, 1)."""
-
-    def __init__(self, cfg: KabadraConfig, seed: int = 0, device="cpu"):
-        self.cfg, self.seed, self.device = cfg, seed, torch.device(device)
-        self._shapes = cfg.tensor_shapes()
-
-    def get(self, name: str) -> torch.Tensor:
-        shape = self._shapes[name]
-        if name.endswith(("norm", "norm1")):
-            return torch.ones(shape, dtype=torch.float32, device=self.device)
-        # small tensors come from the CPU generator so that CPU and GPU runs see the same weights
-        numel = 1
-        for n in shape:
-            numel *= n
-        dev = torch.device("cpu") if numel <= 1 << 24 else self.device
-        g = torch.Generator(device=dev)
-        g.manual_seed(int.from_bytes(hashlib.sha256(f"{self.seed}:{name}".encode()).digest()[:7], "little"))
-        w = torch.empty(shape, dtype=torch.float32, device=dev).normal_(0.0, 1.0, generator=g)
-        if not name.endswith((".sink", "embed", "pos")):
-            w *= shape[-1] ** -0.5
-        return w.to(torch.bfloat16).float().to(self.device)
+def _random_scale(name: str, shape) -> float:
+    """Matrices are scaled by their input size; sinks and embeddings are N(0, 1)."""
+    return 1.0 if name.endswith((".sink", "embed", "pos")) else shape[-1] ** -0.5
 
 
 def make_weights(cfg: KabadraConfig, spec: str, model_dir: str | None, device="cpu"):
-    """`spec` is "random:<seed>" or "hf" (a checkpoint folder)."""
-    if spec.startswith("random"):
-        return KabadraRandomWeights(cfg, int(spec.split(":", 1)[1]) if ":" in spec else 0, device)
-    if spec == "hf":
-        return KabadraWeights(cfg, model_dir, device)
-    raise ValueError(f"unknown weights spec {spec!r}")
+    return make_source(cfg, spec, model_dir, device, _random_scale)
 
 
 def read_config_json(model_dir: str) -> dict:

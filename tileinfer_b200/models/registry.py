@@ -53,7 +53,20 @@ def _kabadra() -> Family:
     return Family("kabadra", lambda: k.PRESETS, k.ARCHITECTURE, k.load_config, k.make_weights, executor, ("w8a16", "bf16", "fp32"))
 
 
-_MAKERS = {"hybrid": _hybrid, "kabadra": _kabadra}
+def _gerivik() -> Family:
+    from . import gerivik as g
+
+    def executor(device):
+        if device == "cuda":
+            from .gated_b200 import B200GatedModel
+            return B200GatedModel
+        from .gated_cpu import TorchGatedModel
+        return TorchGatedModel
+
+    return Family("gerivik", lambda: g.PRESETS, g.ARCHITECTURE, g.load_config, g.make_weights, executor, ("w8a16", "bf16", "fp32"))
+
+
+_MAKERS = {"hybrid": _hybrid, "kabadra": _kabadra, "gerivik": _gerivik}
 
 
 def family(name: str) -> Family:
