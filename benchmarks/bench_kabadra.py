@@ -133,7 +133,7 @@ def _row(name, us, *, flops=0, nbytes=0, like=None):
 def kernels(cfg, prompt, ctx, batch):
     """Rows of the kernel table for one size: a prefill step of `prompt` tokens and a decode step of `batch` sequences."""
     from tileinfer_b200.ops import functional as F
-    F.L("base", "hybrid", "latent")
+    F.L("base", "rows", "attention", "hybrid", "latent")
     m, f = cfg.layers[0].mixer, cfg.layers[0].mlp
     W, H, D, R, ff, win = cfg.hidden_size, m.heads, m.dim, m.kv_rank, f.ff, m.window
     dev, rows = "cuda", []

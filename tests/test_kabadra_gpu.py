@@ -22,7 +22,7 @@ TOL = {"bf16": 0.03, "fp32": 1e-4, "w8a16": 0.03}
 @pytest.fixture(scope="module")
 def F():
     from tileinfer_b200.ops import functional
-    functional.L("base", "latent")
+    functional.L("base", "rows", "latent")
     return functional
 
 

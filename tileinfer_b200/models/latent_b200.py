@@ -20,43 +20,10 @@ from ..ops import functional as F
 from ..ops.functional import LatentAttnParams, LinearW, ptr
 from ..utils.trace import nvtx_end, nvtx_mark
 from .kabadra import GLU_ALPHA, GLU_BIAS, KabadraConfig
+from .products_b200 import Product, pad64, pad_to
 from .runtime_b200 import DeviceRuntime, StepCtx
 
 PAGE = 16
-
-
-def pad64(n: int) -> int:
-    return -(-n // 64) * 64
-
-
-def pad_to(t: torch.Tensor, *shape) -> torch.Tensor:
-    """`t` in the corner of a zero tensor of the given shape."""
-    out = t.new_zeros(shape)
-    out[tuple(slice(0, n) for n in t.shape)] = t
-    return out
-
-
-class Product:
-    """y = x W^T with the epilogues of a fp32-residual model, in one of three weight formats."""
-
-    def __init__(self, w: torch.Tensor, quant: str, dev):
-        self.N, self.K = w.shape
-        self.f32 = quant == "fp32"
-        self.w = w.to(dev, torch.float32).contiguous() if self.f32 else LinearW(w, quant == "w8a16", dev)
-
-    def nbytes(self) -> int:
-        return self.w.numel() * 4 if self.f32 else self.w.nbytes()
-
-    def __call__(self, x, out, epi, ex=None) -> int:
-        """Returns the number of kernels launched."""
-        if self.f32:
-            F.gemm_f32(self.w, x, out=out, epi=F.GEPI_F32 if epi == F.GEPI_STORE else epi, ex=ex)
-            return 1
-        if self.w.wt == F.W_INT8:
-            F.gemm_w8a16(self.w, F.quant_rows(x), out=out, epi=epi, ex=ex)
-            return 2
-        F.gemm_bf16(self.w, x, out=out, epi=epi, ex=ex)
-        return 1
 
 
 class _Layer:
@@ -67,7 +34,7 @@ class B200LatentModel(DeviceRuntime):
     def __init__(self, cfg: KabadraConfig, src, *, quant="bf16", tp=1, rank=0, comm=None, config=None):
         assert torch.cuda.is_available(), "B200LatentModel needs a CUDA device"
         cfg.validate_tp(tp)
-        F.L("base", "latent")              # load (or build) the kernel libraries now: fail loudly if they are missing
+        F.L("base", "rows", "latent")              # load (or build) the kernel libraries now: fail loudly if they are missing
         self.cfg, self.tp, self.rank, self.comm, self.peer = cfg, tp, rank, comm, None
         self.dev = torch.device("cuda", torch.cuda.current_device())
         self.quant, self.f32 = quant, quant == "fp32"

@@ -21,8 +21,12 @@ BUILD = os.path.join(HERE, "build")
 # sampling, pointwise ops) is used by every model family, the others by the family that has the mechanism.
 GROUPS = {
     "base": ("gemm_tcgen05.cu", "lm_head.cu", "pointwise.cu", "sampling.cu", "symm.cu"),
-    "hybrid": ("attn_paged.cu", "attn_prefill.cu", "fused_ar.cu", "gdn.cu", "gdn_chunk.cu", "gemv_w8a16.cu"),
+    "rows": ("row_ops.cu",),
+    "attention": ("attn_paged.cu", "attn_prefill.cu", "attn_general.cu"),
+    "hybrid": ("fused_ar.cu", "gdn.cu", "gdn_chunk.cu", "gemv_w8a16.cu"),
     "latent": ("latent_ops.cu", "latent_attn.cu", "latent_decode.cu", "latent_prefill.cu"),
+    "gla": ("gla.cu",),
+    "moe": ("moe_route.cu", "gemm_grouped.cu"),
 }
 
 

@@ -1,0 +1,215 @@
+// Around the paged attention kernels: the preparation of rotated, root-mean-square normalised heads, and a plain attention
+// kernel for what the tensor-core kernels do not take (32-bit mode, heads wider than 256).
+//
+// Cache layout as in attn_paged.cu, in bf16 or float: K pages [block][kv_head][16 tokens][dp], V pages transposed
+// [block][kv_head][vp][16 tokens].  Head sizes are padded to multiples of 64 with zeros; means divide by the true size.
+#include "row_vec.cuh"
+
+namespace ti {
+
+struct RopeUnitParams {
+  const void* proj;              // [T, ld]: H query heads at q_col, G key heads at k_col (dp each), G value heads at v_col (vp)
+  const float* inv_freq;         // [half] angle per position of pair i, i + half
+  const int* positions;          // [T]
+  const long long* slot_mapping; // [T] flat slot = block * 16 + offset; outside the cache: not stored
+  void* q_out;                   // [T, H, dp]
+  void* kcache;
+  void* vcache;
+  unsigned* status;
+  int T, ld, q_col, k_col, v_col, H, G, dim, dp, vp, half, num_blocks;
+  float eps;
+};
+
+// A warp per (token, head): rotation of the first 2 * half dimensions, then x / sqrt(mean(x^2) + eps); values are only
+// stored.  Everything up to the store is fp32.
+template <typename T, int E>
+__global__ void __launch_bounds__(128) rope_unit_kernel(const __grid_constant__ RopeUnitParams p) {
+  extern __shared__ float sh[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, heads = p.H + 2 * p.G;
+  const long long item = (long long)blockIdx.x * 4 + warp;
+  pdl_trigger();
+  pdl_wait();
+  if (item >= (long long)p.T * heads) return;
+  const int t = (int)(item / heads), head = (int)(item - (long long)t * heads);
+  const T* row = static_cast<const T*>(p.proj) + (size_t)t * p.ld;
+  const long long slot = p.slot_mapping[t], blk = slot >> 4;
+  const int off = (int)(slot & 15);
+  const bool stored = slot >= 0 && blk < p.num_blocks;
+  if (head >= p.H + p.G) {
+    if (!stored) return;
+    const int g = head - p.H - p.G;
+    const T* src = row + p.v_col + (size_t)g * p.vp;
+    T* dst = static_cast<T*>(p.vcache) + ((size_t)blk * p.G + g) * p.vp * 16 + off;
+    for (int c = lane; c < p.vp; c += 32) dst[(size_t)c * 16] = src[c];
+    return;
+  }
+  const bool is_q = head < p.H;
+  if (!is_q && !stored) return;
+  const T* src = row + (is_q ? p.q_col + (size_t)head * p.dp : p.k_col + (size_t)(head - p.H) * p.dp);
+  float* buf = sh + (size_t)warp * p.dp;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < E; ++i) {
+    const int c = lane + 32 * i;
+    if (c < p.dp) {
+      const float v = to_f<T>(src[c]);
+      buf[c] = v;
+      ss += v * v;                                         // a rotation keeps the sum of squares
+    }
+  }
+  __syncwarp();
+  const float rr = rsqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+  const float pos = (float)p.positions[t];
+  for (int i = lane; i < p.half; i += 32) {
+    float sn, cs;
+    sincosf(pos * p.inv_freq[i], &sn, &cs);
+    const float u = buf[i], v = buf[i + p.half];
+    buf[i] = u * cs - v * sn;
+    buf[i + p.half] = v * cs + u * sn;
+  }
+  __syncwarp();
+  T* dst = is_q ? static_cast<T*>(p.q_out) + ((size_t)t * p.H + head) * p.dp
+                : static_cast<T*>(p.kcache) + (((size_t)blk * p.G + head - p.H) * 16 + off) * p.dp;
+#pragma unroll
+  for (int i = 0; i < E; ++i) {
+    const int c = lane + 32 * i;
+    if (c < p.dp) dst[c] = from_f<T>(buf[c] * rr);
+  }
+}
+
+struct AttnGeneralParams {
+  const void* q;           // [T, H, dp]
+  const void* kcache;
+  const void* vcache;
+  const int* block_tables; // [S, max_blocks]
+  const int* positions;    // [T]
+  const int* qg_seq;       // [num_qg] sequence of a query token
+  const int* qg_tok0;      // [num_qg] its flat index
+  const int* qg_ntok;      // [num_qg] 1, or 0: padding
+  void* out;               // [T, ldo], head h at column h * vp
+  unsigned* status;
+  int H, G, dp, vp, max_blocks, num_qg, num_blocks, ldo;
+  float scale, softcap;    // softcap 0: none
+};
+
+// One query token and head per block; the four warps take the pages in turn and keep running maxima, sums and outputs.
+template <typename T, int NV>
+__global__ void __launch_bounds__(128) attn_general_kernel(const __grid_constant__ AttnGeneralParams p) {
+  extern __shared__ float sh[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, qg = blockIdx.x, h = blockIdx.y;
+  float *qs = sh, *acc_s = sh + p.dp, *ml = acc_s + 4 * p.vp, *ps = ml + 8 + warp * 16;
+  pdl_trigger();
+  pdl_wait();
+  if (p.qg_ntok[qg] == 0) return;
+  const int seq = p.qg_seq[qg], tok = p.qg_tok0[qg], g = h / (p.H / p.G), pos = p.positions[tok];
+  for (int c = threadIdx.x; c < p.dp; c += 128) qs[c] = to_f<T>(static_cast<const T*>(p.q)[((size_t)tok * p.H + h) * p.dp + c]);
+  __syncthreads();
+  float acc[NV], m = -1e30f, l = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) acc[i] = 0.f;
+  for (int pg = warp; pg <= pos >> 4; pg += 4) {
+    const int blk = p.block_tables[(size_t)seq * p.max_blocks + pg];
+    if (!TI_CHECK(blk, p.num_blocks, p.status)) continue;
+    const T* kb = static_cast<const T*>(p.kcache) + (((size_t)blk * p.G + g) * 16 + (lane >> 1)) * p.dp;
+    float s = 0.f;
+    for (int c = (lane & 1) * 8; c < p.dp; c += 16) {
+      float v[8];
+      load8(kb + c, v);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) s = fmaf(v[i], qs[c + i], s);
+    }
+    s = (s + __shfl_xor_sync(0xffffffffu, s, 1)) * p.scale;
+    if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+    const bool seen = pg * 16 + (lane >> 1) <= pos;
+    const float mn = fmaxf(m, warp_max(seen ? s : -1e30f));
+    const float e = seen ? expf(s - mn) : 0.f, alpha = expf(m - mn);
+    l = l * alpha + warp_sum((lane & 1) ? 0.f : e);
+    m = mn;
+    __syncwarp();
+    if ((lane & 1) == 0) ps[lane >> 1] = e;
+    __syncwarp();
+    const T* vb = static_cast<const T*>(p.vcache) + ((size_t)blk * p.G + g) * p.vp * 16;
+    const int last = pos - pg * 16;                        // keys past the query may hold anything: they are not multiplied
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = lane + 32 * i;
+      if (c >= p.vp) continue;
+      float a[8], b[8], t = 0.f;
+      load8(vb + (size_t)c * 16, a);
+      load8(vb + (size_t)c * 16 + 8, b);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        if (j <= last) t = fmaf(ps[j], a[j], t);
+        if (j + 8 <= last) t = fmaf(ps[j + 8], b[j], t);
+      }
+      acc[i] = acc[i] * alpha + t;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (lane + 32 * i < p.vp) acc_s[warp * p.vp + lane + 32 * i] = acc[i];
+  if (lane == 0) { ml[warp] = m; ml[4 + warp] = l; }
+  __syncthreads();
+  const float M = fmaxf(fmaxf(ml[0], ml[1]), fmaxf(ml[2], ml[3]));
+  float w[4], L = 0.f;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    w[i] = expf(ml[i] - M);
+    L += w[i] * ml[4 + i];
+  }
+  T* out = static_cast<T*>(p.out) + (size_t)tok * p.ldo + (size_t)h * p.vp;
+  for (int c = threadIdx.x; c < p.vp; c += 128) {
+    float o = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) o = fmaf(w[i], acc_s[i * p.vp + c], o);
+    out[c] = from_f<T>(o / L);
+  }
+}
+
+template <typename T>
+static int launch_rope(const RopeUnitParams& p, cudaStream_t st) {
+  const long long items = (long long)p.T * (p.H + 2 * p.G);
+  const dim3 grid((unsigned)((items + 3) / 4));
+  const size_t smem = (size_t)4 * p.dp * 4;
+  if (p.dp <= 64) launch_kernel(rope_unit_kernel<T, 2>, grid, dim3(128), smem, st, true, p);
+  else if (p.dp <= 128) launch_kernel(rope_unit_kernel<T, 4>, grid, dim3(128), smem, st, true, p);
+  else if (p.dp <= 256) launch_kernel(rope_unit_kernel<T, 8>, grid, dim3(128), smem, st, true, p);
+  else if (p.dp <= 1024) launch_kernel(rope_unit_kernel<T, 32>, grid, dim3(128), smem, st, true, p);
+  else return -3;
+  return (int)cudaGetLastError();
+}
+
+template <typename T>
+static int launch_general(const AttnGeneralParams& p, cudaStream_t st) {
+  const dim3 grid(p.num_qg, p.H);
+  const size_t smem = (size_t)(p.dp + 4 * p.vp + 8 + 64) * 4;
+  if (p.vp <= 64) launch_kernel(attn_general_kernel<T, 2>, grid, dim3(128), smem, st, true, p);
+  else if (p.vp <= 128) launch_kernel(attn_general_kernel<T, 4>, grid, dim3(128), smem, st, true, p);
+  else if (p.vp <= 256) launch_kernel(attn_general_kernel<T, 8>, grid, dim3(128), smem, st, true, p);
+  else if (p.vp <= 1024) launch_kernel(attn_general_kernel<T, 32>, grid, dim3(128), smem, st, true, p);
+  else return -3;
+  return (int)cudaGetLastError();
+}
+
+}  // namespace ti
+
+extern "C" {
+
+int ti_rope_unit_params_size() { return (int)sizeof(ti::RopeUnitParams); }
+int ti_attn_general_params_size() { return (int)sizeof(ti::AttnGeneralParams); }
+
+int ti_rope_unit(const ti::RopeUnitParams* p, int f32, void* stream) {
+  if (p->T <= 0) return 0;
+  if (p->dp % 64 || p->vp % 64 || p->dim > p->dp || 2 * p->half > p->dim || p->num_blocks < 1) return -2;
+  return f32 ? ti::launch_rope<float>(*p, (cudaStream_t)stream) : ti::launch_rope<ti::bf16>(*p, (cudaStream_t)stream);
+}
+
+int ti_attn_general(const ti::AttnGeneralParams* p, int f32, void* stream) {
+  if (p->num_qg <= 0) return 0;
+  if (p->dp % 64 || p->vp % 64 || p->H % p->G || p->num_blocks < 1 ||
+      (((uintptr_t)p->kcache | (uintptr_t)p->vcache) & 15))
+    return -2;
+  return f32 ? ti::launch_general<float>(*p, (cudaStream_t)stream) : ti::launch_general<ti::bf16>(*p, (cudaStream_t)stream);
+}
+
+}  // extern "C"

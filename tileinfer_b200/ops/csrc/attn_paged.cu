@@ -15,7 +15,8 @@
 // the (up to 16) query rows = (token, head-of-group) pairs as the A operand, online softmax in the
 // exp2 domain in registers, O += P V^T.  Pages are dealt round-robin to the warp streams of a CTA and
 // to `nsplit` CTAs (split-KV); a second kernel merges the partial (O, max, sum) triples and applies
-// the sigmoid gate.  All sizes (batch, context, block-table width) are run-time values.
+// the sigmoid gate.  All sizes (batch, context, block-table width) are run-time values.  Values may be of another size
+// than queries and keys, scores may be capped by cap * tanh(score / cap), and the gate may be absent.
 #include "common.cuh"
 
 namespace ti {
@@ -117,7 +118,14 @@ struct AttnParams {
   float scale_log2e;
   int num_blocks;                // pages in the cache (checked builds verify block-table entries; 0: unknown)
   unsigned* status;
+  float cap_in, cap_out;         // cap_out > 0: score = cap_out * tanh(q.k * cap_in / 2), in log2 units
+  int rep;                       // blocks per KV head, each with hq / (hkv * rep) of its query heads
 };
+
+TI_DEVICE float attn_score(const AttnParams& p, float qk) {
+  // tanh(y) = 1 - 2 / (1 + exp(2 y)): absolute error of a few 1e-7, what a score needs
+  return p.cap_out > 0.f ? p.cap_out * (1.f - __fdividef(2.f, 1.f + exp2f(qk * p.cap_in))) : qk * p.scale_log2e;
+}
 
 constexpr float kNegBig = -1e30f;
 
@@ -292,14 +300,14 @@ TI_DEVICE uint4 lds128a(uint32_t addr) {
 
 constexpr int kPipe = 3;       // ring stages per page stream
 
-template <int D, int DSPLIT>
+template <int D, int DV, int DSPLIT>
 __global__ void __launch_bounds__(128) attn_pipe_kernel(const __grid_constant__ AttnParams p) {
   constexpr int NSTREAM = 4 / DSPLIT;
-  constexpr int DH = D / DSPLIT;
+  constexpr int DH = DV / DSPLIT;
   constexpr int NT_O = DH / 8;
   constexpr int NCH = D / 32;
-  constexpr int kPage = 16 * D * 2;                     // bytes of a K page (and of a V page)
-  constexpr int kStage = 2 * kPage;
+  constexpr int kPage = 16 * D * 2, kPageV = 16 * DV * 2;      // bytes of a K page and of a V page
+  constexpr int kStage = kPage + kPageV;
   constexpr int TS = 32 * DSPLIT;                       // threads of a stream
   extern __shared__ __align__(128) uint8_t ring_raw[];  // [NSTREAM][kPipe][K page | V page]; reused for the merge
   __shared__ float MLsm[NSTREAM][16][2];
@@ -311,7 +319,7 @@ __global__ void __launch_bounds__(128) attn_pipe_kernel(const __grid_constant__ 
   if (pr.ntok == 0) return;
   const int p0 = sp * pr.pps, p1 = min(pr.npages, p0 + pr.pps);
   if (p0 >= p1) return;
-  const int G = p.hq / p.hkv;
+  const int G = p.hq / (p.hkv * p.rep), kvh = kh / p.rep;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const int stream = warp / DSPLIT, dpart = warp % DSPLIT;
   const int st_tid = tid - stream * TS;                 // thread index inside the stream
@@ -345,15 +353,19 @@ __global__ void __launch_bounds__(128) attn_pipe_kernel(const __grid_constant__ 
       const int pg = p0 + stream + k * NSTREAM;
       int blk = p.block_tables[(size_t)pr.seq * p.max_blocks + pg];
       if (p.num_blocks > 0 && !TI_CHECK(blk, p.num_blocks, p.status)) blk = 0;    // checked build: never leave the cache
-      const uint8_t* kg = reinterpret_cast<const uint8_t*>(p.kcache + ((size_t)blk * p.hkv + kh) * 16 * D);
-      const uint8_t* vg = reinterpret_cast<const uint8_t*>(p.vcache + ((size_t)blk * p.hkv + kh) * D * 16);
+      const uint8_t* kg = reinterpret_cast<const uint8_t*>(p.kcache + ((size_t)blk * p.hkv + kvh) * 16 * D);
+      const uint8_t* vg = reinterpret_cast<const uint8_t*>(p.vcache + ((size_t)blk * p.hkv + kvh) * DV * 16);
       const uint32_t ks = ring + (uint32_t)(k % kPipe) * kStage, vs = ks + kPage;
       constexpr int kChunks = kPage / 16, kRowChunks = D * 2 / 16;     // 16-byte chunks per page / per token row
 #pragma unroll
       for (int c = st_tid; c < kChunks; c += TS) {
         const int tok = c / kRowChunks, cc = c - tok * kRowChunks;
         cp_async16(ks + (uint32_t)(tok * kRowChunks + (cc ^ ((tok & 1) << 2))) * 16u, kg + (size_t)c * 16);
-        cp_async16(vs + (uint32_t)c * 16u, vg + (size_t)c * 16);
+        if (DV == D) cp_async16(vs + (uint32_t)c * 16u, vg + (size_t)c * 16);
+      }
+      if (DV != D) {
+#pragma unroll
+        for (int c = st_tid; c < kPageV / 16; c += TS) cp_async16(vs + (uint32_t)c * 16u, vg + (size_t)c * 16);
       }
     }
     cp_async_commit();
@@ -390,7 +402,7 @@ __global__ void __launch_bounds__(128) attn_pipe_kernel(const __grid_constant__ 
       float mx = kNegBig;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        sc[e] = (j0 + e <= pos[h]) ? sc[e] * p.scale_log2e : kNegBig;
+        sc[e] = (j0 + e <= pos[h]) ? attn_score(p, sc[e]) : kNegBig;
         mx = fmaxf(mx, sc[e]);
       }
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -423,7 +435,7 @@ __global__ void __launch_bounds__(128) attn_pipe_kernel(const __grid_constant__ 
     l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
   }
   __syncthreads();                                       // every stream is done with its ring: reuse it for the merge
-  float(*Osm)[16][D] = reinterpret_cast<float(*)[16][D]>(ring_raw);
+  float(*Osm)[16][DV] = reinterpret_cast<float(*)[16][DV]>(ring_raw);
 #pragma unroll
   for (int n = 0; n < NT_O; ++n) {
     const int d = dpart * DH + n * 8 + 2 * t;
@@ -435,16 +447,16 @@ __global__ void __launch_bounds__(128) attn_pipe_kernel(const __grid_constant__ 
     MLsm[stream][g + 8][0] = m[1]; MLsm[stream][g + 8][1] = l[1];
   }
   __syncthreads();
-  const size_t item = ((size_t)qg * p.hkv + kh) * p.nsplit + sp;
-  for (int idx = tid; idx < 16 * D; idx += 128) {
-    const int r = idx / D, d = idx - r * D;
+  const size_t item = ((size_t)qg * p.hkv * p.rep + kh) * p.nsplit + sp;
+  for (int idx = tid; idx < 16 * DV; idx += 128) {
+    const int r = idx / DV, d = idx - r * DV;
     float M = kNegBig;
 #pragma unroll
     for (int s = 0; s < NSTREAM; ++s) M = fmaxf(M, MLsm[s][r][0]);
     float acc = 0.f;
 #pragma unroll
     for (int s = 0; s < NSTREAM; ++s) acc += exp2f(MLsm[s][r][0] - M) * Osm[s][r][d];
-    p.o_part[(item * 16 + r) * D + d] = acc;
+    p.o_part[(item * 16 + r) * DV + d] = acc;
   }
   if (tid < 16) {
     float M = kNegBig, L = 0.f;
@@ -469,10 +481,10 @@ __global__ void __launch_bounds__(D / 2) attn_merge_kernel(const __grid_constant
   pdl_trigger();
   pdl_wait();
   const PageRange pr = page_range(p, qg);
-  const int G = p.hq / p.hkv;
+  const int G = p.hq / (p.hkv * p.rep);
   if (pr.ntok == 0 || r >= pr.ntok * G) return;
   const int nact = (pr.npages + pr.pps - 1) / pr.pps;
-  const size_t item0 = ((size_t)qg * p.hkv + kh) * p.nsplit;
+  const size_t item0 = ((size_t)qg * p.hkv * p.rep + kh) * p.nsplit;
   for (int s = tid; s < nact; s += D / 2) {
     const float2 ml = *reinterpret_cast<const float2*>(p.ml_part + ((item0 + s) * 16 + r) * 2);
     w_s[s] = ml.x;
@@ -500,19 +512,25 @@ __global__ void __launch_bounds__(D / 2) attn_merge_kernel(const __grid_constant
   }
   const int tk = r / G, hg = r - tk * G;
   const int tok = pr.tok0 + tk, head = kh * G + hg;
-  const uint32_t gw = *reinterpret_cast<const uint32_t*>(p.gate_src + (size_t)tok * p.ld + (size_t)head * 2 * D + D + d);
   const float inv = 1.f / L;
+  float g0 = 1.f, g1 = 1.f;
+  if (p.gate_src != nullptr) {
+    const uint32_t gw = *reinterpret_cast<const uint32_t*>(p.gate_src + (size_t)tok * p.ld + (size_t)head * 2 * D + D + d);
+    g0 = sigmoid_f(bf16lo(gw));
+    g1 = sigmoid_f(bf16hi(gw));
+  }
   *reinterpret_cast<uint32_t*>(p.out + (size_t)tok * p.hq * D + (size_t)head * D + d) =
-      pack_bf16(a0 * inv * sigmoid_f(bf16lo(gw)), a1 * inv * sigmoid_f(bf16hi(gw)));
+      pack_bf16(a0 * inv * g0, a1 * inv * g1);
 }
 
 }  // namespace ti
 
-template <int D, int DSPLIT>
+template <int D, int DV>
 static void launch_attn_pipe(const ti::AttnParams& p, dim3 grid, cudaStream_t st) {
-  constexpr size_t smem = (size_t)(4 / DSPLIT) * ti::kPipe * 2 * 16 * D * 2;
+  constexpr int DSPLIT = D == 256 || DV == 256 ? 2 : 1;       // two warps share a page when a row is too wide for one
+  constexpr size_t smem = (size_t)(4 / DSPLIT) * ti::kPipe * 16 * (D + DV) * 2;
   static bool configured = false;
-  auto k = ti::attn_pipe_kernel<D, DSPLIT>;
+  auto k = ti::attn_pipe_kernel<D, DV, DSPLIT>;
   if (!configured) {
     cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     configured = true;
@@ -537,47 +555,37 @@ int ti_qkv_prep(const ti::QkvPrepParams* p, int T, int D, void* stream) {
   return (int)cudaGetLastError();
 }
 
-// Launches the split-KV attention kernel and the merge/gate kernel.  The cp.async-pipelined kernel is the default
-// (measured faster from batch 1 / 256 tokens of context to batch 64 / 8192); TI_ATTN_PIPE=0 selects the direct-load
-// kernel.
-int ti_attn_paged(const ti::AttnParams* p, int D, void* stream) {
+// Launches the split-KV attention kernel and the merge/gate kernel.  D: size of a query / key head, DV of a value head.
+// The cp.async-pipelined kernel is the default (measured faster from batch 1 / 256 tokens of context to batch 64 / 8192);
+// TI_ATTN_PIPE=0 selects the direct-load kernel, which takes neither a cap nor values of another size.
+int ti_attn_paged(const ti::AttnParams* p, int D, int DV, void* stream) {
   if (p->num_qg <= 0) return 0;
-  const int G = p->hq / p->hkv;
-  if (p->hq % p->hkv || G > 16 || p->nsplit < 1 || p->nsplit > ti::kMaxSplit) return -2;
-  dim3 grid(p->num_qg, p->hkv, p->nsplit), mgrid(p->num_qg, p->hkv, 16);
+  const int rep = p->rep < 1 ? 1 : p->rep;
+  if (p->hq % (p->hkv * rep) || p->hq / (p->hkv * rep) > 16 || p->nsplit < 1 || p->nsplit > ti::kMaxSplit) return -2;
+  ti::AttnParams a = *p;
+  a.rep = rep;
+  dim3 grid(p->num_qg, p->hkv * rep, p->nsplit), mgrid(p->num_qg, p->hkv * rep, 16);
   cudaStream_t st = (cudaStream_t)stream;
   static const int pipe_mode = [] {
     const char* e = getenv("TI_ATTN_PIPE");
     return e == nullptr ? -1 : atoi(e);
   }();
-  const bool pipe = pipe_mode != 0;
-  if (pipe) {
-    if (D == 256) {
-      launch_attn_pipe<256, 2>(*p, grid, st);
-      ti::launch_kernel(ti::attn_merge_kernel<256>, mgrid, dim3(128), 0, st, true, *p);
-    } else if (D == 128) {
-      launch_attn_pipe<128, 1>(*p, grid, st);
-      ti::launch_kernel(ti::attn_merge_kernel<128>, mgrid, dim3(64), 0, st, true, *p);
-    } else if (D == 64) {
-      launch_attn_pipe<64, 1>(*p, grid, st);
-      ti::launch_kernel(ti::attn_merge_kernel<64>, mgrid, dim3(32), 0, st, true, *p);
-    } else {
-      return -3;
-    }
-    return (int)cudaGetLastError();
-  }
-  if (D == 256) {
-    ti::launch_kernel(ti::attn_kernel<256, 2>, grid, dim3(128), 0, st, true, *p);
-    ti::launch_kernel(ti::attn_merge_kernel<256>, mgrid, dim3(128), 0, st, true, *p);
-  } else if (D == 128) {
-    ti::launch_kernel(ti::attn_kernel<128, 1>, grid, dim3(128), 0, st, true, *p);
-    ti::launch_kernel(ti::attn_merge_kernel<128>, mgrid, dim3(64), 0, st, true, *p);
-  } else if (D == 64) {
-    ti::launch_kernel(ti::attn_kernel<64, 1>, grid, dim3(128), 0, st, true, *p);
-    ti::launch_kernel(ti::attn_merge_kernel<64>, mgrid, dim3(32), 0, st, true, *p);
+  if (pipe_mode == 0 && D == DV && rep == 1 && !(p->cap_out > 0.f)) {
+    if (D == 256) ti::launch_kernel(ti::attn_kernel<256, 2>, grid, dim3(128), 0, st, true, a);
+    else if (D == 128) ti::launch_kernel(ti::attn_kernel<128, 1>, grid, dim3(128), 0, st, true, a);
+    else if (D == 64) ti::launch_kernel(ti::attn_kernel<64, 1>, grid, dim3(128), 0, st, true, a);
+    else return -3;
   } else {
-    return -3;
+#define TI_PIPE(A, B) if (D == A && DV == B) launch_attn_pipe<A, B>(a, grid, st)
+    TI_PIPE(64, 64); else TI_PIPE(64, 128); else TI_PIPE(64, 256);
+    else TI_PIPE(128, 64); else TI_PIPE(128, 128); else TI_PIPE(128, 256);
+    else TI_PIPE(256, 64); else TI_PIPE(256, 128); else TI_PIPE(256, 256);
+    else return -3;
+#undef TI_PIPE
   }
+  if (DV == 256) ti::launch_kernel(ti::attn_merge_kernel<256>, mgrid, dim3(128), 0, st, true, a);
+  else if (DV == 128) ti::launch_kernel(ti::attn_merge_kernel<128>, mgrid, dim3(64), 0, st, true, a);
+  else ti::launch_kernel(ti::attn_merge_kernel<64>, mgrid, dim3(32), 0, st, true, a);
   return (int)cudaGetLastError();
 }
 

@@ -18,7 +18,10 @@
 //
 // TMEM: S0 | S1 | O = 128 + 128 + D columns (512 allocated).  Shared memory at D = 256: Q 64 KB, K 64 KB,
 // V 64 KB, P 32 KB.  Causal alignment is by absolute position (bottom-right): a chunk that continues a cached
-// prefix sees all of it.  Every wait is bounded; on expiry the status word is set, all roles leave their loops
+// prefix sees all of it.  Values may be of another size than queries and keys, and the gate may be absent.  Scores may be
+// capped by cap * tanh(score / cap); where |score / cap| is known to stay small (normalised queries and keys) the tanh is
+// its power series and the softmax needs no running maximum at all: exp2 of a bounded score neither overflows nor
+// vanishes, so the scores of a tile are read once.  Every wait is bounded; on expiry the status word is set, all roles leave their loops
 // and TMEM is freed.  No load carries a cluster-multicast qualifier.
 #include "tensor_map.cuh"
 
@@ -38,7 +41,33 @@ struct AttnPrefillParams {
   unsigned* status;
   int hq, hkv, max_blocks, ld;
   float scale_log2e;
+  float cap_in, cap_out;           // score = cap_out * tanh(q.k * cap_in), in log2 units
 };
+
+// How a score follows from q.k: scaled; capped with the series, reference 0 instead of a running maximum; capped
+enum { SCORE_PLAIN = 0, SCORE_SERIES = 1, SCORE_CAPPED = 2 };
+constexpr float kSeriesMax = 0.5f;       // largest |argument| the series serves (error below 1e-6 there)
+
+// tanh(y) = y - y^3/3 + 2 y^5/15 - 17 y^7/315 + 62 y^9/2835 - 1382 y^11/155925 + ...
+TI_DEVICE float tanh_series(float y) {
+  const float z = y * y;
+  float s = fmaf(z, 21844.f / 6081075.f, -1382.f / 155925.f);
+  s = fmaf(s, z, 62.f / 2835.f);
+  s = fmaf(s, z, -17.f / 315.f);
+  s = fmaf(s, z, 2.f / 15.f);
+  s = fmaf(s, z, -1.f / 3.f);
+  return fmaf(y * z, s, y);
+}
+TI_DEVICE float ex2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+  return y;
+}
+template <int MODE> TI_DEVICE float prefill_score(const AttnPrefillParams& p, float qk) {
+  if (MODE == SCORE_SERIES) return p.cap_out * tanh_series(qk * p.cap_in);
+  if (MODE == SCORE_CAPPED) return p.cap_out * (1.f - __fdividef(2.f, 1.f + ex2_approx(qk * p.cap_in * 2.8853900817779268f)));
+  return qk * p.scale_log2e;
+}
 
 constexpr unsigned long long kAttnWaitNs = 500000000ull;
 constexpr int kAttnThreads = 224;        // warp 0: Q/K producer, 1: MMA issuer, 2..5: softmax, 6: V producer
@@ -46,11 +75,11 @@ constexpr int kAttnProducerV = 6;
 constexpr float kMaskVal = -1e30f;
 constexpr float kRescaleGap = 8.f;       // log2 units the running maximum may lag behind before O is rescaled
 
-template <int D> struct AttnPrefillGeom {
+template <int D, int DV> struct AttnPrefillGeom {
   static constexpr int kSlabs = D / 64;
   static constexpr int kQBytes = kSlabs * 128 * 128;
   static constexpr int kKBytes = kSlabs * 128 * 128;
-  static constexpr int kVPage = D * 32;
+  static constexpr int kVPage = DV * 32;
   static constexpr int kVBytes = 8 * kVPage;
   static constexpr int kPBytes = 2 * 128 * 128;
   static constexpr int kBarBytes = 128;
@@ -59,9 +88,9 @@ template <int D> struct AttnPrefillGeom {
   static constexpr size_t kSmem = kNeeded > 120 * 1024 ? kNeeded : 120 * 1024;
 };
 
-template <int D>
+template <int D, int DV, int MODE>
 __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __grid_constant__ AttnPrefillParams p) {
-  using G = AttnPrefillGeom<D>;
+  using G = AttnPrefillGeom<D, DV>;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   const uint32_t q_s = smem_u32(smem), k_s = q_s + G::kQBytes, v_s = k_s + G::kKBytes, p_s = v_s + G::kVBytes;
@@ -132,14 +161,14 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
           if (j > 0 && !mbar_wait(v_empty, (uint32_t)((j - 1) & 1), kAttnWaitNs, p.status)) { *abort_flag = 1; break; }
           mbar_expect_tx(v_full, G::kVBytes);
 #pragma unroll
-          for (int g = 0; g < 8; ++g) tma_load_2d(v_s + g * G::kVPage, &p.map_v, 0, (blk[g] * p.hkv + kh) * D, v_full);
+          for (int g = 0; g < 8; ++g) tma_load_2d(v_s + g * G::kVPage, &p.map_v, 0, (blk[g] * p.hkv + kh) * DV, v_full);
         }
       }
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------ MMA issuer
     if (elect_one()) {
-      constexpr uint32_t idesc_s = idesc_f16_bf16(128, 128), idesc_o = idesc_f16_bf16(128, D);
+      constexpr uint32_t idesc_s = idesc_f16_bf16(128, 128), idesc_o = idesc_f16_bf16(128, DV);
       auto issue_qk = [&](int j) {
         const uint32_t d = tmem_base + (uint32_t)(j & 1) * 128u;
 #pragma unroll
@@ -182,7 +211,7 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
     const bool valid = r < ntok;
     const int pos = p.positions[tok0 + (valid ? r : ntok - 1)];
     const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
-    float m_used = kMaskVal, l = 0.f;
+    float m_used = MODE == SCORE_SERIES ? 0.f : kMaskVal, l = 0.f;
     bool ok = true;
     for (int j = 0; j < ntiles; ++j) {
       ok = ok && !*abort_flag && mbar_wait(s_full0 + 8 * (j & 1), (uint32_t)((j >> 1) & 1), kAttnWaitNs, p.status);
@@ -195,19 +224,19 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
       // ---- pass 1: row maximum
       float mx = kMaskVal;
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < (MODE == SCORE_SERIES ? 0 : 4); ++c) {
         uint32_t v[32];
         tmem_ld32(s_addr + c * 32, v);
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          float s = __uint_as_float(v[i]) * p.scale_log2e;
+          float s = prefill_score<MODE>(p, __uint_as_float(v[i]));
           if (need_mask && key0 + c * 32 + i > pos) s = kMaskVal;
           mx = fmaxf(mx, s);
         }
       }
-      const float m_new = fmaxf(m_used, mx);
-      const bool resc = m_new - m_used > kRescaleGap;
+      const float m_new = MODE == SCORE_SERIES ? 0.f : fmaxf(m_used, mx);
+      const bool resc = MODE != SCORE_SERIES && m_new - m_used > kRescaleGap;
       float alpha = 1.f;
       if (resc) {
         alpha = exp2f(m_used - m_new);
@@ -222,7 +251,7 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
         tc_fence_after();
         if (__any_sync(0xffffffffu, resc)) {
 #pragma unroll 1
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             uint32_t v[32];
             tmem_ld32(lane_base + 256u + c * 32, v);
             tmem_ld_wait();
@@ -243,12 +272,12 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          float s0 = __uint_as_float(v[i]) * p.scale_log2e, s1 = __uint_as_float(v[i + 1]) * p.scale_log2e;
+          float s0 = prefill_score<MODE>(p, __uint_as_float(v[i])), s1 = prefill_score<MODE>(p, __uint_as_float(v[i + 1]));
           if (need_mask) {
             if (key0 + c * 32 + i > pos) s0 = kMaskVal;
             if (key0 + c * 32 + i + 1 > pos) s1 = kMaskVal;
           }
-          const float p0 = exp2f(s0 - m_used), p1 = exp2f(s1 - m_used);
+          const float p0 = MODE == SCORE_SERIES ? ex2_approx(s0) : exp2f(s0 - m_used), p1 = MODE == SCORE_SERIES ? ex2_approx(s1) : exp2f(s1 - m_used);
           sum += p0 + p1;
           pk[i >> 1] = pack_bf16(p0, p1);
         }
@@ -276,22 +305,30 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
       const float inv = 1.f / l;
       const size_t tok = (size_t)tok0 + (valid ? r : 0);
       const __nv_bfloat16* gate = p.gate_src + tok * p.ld + (size_t)head * 2 * D + D;
-      __nv_bfloat16* dst = p.out + tok * ((size_t)p.hq * D) + (size_t)head * D;
+      __nv_bfloat16* dst = p.out + tok * ((size_t)p.hq * DV) + (size_t)head * DV;
 #pragma unroll 1
-      for (int c = 0; c < D / 32; ++c) {
+      for (int c = 0; c < DV / 32; ++c) {
         uint32_t v[32];
         tmem_ld32(lane_base + 256u + c * 32, v);
         tmem_ld_wait();
         if (valid) {
 #pragma unroll
           for (int q4 = 0; q4 < 4; ++q4) {
-            const uint4 gw = *reinterpret_cast<const uint4*>(gate + c * 32 + q4 * 8);
-            const uint32_t g4[4] = {gw.x, gw.y, gw.z, gw.w};
+            float f[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(v[q4 * 8 + e]) * inv;
+            if (p.gate_src != nullptr) {
+              const uint4 gw = *reinterpret_cast<const uint4*>(gate + c * 32 + q4 * 8);
+              const uint32_t g4[4] = {gw.x, gw.y, gw.z, gw.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                f[2 * e] *= sigmoid_f(bf16lo(g4[e]));
+                f[2 * e + 1] *= sigmoid_f(bf16hi(g4[e]));
+              }
+            }
             uint32_t o4[4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e)
-              o4[e] = pack_bf16(__uint_as_float(v[q4 * 8 + 2 * e]) * inv * sigmoid_f(bf16lo(g4[e])),
-                                __uint_as_float(v[q4 * 8 + 2 * e + 1]) * inv * sigmoid_f(bf16hi(g4[e])));
+            for (int e = 0; e < 4; ++e) o4[e] = pack_bf16(f[2 * e], f[2 * e + 1]);
             *reinterpret_cast<uint4*>(dst + c * 32 + q4 * 8) = make_uint4(o4[0], o4[1], o4[2], o4[3]);
           }
         }
@@ -308,40 +345,58 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
   }
 }
 
-template <int D>
-static int launch_attn_prefill(const AttnPrefillParams& p, int num_tiles, cudaStream_t st) {
+template <int D, int DV, int MODE>
+static int launch_mode(const AttnPrefillParams& p, int num_tiles, cudaStream_t st) {
   static bool configured = false;
-  auto k = attn_prefill_kernel<D>;
+  auto k = attn_prefill_kernel<D, DV, MODE>;
   if (!configured) {
-    cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)AttnPrefillGeom<D>::kSmem);
+    cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)AttnPrefillGeom<D, DV>::kSmem);
     configured = true;
   }
-  k<<<dim3(num_tiles, p.hq), kAttnThreads, AttnPrefillGeom<D>::kSmem, st>>>(p);
+  k<<<dim3(num_tiles, p.hq), kAttnThreads, AttnPrefillGeom<D, DV>::kSmem, st>>>(p);
   return (int)cudaGetLastError();
+}
+
+template <int D, int DV>
+static int launch_attn_prefill(const AttnPrefillParams& p, int num_tiles, int mode, cudaStream_t st) {
+  if (mode == SCORE_SERIES) return launch_mode<D, DV, SCORE_SERIES>(p, num_tiles, st);
+  if (mode == SCORE_CAPPED) return launch_mode<D, DV, SCORE_CAPPED>(p, num_tiles, st);
+  if constexpr (D == DV) return launch_mode<D, DV, SCORE_PLAIN>(p, num_tiles, st);
+  return -3;
 }
 
 }  // namespace ti
 
 extern "C" {
 
-// out[tok, head*D + d] = softmax(q k^T / sqrt(D), causal by position) v * sigmoid(gate) for the tokens of the listed
-// query tiles (up to 128 consecutive tokens of one sequence each; longest first gives the best balance).
+// out[tok, head*DV + d] = softmax(score(q k^T), causal by position) v * sigmoid(gate) for the tokens of the listed query
+// tiles (up to 128 consecutive tokens of one sequence each; longest first gives the best balance).
 // q: bf16 [T, hq, D] (normalised, rotated); kcache / vcache: the paged cache of this layer, `num_blocks` pages;
-// positions: absolute position of every flat token; gate_src: the projection rows [T, ld] holding the gates.
+// positions: absolute position of every flat token; gate_src: the projection rows [T, ld] holding the gates, or null.
+// score(x) = scale x, or with softcap > 0 softcap * tanh(scale x / softcap).  `qk_max`: a bound of |q.k|, or <= 0.
 int ti_attn_prefill(const void* q, int T, const void* kcache, const void* vcache, int num_blocks, const void* block_tables,
                     const void* positions, const void* qt_seq, const void* qt_tok0, const void* qt_ntok, int num_tiles,
-                    const void* gate_src, void* out, int hq, int hkv, int max_blocks, int ld, float scale_log2e, int D,
-                    void* status, void* stream) {
+                    const void* gate_src, void* out, int hq, int hkv, int max_blocks, int ld, float scale, int D, int DV,
+                    float softcap, float qk_max, void* status, void* stream) {
   if (num_tiles <= 0) return 0;
-  if (hq % hkv || (D != 64 && D != 128 && D != 256) || T < 1 || num_blocks < 1) return -2;
+  if (hq % hkv || T < 1 || num_blocks < 1 || (gate_src != nullptr && D != DV)) return -2;
   // the gate and the output are read / written 16 bytes at a time: refuse layouts that would make those accesses misaligned
   if ((ld & 7) || (reinterpret_cast<uintptr_t>(gate_src) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return -4;
+  if ((D != 64 && D != 128 && D != 256) || (DV != 64 && DV != 128 && DV != 256)) return -3;
+  constexpr float kLog2e = 1.4426950408889634f;
   ti::AttnPrefillParams p = {};
+  int mode = ti::SCORE_PLAIN;
+  if (softcap > 0.f) {
+    p.cap_in = scale / softcap;
+    p.cap_out = softcap * kLog2e;
+    const float y = qk_max * p.cap_in;
+    mode = qk_max > 0.f && y > -ti::kSeriesMax && y < ti::kSeriesMax && (y < 0.f ? -y : y) * p.cap_out < 60.f ? ti::SCORE_SERIES : ti::SCORE_CAPPED;
+  }
   int rc = ti::bf16_map_2d(&p.map_q, q, (long long)hq * D, T, 64, 128, CU_TENSOR_MAP_SWIZZLE_128B);
   if (rc) return rc;
   rc = ti::bf16_map_groups(&p.map_k, kcache, D, (long long)num_blocks * hkv * 16, D / 64, 2);
   if (rc) return rc;
-  rc = ti::bf16_map_2d(&p.map_v, vcache, 16, (long long)num_blocks * hkv * D, 16, D, CU_TENSOR_MAP_SWIZZLE_32B);
+  rc = ti::bf16_map_2d(&p.map_v, vcache, 16, (long long)num_blocks * hkv * DV, 16, DV, CU_TENSOR_MAP_SWIZZLE_32B);
   if (rc) return rc;
   p.block_tables = (const int*)block_tables;
   p.positions = (const int*)positions;
@@ -355,11 +410,14 @@ int ti_attn_prefill(const void* q, int T, const void* kcache, const void* vcache
   p.hkv = hkv;
   p.max_blocks = max_blocks;
   p.ld = ld;
-  p.scale_log2e = scale_log2e;
+  p.scale_log2e = scale * kLog2e;
   cudaStream_t st = (cudaStream_t)stream;
-  if (D == 256) return ti::launch_attn_prefill<256>(p, num_tiles, st);
-  if (D == 128) return ti::launch_attn_prefill<128>(p, num_tiles, st);
-  return ti::launch_attn_prefill<64>(p, num_tiles, st);
+#define TI_AP(A, B) if (D == A && DV == B) return ti::launch_attn_prefill<A, B>(p, num_tiles, mode, st)
+  TI_AP(64, 64); TI_AP(64, 128); TI_AP(64, 256);
+  TI_AP(128, 64); TI_AP(128, 128); TI_AP(128, 256);
+  TI_AP(256, 64); TI_AP(256, 128); TI_AP(256, 256);
+#undef TI_AP
+  return -3;
 }
 
 }  // extern "C"

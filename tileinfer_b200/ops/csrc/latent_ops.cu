@@ -1,138 +1,12 @@
-// Row operations and small products around latent attention and an fp32 residual stream: token + position embedding
-// with a norm, plain RMSNorm of fp32 rows, the latent's norm and its store into cache pages, the per-head products that
-// absorb W_uk into the query and W_uv into the output, and the fp32 matrix product of the 32-bit mode.
+// Row operations and small products around latent attention: the latent's norm and its store into cache pages, and the
+// per-head products that absorb W_uk into the query and W_uv into the output.
 //
 // Every kernel is templated on the activation type (bf16, or float in 32-bit mode).  Row pitches are padded to
 // multiples of 64 elements and the pad columns hold zeros (zero weight rows, zero norm weights), so that rows are read
 // in whole vectors; means divide by the true length.
-#include "common.cuh"
+#include "row_vec.cuh"
 
 namespace ti {
-
-typedef __nv_bfloat16 bf16;
-
-template <typename T> TI_DEVICE void load8(const T* p, float (&v)[8]);
-template <> TI_DEVICE void load8<bf16>(const bf16* p, float (&v)[8]) {
-  const uint4 q = *reinterpret_cast<const uint4*>(p);
-  const uint32_t w[4] = {q.x, q.y, q.z, q.w};
-#pragma unroll
-  for (int i = 0; i < 4; ++i) { v[2 * i] = bf16lo(w[i]); v[2 * i + 1] = bf16hi(w[i]); }
-}
-template <> TI_DEVICE void load8<float>(const float* p, float (&v)[8]) {
-  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-template <typename T> TI_DEVICE void store8(T* p, const float (&v)[8]);
-template <> TI_DEVICE void store8<bf16>(bf16* p, const float (&v)[8]) {
-  *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
-}
-template <> TI_DEVICE void store8<float>(float* p, const float (&v)[8]) {
-  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
-}
-template <typename T> TI_DEVICE float to_f(T v);
-template <> TI_DEVICE float to_f<bf16>(bf16 v) { return __bfloat162float(v); }
-template <> TI_DEVICE float to_f<float>(float v) { return v; }
-TI_DEVICE float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
-
-TI_DEVICE float block_sum32(float v, float* red) {
-  v = warp_sum(v);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  if (lane == 0) red[warp] = v;
-  __syncthreads();
-  float t = 0.f;
-  for (int w = 0; w < nw; ++w) t += red[w];
-  return t;
-}
-
-// ---------------------------------------------------------------- embedding
-// x[m, :] = rmsnorm(embed[ids[m]] + pos[positions[m]]) * w in fp32.  Either of `pos` and `w` may be null.  Block 0 also
-// advances the device step counter.
-template <typename T>
-__global__ void __launch_bounds__(256) embed_pos_kernel(const long long* __restrict__ ids, const int* __restrict__ positions,
-                                                        const T* __restrict__ embed, const T* __restrict__ pos,
-                                                        const float* __restrict__ w, float* __restrict__ x, int W, int P,
-                                                        int vocab, int max_pos, float eps, unsigned* step) {
-  __shared__ float red[8];
-  pdl_trigger();
-  pdl_wait();
-  const int m = blockIdx.x;
-  long long id = ids[m];
-  if (id < 0 || id >= vocab) id = 0;
-  const int ps = min(max(positions[m], 0), max_pos - 1);
-  const T* e = embed + (size_t)id * P;
-  const T* q = pos == nullptr ? nullptr : pos + (size_t)ps * P;
-  float ss = 0.f;
-  for (int c = threadIdx.x * 8; c < P; c += blockDim.x * 8) {
-    float a[8], b[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    load8(e + c, a);
-    if (q != nullptr) load8(q + c, b);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) { const float v = a[i] + b[i]; ss += v * v; }
-  }
-  const float rr = w == nullptr ? 1.f : rsqrtf(block_sum32(ss, red) / (float)W + eps);
-  for (int c = threadIdx.x * 8; c < P; c += blockDim.x * 8) {
-    float a[8], b[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, g[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
-    load8(e + c, a);
-    if (q != nullptr) load8(q + c, b);
-    if (w != nullptr) load8(w + c, g);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) a[i] = (a[i] + b[i]) * rr * g[i];
-    store8(x + (size_t)m * P + c, a);
-  }
-  if (step != nullptr && m == 0 && threadIdx.x == 0) *step = *step + 1u;
-}
-
-// ---------------------------------------------------------------- RMSNorm of fp32 rows
-// y[m, :] = x[m, :] / sqrt(mean(x^2) + eps) * w.  The row is kept in registers between the two passes when it fits.
-template <typename T>
-__global__ void __launch_bounds__(256) rmsnorm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w,
-                                                          T* __restrict__ y, int W, int P, float eps) {
-  __shared__ float red[8];
-  constexpr int kKeep = 4;                                // 256 threads x 4 x 8 = 8192 columns
-  pdl_trigger();
-  pdl_wait();
-  const float* row = x + (size_t)blockIdx.x * P;
-  T* out = y + (size_t)blockIdx.x * P;
-  const int step = blockDim.x * 8;
-  float keep[kKeep][8];
-  float ss = 0.f;
-#pragma unroll
-  for (int j = 0; j < kKeep; ++j) {
-    const int c = threadIdx.x * 8 + j * step;
-    if (c < P) {
-      load8(row + c, keep[j]);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) ss += keep[j][i] * keep[j][i];
-    }
-  }
-  for (int c = threadIdx.x * 8 + kKeep * step; c < P; c += step) {
-    float v[8];
-    load8(row + c, v);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) ss += v[i] * v[i];
-  }
-  const float rr = rsqrtf(block_sum32(ss, red) / (float)W + eps);
-#pragma unroll
-  for (int j = 0; j < kKeep; ++j) {
-    const int c = threadIdx.x * 8 + j * step;
-    if (c < P) {
-      float g[8];
-      load8(w + c, g);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) g[i] *= keep[j][i] * rr;
-      store8(out + c, g);
-    }
-  }
-  for (int c = threadIdx.x * 8 + kKeep * step; c < P; c += step) {
-    float v[8], g[8];
-    load8(row + c, v);
-    load8(w + c, g);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] *= rr * g[i];
-    store8(out + c, v);
-  }
-}
 
 // ---------------------------------------------------------------- latent -> cache
 // One warp per token: c = rmsnorm(proj[t, col0 : col0 + R]) * w into the token's cache slot (pages of 16 rows of Rp
@@ -264,98 +138,9 @@ __global__ void __launch_bounds__(128) head_product_f32_kernel(const __grid_cons
   }
 }
 
-// ---------------------------------------------------------------- fp32 matrix product (32-bit mode)
-// y[M, N] = x[M, K] W[N, K]^T in plain fp32 FMAs, 64 x 64 tiles, with the epilogues of the tcgen05 product that an fp32
-// residual stream uses.  K a multiple of 16.
-struct GemmF32Params {
-  const float* w;       // [N][K]
-  const float* x;       // [M][ldx]
-  const float* resid;   // epi 4: [M][ldo]
-  float* out;           // [M][ldo]
-  float* out2;          // epi 5: [M][ldo2], column (n - n_split) / 2 for the pairs of rows from n_split on
-  int M, N, K, ldx, ldo, ldo2, n_split, epi;
-  float scale, glu_limit, glu_alpha, glu_bias;
-};
-
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ GemmF32Params p) {
-  __shared__ float xs[16][68], ws[16][68];
-  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
-  const int lr = tid >> 2, lk = (tid & 3) * 4;
-  const float* xrow = p.x + (size_t)min(m0 + lr, p.M - 1) * p.ldx;
-  const float* wrow = p.w + (size_t)min(n0 + lr, p.N - 1) * p.K;
-  pdl_trigger();
-  pdl_wait();
-  float acc[4][4] = {};
-  for (int k0 = 0; k0 < p.K; k0 += 16) {
-    const float4 a = *reinterpret_cast<const float4*>(xrow + k0 + lk), b = *reinterpret_cast<const float4*>(wrow + k0 + lk);
-    xs[lk][lr] = a.x; xs[lk + 1][lr] = a.y; xs[lk + 2][lr] = a.z; xs[lk + 3][lr] = a.w;
-    ws[lk][lr] = b.x; ws[lk + 1][lr] = b.y; ws[lk + 2][lr] = b.z; ws[lk + 3][lr] = b.w;
-    __syncthreads();
-#pragma unroll
-    for (int k = 0; k < 16; ++k) {
-      const float4 u = *reinterpret_cast<const float4*>(&xs[k][ty * 4]), v = *reinterpret_cast<const float4*>(&ws[k][tx * 4]);
-      const float xm[4] = {u.x, u.y, u.z, u.w}, wn[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xm[i], wn[j], acc[i][j]);
-    }
-    __syncthreads();
-  }
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const int m = m0 + ty * 4 + i;
-    if (m >= p.M) continue;
-#pragma unroll
-    for (int j = 0; j < 4; j += 2) {
-      const int n = n0 + tx * 4 + j;
-      if (n >= p.N) continue;
-      if (p.epi == 5 && n >= p.n_split) {               // (gate, up) pair
-        const float g = fminf(acc[i][j], p.glu_limit), u = fminf(fmaxf(acc[i][j + 1], -p.glu_limit), p.glu_limit);
-        p.out2[(size_t)m * p.ldo2 + ((n - p.n_split) >> 1)] = g * sigmoid_exact(p.glu_alpha * g) * (u + p.glu_bias);
-        continue;
-      }
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        if (n + e >= p.N) continue;
-        const size_t at = (size_t)m * p.ldo + n + e;
-        p.out[at] = p.epi == 4 ? p.resid[at] + acc[i][j + e] : acc[i][j + e] * p.scale;
-      }
-    }
-  }
-}
-
 }  // namespace ti
 
 extern "C" {
-
-// f32 selects the activation / table type: 0 bf16, 1 float.  P: row pitch (a multiple of 8), W: true width.
-int ti_embed_pos(const void* ids, const void* positions, const void* embed, const void* pos, const void* w, void* x, int M,
-                 int W, int P, int vocab, int max_pos, float eps, void* step, int f32, void* stream) {
-  if (M <= 0) return 0;
-  if (P % 8 || W > P || vocab < 1 || (pos != nullptr && max_pos < 1)) return -2;
-  cudaStream_t st = (cudaStream_t)stream;
-  if (f32)
-    ti::launch_kernel(ti::embed_pos_kernel<float>, dim3(M), dim3(256), 0, st, true, (const long long*)ids, (const int*)positions,
-                      (const float*)embed, (const float*)pos, (const float*)w, (float*)x, W, P, vocab, max_pos, eps, (unsigned*)step);
-  else
-    ti::launch_kernel(ti::embed_pos_kernel<ti::bf16>, dim3(M), dim3(256), 0, st, true, (const long long*)ids, (const int*)positions,
-                      (const ti::bf16*)embed, (const ti::bf16*)pos, (const float*)w, (float*)x, W, P, vocab, max_pos, eps, (unsigned*)step);
-  return (int)cudaGetLastError();
-}
-
-int ti_rmsnorm_f32(const void* x, const void* w, void* y, int M, int W, int P, float eps, int f32, void* stream) {
-  if (M <= 0) return 0;
-  if (P % 8 || W > P) return -2;
-  cudaStream_t st = (cudaStream_t)stream;
-  const dim3 block(P >= 2048 ? 256 : 128);
-  if (f32)
-    ti::launch_kernel(ti::rmsnorm_f32_kernel<float>, dim3(M), block, 0, st, true, (const float*)x, (const float*)w, (float*)y, W, P, eps);
-  else
-    ti::launch_kernel(ti::rmsnorm_f32_kernel<ti::bf16>, dim3(M), block, 0, st, true, (const float*)x, (const float*)w, (ti::bf16*)y, W, P, eps);
-  return (int)cudaGetLastError();
-}
 
 int ti_latent_store(const void* proj, int ld, int col0, const void* w, const void* slots, void* cache, long long num_slots,
                     int M, int R, int Rp, float eps, int f32, void* stream) {
@@ -393,16 +178,6 @@ int ti_head_product(const void* x, const void* w, const void* gate, void* out, i
   ti::HeadProductParams p = {x, w, gate, out, M, H, N, K, ldx, ldo, ldg, gcol};
   const dim3 grid(N / 64, H, (M + 15) / 16);
   ti::launch_kernel(f32 ? ti::head_product_f32_kernel : ti::head_product_bf16_kernel, grid, dim3(128), 0, (cudaStream_t)stream, true, p);
-  return (int)cudaGetLastError();
-}
-
-int ti_gemm_f32(const void* w, const void* x, const void* resid, void* out, void* out2, int M, int N, int K, int ldx, int ldo,
-                int ldo2, int n_split, int epi, float scale, float glu_limit, float glu_alpha, float glu_bias, void* stream) {
-  if (M <= 0) return 0;
-  if (K % 16 || ldx % 4 || n_split % 2 || (epi != 3 && epi != 4 && epi != 5)) return -2;
-  ti::GemmF32Params p = {(const float*)w, (const float*)x, (const float*)resid, (float*)out, (float*)out2, M, N, K, ldx, ldo,
-                         ldo2, n_split, epi, scale, glu_limit, glu_alpha, glu_bias};
-  ti::launch_kernel(ti::gemm_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64), dim3(256), 0, (cudaStream_t)stream, true, p);
   return (int)cudaGetLastError();
 }
 

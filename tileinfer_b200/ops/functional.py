@@ -64,7 +64,8 @@ class AttnParams(ctypes.Structure):
     _fields_ = [("q", _P), ("kcache", _P), ("vcache", _P), ("block_tables", _P), ("positions", _P),
                 ("qg_seq", _P), ("qg_tok0", _P), ("qg_ntok", _P), ("o_part", _P), ("ml_part", _P),
                 ("gate_src", _P), ("out", _P), ("hq", _I), ("hkv", _I), ("max_blocks", _I), ("nsplit", _I),
-                ("ld", _I), ("num_qg", _I), ("scale_log2e", _F), ("num_blocks", _I), ("status", _P)]
+                ("ld", _I), ("num_qg", _I), ("scale_log2e", _F), ("num_blocks", _I), ("status", _P), ("cap_in", _F), ("cap_out", _F),
+                ("rep", _I)]
 
 
 class LatentAttnParams(ctypes.Structure):
@@ -72,6 +73,38 @@ class LatentAttnParams(ctypes.Structure):
                 ("qg_ntok", _P), ("sink", _P), ("o_part", _P), ("ml_part", _P), ("out", _P), ("status", _P),
                 ("H", _I), ("R", _I), ("Rp", _I), ("max_blocks", _I), ("nsplit", _I), ("num_qg", _I), ("window", _I),
                 ("num_blocks", _I), ("scale", _F)]
+
+
+class RopeUnitParams(ctypes.Structure):
+    _fields_ = [("proj", _P), ("inv_freq", _P), ("positions", _P), ("slot_mapping", _P), ("q_out", _P), ("kcache", _P), ("vcache", _P),
+                ("status", _P), ("T", _I), ("ld", _I), ("q_col", _I), ("k_col", _I), ("v_col", _I), ("H", _I), ("G", _I), ("dim", _I),
+                ("dp", _I), ("vp", _I), ("half", _I), ("num_blocks", _I), ("eps", _F)]
+
+
+class AttnGeneralParams(ctypes.Structure):
+    _fields_ = [("q", _P), ("kcache", _P), ("vcache", _P), ("block_tables", _P), ("positions", _P), ("qg_seq", _P), ("qg_tok0", _P),
+                ("qg_ntok", _P), ("out", _P), ("status", _P), ("H", _I), ("G", _I), ("dp", _I), ("vp", _I), ("max_blocks", _I),
+                ("num_qg", _I), ("num_blocks", _I), ("ldo", _I), ("scale", _F), ("softcap", _F)]
+
+
+class GlaParams(ctypes.Structure):
+    _fields_ = [("proj", _P), ("a2", _P), ("a2_bias", _P), ("norm", _P), ("state", _P), ("slots", _P), ("cu", _P), ("seqs", _P),
+                ("o", _P), ("out", _P), ("snap_rel", _P), ("snap_idx", _P), ("snap", _P),
+                ("ld", _I), ("ldo", _I), ("H", _I), ("R", _I), ("q_col", _I), ("k_col", _I), ("v_col", _I), ("g_col", _I), ("a_col", _I),
+                ("num_snap", _I), ("vdim", _I), ("q_scale", _F), ("inv_tau", _F), ("eps", _F),
+                ("ck_seq", _P), ("ck_tok0", _P), ("ck_ntok", _P), ("ck_snap", _P), ("seq_ck", _P), ("g_ws", _P), ("s_ws", _P),
+                ("nc", _I), ("num_long", _I)]
+
+
+class MoeRouteParams(ctypes.Structure):
+    _fields_ = [("logits", _P), ("correction", _P), ("valid", _P), ("ids", _P), ("weight", _P), ("pos", _P), ("counts", _P),
+                ("ticket", _P), ("first", _P), ("tiles", _P), ("num_tiles", _P), ("M", _I), ("E", _I), ("identity", _I), ("top", _I),
+                ("groups", _I), ("keep", _I), ("ldl", _I), ("tile_rows", _I), ("max_tiles", _I)]
+
+
+class ResidNormParams(ctypes.Structure):
+    _fields_ = [("y", _P), ("x", _P), ("w_out", _P), ("w_next", _P), ("h", _P), ("slot", _P), ("weight", _P), ("h_in", _P),
+                ("W", _I), ("P", _I), ("ldy", _I), ("top", _I), ("eps", _F)]
 
 
 class GemmEpilogue(ctypes.Structure):
@@ -120,11 +153,26 @@ _l.register("ti_gdn_step", _I, [ctypes.POINTER(GdnParams), _I, _I, _I, _I, _I, _
 _l.register("ti_gdn_chunk_params_size", _I, [], "hybrid")
 _l.register("ti_gdn_chunk_ws_bytes", _I, [_I, _I, _I], "hybrid")
 _l.register("ti_gdn_chunked", _I, [ctypes.POINTER(GdnChunkParams), _I, _I, _I, _I, _I, _P], "hybrid")
-_l.register("ti_qkv_prep_params_size", _I, [], "hybrid")
-_l.register("ti_attn_params_size", _I, [], "hybrid")
-_l.register("ti_qkv_prep", _I, [ctypes.POINTER(QkvPrepParams), _I, _I, _P], "hybrid")
-_l.register("ti_attn_paged", _I, [ctypes.POINTER(AttnParams), _I, _P], "hybrid")
-_l.register("ti_attn_prefill", _I, [_P, _I, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _P, _P], "hybrid")
+_l.register("ti_qkv_prep_params_size", _I, [], "attention")
+_l.register("ti_attn_params_size", _I, [], "attention")
+_l.register("ti_qkv_prep", _I, [ctypes.POINTER(QkvPrepParams), _I, _I, _P], "attention")
+_l.register("ti_attn_paged", _I, [ctypes.POINTER(AttnParams), _I, _I, _P], "attention")
+_l.register("ti_attn_prefill", _I, [_P, _I, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _F, _P, _P],
+            "attention")
+_l.register("ti_rope_unit_params_size", _I, [], "attention")
+_l.register("ti_rope_unit", _I, [ctypes.POINTER(RopeUnitParams), _I, _P], "attention")
+_l.register("ti_attn_general_params_size", _I, [], "attention")
+_l.register("ti_attn_general", _I, [ctypes.POINTER(AttnGeneralParams), _I, _P], "attention")
+_l.register("ti_gla_params_size", _I, [], "gla")
+_l.register("ti_gla_step", _I, [ctypes.POINTER(GlaParams), _I, _I, _I, _I, _P], "gla")
+_l.register("ti_gla_finish", _I, [ctypes.POINTER(GlaParams), _I, _I, _I, _P], "gla")
+_l.register("ti_moe_route_params_size", _I, [], "moe")
+_l.register("ti_moe_route", _I, [ctypes.POINTER(MoeRouteParams), _P], "moe")
+_l.register("ti_moe_permute", _I, [_P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P], "moe")
+_l.register("ti_gemm_grouped_bf16", _I, [_P, _I, _I, _I, _I, _P, _I, _P, _P, _I, _I, _P, _I, _I, _P, _P, _P], "moe")
+_l.register("ti_gemm_grouped_w8a16", _I, [_P, _P, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _P, _I, _I, _P, _P, _P], "moe")
+_l.register("ti_resid_norm_params_size", _I, [], "rows")
+_l.register("ti_resid_norm", _I, [ctypes.POINTER(ResidNormParams), _I, _I, _P], "rows")
 _l.register("ti_topk_params_size", _I, [])
 _l.register("ti_topk", _I, [ctypes.POINTER(TopkParams), _P])
 _l.register("ti_topk_merge", _I, [ctypes.POINTER(TopkParams), _P])
@@ -145,28 +193,32 @@ _l.register("ti_latent_attn_params_size", _I, [], "latent")
 _l.register("ti_latent_attn_max_split_rank", _I, [], "latent")
 _l.register("ti_latent_attn", _I, [ctypes.POINTER(LatentAttnParams), _I, _P], "latent")
 _l.register("ti_latent_prefill", _I, [_P, _I, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P], "latent")
-_l.register("ti_embed_pos", _I, [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _P, _I, _P], "latent")
-_l.register("ti_rmsnorm_f32", _I, [_P, _P, _P, _I, _I, _I, _F, _I, _P], "latent")
+_l.register("ti_embed_pos", _I, [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P, _I, _P], "rows")
+_l.register("ti_rmsnorm_f32", _I, [_P, _P, _P, _I, _I, _I, _F, _I, _P], "rows")
 _l.register("ti_latent_store", _I, [_P, _I, _I, _P, _P, _P, _LL, _I, _I, _I, _F, _I, _P], "latent")
 _l.register("ti_latent_gather", _I, [_P, _P, _LL, _P, _I, _I, _I, _P], "latent")
 _l.register("ti_head_product", _I, [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P], "latent")
-_l.register("ti_gemm_f32", _I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P], "latent")
+_l.register("ti_gemm_f32", _I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P, _P, _I, _P], "rows")
 
 _PARAM_SIZES = {"base": (("ti_topk_params_size", TopkParams), ("ti_edit_params_size", EditParams),
                          ("ti_sample_params_size", SampleParams), ("ti_gemm_epilogue_size", GemmEpilogue)),
                 "latent": (("ti_latent_attn_params_size", LatentAttnParams),),
+                "rows": (("ti_resid_norm_params_size", ResidNormParams),),
+                "attention": (("ti_qkv_prep_params_size", QkvPrepParams), ("ti_attn_params_size", AttnParams),
+                              ("ti_rope_unit_params_size", RopeUnitParams), ("ti_attn_general_params_size", AttnGeneralParams)),
+                "gla": (("ti_gla_params_size", GlaParams),),
+                "moe": (("ti_moe_route_params_size", MoeRouteParams),),
                 "hybrid": (("ti_gdn_params_size", GdnParams), ("ti_gdn_chunk_params_size", GdnChunkParams),
-                           ("ti_qkv_prep_params_size", QkvPrepParams), ("ti_attn_params_size", AttnParams),
                            ("ti_ar_rows_params_size", ArRowsParams), ("ti_gemv_params_size", GemvParams),
                            ("ti_chain_params_size", ChainParams))}
 _checked = set()
 
 
 def L(*groups: str):
-    """The kernel libraries; the named groups (default: "base" and "hybrid") are loaded now, with their parameter
+    """The kernel libraries; the named groups (default: what the hybrid family uses) are loaded now, with their parameter
     blocks checked against the Python structures."""
     lib = _l.lib()
-    groups = groups or ("base", "hybrid")
+    groups = groups or ("base", "attention", "hybrid")
     if not _checked.issuperset(groups):
         _l.build_groups(*groups)
         for g in groups:
@@ -517,21 +569,25 @@ def qkv_prep(p: QkvPrepParams, T: int, D: int):
     check(_l.lib().ti_qkv_prep(ctypes.byref(p), T, D, stream()), "ti_qkv_prep")
 
 
-def attn_paged(p: AttnParams, D: int):
+def attn_paged(p: AttnParams, D: int, DV: int = None):
+    """D, DV: sizes of a query / key head and of a value head (64, 128 or 256)."""
     if not p.status:
         p.status = status_ptr()
-    check(_l.lib().ti_attn_paged(ctypes.byref(p), D, stream()), "ti_attn_paged")
+    check(_l.lib().ti_attn_paged(ctypes.byref(p), D, D if DV is None else DV, stream()), "ti_attn_paged")
 
 
 def attn_prefill(q, kcache, vcache, num_blocks, block_tables, positions, tiles, gate_src, out, *, hq, hkv, D,
-                 max_blocks, ld):
+                 max_blocks, ld, DV=None, scale=None, softcap=0.0, qk_max=0.0):
     """Causal GQA attention of prefill query tiles on the tcgen05 tensor cores (ops/csrc/attn_prefill.cu).
-    `tiles`: int32 [3, n] = (sequence, first flat token, tokens <= 128) per tile, longest KV first."""
+    `tiles`: int32 [3, n] = (sequence, first flat token, tokens <= 128) per tile, longest KV first.  DV: size of a value
+    head (default D); softcap: scores become softcap * tanh(scale q.k / softcap); qk_max: a bound of |q.k| where there is
+    one (it selects a cheaper softmax); gate_src None: no output gate."""
     n = tiles.shape[1]
-    scale = D ** -0.5 * 1.4426950408889634
+    scale = D ** -0.5 if scale is None else scale
     check(_l.lib().ti_attn_prefill(ptr(q), q.shape[0], ptr(kcache), ptr(vcache), num_blocks, ptr(block_tables), ptr(positions),
                               ptr(tiles[0]), ptr(tiles[1]), ptr(tiles[2]), n, ptr(gate_src), ptr(out), hq, hkv,
-                              max_blocks, ld, scale, D, status_ptr(), stream()), "ti_attn_prefill")
+                              max_blocks, ld, scale, D, D if DV is None else DV, softcap, qk_max, status_ptr(), stream()),
+          "ti_attn_prefill")
 
 
 AR_NONE, AR_LIMBS, AR_BF16 = 0, 1, 2
@@ -659,10 +715,10 @@ def _f32(t) -> int:
     return int(t.dtype == torch.float32)
 
 
-def embed_pos(ids, positions, embed, pos, norm_w, x, W, eps, step_ptr=0):
-    """x[m] (fp32) = rmsnorm(embed[ids[m]] + pos[positions[m]]) * norm_w; `pos` and `norm_w` may be None."""
+def embed_pos(ids, positions, embed, pos, norm_w, x, W, eps, step_ptr=0, scale=1.0):
+    """x[m] (fp32) = rmsnorm(embed[ids[m]] + pos[positions[m]]) * norm_w * scale; `pos` and `norm_w` (no norm) may be None."""
     check(_l.lib().ti_embed_pos(ptr(ids), ptr(positions), ptr(embed), ptr(pos), ptr(norm_w), ptr(x), x.shape[0], W, x.stride(0),
-                                embed.shape[0], 0 if pos is None else pos.shape[0], eps, step_ptr, _f32(embed), stream()), "ti_embed_pos")
+                                embed.shape[0], 0 if pos is None else pos.shape[0], eps, scale, step_ptr, _f32(embed), stream()), "ti_embed_pos")
 
 
 def rmsnorm_f32(x, norm_w, y, W, eps):
@@ -725,9 +781,101 @@ def latent_prefill(q, kv, tiles, out, *, H, dp, vp, window, scale, sink=None, ga
                                      H, dp, vp, H * dp, window, scale, status or status_ptr(), stream()), "ti_latent_prefill")
 
 
-def gemm_f32(w, x, *, out, epi=GEPI_F32, ex=None):
-    """y = x W^T in fp32 FMAs (w [N, K] row-major) with the GEPI_F32 / GEPI_RESID32 / GEPI_SPLIT_GLU epilogues."""
+def gemm_f32(w, x, *, out, epi=GEPI_F32, ex=None, groups=None):
+    """y = x W^T in fp32 FMAs (w [N, K] row-major) with the GEPI_F32 / GEPI_RESID32 / GEPI_SPLIT_GLU epilogues.  With
+    `groups` w is [E, N, K] and the rows of x meet the matrices of the token tiles (of at most 64 rows)."""
     e = ex if ex is not None else gemm_epilogue()
-    N, K = w.shape
-    check(_l.lib().ti_gemm_f32(ptr(w), ptr(x), e.resid32, ptr(out), e.out2, x.shape[0], N, K, x.stride(0), out.stride(0), e.ldo2,
-                               e.n_split, epi, e.scale, e.glu_limit, e.glu_alpha, e.glu_bias, stream()), "ti_gemm_f32")
+    N, K = w.shape[-2:]
+    check(_l.lib().ti_gemm_f32(ptr(w), ptr(x), e.resid32, ptr(out), e.out2, x.shape[0], N, K, x.stride(0), 0 if out is None else out.stride(0), e.ldo2,
+                               e.n_split, epi, e.scale, e.glu_limit, e.glu_alpha, e.glu_bias,
+                               *((0, 0, 0) if groups is None else (ptr(groups.tiles), ptr(groups.num_tiles), groups.tiles.shape[1])),
+                               stream()), "ti_gemm_f32")
+
+
+def resid_norm(y, x, w_out, h, w_next, W, eps, routed=None):
+    """x += rmsnorm(y) * w_out (fp32 rows), then h = rmsnorm(x) * w_next unless w_next is None.  With `routed` (a
+    TokenGroups after `moe_permute`) y holds the experts' rows and h the input of the identity experts."""
+    p = ResidNormParams()
+    p.y, p.x, p.w_out, p.w_next, p.h = ptr(y), ptr(x), ptr(w_out), ptr(w_next), ptr(h)
+    if routed is not None:
+        p.slot, p.weight, p.h_in, p.top = ptr(routed.slot), ptr(routed.weight), ptr(h), routed.top
+    p.W, p.P, p.ldy, p.eps = W, x.stride(0), y.stride(0), eps
+    check(_l.lib().ti_resid_norm(ctypes.byref(p), x.shape[0], _f32(y), stream()), "ti_resid_norm")
+
+
+# ------------------------------------------------------------------------------------ rotated unit heads, plain attention
+def rope_unit(p: RopeUnitParams, f32: bool):
+    if not p.status:
+        p.status = status_ptr()
+    check(_l.lib().ti_rope_unit(ctypes.byref(p), int(f32), stream()), "ti_rope_unit")
+
+
+def attn_general(p: AttnGeneralParams, f32: bool):
+    if not p.status:
+        p.status = status_ptr()
+    check(_l.lib().ti_attn_general(ctypes.byref(p), int(f32), stream()), "ti_attn_general")
+
+
+# ------------------------------------------------------------------------------------ gated linear attention
+GLA_KEY_SIZES = (64, 128, 192, 256, 384, 512)     # key sizes the kernels are built for
+
+
+def gla_step(p: GlaParams, num_seqs: int, dk: int, dv: int, f32: bool):
+    check(_l.lib().ti_gla_step(ctypes.byref(p), num_seqs, dk, dv, int(f32), stream()), "ti_gla_step")
+
+
+def gla_finish(p: GlaParams, T: int, dv: int, f32: bool):
+    check(_l.lib().ti_gla_finish(ctypes.byref(p), T, dv, int(f32), stream()), "ti_gla_finish")
+
+
+# ------------------------------------------------------------------------------------ experts
+class TokenGroups:
+    """Routing of up to T tokens to `top` of E experts: chosen experts, weights, rows, and the table of token tiles the
+    grouped products run on.  `counters` (see `moe_counters`) may be shared by everything on one stream."""
+
+    def __init__(self, T: int, E: int, choices: int, top: int, counters, f32: bool, device):
+        self.T, self.E, self.choices, self.top, self.counters, self.rows = T, E, choices, top, counters, T * top
+        mean = T * top / choices                           # rows of an expert
+        self.tile = 64 if f32 else 32 if mean <= 24 else 64 if mean <= 96 else 128
+        n = T * top // self.tile + min(E, T * top)
+        self.buf = torch.zeros(4, T * top, dtype=torch.int32, device=device)
+        self.ids, self.pos, self.slot = self.buf[0], self.buf[1], self.buf[2]
+        self.weight = self.buf[3].view(torch.float32)
+        self.tiles = torch.zeros(3, n, dtype=torch.int32, device=device)
+        self.num_tiles = torch.zeros(1, dtype=torch.int32, device=device)
+        self.first = torch.zeros(E, dtype=torch.int32, device=device)
+
+
+def moe_counters(max_experts: int, device):
+    """Arrival counters of the routing kernel, zero between launches."""
+    return torch.zeros(max_experts + 1, dtype=torch.int32, device=device)
+
+
+def moe_route(g: TokenGroups, logits, correction, groups: int, keep: int, valid=None):
+    """Chooses the experts of every row of `logits` [T, >= choices] (fp32) and lays out the token tiles."""
+    p = MoeRouteParams()
+    p.logits, p.correction, p.valid, p.ids, p.weight, p.pos = ptr(logits), ptr(correction), ptr(valid), ptr(g.ids), ptr(g.weight), ptr(g.pos)
+    p.counts, p.ticket, p.first, p.tiles, p.num_tiles = ptr(g.counters) + 4, ptr(g.counters), ptr(g.first), ptr(g.tiles), ptr(g.num_tiles)
+    p.M, p.E, p.identity, p.top, p.groups, p.keep, p.ldl = g.T, g.E, g.choices - g.E, g.top, groups, keep, logits.stride(0)
+    p.tile_rows, p.max_tiles = g.tile, g.tiles.shape[1]
+    check(_l.lib().ti_moe_route(ctypes.byref(p), stream()), "ti_moe_route")
+
+
+def moe_permute(g: TokenGroups, h, xs):
+    """Rows of h [T, P] to their places in xs [T * top, P]."""
+    check(_l.lib().ti_moe_permute(ptr(h), g.T, h.stride(0), ptr(g.ids), ptr(g.pos), ptr(g.first), ptr(g.slot), ptr(xs), g.E, g.top,
+                                  xs.shape[0], _f32(h), stream()), "ti_moe_permute")
+
+
+def gemm_grouped(W: "LinearW", E: int, x, g: TokenGroups, *, out, epi=GEPI_STORE, ex=None):
+    """y[r] = x[r] W_e^T for the rows of every token tile; W holds the E matrices one after the other.  x: bf16 rows, or
+    their limb planes for int8 matrices."""
+    N, nt, tab = W.N // E, W.n_tiles // E, (ptr(g.tiles), ptr(g.num_tiles), g.tiles.shape[1], g.tile)
+    assert W.N == N * E and N % 8 == 0
+    ldo = 0 if out is None else out.stride(0)
+    if W.wt == W_BF16:
+        check(_l.lib().ti_gemm_grouped_bf16(ptr(W.tiles), E, nt, N, W.K, ptr(x), x.shape[0], *tab, ptr(out), ldo, epi, status_ptr(),
+                                            _ref(ex), stream()), "ti_gemm_grouped_bf16")
+    else:
+        check(_l.lib().ti_gemm_grouped_w8a16(ptr(W.tiles), ptr(W.scale), E, nt, N, W.K, ptr(x.hi), ptr(x.lo), ptr(x.scale), x.M, *tab,
+                                             ptr(out), ldo, epi, status_ptr(), _ref(ex), stream()), "ti_gemm_grouped_w8a16")
