@@ -63,7 +63,9 @@ class B200GatedModel(DeviceRuntime):
         self.PREFILL_ATTN_MIN_TOKENS = 16 if tiled else 1 << 30
         self._group_tokens = 2 if tiled and all(L.heads // (L.G * L.rep) * 2 <= 16 for L in attn) else 1
         # sequences with at least this many tokens in a step run the recurrence in chunks
-        self.gla_chunk_min_tokens = 1 << 30
+        chunked = not self.f32 and all(F.gla_chunk_size(self.layers[i].dp) for i in cfg.gla_layers)
+        self.gla_chunk_min_tokens = 32 if chunked else 1 << 30
+        self.gla_ws = F.GlaWorkspace(self.dev)
         self.counters = F.moe_counters(max((L.mlp.experts for L in cfg.layers if L.mlp is not None), default=1), self.dev)
         self.block_size, self.cache, self.state = PAGE, {}, {}
         self.graphs, self.snapshots, self.host_steps = {}, {}, 0
@@ -246,7 +248,7 @@ class B200GatedModel(DeviceRuntime):
                 key = (L.moe.experts, L.moe.choices, L.moe.top)
                 if key not in x.groups:
                     x.groups[key] = F.TokenGroups(T, *key, self.counters, self.f32, dev)
-        x.long, x.short, x.ck, x.snaps = 0, None, None, []
+        x.snaps, x.chunks, x.short = [], {}, None          # chunks: chunk size -> (table, ranges); short: the other sequences
         return x
 
     def _prepare_step(self, x: StepCtx, batch):
@@ -266,6 +268,15 @@ class B200GatedModel(DeviceRuntime):
             x.snap_rel, x.snap_idx, x.num_snap = rel.to(self.dev), idx.to(self.dev), ns
             x.snap_state = {i: torch.empty(len(x.snaps), *self.state[i].shape[1:], dtype=torch.float32, device=self.dev)
                             for i in self.cfg.gla_layers}
+        lens = [b - a for a, b in zip(batch.cu_seqlens[:-1], batch.cu_seqlens[1:])]
+        longs = [s for s in range(S) if lens[s] >= self.gla_chunk_min_tokens]
+        if longs:
+            up = lambda v: torch.tensor(v, dtype=torch.int32).to(self.dev, non_blocking=True)
+            x.short, x.longs = up([s for s in range(S) if lens[s] < self.gla_chunk_min_tokens]), up(longs)
+            entries = [{int(r): int(e) for r, e in zip(rel[s, :len(points[s])], idx[s])} for s in range(S)]
+            for n in {F.gla_chunk_size(self.layers[i].dp) for i in self.cfg.gla_layers}:
+                ck, rng = F.gla_chunk_table(batch.cu_seqlens, longs, n, entries)
+                x.chunks[n] = (ck.to(self.dev, non_blocking=True), rng.to(self.dev, non_blocking=True))
 
     def _finish_step(self, x: StepCtx):
         for k, key in enumerate(x.snaps):                  # snapshots stay on the device
@@ -317,9 +328,19 @@ class B200GatedModel(DeviceRuntime):
 
     def _gla(self, i: int, L, x: StepCtx, proj, mix):
         p = self._gla_params(i, L, x, proj, mix)
-        F.gla_step(p, x.S, L.dp, L.vp, self.f32)
+        if x.short is not None:
+            ck, rng = x.chunks[F.gla_chunk_size(L.dp)]
+            p.ck_seq, p.ck_tok0, p.ck_ntok, p.ck_snap = (ptr(r) for r in ck)
+            p.long_seq, p.long_ck, p.nc, p.num_long = ptr(x.longs), ptr(rng), ck.shape[1], x.longs.numel()
+            p.g_ws, p.s_ws = (ptr(w) for w in self.gla_ws.get(p.nc, L.heads, L.dp, L.vp))
+            F.gla_chunked(p, L.dp, L.vp)
+            p.seqs = ptr(x.short)
+            self._launches += 3
+        num = x.S if x.short is None else x.short.numel()
+        if num:
+            F.gla_step(p, num, L.dp, L.vp, self.f32)
         F.gla_finish(p, x.T, L.vp, self.f32)
-        self._launches += 2
+        self._launches += 1 + bool(num)
 
     def _experts(self, L, x: StepCtx):
         """Routed experts of x.h; returns (their rows, the groups that say which rows a token sums up)."""

@@ -105,9 +105,7 @@ static int launch_step(const GlaParams& p, int S, int DK, int dv, cudaStream_t s
   switch (DK) {
     case 64: launch_kernel(gla_step_kernel<T, 4>, grid, dim3(256), 0, st, true, p); break;
     case 128: launch_kernel(gla_step_kernel<T, 8>, grid, dim3(256), 0, st, true, p); break;
-    case 192: launch_kernel(gla_step_kernel<T, 12>, grid, dim3(256), 0, st, true, p); break;
     case 256: launch_kernel(gla_step_kernel<T, 16>, grid, dim3(256), 0, st, true, p); break;
-    case 384: launch_kernel(gla_step_kernel<T, 24>, grid, dim3(256), 0, st, true, p); break;
     case 512: launch_kernel(gla_step_kernel<T, 32>, grid, dim3(256), 0, st, true, p); break;
     default: return -3;
   }

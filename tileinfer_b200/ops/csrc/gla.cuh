@@ -25,8 +25,9 @@ struct GlaParams {
   const int* ck_tok0;      // [nc] first flat token
   const int* ck_ntok;      // [nc]
   const int* ck_snap;      // [nc] entry of `snap` written after the chunk, or -1
-  const int* seq_ck;       // [2][num_long] sequence and first chunk of those that run in chunks, + [1] nc
-  float* g_ws;             // [nc][H][C][dk] running log decay inside the chunk
+  const int* long_seq;     // [num_long] sequences that run in chunks
+  const int* long_ck;      // [num_long + 1] their chunk ranges
+  float* g_ws;             // [nc][H][C][dk] running log2 decay inside the chunk
   float* s_ws;             // [nc][H][dk][dv] what the chunk adds to the state, then the state before it
   int nc, num_long;
 };

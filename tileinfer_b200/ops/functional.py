@@ -92,8 +92,8 @@ class GlaParams(ctypes.Structure):
                 ("o", _P), ("out", _P), ("snap_rel", _P), ("snap_idx", _P), ("snap", _P),
                 ("ld", _I), ("ldo", _I), ("H", _I), ("R", _I), ("q_col", _I), ("k_col", _I), ("v_col", _I), ("g_col", _I), ("a_col", _I),
                 ("num_snap", _I), ("vdim", _I), ("q_scale", _F), ("inv_tau", _F), ("eps", _F),
-                ("ck_seq", _P), ("ck_tok0", _P), ("ck_ntok", _P), ("ck_snap", _P), ("seq_ck", _P), ("g_ws", _P), ("s_ws", _P),
-                ("nc", _I), ("num_long", _I)]
+                ("ck_seq", _P), ("ck_tok0", _P), ("ck_ntok", _P), ("ck_snap", _P), ("long_seq", _P), ("long_ck", _P), ("g_ws", _P),
+                ("s_ws", _P), ("nc", _I), ("num_long", _I)]
 
 
 class MoeRouteParams(ctypes.Structure):
@@ -165,6 +165,8 @@ _l.register("ti_attn_general_params_size", _I, [], "attention")
 _l.register("ti_attn_general", _I, [ctypes.POINTER(AttnGeneralParams), _I, _P], "attention")
 _l.register("ti_gla_params_size", _I, [], "gla")
 _l.register("ti_gla_step", _I, [ctypes.POINTER(GlaParams), _I, _I, _I, _I, _P], "gla")
+_l.register("ti_gla_chunk_size", _I, [_I], "gla")
+_l.register("ti_gla_chunked", _I, [ctypes.POINTER(GlaParams), _I, _I, _P], "gla")
 _l.register("ti_gla_finish", _I, [ctypes.POINTER(GlaParams), _I, _I, _I, _P], "gla")
 _l.register("ti_moe_route_params_size", _I, [], "moe")
 _l.register("ti_moe_route", _I, [ctypes.POINTER(MoeRouteParams), _P], "moe")
@@ -817,11 +819,53 @@ def attn_general(p: AttnGeneralParams, f32: bool):
 
 
 # ------------------------------------------------------------------------------------ gated linear attention
-GLA_KEY_SIZES = (64, 128, 192, 256, 384, 512)     # key sizes the kernels are built for
+GLA_KEY_SIZES = (64, 128, 256, 512)     # key sizes the kernels are built for
 
 
 def gla_step(p: GlaParams, num_seqs: int, dk: int, dv: int, f32: bool):
     check(_l.lib().ti_gla_step(ctypes.byref(p), num_seqs, dk, dv, int(f32), stream()), "ti_gla_step")
+
+
+def gla_chunk_size(dk: int) -> int:
+    """Tokens of a chunk for this key size (0: no chunked form)."""
+    return _l.lib().ti_gla_chunk_size(dk)
+
+
+def gla_chunk_table(cu_seqlens, seqs, chunk: int, snapshot_points=None):
+    """Chunks of the listed sequences: every one is cut after `chunk` tokens, and where a state snapshot is wanted
+    (`snapshot_points[s]`: {tokens into the step: entry of the snapshot buffers}).  Returns int32 tensors (ck [4, nc] =
+    sequence | first flat token | tokens | snapshot entry or -1, rng [num_long + 1] = chunk range of every listed sequence)."""
+    rows, rng = [], [0]
+    for s in seqs:
+        t0, n = cu_seqlens[s], cu_seqlens[s + 1] - cu_seqlens[s]
+        pts = snapshot_points[s] if snapshot_points else {}
+        a = 0
+        while a < n:
+            b = min([a + chunk, n] + [x for x in pts if a < x])
+            rows.append((s, t0 + a, b - a, pts.get(b, -1)))
+            a = b
+        rng.append(len(rows))
+    return torch.tensor(rows, dtype=torch.int32).t().contiguous(), torch.tensor(rng, dtype=torch.int32)
+
+
+class GlaWorkspace:
+    """Running decays and chunk states of the chunked form; grows on demand."""
+
+    def __init__(self, device):
+        self.device, self.g, self.s = device, None, None
+
+    def get(self, nc: int, H: int, dk: int, dv: int):
+        ng, ns = nc * H * gla_chunk_size(dk) * dk, nc * H * dk * dv
+        if self.g is None or self.g.numel() < ng:
+            self.g = torch.empty(ng, dtype=torch.float32, device=self.device)
+        if self.s is None or self.s.numel() < ns:
+            self.s = torch.empty(ns, dtype=torch.float32, device=self.device)
+        return self.g, self.s
+
+
+def gla_chunked(p: GlaParams, dk: int, dv: int):
+    """Outputs and states of the sequences with chunks (bf16 projections); three kernels."""
+    check(_l.lib().ti_gla_chunked(ctypes.byref(p), dk, dv, stream()), "ti_gla_chunked")
 
 
 def gla_finish(p: GlaParams, T: int, dv: int, f32: bool):
