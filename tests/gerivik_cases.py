@@ -6,6 +6,7 @@ import gerivik_oracle as oracle
 from kabadra_cases import cut, engine, replay, rms_error, tokens  # noqa: F401  (engine and schedule helpers)
 
 
+
 def moe(experts, top, ff, limit, identity=0, count=1, keep=1):
     return {"kind": "moe", "expert": {"ff": ff, "limit": limit},
             "router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": count, "keep": keep}}}
@@ -77,3 +78,22 @@ def quantised(weights):
             w = (w / s).round().clamp(-128, 127) * s
         out[n] = w
     return out
+
+
+def errors(got, want):
+    """Error of every position: root mean square of the difference (mean over the vocabulary taken off) over that of the
+    wanted logits."""
+    d, w = got.float() - want.float(), want.float() - want.float().mean(-1, keepdim=True)
+    return (d - d.mean(-1, keepdim=True)).pow(2).mean(-1).sqrt() / w.pow(2).mean().sqrt()
+
+
+def assert_close(got, want, quant):
+    """32-bit: every position to 1e-4.  16-bit: about a hundredth at most positions; where a head's output nearly cancels
+    its norm scales the rounding up again, so single positions may be several times worse (a bf16 run of the same equations
+    shows the same)."""
+    e = errors(got, want)
+    if quant == "fp32":
+        assert e.max() < 1e-4, float(e.max())
+    else:
+        q = [float(e.quantile(x)) for x in (0.5, 0.9, 1.0)]
+        assert q[0] < 0.02 and q[1] < 0.04 and q[2] < 0.15, q
