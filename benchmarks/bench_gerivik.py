@@ -111,12 +111,16 @@ def kernel_rows(cfg, tag, lens, ctxs, prompt, ctx):
     n = -(-f.choices // 8) * 8
     logits = x.logits[:T * n].view(T, n)
     xs, act = x.xs[:g.rows * m.Wp].view(g.rows, m.Wp), x.act[:g.rows * L.ff].view(g.rows, L.ff)
-    small(lambda: L.router(x.h, logits, F.GEPI_F32))
-    row("router product", small(lambda: L.router(x.h, logits, F.GEPI_F32)), **gemm(f.choices, W, 4))
-    row("routing", small(lambda: F.moe_route(g, logits, L.correction, f.groups, f.keep)), nbytes=T * (4 * f.choices + 12 * f.top))
+    if g.row_stride:
+        row("norm + residual + next norm + router + routing + rows to experts", small(lambda: m._norm_and_route(L, x)),
+            nbytes=12 * W * T + 2 * W * (f.choices + T * f.top), like="rmsnorm")
+    else:
+        row("router product", small(lambda: L.router(x.h, logits, F.GEPI_F32)), **gemm(f.choices, W, 4))
+        row("routing", small(lambda: F.moe_route(g, logits, L.correction, f.groups, f.keep)), nbytes=T * (4 * f.choices + 12 * f.top))
+        row("token rows to experts", small(lambda: F.moe_permute(g, x.h, xs)), nbytes=2 * W * T * (1 + f.top), like="rmsnorm")
+        row("norm + residual + next norm", small(lambda: F.resid_norm(x.y, x.x, L.norm1b, x.h, L.norm2, W, 1e-6)), nbytes=12 * W * T, like="rmsnorm")
     live = int((g.ids < f.experts).sum())
     used = int(torch.unique(g.ids[g.ids < f.experts]).numel())
-    row("token rows to experts", small(lambda: F.moe_permute(g, x.h, xs)), nbytes=2 * W * (T + live), like="rmsnorm")
     ex = F.gemm_epilogue(out2=act, n_split=0, glu=(f.limit, 1.702, 1.0))
     row(f"experts gate/up + gated unit ({used} experts, {live} rows)", timed(lambda: L.w_up(xs, g, None, F.GEPI_SPLIT_GLU, ex)), flops=4 * live * W * L.ff,
         nbytes=2 * (used * 2 * L.ff * W + live * (W + L.ff)), like="gate_up")
@@ -124,7 +128,6 @@ def kernel_rows(cfg, tag, lens, ctxs, prompt, ctx):
     row("experts down", timed(lambda: L.w_down(act, g, ye, F.GEPI_STORE)), flops=2 * live * W * L.ff, nbytes=2 * (used * L.ff * W + live * (W + L.ff)), like="down")
     row("experts' sum + norm + residual + next norm", small(lambda: F.resid_norm(ye, x.x, L.norm2b, x.h, L.norm1, W, 1e-6, routed=g)),
         nbytes=2 * W * (live + 2 * T) + 8 * W * T, like="rmsnorm")
-    row("norm + residual + next norm", small(lambda: F.resid_norm(x.y, x.x, L.norm1b, x.h, L.norm2, W, 1e-6)), nbytes=12 * W * T, like="rmsnorm")
     nw = rnd(W)
     row("rmsnorm (other model)", small(lambda: F.rmsnorm(hb, nw, 1e-6, out=x.h)), nbytes=4 * T * W)
     # ---- gated linear attention

@@ -389,6 +389,33 @@ def test_routing_and_permutation(F, T, E, identity, top, count, keep):
         assert expert == dict(used)
 
 
+@pytest.mark.parametrize("dtype", [BF16, F32])
+@pytest.mark.parametrize("T,W,E,identity,top,count,keep", [(1, 40, 1, 0, 1, 1, 1), (5, 320, 6, 2, 3, 4, 2), (64, 1500, 70, 10, 9, 8, 3), (3, 8192, 30, 2, 4, 1, 1)])
+def test_norm_and_routing_in_one_kernel(F, dtype, T, W, E, identity, top, count, keep):
+    """The same residual, row, choice and placed rows as the four kernels it stands for."""
+    torch.manual_seed(W)
+    P, n = pad64(W), E + identity
+    y, x = _rows(torch.randn(T, W, device="cuda").to(dtype), P), _rows(torch.randn(T, W, device="cuda") * 3, P)
+    a, b = (_rows(torch.rand(W, device="cuda") + 0.5, P) for _ in range(2))
+    router = _rows((torch.randn(n, W, device="cuda") / math.sqrt(W)).to(dtype), P)
+    corr, ctr = -1.0 - torch.rand(n, device="cuda"), F.moe_counters(E, "cuda")
+    x2, h, h2 = x.clone(), torch.zeros(T, P, dtype=dtype, device="cuda"), torch.zeros(T, P, dtype=dtype, device="cuda")
+    F.resid_norm(y, x, a, h, b, W, 1e-4)
+    g = F.TokenGroups(T, E, n, top, ctr, False, "cuda", fixed=True)
+    xs = torch.zeros(g.rows, P, dtype=dtype, device="cuda")
+    F.moe_norm_route(y, x2, a, h2, b, W, 1e-4, g, router, corr, count, keep, xs)
+    assert rel(x2, x) < 1e-6 and rel(h2, h) < 1e-3 and not ctr.any()               # sums in another order
+    logits = (h2.double() @ router.double().t()).float().cpu()
+    want, weight = oracle.route(logits, torch.eye(n), corr.cpu(), {"experts": E, "identity": identity, "top": top, "groups": {"count": count, "keep": keep}})
+    assert torch.equal(g.ids.view(T, top).cpu(), want.int())
+    torch.testing.assert_close(g.weight.view(T, top).cpu(), weight, rtol=1e-4, atol=1e-7)
+    rows = [(e, r) for e, r0, k in g.tiles[:, :int(g.num_tiles)].t().tolist() for r in range(r0, r0 + k)]
+    slot = g.slot.view(T, top).cpu()
+    placed = [(int(want[t, k]), int(slot[t, k])) for t in range(T) for k in range(top) if want[t, k] < E]
+    assert sorted(rows) == sorted(placed) and bool((slot[want >= E] == -1).all())
+    assert all(torch.equal(xs[slot[t, k]], h2[t]) for t in range(T) for k in range(top) if want[t, k] < E)
+
+
 @pytest.mark.parametrize("quant", ["bf16", "w8a16", "fp32"])
 @pytest.mark.parametrize("T,E,top,W,ff", [(1, 5, 2, 64, 64), (40, 7, 3, 192, 128), (333, 4, 2, 128, 320), (700, 3, 2, 320, 64), (3000, 2, 2, 64, 192)])
 def test_grouped_products(F, quant, T, E, top, W, ff):

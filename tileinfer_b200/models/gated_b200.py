@@ -4,9 +4,8 @@ Per layer a decode step launches
 
   input product -> attention: rotation + unit heads + cache store -> paged attention with capped scores (+ merge)
                    gated linear attention: state step -> head norm + silu gate
-  -> output product -> [norm, residual add, next norm]
-  -> router product -> routing -> token rows to their experts -> gate/up product [clamped gated unit in the epilogue]
-  -> down product -> [weighted sum of the experts, norm, residual add, next layer's norm]
+  -> output product -> [norm, residual add, next norm, router product, routing, token rows to their experts]
+  -> gate/up product [clamped gated unit in the epilogue] -> down product -> [weighted sum of the experts, norm, residual add, next layer's norm]
 
 A layer that reuses another one's tensors shares its weights object and has a cache or state of its own.  Long portions of
 prompts run the tcgen05 attention over the paged cache and the chunked form of the recurrence.  Head sizes are padded with
@@ -122,9 +121,12 @@ class B200GatedModel(DeviceRuntime):
         L.moe = None
         if spec.mlp is not None:
             f, L.ff = spec.mlp, pad64(spec.mlp.ff)
+            if f.choices > 1024:
+                raise ValueError(f"the router takes at most 1024 experts, got {f.choices}")
             L.moe = f
             L.norm2, L.norm2b = self._norm(get(p + "norm2"), Wp), self._norm(get(p + "norm2b"), Wp)
-            L.router = Product(pad_to(get(p + "mlp.router"), f.choices, Wp), "fp32" if self.f32 else "bf16", dev)
+            router = pad_to(get(p + "mlp.router"), f.choices, Wp)
+            L.router, L.router_rows = Product(router, "fp32" if self.f32 else "bf16", dev), router.to(self.dtype).contiguous()
             L.correction = get(p + "mlp.correction").float().contiguous()
             up, down = [], []
             for e in range(f.experts):
@@ -240,14 +242,16 @@ class B200GatedModel(DeviceRuntime):
             x.o = new(T * max(L.n_mix for L in gla), dtype=torch.float32, device=dev)
         x.groups, moe = {}, [L for L in Ls if L.moe is not None]
         if moe:
-            rows = T * max(L.moe.top for L in moe)
-            x.logits = new(T * max(-(-L.moe.choices // 8) * 8 for L in moe), dtype=torch.float32, device=dev)
-            x.xs = new(rows * self.Wp, dtype=dt, device=dev)          # token rows by expert, then the experts' outputs
-            x.act = new(rows * max(L.ff for L in moe), dtype=dt, device=dev)
+            few = T <= self.FEW_TOKENS and self.Wp <= F.NORM_ROUTE_MAX_WIDTH
             for L in moe:
                 key = (L.moe.experts, L.moe.choices, L.moe.top)
                 if key not in x.groups:
-                    x.groups[key] = F.TokenGroups(T, *key, self.counters, self.f32, dev)
+                    fixed = few and L.moe.experts * T * self.Wp <= 1 << 26
+                    x.groups[key] = F.TokenGroups(T, *key, self.counters, self.f32, dev, fixed)
+            rows = max(g.rows for g in x.groups.values())
+            x.logits = new(T * max(-(-L.moe.choices // 8) * 8 for L in moe), dtype=torch.float32, device=dev)
+            x.xs = new(rows * self.Wp, dtype=dt, device=dev)          # token rows by expert, then the experts' outputs
+            x.act = new(rows * max(L.ff for L in moe), dtype=dt, device=dev)
         x.snaps, x.chunks, x.short = [], {}, None          # chunks: chunk size -> (table, ranges); short: the other sequences
         return x
 
@@ -342,20 +346,31 @@ class B200GatedModel(DeviceRuntime):
         F.gla_finish(p, x.T, L.vp, self.f32)
         self._launches += 1 + bool(num)
 
-    def _experts(self, L, x: StepCtx):
-        """Routed experts of x.h; returns (their rows, the groups that say which rows a token sums up)."""
-        f, T, Wp = L.moe, x.T, self.Wp
+    FEW_TOKENS = 128                 # up to this many tokens the norm kernel routes the rows it makes
+
+    def _norm_and_route(self, L, x: StepCtx):
+        """The mixer's output into the residual, the experts' input x.h, its routing and its rows by expert."""
+        f, T, c, Wp = L.moe, x.T, self.cfg, self.Wp
         g = x.groups[(f.experts, f.choices, f.top)]
-        n = -(-f.choices // 8) * 8
-        logits = x.logits[:T * n].view(T, n)
-        k = L.router(x.h, logits, F.GEPI_F32)
-        F.moe_route(g, logits, L.correction, f.groups, f.keep, valid=x.slot_mapping)
-        xs, act = x.xs[:g.rows * Wp].view(g.rows, Wp), x.act[:g.rows * L.ff].view(g.rows, L.ff)
-        F.moe_permute(g, x.h, xs)
-        k += L.w_up(xs, g, None, F.GEPI_SPLIT_GLU, F.gemm_epilogue(out2=act, n_split=0, glu=(f.limit, GLU_ALPHA, GLU_BIAS)))
-        k += L.w_down(act, g, xs, F.GEPI_STORE)            # the token rows have been read: their buffer takes the outputs
-        self._launches += k + 2
-        return xs, g
+        xs = x.xs[:g.rows * Wp].view(g.rows, Wp)
+        if g.row_stride:
+            F.moe_norm_route(x.y, x.x, L.norm1b, x.h, L.norm2, self.W, c.rms_eps, g, L.router_rows, L.correction, f.groups, f.keep, xs,
+                             valid=x.slot_mapping)
+            self._launches += 1
+        else:
+            F.resid_norm(x.y, x.x, L.norm1b, x.h, L.norm2, self.W, c.rms_eps)
+            n = -(-f.choices // 8) * 8
+            logits = x.logits[:T * n].view(T, n)
+            self._launches += 3 + L.router(x.h, logits, F.GEPI_F32)
+            F.moe_route(g, logits, L.correction, f.groups, f.keep, valid=x.slot_mapping)
+            F.moe_permute(g, x.h, xs)
+        return g, xs
+
+    def _experts(self, L, x: StepCtx, g, xs):
+        """The experts' outputs, in the place of their rows."""
+        f, act = L.moe, x.act[:g.rows * L.ff].view(g.rows, L.ff)
+        ex = F.gemm_epilogue(out2=act, n_split=0, glu=(f.limit, GLU_ALPHA, GLU_BIAS))
+        self._launches += L.w_up(xs, g, None, F.GEPI_SPLIT_GLU, ex) + L.w_down(act, g, xs, F.GEPI_STORE)
 
     def _run_layers(self, x: StepCtx):
         c, T = self.cfg, x.T
@@ -369,10 +384,13 @@ class B200GatedModel(DeviceRuntime):
             (self._gla if L.is_gla else self._attention)(i, L, x, proj, mix)
             n += L.w_o(mix, x.y, F.GEPI_STORE)
             after = self.layers[i + 1].norm1 if i + 1 < len(self.layers) else None
-            F.resid_norm(x.y, x.x, L.norm1b, x.h, after if L.moe is None else L.norm2, self.W, c.rms_eps)
-            self._launches += n + 1
-            if L.moe is not None:
-                rows, g = self._experts(L, x)
+            self._launches += n
+            if L.moe is None:
+                F.resid_norm(x.y, x.x, L.norm1b, x.h, after, self.W, c.rms_eps)
+                self._launches += 1
+            else:
+                g, rows = self._norm_and_route(L, x)
+                self._experts(L, x, g, rows)
                 F.resid_norm(rows, x.x, L.norm2b, x.h, after, self.W, c.rms_eps, routed=g)
                 self._launches += 1
         nvtx_end()

@@ -16,8 +16,10 @@ static int run_grouped(GemmParams& p, int BN, int BMH, cudaStream_t st) {
   const dim3 grid((p.max_tiles + p.group_m - 1) / p.group_m * p.group_m * p.tiles_n, 1, 1);
   if (BN == 32) return launch_gemm<32, BF16, 1, kGemmShortRingKb, true>(p, grid, st);
   if (BN == 64) return launch_gemm<64, BF16, 1, kGemmShortRingKb, true>(p, grid, st);
-  if (BMH == 2) return launch_gemm<128, BF16, 2, TI_GEMM_RING_KB, true>(p, grid, st);
-  return launch_gemm<128, BF16, 1, TI_GEMM_RING_KB, true>(p, grid, st);
+  // two CTAs per SM (bf16: 2 x 256 TMEM columns): the epilogue of one overlaps the main loop of the other
+  constexpr int RK = BF16 ? kGemmShortRingKb : TI_GEMM_RING_KB;
+  if (BMH == 2) return launch_gemm<128, BF16, 2, RK, true>(p, grid, st);
+  return launch_gemm<128, BF16, 1, RK, true>(p, grid, st);
 }
 
 static int prepare_grouped(GemmParams& p, const void* w, int E, int KB, int BN, int BMH) {

@@ -220,7 +220,8 @@ int ti_gemm_bf16(const void* w, int n_tiles, int N, int K, const void* x, int M,
   if (K % 32 || N < 1 || epi < 0 || epi > 5) return -2;
   ti::GemmParams p = {};
   const int KB = K / 32, KS = (KB + ti::kKS - 1) / ti::kKS;    // 64-byte slabs; 128-byte stages
-  const int BN = M <= 32 ? 32 : (M <= 64 ? 64 : 128);
+  // a single weight tile (a router): smaller token tiles, so that there are enough of them for all SMs
+  const int BN = M <= 32 || (N <= 128 && M <= 64 * 148) ? 32 : (M <= 64 || N <= 128 ? 64 : 128);
   const int BMH = ti::pick_bmh(M, n_tiles);
   int rc = ti::cached_map(&p.map_w, w, KB, n_tiles, BMH == 2 ? -32 : 0);
   if (rc) return rc;

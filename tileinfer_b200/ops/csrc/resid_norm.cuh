@@ -1,0 +1,100 @@
+// A sublayer's output into the fp32 residual, with the norms on both sides: one row by one block, kept in registers.
+#pragma once
+#include "row_vec.cuh"
+
+namespace ti {
+
+// x[m] += rmsnorm(y[m]) * w_out, then h[m] = rmsnorm(x[m]) * w_next (w_next null: no h).  y[m] is a row, or, with `slot`,
+// the weighted sum over k < top of the rows slot[m, k] of y plus the input row h_in[m] times the weights whose slot is
+// negative (-1; -2 adds nothing).
+struct ResidNormParams {
+  const void* y;           // [rows][ldy]
+  float* x;                // [M][P]
+  const float* w_out;      // [P]
+  const float* w_next;     // [P] or null
+  void* h;                 // [M][P]
+  const int* slot;         // [M][top] or null
+  const float* weight;     // [M][top]
+  const void* h_in;        // [M][P]
+  int W, P, ldy, top;
+  float eps;
+};
+
+// KEEP x 8 columns per thread; on return `y` holds the thread's part of h (fp32, before it was stored as T).  `red`: 64
+// floats of shared memory.
+template <typename T, int KEEP>
+TI_DEVICE void resid_norm_row(const ResidNormParams& p, int m, float (&y)[KEEP][8], float* red) {
+  const int step = blockDim.x * 8;
+  float* xr = p.x + (size_t)m * p.P;
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * 8 + j * step;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[j][i] = 0.f;
+    if (c >= p.P) continue;
+    if (p.slot == nullptr) {
+      load8(static_cast<const T*>(p.y) + (size_t)m * p.ldy + c, y[j]);
+    } else {
+      float own = 0.f;
+      for (int k0 = 0; k0 < p.top; k0 += 4) {              // four rows in flight
+        int sl[4];
+        float a[4], v[4][8];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const bool in = k0 + k < p.top;
+          sl[k] = in ? p.slot[(size_t)m * p.top + k0 + k] : -2;
+          a[k] = in ? p.weight[(size_t)m * p.top + k0 + k] : 0.f;
+        }
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (sl[k] >= 0) load8(static_cast<const T*>(p.y) + (size_t)sl[k] * p.ldy + c, v[k]);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          if (sl[k] == -1) own += a[k];
+          if (sl[k] < 0) continue;
+#pragma unroll
+          for (int i = 0; i < 8; ++i) y[j][i] = fmaf(a[k], v[k][i], y[j][i]);
+        }
+      }
+      if (own != 0.f) {
+        float v[8];
+        load8(static_cast<const T*>(p.h_in) + (size_t)m * p.P + c, v);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) y[j][i] = fmaf(own, v[i], y[j][i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss += y[j][i] * y[j][i];
+  }
+  const float ry = rsqrtf(block_sum32(ss, red) / (float)p.W + p.eps);
+  ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * 8 + j * step;
+    if (c >= p.P) continue;
+    float v[8], g[8];
+    load8(xr + c, v);
+    load8(p.w_out + c, g);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      y[j][i] = v[i] + y[j][i] * ry * g[i];
+      ss += y[j][i] * y[j][i];
+    }
+    store8(xr + c, y[j]);
+  }
+  if (p.w_next == nullptr) return;
+  const float rx = rsqrtf(block_sum32(ss, red + 32) / (float)p.W + p.eps);
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * 8 + j * step;
+    if (c >= p.P) continue;
+    float g[8];
+    load8(p.w_next + c, g);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[j][i] *= rx * g[i];
+    store8(static_cast<T*>(p.h) + (size_t)m * p.P + c, y[j]);
+  }
+}
+
+}  // namespace ti

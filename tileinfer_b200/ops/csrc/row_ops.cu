@@ -4,7 +4,7 @@
 // Every kernel is templated on the activation type (bf16, or float in 32-bit mode).  Row pitches are padded to
 // multiples of 64 elements and the pad columns hold zeros (zero weight rows, zero norm weights), so that rows are read
 // in whole vectors; means divide by the true length.
-#include "row_vec.cuh"
+#include "resid_norm.cuh"
 
 namespace ti {
 
@@ -98,90 +98,13 @@ __global__ void __launch_bounds__(256) rmsnorm_f32_kernel(const float* __restric
 }
 
 // ---------------------------------------------------------------- sublayer output -> residual -> next sublayer's input
-// x[m] += rmsnorm(y[m]) * w_out, then h[m] = rmsnorm(x[m]) * w_next (w_next null: no h).  y[m] is a row, or, with `slot`,
-// the weighted sum over k < top of the rows slot[m, k] of y plus the input row h_in[m] times the weights whose slot is
-// negative (-1; -2 adds nothing).
-struct ResidNormParams {
-  const void* y;           // [rows][ldy]
-  float* x;                // [M][P]
-  const float* w_out;      // [P]
-  const float* w_next;     // [P] or null
-  void* h;                 // [M][P]
-  const int* slot;         // [M][top] or null
-  const float* weight;     // [M][top]
-  const void* h_in;        // [M][P]
-  int W, P, ldy, top;
-  float eps;
-};
-
-// The row stays in registers: KEEP x 8 columns per thread.
 template <typename T, int KEEP>
 __global__ void __launch_bounds__(256) resid_norm_kernel(const __grid_constant__ ResidNormParams p) {
-  __shared__ float red[2][8];
-  const int m = blockIdx.x, step = blockDim.x * 8;
-  float* xr = p.x + (size_t)m * p.P;
+  __shared__ float red[64];
+  float y[KEEP][8];
   pdl_trigger();
   pdl_wait();
-  float y[KEEP][8];
-  float ss = 0.f;
-#pragma unroll
-  for (int j = 0; j < KEEP; ++j) {
-    const int c = threadIdx.x * 8 + j * step;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) y[j][i] = 0.f;
-    if (c >= p.P) continue;
-    if (p.slot == nullptr) {
-      load8(static_cast<const T*>(p.y) + (size_t)m * p.ldy + c, y[j]);
-    } else {
-      float own = 0.f;
-      for (int k = 0; k < p.top; ++k) {
-        const int s = p.slot[(size_t)m * p.top + k];
-        const float a = p.weight[(size_t)m * p.top + k];
-        if (s == -1) own += a;
-        if (s < 0) continue;
-        float v[8];
-        load8(static_cast<const T*>(p.y) + (size_t)s * p.ldy + c, v);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) y[j][i] = fmaf(a, v[i], y[j][i]);
-      }
-      if (own != 0.f) {
-        float v[8];
-        load8(static_cast<const T*>(p.h_in) + (size_t)m * p.P + c, v);
-#pragma unroll
-        for (int i = 0; i < 8; ++i) y[j][i] = fmaf(own, v[i], y[j][i]);
-      }
-    }
-#pragma unroll
-    for (int i = 0; i < 8; ++i) ss += y[j][i] * y[j][i];
-  }
-  const float ry = rsqrtf(block_sum32(ss, red[0]) / (float)p.W + p.eps);
-  ss = 0.f;
-#pragma unroll
-  for (int j = 0; j < KEEP; ++j) {
-    const int c = threadIdx.x * 8 + j * step;
-    if (c >= p.P) continue;
-    float v[8], g[8];
-    load8(xr + c, v);
-    load8(p.w_out + c, g);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      y[j][i] = v[i] + y[j][i] * ry * g[i];
-      ss += y[j][i] * y[j][i];
-    }
-    store8(xr + c, y[j]);
-  }
-  if (p.w_next == nullptr) return;
-  const float rx = rsqrtf(block_sum32(ss, red[1]) / (float)p.W + p.eps);
-#pragma unroll
-  for (int j = 0; j < KEEP; ++j) {
-    const int c = threadIdx.x * 8 + j * step;
-    if (c >= p.P) continue;
-    float g[8];
-    load8(p.w_next + c, g);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) g[i] *= y[j][i] * rx;
-    store8(static_cast<T*>(p.h) + (size_t)m * p.P + c, g);
-  }
+  resid_norm_row<T, KEEP>(p, blockIdx.x, y, red);
 }
 
 // ---------------------------------------------------------------- fp32 matrix product (32-bit mode)

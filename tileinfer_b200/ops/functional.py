@@ -99,7 +99,7 @@ class GlaParams(ctypes.Structure):
 class MoeRouteParams(ctypes.Structure):
     _fields_ = [("logits", _P), ("correction", _P), ("valid", _P), ("ids", _P), ("weight", _P), ("pos", _P), ("counts", _P),
                 ("ticket", _P), ("first", _P), ("tiles", _P), ("num_tiles", _P), ("M", _I), ("E", _I), ("identity", _I), ("top", _I),
-                ("groups", _I), ("keep", _I), ("ldl", _I), ("tile_rows", _I), ("max_tiles", _I)]
+                ("groups", _I), ("keep", _I), ("ldl", _I), ("tile_rows", _I), ("max_tiles", _I), ("row_stride", _I)]
 
 
 class ResidNormParams(ctypes.Structure):
@@ -170,6 +170,7 @@ _l.register("ti_gla_chunked", _I, [ctypes.POINTER(GlaParams), _I, _I, _P], "gla"
 _l.register("ti_gla_finish", _I, [ctypes.POINTER(GlaParams), _I, _I, _I, _P], "gla")
 _l.register("ti_moe_route_params_size", _I, [], "moe")
 _l.register("ti_moe_route", _I, [ctypes.POINTER(MoeRouteParams), _P], "moe")
+_l.register("ti_moe_norm_route", _I, [ctypes.POINTER(ResidNormParams), ctypes.POINTER(MoeRouteParams), _P, _P, _P, _I, _P], "moe")
 _l.register("ti_moe_permute", _I, [_P, _I, _I, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P], "moe")
 _l.register("ti_gemm_grouped_bf16", _I, [_P, _I, _I, _I, _I, _P, _I, _P, _P, _I, _I, _P, _I, _I, _P, _P, _P], "moe")
 _l.register("ti_gemm_grouped_w8a16", _I, [_P, _P, _I, _I, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _P, _I, _I, _P, _P, _P], "moe")
@@ -797,12 +798,17 @@ def gemm_f32(w, x, *, out, epi=GEPI_F32, ex=None, groups=None):
 def resid_norm(y, x, w_out, h, w_next, W, eps, routed=None):
     """x += rmsnorm(y) * w_out (fp32 rows), then h = rmsnorm(x) * w_next unless w_next is None.  With `routed` (a
     TokenGroups after `moe_permute`) y holds the experts' rows and h the input of the identity experts."""
+    p = _resid_params(y, x, w_out, h, w_next, W, eps, routed)
+    check(_l.lib().ti_resid_norm(ctypes.byref(p), x.shape[0], _f32(y), stream()), "ti_resid_norm")
+
+
+def _resid_params(y, x, w_out, h, w_next, W, eps, routed=None) -> ResidNormParams:
     p = ResidNormParams()
     p.y, p.x, p.w_out, p.w_next, p.h = ptr(y), ptr(x), ptr(w_out), ptr(w_next), ptr(h)
     if routed is not None:
         p.slot, p.weight, p.h_in, p.top = ptr(routed.slot), ptr(routed.weight), ptr(h), routed.top
     p.W, p.P, p.ldy, p.eps = W, x.stride(0), y.stride(0), eps
-    check(_l.lib().ti_resid_norm(ctypes.byref(p), x.shape[0], _f32(y), stream()), "ti_resid_norm")
+    return p
 
 
 # ------------------------------------------------------------------------------------ rotated unit heads, plain attention
@@ -877,8 +883,10 @@ class TokenGroups:
     """Routing of up to T tokens to `top` of E experts: chosen experts, weights, rows, and the table of token tiles the
     grouped products run on.  `counters` (see `moe_counters`) may be shared by everything on one stream."""
 
-    def __init__(self, T: int, E: int, choices: int, top: int, counters, f32: bool, device):
-        self.T, self.E, self.choices, self.top, self.counters, self.rows = T, E, choices, top, counters, T * top
+    def __init__(self, T: int, E: int, choices: int, top: int, counters, f32: bool, device, fixed: bool = False):
+        """`fixed`: every expert has T rows of its own (for `moe_norm_route`), else the experts' rows follow each other."""
+        self.T, self.E, self.choices, self.top, self.counters = T, E, choices, top, counters
+        self.row_stride, self.rows = T if fixed else 0, E * T if fixed else T * top
         mean = T * top / choices                           # rows of an expert
         self.tile = 64 if f32 else 32 if mean <= 24 else 64 if mean <= 96 else 128
         n = T * top // self.tile + min(E, T * top)
@@ -897,12 +905,29 @@ def moe_counters(max_experts: int, device):
 
 def moe_route(g: TokenGroups, logits, correction, groups: int, keep: int, valid=None):
     """Chooses the experts of every row of `logits` [T, >= choices] (fp32) and lays out the token tiles."""
-    p = MoeRouteParams()
-    p.logits, p.correction, p.valid, p.ids, p.weight, p.pos = ptr(logits), ptr(correction), ptr(valid), ptr(g.ids), ptr(g.weight), ptr(g.pos)
-    p.counts, p.ticket, p.first, p.tiles, p.num_tiles = ptr(g.counters) + 4, ptr(g.counters), ptr(g.first), ptr(g.tiles), ptr(g.num_tiles)
-    p.M, p.E, p.identity, p.top, p.groups, p.keep, p.ldl = g.T, g.E, g.choices - g.E, g.top, groups, keep, logits.stride(0)
-    p.tile_rows, p.max_tiles = g.tile, g.tiles.shape[1]
+    p = _route_params(g, correction, groups, keep, valid)
+    p.logits, p.ldl = ptr(logits), logits.stride(0)
     check(_l.lib().ti_moe_route(ctypes.byref(p), stream()), "ti_moe_route")
+
+
+NORM_ROUTE_MAX_WIDTH = 8192      # columns of a row that `moe_norm_route` takes
+
+
+def moe_norm_route(y, x, w_out, h, w_next, W, eps, g: TokenGroups, router, correction, groups: int, keep: int, xs, valid=None):
+    """`resid_norm` and, for the rows h it makes, the router product, `moe_route` and `moe_permute` (into xs) in one kernel,
+    for few tokens and fixed rows.  router: [choices, P] in the type of h."""
+    r, p = _resid_params(y, x, w_out, h, w_next, W, eps), _route_params(g, correction, groups, keep, valid)
+    assert router.shape == (g.choices, x.stride(0)) and router.dtype == h.dtype and xs.shape[0] == g.rows and g.row_stride == g.T
+    check(_l.lib().ti_moe_norm_route(ctypes.byref(r), ctypes.byref(p), ptr(router), ptr(g.slot), ptr(xs), _f32(h), stream()), "ti_moe_norm_route")
+
+
+def _route_params(g: TokenGroups, correction, groups: int, keep: int, valid) -> MoeRouteParams:
+    p = MoeRouteParams()
+    p.correction, p.valid, p.ids, p.weight, p.pos = ptr(correction), ptr(valid), ptr(g.ids), ptr(g.weight), ptr(g.pos)
+    p.counts, p.ticket, p.first, p.tiles, p.num_tiles = ptr(g.counters) + 4, ptr(g.counters), ptr(g.first), ptr(g.tiles), ptr(g.num_tiles)
+    p.M, p.E, p.identity, p.top, p.groups, p.keep = g.T, g.E, g.choices - g.E, g.top, groups, keep
+    p.tile_rows, p.max_tiles, p.row_stride = g.tile, g.tiles.shape[1], g.row_stride
+    return p
 
 
 def moe_permute(g: TokenGroups, h, xs):
