@@ -21,7 +21,8 @@
 // prefix sees all of it.  Values may be of another size than queries and keys, and the gate may be absent.  Scores may be
 // capped by cap * tanh(score / cap); where |score / cap| is known to stay small (normalised queries and keys) the tanh is
 // its power series and the softmax needs no running maximum at all: exp2 of a bounded score neither overflows nor
-// vanishes, so the scores of a tile are read once.  Every wait is bounded; on expiry the status word is set, all roles leave their loops
+// vanishes, so the scores of a tile are read once, two threads can share a query row (eight softmax warps, half of the keys
+// of a tile each), and with shared memory for two P tiles the next one is written while P V of this one runs.  Every wait is bounded; on expiry the status word is set, all roles leave their loops
 // and TMEM is freed.  No load carries a cluster-multicast qualifier.
 #include "tensor_map.cuh"
 
@@ -46,25 +47,56 @@ struct AttnPrefillParams {
 
 // How a score follows from q.k: scaled; capped with the series, reference 0 instead of a running maximum; capped
 enum { SCORE_PLAIN = 0, SCORE_SERIES = 1, SCORE_CAPPED = 2 };
-constexpr float kSeriesMax = 0.5f;       // largest |argument| the series serves (error below 1e-6 there)
+constexpr float kSeriesMax = 0.4f;       // largest |argument| the series serves (error below 1e-7 there)
 
-// tanh(y) = y - y^3/3 + 2 y^5/15 - 17 y^7/315 + 62 y^9/2835 - 1382 y^11/155925 + ...
-TI_DEVICE float tanh_series(float y) {
-  const float z = y * y;
-  float s = fmaf(z, 21844.f / 6081075.f, -1382.f / 155925.f);
-  s = fmaf(s, z, 62.f / 2835.f);
-  s = fmaf(s, z, -17.f / 315.f);
-  s = fmaf(s, z, 2.f / 15.f);
-  s = fmaf(s, z, -1.f / 3.f);
-  return fmaf(y * z, s, y);
+// Packed pairs of floats
+typedef unsigned long long f2;
+TI_DEVICE f2 pack2(float a, float b) {
+  f2 r;
+  asm("mov.b64 %0, {%1, %2};\n" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+TI_DEVICE void unpack2(f2 v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;\n" : "=f"(a), "=f"(b) : "l"(v)); }
+TI_DEVICE f2 fma2(f2 a, f2 b, f2 c) {
+  f2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+TI_DEVICE f2 mul2(f2 a, f2 b) {
+  f2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(r) : "l"(a), "l"(b));
+  return r;
 }
 TI_DEVICE float ex2_approx(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
+// c tanh(k x) = c k x (1 + z (-1/3 + z (2/15 + z (-17/315 + z (62/2835 - z 1382/155925))))) with z = (k x)^2; the powers of
+// k are folded into the coefficients.  tanh y = y - y^3/3 + 2 y^5/15 - 17 y^7/315 + ... (Bernoulli numbers).
+struct TanhSeries {
+  f2 ck, c1, c2, c3, c4, c5;
+  TI_DEVICE TanhSeries(float c, float k) {
+    const float z = k * k;
+    auto two = [](float v) { return pack2(v, v); };
+    ck = two(c * k);
+    c1 = two(-z / 3.f);
+    c2 = two(z * z * (2.f / 15.f));
+    c3 = two(z * z * z * (-17.f / 315.f));
+    c4 = two(z * z * z * z * (62.f / 2835.f));
+    c5 = two(z * z * z * z * z * (-1382.f / 155925.f));
+  }
+  TI_DEVICE f2 operator()(f2 x) const {
+    const f2 a = mul2(x, x);
+    f2 u = fma2(c5, a, c4);
+    u = fma2(u, a, c3);
+    u = fma2(u, a, c2);
+    u = fma2(u, a, c1);
+    const f2 y = mul2(x, ck);
+    return fma2(mul2(u, a), y, y);
+  }
+};
 template <int MODE> TI_DEVICE float prefill_score(const AttnPrefillParams& p, float qk) {
-  if (MODE == SCORE_SERIES) return p.cap_out * tanh_series(qk * p.cap_in);
   if (MODE == SCORE_CAPPED) return p.cap_out * (1.f - __fdividef(2.f, 1.f + ex2_approx(qk * p.cap_in * 2.8853900817779268f)));
   return qk * p.scale_log2e;
 }
@@ -75,29 +107,57 @@ constexpr int kAttnProducerV = 6;
 constexpr float kMaskVal = -1e30f;
 constexpr float kRescaleGap = 8.f;       // log2 units the running maximum may lag behind before O is rescaled
 
-template <int D, int DV> struct AttnPrefillGeom {
+template <int D, int DV, int MODE> struct AttnPrefillGeom {
   static constexpr int kSlabs = D / 64;
   static constexpr int kQBytes = kSlabs * 128 * 128;
   static constexpr int kKBytes = kSlabs * 128 * 128;
   static constexpr int kVPage = DV * 32;
   static constexpr int kVBytes = 8 * kVPage;
-  static constexpr int kPBytes = 2 * 128 * 128;
+  static constexpr int kP = 2 * 128 * 128;                          // one P tile
   static constexpr int kBarBytes = 128;
+  static constexpr int kPTiles = MODE == SCORE_SERIES && kQBytes + kKBytes + kVBytes + 2 * kP + kBarBytes + 1024 + 1024 <= 227 * 1024 ? 2 : 1;
+  static constexpr int kPBytes = kPTiles * kP;
+  static constexpr int kHalves = MODE == SCORE_SERIES ? 2 : 1;      // threads that share a query row
+  static constexpr int kThreads = MODE == SCORE_SERIES ? 384 : kAttnThreads;
   static constexpr size_t kNeeded = (size_t)kQBytes + kKBytes + kVBytes + kPBytes + kBarBytes + 1024;
   // one CTA per SM (the kernel takes all 512 TMEM columns)
   static constexpr size_t kSmem = kNeeded > 120 * 1024 ? kNeeded : 120 * 1024;
 };
 
+// 32 output columns of a row: times 1 / l and the sigmoid gate, as bf16
+TI_DEVICE void store_rows32(const AttnPrefillParams& p, const uint32_t (&v)[32], float inv, const __nv_bfloat16* gate, __nv_bfloat16* dst, int c) {
+#pragma unroll
+  for (int q4 = 0; q4 < 4; ++q4) {
+    float f[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(v[q4 * 8 + e]) * inv;
+    if (p.gate_src != nullptr) {
+      const uint4 gw = *reinterpret_cast<const uint4*>(gate + c * 32 + q4 * 8);
+      const uint32_t g4[4] = {gw.x, gw.y, gw.z, gw.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        f[2 * e] *= sigmoid_f(bf16lo(g4[e]));
+        f[2 * e + 1] *= sigmoid_f(bf16hi(g4[e]));
+      }
+    }
+    uint32_t o4[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o4[e] = pack_bf16(f[2 * e], f[2 * e + 1]);
+    *reinterpret_cast<uint4*>(dst + c * 32 + q4 * 8) = make_uint4(o4[0], o4[1], o4[2], o4[3]);
+  }
+}
+
 template <int D, int DV, int MODE>
-__global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __grid_constant__ AttnPrefillParams p) {
-  using G = AttnPrefillGeom<D, DV>;
+__global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) attn_prefill_kernel(const __grid_constant__ AttnPrefillParams p) {
+  using G = AttnPrefillGeom<D, DV, MODE>;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   const uint32_t q_s = smem_u32(smem), k_s = q_s + G::kQBytes, v_s = k_s + G::kKBytes, p_s = v_s + G::kVBytes;
   const uint32_t bars = p_s + G::kPBytes;
   const uint32_t q_full = bars, k_full = bars + 8, k_empty = bars + 16, v_full = bars + 24, v_empty = bars + 32,
-                 s_full0 = bars + 40, p_full = bars + 56, p_empty = bars + 64, tmem_slot = bars + 72;
-  uint32_t* tmem_slot_ptr = reinterpret_cast<uint32_t*>(smem + G::kQBytes + G::kKBytes + G::kVBytes + G::kPBytes + 72);
+                 s_full0 = bars + 40, p_full = bars + 56, p_empty = bars + 72, tmem_slot = bars + 88;    // p: one per P tile
+  uint32_t* tmem_slot_ptr = reinterpret_cast<uint32_t*>(smem + G::kQBytes + G::kKBytes + G::kVBytes + G::kPBytes + 88);
+  constexpr int NP = G::kPTiles;
   __shared__ int s_abort;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -119,8 +179,10 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
     mbar_init(v_empty, 1);
     mbar_init(s_full0, 1);
     mbar_init(s_full0 + 8, 1);
-    mbar_init(p_full, 128);
-    mbar_init(p_empty, 1);
+    for (int i = 0; i < NP; ++i) {
+      mbar_init(p_full + 8 * i, 128 * G::kHalves);
+      mbar_init(p_empty + 8 * i, 1);
+    }
     fence_mbar_init();
   }
   if (warp == 1) {
@@ -192,17 +254,97 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
           tc_fence_after();
           issue_qk(j + 1);
         }
-        ok = mbar_wait(p_full, (uint32_t)(j & 1), kAttnWaitNs, p.status) && mbar_wait(v_full, (uint32_t)(j & 1), kAttnWaitNs, p.status);
+        ok = mbar_wait(p_full + 8 * (j % NP), (uint32_t)((j / NP) & 1), kAttnWaitNs, p.status) && mbar_wait(v_full, (uint32_t)(j & 1), kAttnWaitNs, p.status);
         if (!ok) break;
         tc_fence_after();
 #pragma unroll
         for (int g = 0; g < 8; ++g)
-          umma_bf16(tmem_base + 256u, smem_desc_sw128(p_s + (g >> 2) * (128 * 128) + (g & 3) * 32),
+          umma_bf16(tmem_base + 256u, smem_desc_sw128(p_s + (j % NP) * G::kP + (g >> 2) * (128 * 128) + (g & 3) * 32),
                     smem_desc_sw32(v_s + g * G::kVPage), idesc_o, (j | g) ? 1u : 0u);
         umma_commit(v_empty);
-        umma_commit(p_empty);
+        umma_commit(p_empty + 8 * (j % NP));
       }
       if (!ok) *abort_flag = 1;
+    }
+  } else if (MODE == SCORE_SERIES) {
+    // ------------------------------------------------------------ softmax + epilogue, bounded scores: two threads (in
+    // warps 2-5 and 8-11) per query row, each half of the keys of a tile and half of the output columns
+    if (warp < 6 || warp >= 8) {
+      const int quarter = warp & 3, half = warp >= 8 ? 1 : 0, r = quarter * 32 + lane;
+      const bool valid = r < ntok;
+      const int pos = p.positions[tok0 + (valid ? r : ntok - 1)];
+      const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
+      const TanhSeries series(p.cap_out, p.cap_in);
+      f2 sum2 = pack2(0.f, 0.f);
+      const f2 one2 = pack2(1.f, 1.f);
+      bool ok = true;
+      for (int j = 0; j < ntiles; ++j) {
+        ok = ok && !*abort_flag && mbar_wait(s_full0 + 8 * (j & 1), (uint32_t)((j >> 1) & 1), kAttnWaitNs, p.status);
+        if (ok && j >= NP) ok = mbar_wait(p_empty + 8 * (j % NP), (uint32_t)((j / NP - 1) & 1), kAttnWaitNs, p.status);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        tc_fence_after();
+        const uint32_t s_addr = lane_base + (uint32_t)(j & 1) * 128u + (uint32_t)half * 64u;
+        const int key0 = j * 128 + half * 64;
+        const bool need_mask = key0 + 63 > pos;
+        uint32_t v[2][32];
+        tmem_ld32(s_addr, v[0]);
+        tmem_ld32(s_addr + 32, v[1]);
+        tmem_ld_wait();
+        const uint32_t row_addr = p_s + (uint32_t)(j % NP) * G::kP + (uint32_t)half * (128 * 128) + (uint32_t)r * 128u;
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          uint32_t pk[16];
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) {
+            float s0, s1;
+            unpack2(series(pack2(__uint_as_float(v[c][i]), __uint_as_float(v[c][i + 1]))), s0, s1);
+            if (need_mask) {
+              if (key0 + c * 32 + i > pos) s0 = kMaskVal;
+              if (key0 + c * 32 + i + 1 > pos) s1 = kMaskVal;
+            }
+            const float p0 = ex2_approx(s0), p1 = ex2_approx(s1);
+            sum2 = fma2(pack2(p0, p1), one2, sum2);
+            pk[i >> 1] = pack_bf16(p0, p1);
+          }
+#pragma unroll
+          for (int q4 = 0; q4 < 4; ++q4) {
+            const uint32_t chunk = (uint32_t)(c * 4 + q4) ^ (uint32_t)(r & 7);
+            asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};\n" ::"r"(row_addr + chunk * 16u), "r"(pk[4 * q4]),
+                         "r"(pk[4 * q4 + 1]), "r"(pk[4 * q4 + 2]), "r"(pk[4 * q4 + 3])
+                         : "memory");
+          }
+        }
+        tc_fence_before();
+        fence_proxy_async();
+        asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(p_full + 8 * (j % NP)) : "memory");
+      }
+      if (ok) {                                            // every P V has completed: they complete in order
+        ok = mbar_wait(p_empty + 8 * ((ntiles - 1) % NP), (uint32_t)(((ntiles - 1) / NP) & 1), kAttnWaitNs, p.status);
+        ok = __all_sync(0xffffffffu, ok);
+      }
+      if (!ok) *abort_flag = 1;
+      // the sums of the two halves meet in the idle P tile; a warp that gave up still takes part in the barrier
+      float a, b;
+      unpack2(sum2, a, b);
+      float* l_s = reinterpret_cast<float*>(smem + (p_s - q_s));
+      l_s[half * 128 + r] = a + b;
+      asm volatile("bar.sync 1, 256;\n" ::: "memory");
+      if (ok) {
+        tc_fence_after();
+        const float inv = 1.f / (l_s[r] + l_s[128 + r]);
+        const size_t tok = (size_t)tok0 + (valid ? r : 0);
+        const __nv_bfloat16* gate = p.gate_src + tok * p.ld + (size_t)head * 2 * D + D;
+        __nv_bfloat16* dst = p.out + tok * ((size_t)p.hq * DV) + (size_t)head * DV;
+#pragma unroll 1
+        for (int c = half * (DV / 64); c < (half + 1) * (DV / 64); ++c) {
+          uint32_t v[32];
+          tmem_ld32(lane_base + 256u + c * 32, v);
+          tmem_ld_wait();
+          if (valid) store_rows32(p, v, inv, gate, dst, c);
+        }
+      }
+      tc_fence_before();
     }
   } else {
     // ------------------------------------------------------------ softmax + epilogue: thread = query row
@@ -211,7 +353,7 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
     const bool valid = r < ntok;
     const int pos = p.positions[tok0 + (valid ? r : ntok - 1)];
     const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
-    float m_used = MODE == SCORE_SERIES ? 0.f : kMaskVal, l = 0.f;
+    float m_used = kMaskVal, l = 0.f;
     bool ok = true;
     for (int j = 0; j < ntiles; ++j) {
       ok = ok && !*abort_flag && mbar_wait(s_full0 + 8 * (j & 1), (uint32_t)((j >> 1) & 1), kAttnWaitNs, p.status);
@@ -224,7 +366,7 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
       // ---- pass 1: row maximum
       float mx = kMaskVal;
 #pragma unroll
-      for (int c = 0; c < (MODE == SCORE_SERIES ? 0 : 4); ++c) {
+      for (int c = 0; c < 4; ++c) {
         uint32_t v[32];
         tmem_ld32(s_addr + c * 32, v);
         tmem_ld_wait();
@@ -235,8 +377,8 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
           mx = fmaxf(mx, s);
         }
       }
-      const float m_new = MODE == SCORE_SERIES ? 0.f : fmaxf(m_used, mx);
-      const bool resc = MODE != SCORE_SERIES && m_new - m_used > kRescaleGap;
+      const float m_new = fmaxf(m_used, mx);
+      const bool resc = m_new - m_used > kRescaleGap;
       float alpha = 1.f;
       if (resc) {
         alpha = exp2f(m_used - m_new);
@@ -277,7 +419,7 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
             if (key0 + c * 32 + i > pos) s0 = kMaskVal;
             if (key0 + c * 32 + i + 1 > pos) s1 = kMaskVal;
           }
-          const float p0 = MODE == SCORE_SERIES ? ex2_approx(s0) : exp2f(s0 - m_used), p1 = MODE == SCORE_SERIES ? ex2_approx(s1) : exp2f(s1 - m_used);
+          const float p0 = exp2f(s0 - m_used), p1 = exp2f(s1 - m_used);
           sum += p0 + p1;
           pk[i >> 1] = pack_bf16(p0, p1);
         }
@@ -312,25 +454,7 @@ __global__ void __launch_bounds__(kAttnThreads, 1) attn_prefill_kernel(const __g
         tmem_ld32(lane_base + 256u + c * 32, v);
         tmem_ld_wait();
         if (valid) {
-#pragma unroll
-          for (int q4 = 0; q4 < 4; ++q4) {
-            float f[8];
-#pragma unroll
-            for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(v[q4 * 8 + e]) * inv;
-            if (p.gate_src != nullptr) {
-              const uint4 gw = *reinterpret_cast<const uint4*>(gate + c * 32 + q4 * 8);
-              const uint32_t g4[4] = {gw.x, gw.y, gw.z, gw.w};
-#pragma unroll
-              for (int e = 0; e < 4; ++e) {
-                f[2 * e] *= sigmoid_f(bf16lo(g4[e]));
-                f[2 * e + 1] *= sigmoid_f(bf16hi(g4[e]));
-              }
-            }
-            uint32_t o4[4];
-#pragma unroll
-            for (int e = 0; e < 4; ++e) o4[e] = pack_bf16(f[2 * e], f[2 * e + 1]);
-            *reinterpret_cast<uint4*>(dst + c * 32 + q4 * 8) = make_uint4(o4[0], o4[1], o4[2], o4[3]);
-          }
+          store_rows32(p, v, inv, gate, dst, c);
         }
       }
     } else {
@@ -350,10 +474,10 @@ static int launch_mode(const AttnPrefillParams& p, int num_tiles, cudaStream_t s
   static bool configured = false;
   auto k = attn_prefill_kernel<D, DV, MODE>;
   if (!configured) {
-    cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)AttnPrefillGeom<D, DV>::kSmem);
+    cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)AttnPrefillGeom<D, DV, MODE>::kSmem);
     configured = true;
   }
-  k<<<dim3(num_tiles, p.hq), kAttnThreads, AttnPrefillGeom<D, DV>::kSmem, st>>>(p);
+  k<<<dim3(num_tiles, p.hq), AttnPrefillGeom<D, DV, MODE>::kThreads, AttnPrefillGeom<D, DV, MODE>::kSmem, st>>>(p);
   return (int)cudaGetLastError();
 }
 

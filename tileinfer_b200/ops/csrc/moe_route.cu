@@ -192,7 +192,7 @@ __global__ void __launch_bounds__(1024) moe_norm_route_kernel(const __grid_const
   float y[1][8];
   pdl_trigger();
   pdl_wait();
-  resid_norm_row<T, 1>(r, m, y, red);
+  resid_norm_row<T, 1, false>(r, m, y, red);
   if (tid * 8 < r.P) {
     float v[8];
 #pragma unroll

@@ -22,40 +22,31 @@ struct ResidNormParams {
 
 // KEEP x 8 columns per thread; on return `y` holds the thread's part of h (fp32, before it was stored as T).  `red`: 64
 // floats of shared memory.
-template <typename T, int KEEP>
+template <typename T, int KEEP, bool ROUTED>
 TI_DEVICE void resid_norm_row(const ResidNormParams& p, int m, float (&y)[KEEP][8], float* red) {
   const int step = blockDim.x * 8;
   float* xr = p.x + (size_t)m * p.P;
-  float ss = 0.f;
+  float ss = 0.f, x[KEEP][8];
 #pragma unroll
   for (int j = 0; j < KEEP; ++j) {
     const int c = threadIdx.x * 8 + j * step;
 #pragma unroll
     for (int i = 0; i < 8; ++i) y[j][i] = 0.f;
     if (c >= p.P) continue;
-    if (p.slot == nullptr) {
+    if (!ROUTED) {
+      load8(xr + c, x[j]);
       load8(static_cast<const T*>(p.y) + (size_t)m * p.ldy + c, y[j]);
     } else {
       float own = 0.f;
-      for (int k0 = 0; k0 < p.top; k0 += 4) {              // four rows in flight
-        int sl[4];
-        float a[4], v[4][8];
+      for (int k = 0; k < p.top; ++k) {
+        const int sl = p.slot[(size_t)m * p.top + k];
+        const float a = p.weight[(size_t)m * p.top + k];
+        if (sl == -1) own += a;
+        if (sl < 0) continue;
+        float v[8];
+        load8(static_cast<const T*>(p.y) + (size_t)sl * p.ldy + c, v);
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const bool in = k0 + k < p.top;
-          sl[k] = in ? p.slot[(size_t)m * p.top + k0 + k] : -2;
-          a[k] = in ? p.weight[(size_t)m * p.top + k0 + k] : 0.f;
-        }
-#pragma unroll
-        for (int k = 0; k < 4; ++k)
-          if (sl[k] >= 0) load8(static_cast<const T*>(p.y) + (size_t)sl[k] * p.ldy + c, v[k]);
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          if (sl[k] == -1) own += a[k];
-          if (sl[k] < 0) continue;
-#pragma unroll
-          for (int i = 0; i < 8; ++i) y[j][i] = fmaf(a[k], v[k][i], y[j][i]);
-        }
+        for (int i = 0; i < 8; ++i) y[j][i] = fmaf(a, v[i], y[j][i]);
       }
       if (own != 0.f) {
         float v[8];
@@ -73,12 +64,12 @@ TI_DEVICE void resid_norm_row(const ResidNormParams& p, int m, float (&y)[KEEP][
   for (int j = 0; j < KEEP; ++j) {
     const int c = threadIdx.x * 8 + j * step;
     if (c >= p.P) continue;
-    float v[8], g[8];
-    load8(xr + c, v);
+    float g[8];
+    if (ROUTED) load8(xr + c, x[j]);                       // later: the sum above needs the registers
     load8(p.w_out + c, g);
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      y[j][i] = v[i] + y[j][i] * ry * g[i];
+      y[j][i] = x[j][i] + y[j][i] * ry * g[i];
       ss += y[j][i] * y[j][i];
     }
     store8(xr + c, y[j]);
