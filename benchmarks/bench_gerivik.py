@@ -95,10 +95,19 @@ def kernel_rows(cfg, tag, lens, ctxs, prompt, ctx):
     lin = lambda n, k: F.LinearW(torch.randn(n, k, device="cuda").to(BF16) * k ** -0.5, False, "cuda")
     rnd = lambda *z: torch.randn(*z, device="cuda").to(BF16)
     # ---- dense products (the other model's like kernels: gate_up and down)
+    mc = closest(cfg)
+    kd, vd = mc.gdn_num_k_heads * 128, mc.gdn_num_v_heads * 128
+    like = {"gla": (2 * kd + 2 * vd + 2 * mc.gdn_num_v_heads, vd), "attention": ((2 * mc.num_q_heads + 2 * mc.num_kv_heads) * mc.head_dim, mc.num_q_heads * mc.head_dim)}
     for name, L in (("gla", s.g), ("attention", s.a)):
         proj, mix = s.bufs(L)
-        row(f"input product ({name})", timed(lambda: L.w_in(x.h, proj, F.GEPI_STORE)), **gemm(L.n_proj, W), like="gate_up")
-        row(f"output product ({name})", timed(lambda: L.w_o(mix, x.y, F.GEPI_STORE)), **gemm(W, L.n_mix), like="down")
+        row(f"input product ({name})", timed(lambda: L.w_in(x.h, proj, F.GEPI_STORE)), **gemm(L.n_proj, W), like="input product")
+        row(f"output product ({name})", timed(lambda: L.w_o(mix, x.y, F.GEPI_STORE)), **gemm(W, L.n_mix), like="output product")
+        n, k = like[name]
+        a, b, xa = lin(n, W), lin(W, k), rnd(T, k)
+        ya, yb = torch.empty(T, n, dtype=BF16, device="cuda"), rnd(T, W)
+        row(f"input product ({name}, other model)", timed(lambda: F.gemm_bf16(a, x.h, out=ya)), **gemm(n, W))
+        row(f"output product ({name}, other model)", timed(lambda: F.gemm_bf16(b, xa, out=yb, epi=F.GEPI_ROWPAR, resid=yb)), **gemm(W, k, 4))
+        del a, b, xa, ya, yb
     f = s.g.moe
     ff = f.top * f.ff
     up, down, act, hb = lin(2 * ff, W), lin(W, ff), rnd(T, ff), rnd(T, W)
@@ -151,6 +160,17 @@ def kernel_rows(cfg, tag, lens, ctxs, prompt, ctx):
     keys = sum(c * n - n * (n - 1) // 2 for n, c in zip(lens, ctxs))
     full = {"flops": 4 * keys * H * D, "nbytes": 2 * (T * (2 * H + 2 * G) * D + 2 * sum(ctxs) * G * D)}
     row("attention with rotation and store", timed(lambda: m._attention(1, s.a, x, proj, mix)), **full)
+    prep = 2 * T * (2 * H + 4 * G) * D
+    row("  of it: rotation, unit heads, store", small(lambda: m._rotate_and_store(1, s.a, x, proj)), nbytes=prep, like="qk norm")
+    r, gq = F.QkvPrepParams(), rnd(T, (2 * H + 2 * G) * D)
+    nw = torch.zeros(D, dtype=BF16, device="cuda")
+    kc0, vc0 = (torch.zeros_like(t) for t in m.cache[1])
+    qq = rnd(T, H * D)
+    r.proj, r.q_norm, r.k_norm, r.positions, r.slot_mapping, r.q_out, r.kcache, r.vcache = (
+        t.data_ptr() for t in (gq, nw, nw, x.positions, x.slot_mapping, qq, kc0, vc0))
+    r.ld, r.hq, r.hkv, r.rotary_dim, r.eps, r.log2_theta, r.num_blocks = gq.shape[1], H, G, s.ma.rot_dims, 1e-6, math.log2(s.ma.rot_base), m.num_blocks
+    row("qk norm, rotation, store (other model)", small(lambda: F.qkv_prep(r, T, D)), nbytes=prep)
+    del kc0, vc0, gq, qq
     q, (kc, vc) = x.q[:T * H * D].view(T, H * D), m.cache[1]
     a = s.ma
     if pre:

@@ -286,7 +286,8 @@ class B200GatedModel(DeviceRuntime):
         for k, key in enumerate(x.snaps):                  # snapshots stay on the device
             self.snapshots[key] = torch.cat([t[k].flatten() for t in x.snap_state.values()])
 
-    def _attention(self, i: int, L, x: StepCtx, proj, mix):
+    def _rotate_and_store(self, i: int, L, x: StepCtx, proj):
+        """Rotated unit heads of the queries (returned) and of the keys, and the values, into the cache pages."""
         m, (kc, vc), T = self.cfg.layers[i].mixer, self.cache[i], x.T
         q = x.q[:T * L.heads * L.dp].view(T, L.heads * L.dp)
         r = RopeUnitParams()
@@ -296,6 +297,11 @@ class B200GatedModel(DeviceRuntime):
         r.dim, r.dp, r.vp, r.half, r.num_blocks, r.eps = m.dim, L.dp, L.vp, m.rot_dims // 2, self.num_blocks, self.cfg.rms_eps
         F.rope_unit(r, self.f32)
         self._launches += 1
+        return q
+
+    def _attention(self, i: int, L, x: StepCtx, proj, mix):
+        m, (kc, vc) = self.cfg.layers[i].mixer, self.cache[i]
+        q = self._rotate_and_store(i, L, x, proj)
         if x.num_qg and (self.f32 or max(L.dp, L.vp) > 256):
             a = AttnGeneralParams()
             a.q, a.kcache, a.vcache, a.block_tables, a.positions = ptr(q), ptr(kc), ptr(vc), ptr(x.block_tables), ptr(x.positions)

@@ -244,6 +244,7 @@ int ti_gemm_bf16(const void* w, int n_tiles, int N, int K, const void* x, int M,
   cudaStream_t st = (cudaStream_t)stream;
   if (S == 1 && ti::short_k(KS, BN, (long long)tiles_n * tiles_m))
     return BMH == 2 ? ti::launch_gemm<128, true, 2, ti::kGemmShortRingKb>(p, grid, st) : ti::launch_gemm<128, true, 1, ti::kGemmShortRingKb>(p, grid, st);
+  if (N <= 128 && M > 64 && BN == 32) return ti::launch_gemm<32, true, 1, ti::kGemmShortRingKb>(p, grid, st);   // two CTAs per SM
   if (BMH == 2 && BN == 32) return ti::launch_gemm<32, true, 2>(p, grid, st);
   if (BMH == 2 && BN == 64) return ti::launch_gemm<64, true, 2>(p, grid, st);
   if (BMH == 2) return ti::launch_gemm<128, true, 2>(p, grid, st);

@@ -108,12 +108,15 @@ TI_DEVICE void route_token(const MoeRouteParams& p, int m, float* s, unsigned* k
 // Counters -> first rows and token tiles; counters cleared.  By the last block of the grid to get here.
 TI_DEVICE void route_finish(const MoeRouteParams& p) {
   __shared__ int s_last, s_rows[32], s_tiles[32];
-  __threadfence();
   __syncthreads();
-  if (threadIdx.x == 0) s_last = atomicAdd(p.ticket, 1u) + 1u == gridDim.x;
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
+  if (gridDim.x > 1) {
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) s_last = atomicAdd(p.ticket, 1u) + 1u == gridDim.x;
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+  }
   const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, warp = tid >> 5, per = (p.E + nt - 1) / nt;
   const int e0 = min(tid * per, p.E), e1 = min(e0 + per, p.E);
   int rows = 0, tiles = 0;
@@ -289,7 +292,7 @@ int ti_moe_route(const ti::MoeRouteParams* p, void* stream) {
 int ti_moe_norm_route(const ti::ResidNormParams* r, const ti::MoeRouteParams* p, const void* w, void* slot, void* xs, int f32, void* stream) {
   if (p->M <= 0) return 0;
   if (check_route(p) || r->P % 8 || r->ldy % 8 || r->W > r->P || r->P > 8192 || r->w_next == nullptr || p->row_stride < p->M) return -2;
-  const int threads = std::max(512, (r->P / 8 + 31) / 32 * 32);
+  const int threads = r->P <= 512 ? 256 : 1024;
   const size_t smem = ((size_t)2 * (p->E + p->identity) + p->groups + p->top + r->P) * 4;
   cudaStream_t st = (cudaStream_t)stream;
   static bool configured = false;

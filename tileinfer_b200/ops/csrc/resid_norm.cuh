@@ -22,7 +22,7 @@ struct ResidNormParams {
 
 // KEEP x 8 columns per thread; on return `y` holds the thread's part of h (fp32, before it was stored as T).  `red`: 64
 // floats of shared memory.
-template <typename T, int KEEP, bool ROUTED>
+template <typename T, int KEEP, bool ROUTED, bool FEW = false>
 TI_DEVICE void resid_norm_row(const ResidNormParams& p, int m, float (&y)[KEEP][8], float* red) {
   const int step = blockDim.x * 8;
   float* xr = p.x + (size_t)m * p.P;
@@ -38,7 +38,28 @@ TI_DEVICE void resid_norm_row(const ResidNormParams& p, int m, float (&y)[KEEP][
       load8(static_cast<const T*>(p.y) + (size_t)m * p.ldy + c, y[j]);
     } else {
       float own = 0.f;
-      for (int k = 0; k < p.top; ++k) {
+      int k0 = 0;
+      if (FEW) {                                           // four rows in flight: a chain of loads is all such a step is
+        for (; k0 + 4 <= p.top; k0 += 4) {
+          int sl[4];
+          float a[4], v[4][8];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            sl[k] = p.slot[(size_t)m * p.top + k0 + k];
+            a[k] = p.weight[(size_t)m * p.top + k0 + k];
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k) load8(static_cast<const T*>(p.y) + (size_t)max(sl[k], 0) * p.ldy + c, v[k]);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            own += sl[k] == -1 ? a[k] : 0.f;
+            // a row that is not the token's may hold anything
+#pragma unroll
+            for (int i = 0; i < 8; ++i) y[j][i] = sl[k] < 0 ? y[j][i] : fmaf(a[k], v[k][i], y[j][i]);
+          }
+        }
+      }
+      for (int k = k0; k < p.top; ++k) {
         const int sl = p.slot[(size_t)m * p.top + k];
         const float a = p.weight[(size_t)m * p.top + k];
         if (sl == -1) own += a;

@@ -98,13 +98,13 @@ __global__ void __launch_bounds__(256) rmsnorm_f32_kernel(const float* __restric
 }
 
 // ---------------------------------------------------------------- sublayer output -> residual -> next sublayer's input
-template <typename T, int KEEP, bool ROUTED>
+template <typename T, int KEEP, bool ROUTED, bool FEW>
 __global__ void __launch_bounds__(256) resid_norm_kernel(const __grid_constant__ ResidNormParams p) {
   __shared__ float red[64];
   float y[KEEP][8];
   pdl_trigger();
   pdl_wait();
-  resid_norm_row<T, KEEP, ROUTED>(p, blockIdx.x, y, red);
+  resid_norm_row<T, KEEP, ROUTED, FEW>(p, blockIdx.x, y, red);
 }
 
 // ---------------------------------------------------------------- fp32 matrix product (32-bit mode)
@@ -221,9 +221,10 @@ int ti_resid_norm(const ti::ResidNormParams* p, int M, int f32, void* stream) {
   // one, two, four or eight vectors per thread
   const int threads = p->P >= 2048 ? 256 : (p->P / 8 + 31) / 32 * 32, keep = (p->P / 8 + threads - 1) / threads;
   const dim3 grid(M), block(threads);
-#define TI_RN(T, K)                                                                                  \
-  (p->slot != nullptr ? ti::launch_kernel(ti::resid_norm_kernel<T, K, true>, grid, block, 0, st, true, *p) \
-                      : ti::launch_kernel(ti::resid_norm_kernel<T, K, false>, grid, block, 0, st, true, *p))
+#define TI_RN(T, K)                                                                                                             \
+  (p->slot == nullptr ? ti::launch_kernel(ti::resid_norm_kernel<T, K, false, false>, grid, block, 0, st, true, *p)             \
+   : M <= 512         ? ti::launch_kernel(ti::resid_norm_kernel<T, K, true, true>, grid, block, 0, st, true, *p)               \
+                      : ti::launch_kernel(ti::resid_norm_kernel<T, K, true, false>, grid, block, 0, st, true, *p))
   if (f32) {
     if (keep <= 1) TI_RN(float, 1); else if (keep <= 2) TI_RN(float, 2); else if (keep <= 4) TI_RN(float, 4); else TI_RN(float, 8);
   } else {
