@@ -14,12 +14,10 @@ The residual, norms, router scores, rotations, attention scores, decays and stat
 """
 from __future__ import annotations
 
-import math
-
 import torch
 
 from ..ops import functional as F
-from ..ops.functional import AttnGeneralParams, AttnParams, GlaParams, LinearW, RopeUnitParams, ptr
+from ..ops.functional import AttnGeneralParams, AttnParams, GlaParams, RopeUnitParams, ptr
 from ..utils.trace import nvtx_end, nvtx_mark
 from .gerivik import GLU_ALPHA, GLU_BIAS, GerivikConfig
 from .products_b200 import GroupedProduct, Product, pad64, pad_to
@@ -159,7 +157,7 @@ class B200GatedModel(DeviceRuntime):
 
     def auto_num_blocks(self, util, block_size, num_slots, max_num_seqs, max_model_len) -> int:
         free, total = torch.cuda.mem_get_info()
-        budget = free - (1.0 - util) * total - num_slots * self._state_bytes_per_slot() - (4 << 30)
+        budget = free - (1.0 - util) * total - num_slots * self._state_bytes_per_slot() - (6 << 30)        # room for the activations of a long step
         n = min(int(budget // max(1, self._bytes_per_block())), max_num_seqs * (max_model_len // block_size + 2) + 64)
         if n < max_model_len // block_size + 2:
             raise RuntimeError(f"not enough GPU memory for one sequence of {max_model_len} tokens ({n} cache blocks)")

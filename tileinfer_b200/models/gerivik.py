@@ -223,16 +223,16 @@ def stack(pattern: tuple, repeats: int = 1, shared: int = 0) -> tuple:
     return own + tuple(replace(L, weights_of=i) for _ in range(shared) for i, L in enumerate(pattern))
 
 
-def _pattern(heads, kv, dim, gla_heads, gla_vdim, mlp, softcap=30.0):
-    a = GerivikLayer(CappedAttention(heads=heads, kv_heads=kv, dim=dim, vdim=dim, rot_base=1e6, rot_dims=dim // 4, scale=dim ** -0.5,
+def _pattern(heads, kv, dim, gla_heads, gla_vdim, mlp, softcap=40.0):
+    a = GerivikLayer(CappedAttention(heads=heads, kv_heads=kv, dim=dim, vdim=dim, rot_base=5e5, rot_dims=dim // 4, scale=dim ** -0.5,
                                      softcap=softcap), mlp)
-    g = GerivikLayer(GatedLinearAttention(heads=gla_heads, dim=dim, vdim=gla_vdim, tau=16.0), mlp)
+    g = GerivikLayer(GatedLinearAttention(heads=gla_heads, dim=dim, vdim=gla_vdim, tau=12.0), mlp)
     return (g, g, a, g)
 
 
 TINY = GerivikConfig(
     name="tiny-gerivik", vocab_size=1024, hidden_size=256, rms_eps=1e-6, embedding_scale=16.0, max_position_embeddings=8192,
-    layers=stack(_pattern(4, 2, 64, 2, 128, RoutedExperts(experts=14, identity=2, top=3, groups=4, keep=2, ff=128, limit=7.0)), shared=1),
+    layers=stack(_pattern(6, 2, 64, 3, 128, RoutedExperts(experts=14, identity=2, top=3, groups=4, keep=2, ff=128, limit=7.0)), shared=1),
     eos_token_ids=(1023,))
 
 # Layers of the size of a few-billion-parameter models; the benchmark takes as many as it needs.
