@@ -48,17 +48,19 @@ class CheckpointWeights:
 
 
 class RandomWeights:
-    """Deterministic weights of the architecture: every tensor has its own generator stream.  Norm weights are 1; the
-    N(0, 1) draws of the others go through `scale_of(name, shape)` and are rounded to bf16."""
+    """Deterministic weights of the architecture: every tensor has its own generator stream.  Norm weights are 1
+    (those that `zero_norm(name)` says are stored around zero: 0); the N(0, 1) draws of the others go through
+    `scale_of(name, shape)` and are rounded to bf16."""
 
-    def __init__(self, cfg, seed: int, device, scale_of):
+    def __init__(self, cfg, seed: int, device, scale_of, zero_norm=None):
         self.cfg, self.seed, self.device, self._scale_of = cfg, seed, torch.device(device), scale_of
+        self._zero_norm = zero_norm or (lambda name: False)
         self._shapes = cfg.tensor_shapes()
 
     def get(self, name: str) -> torch.Tensor:
         shape = self._shapes[name]
         if "norm" in name.rsplit(".", 1)[-1]:
-            return torch.ones(shape, dtype=torch.float32, device=self.device)
+            return torch.full(shape, 0.0 if self._zero_norm(name) else 1.0, dtype=torch.float32, device=self.device)
         # small tensors come from the CPU generator so that CPU and GPU runs see the same weights
         numel = 1
         for n in shape:
@@ -70,10 +72,10 @@ class RandomWeights:
         return w.to(torch.bfloat16).float().to(self.device)
 
 
-def make_source(cfg, spec: str, model_dir, device, scale_of):
+def make_source(cfg, spec: str, model_dir, device, scale_of, zero_norm=None):
     """`spec` is "random:<seed>" or "hf" (a checkpoint folder)."""
     if spec.startswith("random"):
-        return RandomWeights(cfg, int(spec.split(":", 1)[1]) if ":" in spec else 0, device, scale_of)
+        return RandomWeights(cfg, int(spec.split(":", 1)[1]) if ":" in spec else 0, device, scale_of, zero_norm)
     if spec == "hf":
         return CheckpointWeights(cfg, model_dir, device)
     raise ValueError(f"unknown weights spec {spec!r}")

@@ -66,7 +66,20 @@ def _gerivik() -> Family:
     return Family("gerivik", lambda: g.PRESETS, g.ARCHITECTURE, g.load_config, g.make_weights, executor, ("w8a16", "bf16", "fp32"))
 
 
-_MAKERS = {"hybrid": _hybrid, "kabadra": _kabadra, "gerivik": _gerivik}
+def _nogidra() -> Family:
+    from . import nogidra as n
+
+    def executor(device):
+        if device == "cuda":
+            from .mixed_b200 import B200MixedModel
+            return B200MixedModel
+        from .mixed_cpu import TorchMixedModel
+        return TorchMixedModel
+
+    return Family("nogidra", lambda: n.PRESETS, n.ARCHITECTURE, n.load_config, n.make_weights, executor, ("w8a16", "bf16", "fp32"))
+
+
+_MAKERS = {"hybrid": _hybrid, "kabadra": _kabadra, "gerivik": _gerivik, "nogidra": _nogidra}
 
 
 def family(name: str) -> Family:
