@@ -90,6 +90,11 @@ struct AttnGeneralParams {
   unsigned* status;
   int H, G, dp, vp, max_blocks, num_qg, num_blocks, ldo;
   float scale, softcap;    // softcap 0: none
+  int window;              // keys seen, the token itself included (0: all earlier ones)
+  const float* slopes;     // null, or [H]: taken off a score per token of distance
+  const void* head_gate;   // null, or [T, ldg]: the sigmoid of column gcol + h scales head h
+  int ldg, gcol;
+  float out_scale;         // factor of the output
 };
 
 // One query token and head per block; the four warps take the pages in turn and keep running maxima, sums and outputs.
@@ -107,7 +112,9 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const __grid_constant
   float acc[NV], m = -1e30f, l = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) acc[i] = 0.f;
-  for (int pg = warp; pg <= pos >> 4; pg += 4) {
+  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const float slope = p.slopes != nullptr ? p.slopes[h] : 0.f;
+  for (int pg = (lo >> 4) + warp; pg <= pos >> 4; pg += 4) {
     const int blk = p.block_tables[(size_t)seq * p.max_blocks + pg];
     if (!TI_CHECK(blk, p.num_blocks, p.status)) continue;
     const T* kb = static_cast<const T*>(p.kcache) + (((size_t)blk * p.G + g) * 16 + (lane >> 1)) * p.dp;
@@ -120,7 +127,9 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const __grid_constant
     }
     s = (s + __shfl_xor_sync(0xffffffffu, s, 1)) * p.scale;
     if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
-    const bool seen = pg * 16 + (lane >> 1) <= pos;
+    const int key = pg * 16 + (lane >> 1);
+    s -= slope * (float)(pos - key);
+    const bool seen = key <= pos && key >= lo;
     const float mn = fmaxf(m, warp_max(seen ? s : -1e30f));
     const float e = seen ? expf(s - mn) : 0.f, alpha = expf(m - mn);
     l = l * alpha + warp_sum((lane & 1) ? 0.f : e);
@@ -157,12 +166,14 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const __grid_constant
     w[i] = expf(ml[i] - M);
     L += w[i] * ml[4 + i];
   }
+  float f = p.out_scale / L;
+  if (p.head_gate != nullptr) f *= sigmoid_exact(to_f<T>(static_cast<const T*>(p.head_gate)[(size_t)tok * p.ldg + p.gcol + h]));
   T* out = static_cast<T*>(p.out) + (size_t)tok * p.ldo + (size_t)h * p.vp;
   for (int c = threadIdx.x; c < p.vp; c += 128) {
     float o = 0.f;
 #pragma unroll
     for (int i = 0; i < 4; ++i) o = fmaf(w[i], acc_s[i * p.vp + c], o);
-    out[c] = from_f<T>(o / L);
+    out[c] = from_f<T>(o * f);
   }
 }
 
@@ -206,7 +217,7 @@ int ti_rope_unit(const ti::RopeUnitParams* p, int f32, void* stream) {
 
 int ti_attn_general(const ti::AttnGeneralParams* p, int f32, void* stream) {
   if (p->num_qg <= 0) return 0;
-  if (p->dp % 64 || p->vp % 64 || p->H % p->G || p->num_blocks < 1 ||
+  if (p->dp % 64 || p->vp % 64 || p->H % p->G || p->num_blocks < 1 || p->window < 0 ||
       (((uintptr_t)p->kcache | (uintptr_t)p->vcache) & 15))
     return -2;
   return f32 ? ti::launch_general<float>(*p, (cudaStream_t)stream) : ti::launch_general<ti::bf16>(*p, (cudaStream_t)stream);

@@ -16,7 +16,8 @@
 // exp2 domain in registers, O += P V^T.  Pages are dealt round-robin to the warp streams of a CTA and
 // to `nsplit` CTAs (split-KV); a second kernel merges the partial (O, max, sum) triples and applies
 // the sigmoid gate.  All sizes (batch, context, block-table width) are run-time values.  Values may be of another size
-// than queries and keys, scores may be capped by cap * tanh(score / cap), and the gate may be absent.
+// than queries and keys, scores may be capped by cap * tanh(score / cap) or lose a slope per head times the distance of the
+// key, a window may limit the keys, and the gate may be absent, per dimension or per head.
 #include "common.cuh"
 
 namespace ti {
@@ -120,6 +121,11 @@ struct AttnParams {
   unsigned* status;
   float cap_in, cap_out;         // cap_out > 0: score = cap_out * tanh(q.k * cap_in / 2), in log2 units
   int rep;                       // blocks per KV head, each with hq / (hkv * rep) of its query heads
+  int window;                    // keys seen, the token itself included (0: all earlier ones)
+  const float* slopes;           // null, or [hq]: taken off a score per token of distance
+  const __nv_bfloat16* head_gate;// merge: null, or [T, ldg]: gate of head h at column gcol + h
+  int ldg, gcol, ldo;            // ldo: row pitch of `out` (0: hq*D)
+  float out_scale;               // merge: factor of the output
 };
 
 TI_DEVICE float attn_score(const AttnParams& p, float qk) {
@@ -132,7 +138,7 @@ constexpr float kNegBig = -1e30f;
 TI_DEVICE uint4 ldg_nc16(const void* p) { return __ldg(reinterpret_cast<const uint4*>(p)); }
 TI_DEVICE uint2 ldg_nc8(const void* p) { return __ldg(reinterpret_cast<const uint2*>(p)); }
 
-struct PageRange { int seq, tok0, ntok, npages, pps; };
+struct PageRange { int seq, tok0, ntok, page0, npages, pps; };    // pages page0 .. npages - 1
 
 TI_DEVICE PageRange page_range(const AttnParams& p, int qg) {
   PageRange r;
@@ -141,7 +147,8 @@ TI_DEVICE PageRange page_range(const AttnParams& p, int qg) {
   r.tok0 = p.qg_tok0[qg];
   const int kvlen = r.ntok > 0 ? p.positions[r.tok0 + r.ntok - 1] + 1 : 0;
   r.npages = (kvlen + 15) >> 4;
-  r.pps = max(1, (r.npages + p.nsplit - 1) / p.nsplit);
+  r.page0 = p.window > 0 && r.ntok > 0 ? max(0, p.positions[r.tok0] - p.window + 1) >> 4 : 0;
+  r.pps = max(1, (r.npages - r.page0 + p.nsplit - 1) / p.nsplit);
   return r;
 }
 
@@ -317,14 +324,15 @@ __global__ void __launch_bounds__(128) attn_pipe_kernel(const __grid_constant__ 
   pdl_wait();
   const PageRange pr = page_range(p, qg);
   if (pr.ntok == 0) return;
-  const int p0 = sp * pr.pps, p1 = min(pr.npages, p0 + pr.pps);
+  const int p0 = pr.page0 + sp * pr.pps, p1 = min(pr.npages, p0 + pr.pps);
   if (p0 >= p1) return;
   const int G = p.hq / (p.hkv * p.rep), kvh = kh / p.rep;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const int stream = warp / DSPLIT, dpart = warp % DSPLIT;
   const int st_tid = tid - stream * TS;                 // thread index inside the stream
 
-  int pos[2];
+  int pos[2], lo[2];                                     // last and first key of a row
+  float slope[2];                                        // in log2 units
   uint32_t qf[2][NCH][4];
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
@@ -332,6 +340,8 @@ __global__ void __launch_bounds__(128) attn_pipe_kernel(const __grid_constant__ 
     const int tk = r / G, hg = r - tk * G;
     const bool valid = tk < pr.ntok;
     pos[h] = valid ? p.positions[pr.tok0 + tk] : -1;
+    lo[h] = p.window > 0 ? pos[h] - p.window + 1 : 0;
+    slope[h] = valid && p.slopes != nullptr ? p.slopes[kh * G + hg] * 1.4426950408889634f : 0.f;
     const __nv_bfloat16* qrow = p.q + ((size_t)(pr.tok0 + (valid ? tk : 0)) * p.hq + kh * G + hg) * D;
 #pragma unroll
     for (int i = 0; i < NCH; ++i) {
@@ -402,7 +412,7 @@ __global__ void __launch_bounds__(128) attn_pipe_kernel(const __grid_constant__ 
       float mx = kNegBig;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        sc[e] = (j0 + e <= pos[h]) ? attn_score(p, sc[e]) : kNegBig;
+        sc[e] = (j0 + e <= pos[h] && j0 + e >= lo[h]) ? attn_score(p, sc[e]) - slope[h] * (float)(pos[h] - j0 - e) : kNegBig;
         mx = fmaxf(mx, sc[e]);
       }
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
@@ -483,7 +493,7 @@ __global__ void __launch_bounds__(D / 2) attn_merge_kernel(const __grid_constant
   const PageRange pr = page_range(p, qg);
   const int G = p.hq / (p.hkv * p.rep);
   if (pr.ntok == 0 || r >= pr.ntok * G) return;
-  const int nact = (pr.npages + pr.pps - 1) / pr.pps;
+  const int nact = (pr.npages - pr.page0 + pr.pps - 1) / pr.pps;
   const size_t item0 = ((size_t)qg * p.hkv * p.rep + kh) * p.nsplit;
   for (int s = tid; s < nact; s += D / 2) {
     const float2 ml = *reinterpret_cast<const float2*>(p.ml_part + ((item0 + s) * 16 + r) * 2);
@@ -512,14 +522,15 @@ __global__ void __launch_bounds__(D / 2) attn_merge_kernel(const __grid_constant
   }
   const int tk = r / G, hg = r - tk * G;
   const int tok = pr.tok0 + tk, head = kh * G + hg;
-  const float inv = 1.f / L;
+  float inv = p.out_scale / L;
+  if (p.head_gate != nullptr) inv *= sigmoid_f(__bfloat162float(p.head_gate[(size_t)tok * p.ldg + p.gcol + head]));
   float g0 = 1.f, g1 = 1.f;
   if (p.gate_src != nullptr) {
     const uint32_t gw = *reinterpret_cast<const uint32_t*>(p.gate_src + (size_t)tok * p.ld + (size_t)head * 2 * D + D + d);
     g0 = sigmoid_f(bf16lo(gw));
     g1 = sigmoid_f(bf16hi(gw));
   }
-  *reinterpret_cast<uint32_t*>(p.out + (size_t)tok * p.hq * D + (size_t)head * D + d) =
+  *reinterpret_cast<uint32_t*>(p.out + (size_t)tok * (p.ldo > 0 ? p.ldo : p.hq * D) + (size_t)head * D + d) =
       pack_bf16(a0 * inv * g0, a1 * inv * g1);
 }
 
@@ -557,11 +568,12 @@ int ti_qkv_prep(const ti::QkvPrepParams* p, int T, int D, void* stream) {
 
 // Launches the split-KV attention kernel and the merge/gate kernel.  D: size of a query / key head, DV of a value head.
 // The cp.async-pipelined kernel is the default (measured faster from batch 1 / 256 tokens of context to batch 64 / 8192);
-// TI_ATTN_PIPE=0 selects the direct-load kernel, which takes neither a cap nor values of another size.
+// TI_ATTN_PIPE=0 selects the direct-load kernel, which takes neither a cap, a window or slopes nor values of another size.
 int ti_attn_paged(const ti::AttnParams* p, int D, int DV, void* stream) {
   if (p->num_qg <= 0) return 0;
   const int rep = p->rep < 1 ? 1 : p->rep;
   if (p->hq % (p->hkv * rep) || p->hq / (p->hkv * rep) > 16 || p->nsplit < 1 || p->nsplit > ti::kMaxSplit) return -2;
+  if (p->window < 0 || p->ldo % 2 || (p->gate_src != nullptr && D != DV)) return -2;
   ti::AttnParams a = *p;
   a.rep = rep;
   dim3 grid(p->num_qg, p->hkv * rep, p->nsplit), mgrid(p->num_qg, p->hkv * rep, 16);
@@ -570,7 +582,7 @@ int ti_attn_paged(const ti::AttnParams* p, int D, int DV, void* stream) {
     const char* e = getenv("TI_ATTN_PIPE");
     return e == nullptr ? -1 : atoi(e);
   }();
-  if (pipe_mode == 0 && D == DV && rep == 1 && !(p->cap_out > 0.f)) {
+  if (pipe_mode == 0 && D == DV && rep == 1 && !(p->cap_out > 0.f) && p->window <= 0 && p->slopes == nullptr) {
     if (D == 256) ti::launch_kernel(ti::attn_kernel<256, 2>, grid, dim3(128), 0, st, true, a);
     else if (D == 128) ti::launch_kernel(ti::attn_kernel<128, 1>, grid, dim3(128), 0, st, true, a);
     else if (D == 64) ti::launch_kernel(ti::attn_kernel<64, 1>, grid, dim3(128), 0, st, true, a);

@@ -62,13 +62,15 @@ template <int BN, bool BF16, int BMH = 1, int RK = TI_GEMM_RING_KB> struct GemmG
 };
 constexpr unsigned long long kGemmWaitNs = 2000000000ull;
 
-// Operands of the epilogues for designs with an fp32 residual stream, a clamped gated unit or scaled logits.
+// Operands of the epilogues for designs with an fp32 residual stream, a clamped gated unit, biases, scaled or capped logits.
 struct GemmEpilogue {
   const float* resid32;            // RESID32: [M, ldo] fp32
   __nv_bfloat16* out2;             // SPLIT_GLU: [M, ldo2], column (n - n_split) / 2 of the (gate, up) row pairs
   int ldo2, n_split;               // SPLIT_GLU: rows below n_split are stored as they are, the others are pairs
   float scale;                     // F32: factor of the stored values
   float glu_limit, glu_alpha, glu_bias;   // g = min(g, limit), u = clamp(u, +-limit): g sigmoid(alpha g) (u + bias)
+  float softcap;                   // F32: > 0 stores softcap * tanh(value / softcap)
+  const float* bias;               // null, or [N]: added to the product before anything else
 };
 
 struct GemmParams {
@@ -112,8 +114,17 @@ TI_DEVICE float clamped_glu(const GemmEpilogue& e, float g, float u) {
   return g * sigmoid_f(e.glu_alpha * g) * (u + e.glu_bias);
 }
 
+TI_DEVICE float f32_value(const GemmEpilogue& e, float v) {
+  v *= e.scale;
+  return e.softcap > 0.f ? e.softcap * tanhf(v / e.softcap) : v;
+}
+
 // fused epilogue for four adjacent weight rows n..n+3 of one token (N is a multiple of 4 here): split-k reduction
 TI_DEVICE void gemm_epilogue4(const GemmParams& p, int m, int n, float4 v, uint2 r, float4 r32) {
+  if (p.ex.bias != nullptr) {
+    const float4 b = *reinterpret_cast<const float4*>(p.ex.bias + n);
+    v = make_float4(v.x + b.x, v.y + b.y, v.z + b.z, v.w + b.w);
+  }
   if (p.epi == GEPI_RESID32) {
     *reinterpret_cast<float4*>(static_cast<float*>(p.out) + (size_t)m * p.ldo + n) =
         make_float4(v.x + r32.x, v.y + r32.y, v.z + r32.z, v.w + r32.w);
@@ -131,8 +142,8 @@ TI_DEVICE void gemm_epilogue4(const GemmParams& p, int m, int n, float4 v, uint2
     return;
   }
   if (p.epi == GEPI_F32) {
-    const float sc = p.ex.scale;
-    *reinterpret_cast<float4*>(static_cast<float*>(p.out) + (size_t)m * p.ldo + n) = make_float4(v.x * sc, v.y * sc, v.z * sc, v.w * sc);
+    *reinterpret_cast<float4*>(static_cast<float*>(p.out) + (size_t)m * p.ldo + n) =
+        make_float4(f32_value(p.ex, v.x), f32_value(p.ex, v.y), f32_value(p.ex, v.z), f32_value(p.ex, v.w));
     return;
   }
   if (p.epi == GEPI_ROWPAR) {                      // r: the residual row's four values, loaded by the caller
@@ -147,7 +158,12 @@ TI_DEVICE void gemm_epilogue4(const GemmParams& p, int m, int n, float4 v, uint2
 
 // Eight adjacent weight rows n..n+7 (n a multiple of 8) of one token, straight from the accumulators: split-k
 // partial (fp32), or the fused epilogue.  Rows past N and rows that cannot be stored as one vector go one by one.
-TI_DEVICE void gemm_store8(const GemmParams& p, int m, int n, const float4 a, const float4 b, int S, int split) {
+TI_DEVICE void gemm_store8(const GemmParams& p, int m, int n, float4 a, float4 b, int S, int split) {
+  if (S == 1 && p.ex.bias != nullptr) {            // N is a multiple of 8 here; with a split the reduction adds it
+    const float4 c = __ldg(reinterpret_cast<const float4*>(p.ex.bias + n)), d = __ldg(reinterpret_cast<const float4*>(p.ex.bias + n + 4));
+    a = make_float4(a.x + c.x, a.y + c.y, a.z + c.z, a.w + c.w);
+    b = make_float4(b.x + d.x, b.y + d.y, b.z + d.z, b.w + d.w);
+  }
   const float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
   if (S > 1) {
     float* dst = p.part + ((size_t)split * p.M + m) * p.N + n;
@@ -174,12 +190,14 @@ TI_DEVICE void gemm_store8(const GemmParams& p, int m, int n, const float4 a, co
   }
   if (p.epi == GEPI_F32) {
     float* dst = static_cast<float*>(p.out) + (size_t)m * p.ldo + n;
-    const float sc = p.ex.scale;
+    float o[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) o[i] = f32_value(p.ex, v[i]);
     if (full && (p.ldo & 3) == 0 && (reinterpret_cast<uintptr_t>(p.out) & 15) == 0) {
-      *reinterpret_cast<float4*>(dst) = make_float4(a.x * sc, a.y * sc, a.z * sc, a.w * sc);
-      *reinterpret_cast<float4*>(dst + 4) = make_float4(b.x * sc, b.y * sc, b.z * sc, b.w * sc);
+      *reinterpret_cast<float4*>(dst) = make_float4(o[0], o[1], o[2], o[3]);
+      *reinterpret_cast<float4*>(dst + 4) = make_float4(o[4], o[5], o[6], o[7]);
     } else {
-      for (int i = 0; i < 8 && n + i < p.N; ++i) dst[i] = v[i] * sc;
+      for (int i = 0; i < 8 && n + i < p.N; ++i) dst[i] = o[i];
     }
     return;
   }
@@ -576,6 +594,7 @@ static int set_epilogue(GemmParams& p, const GemmEpilogue* ex) {
   p.ex.scale = 1.f;
   if (ex != nullptr) p.ex = *ex;
   if (p.epi == GEPI_RESID32 && (p.ex.resid32 == nullptr || p.N % 8 || p.ldo % 8 || ((uintptr_t)p.out | (uintptr_t)p.ex.resid32) % 16)) return -2;
+  if (p.ex.bias != nullptr && (p.N % 8 || (uintptr_t)p.ex.bias % 16)) return -2;
   if (p.epi == GEPI_SPLIT_GLU && (p.ex.out2 == nullptr || p.N % 8 || p.ex.n_split % 8 || p.ex.ldo2 % 4 || (uintptr_t)p.ex.out2 % 8)) return -2;
   return 0;
 }

@@ -1,5 +1,5 @@
-// Routing of tokens to experts: softmax scores over experts and identity experts, a corrected choice inside the best
-// groups of neighbouring experts, and the layout the grouped products work on (gemm_grouped.cu).
+// Routing of tokens to experts: softmax scores over experts and identity experts (or over the chosen ones alone), an
+// optionally corrected choice inside the best groups of neighbouring experts, and the layout the grouped products work on (gemm_grouped.cu).
 //
 // `moe_route_kernel` takes a warp per token, from logits that a product has computed.  `moe_norm_route_kernel`, for few
 // tokens, is a block per token that first finishes the sublayer before (norm, residual add, next norm), computes the
@@ -15,7 +15,7 @@ namespace ti {
 
 struct MoeRouteParams {
   const float* logits;     // [M][ldl], E + identity columns
-  const float* correction; // [E + identity]
+  const float* correction; // [E + identity], or null: the weights are a softmax over the chosen logits alone
   const long long* valid;  // null, or [M]: tokens with a negative entry go nowhere (padding of captured steps)
   int* ids;                // [M][top] chosen expert (>= E: identity; -1: token goes nowhere)
   float* weight;           // [M][top] its score
@@ -62,14 +62,18 @@ TI_DEVICE void route_token(const MoeRouteParams& p, int m, float* s, unsigned* k
   float mx = __int_as_float(0xff800000), sum = 0.f;
   for (int e = lane; e < n; e += 32) mx = fmaxf(mx, s[e]);
   mx = warp_max(mx);
+  const bool chosen_only = p.correction == nullptr;
   for (int e = lane; e < n; e += 32) {
+    if (chosen_only) key[e] = order_key(s[e]);
     s[e] = expf(s[e] - mx);
     sum += s[e];
   }
-  sum = warp_sum(sum);
-  for (int e = lane; e < n; e += 32) {
-    s[e] = s[e] / sum;
-    key[e] = order_key(s[e] + p.correction[e]);            // corrected scores may be negative
+  if (!chosen_only) {
+    sum = warp_sum(sum);
+    for (int e = lane; e < n; e += 32) {
+      s[e] = s[e] / sum;
+      key[e] = order_key(s[e] + p.correction[e]);          // corrected scores may be negative
+    }
   }
   __syncwarp();
   unsigned best;
@@ -92,12 +96,18 @@ TI_DEVICE void route_token(const MoeRouteParams& p, int m, float* s, unsigned* k
     if (lane == 0) sel[k] = e;
   }
   __syncwarp();
+  float total = 1.f;
+  if (chosen_only) {                                       // the largest logit is among the chosen ones: total >= 1
+    total = 0.f;
+    for (int k = lane; k < p.top; k += 32) total += s[sel[k]];
+    total = warp_sum(total);
+  }
   const bool goes = p.valid == nullptr || p.valid[m] >= 0;
   for (int k = lane; k < p.top; k += 32) {
     const int e = sel[k];
     const size_t o = (size_t)m * p.top + k;
     p.ids[o] = goes ? e : -1;
-    p.weight[o] = s[e];
+    p.weight[o] = s[e] / total;
     const int pos = goes && e < p.E ? atomicAdd(counts + e, 1) : 0;
     p.pos[o] = pos;
     if (p.row_stride > 0) sel[k] = !goes ? -2 : e >= p.E ? -1 : e * p.row_stride + pos;

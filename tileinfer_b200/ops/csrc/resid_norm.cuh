@@ -4,13 +4,14 @@
 
 namespace ti {
 
-// x[m] += rmsnorm(y[m]) * w_out, then h[m] = rmsnorm(x[m]) * w_next (w_next null: no h).  y[m] is a row, or, with `slot`,
+// x[m] += rmsnorm(y[m]) * w_out (w_out null: x[m] += y[m]; y null as well: x stays), then h[m] = rmsnorm(x[m]) * w_next
+// (w_next null: no h).  y[m] is a row, or, with `slot`,
 // the weighted sum over k < top of the rows slot[m, k] of y plus the input row h_in[m] times the weights whose slot is
 // negative (-1; -2 adds nothing).
 struct ResidNormParams {
-  const void* y;           // [rows][ldy]
+  const void* y;           // [rows][ldy] or null
   float* x;                // [M][P]
-  const float* w_out;      // [P]
+  const float* w_out;      // [P] or null
   const float* w_next;     // [P] or null
   void* h;                 // [M][P]
   const int* slot;         // [M][top] or null
@@ -35,7 +36,7 @@ TI_DEVICE void resid_norm_row(const ResidNormParams& p, int m, float (&y)[KEEP][
     if (c >= p.P) continue;
     if (!ROUTED) {
       load8(xr + c, x[j]);
-      load8(static_cast<const T*>(p.y) + (size_t)m * p.ldy + c, y[j]);
+      if (p.y != nullptr) load8(static_cast<const T*>(p.y) + (size_t)m * p.ldy + c, y[j]);
     } else {
       float own = 0.f;
       int k0 = 0;
@@ -79,7 +80,8 @@ TI_DEVICE void resid_norm_row(const ResidNormParams& p, int m, float (&y)[KEEP][
 #pragma unroll
     for (int i = 0; i < 8; ++i) ss += y[j][i] * y[j][i];
   }
-  const float ry = rsqrtf(block_sum32(ss, red) / (float)p.W + p.eps);
+  const bool normed = p.w_out != nullptr;                  // uniform over the grid
+  const float ry = normed ? rsqrtf(block_sum32(ss, red) / (float)p.W + p.eps) : 1.f;
   ss = 0.f;
 #pragma unroll
   for (int j = 0; j < KEEP; ++j) {
@@ -87,13 +89,17 @@ TI_DEVICE void resid_norm_row(const ResidNormParams& p, int m, float (&y)[KEEP][
     if (c >= p.P) continue;
     float g[8];
     if (ROUTED) load8(xr + c, x[j]);                       // later: the sum above needs the registers
-    load8(p.w_out + c, g);
+    if (normed) {
+      load8(p.w_out + c, g);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[j][i] *= ry * g[i];
+    }
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
-      y[j][i] = x[j][i] + y[j][i] * ry * g[i];
+      y[j][i] = x[j][i] + y[j][i];
       ss += y[j][i] * y[j][i];
     }
-    store8(xr + c, y[j]);
+    if (p.y != nullptr) store8(xr + c, y[j]);
   }
   if (p.w_next == nullptr) return;
   const float rx = rsqrtf(block_sum32(ss, red + 32) / (float)p.W + p.eps);

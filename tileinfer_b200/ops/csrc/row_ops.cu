@@ -122,6 +122,8 @@ struct GemmF32Params {
   const int* tiles;
   const int* num_tiles;
   int max_tiles;
+  float softcap;        // epi 3: > 0 stores softcap * tanh(value / softcap)
+  const float* bias;    // null, or [N]
 };
 
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ GemmF32Params p) {
@@ -166,6 +168,10 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
     for (int j = 0; j < 4; j += 2) {
       const int n = n0 + tx * 4 + j;
       if (n >= p.N) continue;
+      if (p.bias != nullptr) {
+        acc[i][j] += p.bias[n];
+        if (n + 1 < p.N) acc[i][j + 1] += p.bias[n + 1];
+      }
       if (p.epi == 5 && n >= p.n_split) {               // (gate, up) pair
         const float g = fminf(acc[i][j], p.glu_limit), u = fminf(fmaxf(acc[i][j + 1], -p.glu_limit), p.glu_limit);
         p.out2[(size_t)m * p.ldo2 + ((n - p.n_split) >> 1)] = g * sigmoid_exact(p.glu_alpha * g) * (u + p.glu_bias);
@@ -175,7 +181,12 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
       for (int e = 0; e < 2; ++e) {
         if (n + e >= p.N) continue;
         const size_t at = (size_t)m * p.ldo + n + e;
-        p.out[at] = p.epi == 4 ? p.resid[at] + acc[i][j + e] : acc[i][j + e] * p.scale;
+        if (p.epi == 4) {
+          p.out[at] = p.resid[at] + acc[i][j + e];
+        } else {
+          const float v = acc[i][j + e] * p.scale;
+          p.out[at] = p.softcap > 0.f ? p.softcap * tanhf(v / p.softcap) : v;
+        }
       }
     }
   }
@@ -236,11 +247,11 @@ int ti_resid_norm(const ti::ResidNormParams* p, int M, int f32, void* stream) {
 
 int ti_gemm_f32(const void* w, const void* x, const void* resid, void* out, void* out2, int M, int N, int K, int ldx, int ldo,
                 int ldo2, int n_split, int epi, float scale, float glu_limit, float glu_alpha, float glu_bias, const void* tiles,
-                const void* num_tiles, int max_tiles, void* stream) {
+                const void* num_tiles, int max_tiles, float softcap, const void* bias, void* stream) {
   if (M <= 0) return 0;
   if (K % 16 || ldx % 4 || n_split % 2 || (epi != 3 && epi != 4 && epi != 5)) return -2;
   ti::GemmF32Params p = {(const float*)w, (const float*)x, (const float*)resid, (float*)out, (float*)out2, M, N, K, ldx, ldo,
-                         ldo2, n_split, epi, scale, glu_limit, glu_alpha, glu_bias, (const int*)tiles, (const int*)num_tiles, max_tiles};
+                         ldo2, n_split, epi, scale, glu_limit, glu_alpha, glu_bias, (const int*)tiles, (const int*)num_tiles, max_tiles, softcap, (const float*)bias};
   ti::launch_kernel(ti::gemm_f32_kernel, dim3((N + 63) / 64, tiles != nullptr ? max_tiles : (M + 63) / 64), dim3(256), 0, (cudaStream_t)stream, true, p);
   return (int)cudaGetLastError();
 }
