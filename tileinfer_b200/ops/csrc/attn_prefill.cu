@@ -18,7 +18,9 @@
 //
 // TMEM: S0 | S1 | O = 128 + 128 + D columns (512 allocated).  Shared memory at D = 256: Q 64 KB, K 64 KB,
 // V 64 KB, P 32 KB.  Causal alignment is by absolute position (bottom-right): a chunk that continues a cached
-// prefix sees all of it.  Values may be of another size than queries and keys, and the gate may be absent.  Scores may be
+// prefix sees all of it.  Values may be of another size than queries and keys; the gate may be absent, per dimension or per
+// head.  A window limits the keys (the walk starts at the page of the first one any row sees), and scores may lose a slope
+// per head times the distance of the key.  Scores may be
 // capped by cap * tanh(score / cap); where |score / cap| is known to stay small (normalised queries and keys) the tanh is
 // its power series and the softmax needs no running maximum at all: exp2 of a bounded score neither overflows nor
 // vanishes, so the scores of a tile are read once, two threads can share a query row (eight softmax warps, half of the keys
@@ -43,10 +45,16 @@ struct AttnPrefillParams {
   int hq, hkv, max_blocks, ld;
   float scale_log2e;
   float cap_in, cap_out;           // score = cap_out * tanh(q.k * cap_in), in log2 units
+  int window;                      // keys seen, the token itself included (0: all earlier ones)
+  const float* slopes;             // BIASED: [hq], taken off a score per token of distance
+  const __nv_bfloat16* head_gate;  // null, or [T, ldg]: gate of head h at column gcol + h
+  int ldg, gcol, ldo;              // ldo: row pitch of `out`
+  float out_scale;
 };
 
-// How a score follows from q.k: scaled; capped with the series, reference 0 instead of a running maximum; capped
-enum { SCORE_PLAIN = 0, SCORE_SERIES = 1, SCORE_CAPPED = 2 };
+// How a score follows from q.k: scaled; capped with the series, reference 0 instead of a running maximum; capped; scaled,
+// minus a slope times the distance
+enum { SCORE_PLAIN = 0, SCORE_SERIES = 1, SCORE_CAPPED = 2, SCORE_BIASED = 3 };
 constexpr float kSeriesMax = 0.4f;       // largest |argument| the series serves (error below 1e-7 there)
 
 // Packed pairs of floats
@@ -96,7 +104,9 @@ struct TanhSeries {
     return fma2(mul2(u, a), y, y);
   }
 };
-template <int MODE> TI_DEVICE float prefill_score(const AttnPrefillParams& p, float qk) {
+// `ahead`: slope times (key - query) in log2 units
+template <int MODE> TI_DEVICE float prefill_score(const AttnPrefillParams& p, float qk, float ahead) {
+  if (MODE == SCORE_BIASED) return fmaf(qk, p.scale_log2e, ahead);
   if (MODE == SCORE_CAPPED) return p.cap_out * (1.f - __fdividef(2.f, 1.f + ex2_approx(qk * p.cap_in * 2.8853900817779268f)));
   return qk * p.scale_log2e;
 }
@@ -105,6 +115,7 @@ constexpr unsigned long long kAttnWaitNs = 500000000ull;
 constexpr int kAttnThreads = 224;        // warp 0: Q/K producer, 1: MMA issuer, 2..5: softmax, 6: V producer
 constexpr int kAttnProducerV = 6;
 constexpr float kMaskVal = -1e30f;
+constexpr float kFirstMax = -1e29f;      // a row may see no key of its first tile: exp2(kMaskVal - kFirstMax) is 0
 constexpr float kRescaleGap = 8.f;       // log2 units the running maximum may lag behind before O is rescaled
 
 template <int D, int DV, int MODE> struct AttnPrefillGeom {
@@ -123,6 +134,11 @@ template <int D, int DV, int MODE> struct AttnPrefillGeom {
   // one CTA per SM (the kernel takes all 512 TMEM columns)
   static constexpr size_t kSmem = kNeeded > 120 * 1024 ? kNeeded : 120 * 1024;
 };
+
+// What scales a head's output beside 1 / l
+TI_DEVICE float head_factor(const AttnPrefillParams& p, size_t tok, int head) {
+  return p.head_gate == nullptr ? p.out_scale : p.out_scale * sigmoid_f(__bfloat162float(p.head_gate[tok * p.ldg + p.gcol + head]));
+}
 
 // 32 output columns of a row: times 1 / l and the sigmoid gate, as bf16
 TI_DEVICE void store_rows32(const AttnPrefillParams& p, const uint32_t (&v)[32], float inv, const __nv_bfloat16* gate, __nv_bfloat16* dst, int c) {
@@ -167,8 +183,9 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
   const int seq = p.qt_seq[tile], tok0 = p.qt_tok0[tile];
   const int kh = head / (p.hq / p.hkv);
   const int kv_len = p.positions[tok0 + ntok - 1] + 1;
+  const int page0 = p.window > 0 ? max(0, p.positions[tok0] - p.window + 1) >> 4 : 0, first = page0 * 16;    // first key of the walk
   const int npages = (kv_len + 15) >> 4;
-  const int ntiles = (kv_len + 127) >> 7;
+  const int ntiles = (kv_len - first + 127) >> 7;
 
   if (threadIdx.x == 0) {
     s_abort = 0;
@@ -208,7 +225,7 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
         for (int j = 0; j < ntiles && !*abort_flag; ++j) {
           int blk[8];
 #pragma unroll
-          for (int g = 0; g < 8; ++g) blk[g] = bt[min(j * 8 + g, npages - 1)];   // pages past the end repeat the last one (masked)
+          for (int g = 0; g < 8; ++g) blk[g] = bt[min(page0 + j * 8 + g, npages - 1)];   // pages past the end repeat the last one (masked)
           if (j > 0 && !mbar_wait(k_empty, (uint32_t)((j - 1) & 1), kAttnWaitNs, p.status)) { *abort_flag = 1; break; }
           mbar_expect_tx(k_full, G::kKBytes);
 #pragma unroll
@@ -219,7 +236,7 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
         for (int j = 0; j < ntiles && !*abort_flag; ++j) {
           int blk[8];
 #pragma unroll
-          for (int g = 0; g < 8; ++g) blk[g] = bt[min(j * 8 + g, npages - 1)];
+          for (int g = 0; g < 8; ++g) blk[g] = bt[min(page0 + j * 8 + g, npages - 1)];
           if (j > 0 && !mbar_wait(v_empty, (uint32_t)((j - 1) & 1), kAttnWaitNs, p.status)) { *abort_flag = 1; break; }
           mbar_expect_tx(v_full, G::kVBytes);
 #pragma unroll
@@ -332,10 +349,10 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
       asm volatile("bar.sync 1, 256;\n" ::: "memory");
       if (ok) {
         tc_fence_after();
-        const float inv = 1.f / (l_s[r] + l_s[128 + r]);
         const size_t tok = (size_t)tok0 + (valid ? r : 0);
+        const float inv = head_factor(p, tok, head) / (l_s[r] + l_s[128 + r]);
         const __nv_bfloat16* gate = p.gate_src + tok * p.ld + (size_t)head * 2 * D + D;
-        __nv_bfloat16* dst = p.out + tok * ((size_t)p.hq * DV) + (size_t)head * DV;
+        __nv_bfloat16* dst = p.out + tok * (size_t)p.ldo + (size_t)head * DV;
 #pragma unroll 1
         for (int c = half * (DV / 64); c < (half + 1) * (DV / 64); ++c) {
           uint32_t v[32];
@@ -352,8 +369,10 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
     const int r = quarter * 32 + lane;
     const bool valid = r < ntok;
     const int pos = p.positions[tok0 + (valid ? r : ntok - 1)];
+    const int lo = p.window > 0 ? pos - p.window + 1 : 0;
+    const float slope = MODE == SCORE_BIASED ? p.slopes[head] * 1.4426950408889634f : 0.f;
     const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
-    float m_used = kMaskVal, l = 0.f;
+    float m_used = kFirstMax, l = 0.f;
     bool ok = true;
     for (int j = 0; j < ntiles; ++j) {
       ok = ok && !*abort_flag && mbar_wait(s_full0 + 8 * (j & 1), (uint32_t)((j >> 1) & 1), kAttnWaitNs, p.status);
@@ -361,8 +380,9 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
       if (!ok) break;
       tc_fence_after();
       const uint32_t s_addr = lane_base + (uint32_t)(j & 1) * 128u;
-      const int key0 = j * 128;
-      const bool need_mask = key0 + 127 > pos;
+      const int key0 = first + j * 128, from = lo - key0, to = pos - key0;       // the row sees keys from .. to of the tile
+      const bool need_mask = to < 127 || from > 0;
+      const float ahead = slope * (float)-to;
       // ---- pass 1: row maximum
       float mx = kMaskVal;
 #pragma unroll
@@ -372,8 +392,8 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
         tmem_ld_wait();
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
-          float s = prefill_score<MODE>(p, __uint_as_float(v[i]));
-          if (need_mask && key0 + c * 32 + i > pos) s = kMaskVal;
+          float s = prefill_score<MODE>(p, __uint_as_float(v[i]), fmaf(slope, (float)(c * 32 + i), ahead));
+          if (need_mask && (c * 32 + i > to || c * 32 + i < from)) s = kMaskVal;
           mx = fmaxf(mx, s);
         }
       }
@@ -414,10 +434,11 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          float s0 = prefill_score<MODE>(p, __uint_as_float(v[i])), s1 = prefill_score<MODE>(p, __uint_as_float(v[i + 1]));
+          float s0 = prefill_score<MODE>(p, __uint_as_float(v[i]), fmaf(slope, (float)(c * 32 + i), ahead));
+          float s1 = prefill_score<MODE>(p, __uint_as_float(v[i + 1]), fmaf(slope, (float)(c * 32 + i + 1), ahead));
           if (need_mask) {
-            if (key0 + c * 32 + i > pos) s0 = kMaskVal;
-            if (key0 + c * 32 + i + 1 > pos) s1 = kMaskVal;
+            if (c * 32 + i > to || c * 32 + i < from) s0 = kMaskVal;
+            if (c * 32 + i + 1 > to || c * 32 + i + 1 < from) s1 = kMaskVal;
           }
           const float p0 = exp2f(s0 - m_used), p1 = exp2f(s1 - m_used);
           sum += p0 + p1;
@@ -444,10 +465,10 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
     }
     if (ok) {
       tc_fence_after();
-      const float inv = 1.f / l;
       const size_t tok = (size_t)tok0 + (valid ? r : 0);
+      const float inv = head_factor(p, tok, head) / l;
       const __nv_bfloat16* gate = p.gate_src + tok * p.ld + (size_t)head * 2 * D + D;
-      __nv_bfloat16* dst = p.out + tok * ((size_t)p.hq * DV) + (size_t)head * DV;
+      __nv_bfloat16* dst = p.out + tok * (size_t)p.ldo + (size_t)head * DV;
 #pragma unroll 1
       for (int c = 0; c < DV / 32; ++c) {
         uint32_t v[32];
@@ -485,8 +506,8 @@ template <int D, int DV>
 static int launch_attn_prefill(const AttnPrefillParams& p, int num_tiles, int mode, cudaStream_t st) {
   if (mode == SCORE_SERIES) return launch_mode<D, DV, SCORE_SERIES>(p, num_tiles, st);
   if (mode == SCORE_CAPPED) return launch_mode<D, DV, SCORE_CAPPED>(p, num_tiles, st);
-  if constexpr (D == DV) return launch_mode<D, DV, SCORE_PLAIN>(p, num_tiles, st);
-  return -3;
+  if (mode == SCORE_BIASED) return launch_mode<D, DV, SCORE_BIASED>(p, num_tiles, st);
+  return launch_mode<D, DV, SCORE_PLAIN>(p, num_tiles, st);
 }
 
 }  // namespace ti
@@ -497,19 +518,23 @@ extern "C" {
 // tiles (up to 128 consecutive tokens of one sequence each; longest first gives the best balance).
 // q: bf16 [T, hq, D] (normalised, rotated); kcache / vcache: the paged cache of this layer, `num_blocks` pages;
 // positions: absolute position of every flat token; gate_src: the projection rows [T, ld] holding the gates, or null.
-// score(x) = scale x, or with softcap > 0 softcap * tanh(scale x / softcap).  `qk_max`: a bound of |q.k|, or <= 0.
+// score(x) = scale x, or with softcap > 0 softcap * tanh(scale x / softcap).  `qk_max`: a bound of |q.k|, or <= 0.  With
+// `slopes` [hq] a score loses slopes[h] per token of distance; `window`, `head_gate` [T, ldg], `ldo` (row pitch of out) and
+// `out_scale` as in AttnPrefillParams.
 int ti_attn_prefill(const void* q, int T, const void* kcache, const void* vcache, int num_blocks, const void* block_tables,
                     const void* positions, const void* qt_seq, const void* qt_tok0, const void* qt_ntok, int num_tiles,
                     const void* gate_src, void* out, int hq, int hkv, int max_blocks, int ld, float scale, int D, int DV,
-                    float softcap, float qk_max, void* status, void* stream) {
+                    float softcap, float qk_max, int window, const void* slopes, const void* head_gate, int ldg, int gcol, int ldo,
+                    float out_scale, void* status, void* stream) {
   if (num_tiles <= 0) return 0;
   if (hq % hkv || T < 1 || num_blocks < 1 || (gate_src != nullptr && D != DV)) return -2;
   // the gate and the output are read / written 16 bytes at a time: refuse layouts that would make those accesses misaligned
-  if ((ld & 7) || (reinterpret_cast<uintptr_t>(gate_src) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return -4;
+  if ((ld & 7) || (ldo & 7) || (reinterpret_cast<uintptr_t>(gate_src) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return -4;
+  if (window < 0 || (softcap > 0.f && (window > 0 || slopes != nullptr))) return -2;     // caps come without windows and slopes
   if ((D != 64 && D != 128 && D != 256) || (DV != 64 && DV != 128 && DV != 256)) return -3;
   constexpr float kLog2e = 1.4426950408889634f;
   ti::AttnPrefillParams p = {};
-  int mode = ti::SCORE_PLAIN;
+  int mode = slopes != nullptr ? ti::SCORE_BIASED : ti::SCORE_PLAIN;
   if (softcap > 0.f) {
     p.cap_in = scale / softcap;
     p.cap_out = softcap * kLog2e;
@@ -535,6 +560,13 @@ int ti_attn_prefill(const void* q, int T, const void* kcache, const void* vcache
   p.max_blocks = max_blocks;
   p.ld = ld;
   p.scale_log2e = scale * kLog2e;
+  p.window = window;
+  p.slopes = (const float*)slopes;
+  p.head_gate = (const __nv_bfloat16*)head_gate;
+  p.ldg = ldg;
+  p.gcol = gcol;
+  p.ldo = ldo > 0 ? ldo : hq * DV;
+  p.out_scale = out_scale;
   cudaStream_t st = (cudaStream_t)stream;
 #define TI_AP(A, B) if (D == A && DV == B) return ti::launch_attn_prefill<A, B>(p, num_tiles, mode, st)
   TI_AP(64, 64); TI_AP(64, 128); TI_AP(64, 256);

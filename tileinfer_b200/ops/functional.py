@@ -65,7 +65,11 @@ class AttnParams(ctypes.Structure):
                 ("qg_seq", _P), ("qg_tok0", _P), ("qg_ntok", _P), ("o_part", _P), ("ml_part", _P),
                 ("gate_src", _P), ("out", _P), ("hq", _I), ("hkv", _I), ("max_blocks", _I), ("nsplit", _I),
                 ("ld", _I), ("num_qg", _I), ("scale_log2e", _F), ("num_blocks", _I), ("status", _P), ("cap_in", _F), ("cap_out", _F),
-                ("rep", _I)]
+                ("rep", _I), ("window", _I), ("slopes", _P), ("head_gate", _P), ("ldg", _I), ("gcol", _I), ("ldo", _I), ("out_scale", _F)]
+
+    def __init__(self, *args, **kw):
+        super().__init__(*args, **kw)
+        self.out_scale = kw.get("out_scale", 1.0)
 
 
 class LatentAttnParams(ctypes.Structure):
@@ -84,7 +88,12 @@ class RopeUnitParams(ctypes.Structure):
 class AttnGeneralParams(ctypes.Structure):
     _fields_ = [("q", _P), ("kcache", _P), ("vcache", _P), ("block_tables", _P), ("positions", _P), ("qg_seq", _P), ("qg_tok0", _P),
                 ("qg_ntok", _P), ("out", _P), ("status", _P), ("H", _I), ("G", _I), ("dp", _I), ("vp", _I), ("max_blocks", _I),
-                ("num_qg", _I), ("num_blocks", _I), ("ldo", _I), ("scale", _F), ("softcap", _F)]
+                ("num_qg", _I), ("num_blocks", _I), ("ldo", _I), ("scale", _F), ("softcap", _F), ("window", _I), ("slopes", _P),
+                ("head_gate", _P), ("ldg", _I), ("gcol", _I), ("out_scale", _F)]
+
+    def __init__(self, *args, **kw):
+        super().__init__(*args, **kw)
+        self.out_scale = kw.get("out_scale", 1.0)
 
 
 class GlaParams(ctypes.Structure):
@@ -109,7 +118,7 @@ class ResidNormParams(ctypes.Structure):
 
 class GemmEpilogue(ctypes.Structure):
     _fields_ = [("resid32", _P), ("out2", _P), ("ldo2", _I), ("n_split", _I), ("scale", _F), ("glu_limit", _F),
-                ("glu_alpha", _F), ("glu_bias", _F)]
+                ("glu_alpha", _F), ("glu_bias", _F), ("softcap", _F), ("bias", _P)]
 
 
 class TopkParams(ctypes.Structure):
@@ -157,8 +166,8 @@ _l.register("ti_qkv_prep_params_size", _I, [], "attention")
 _l.register("ti_attn_params_size", _I, [], "attention")
 _l.register("ti_qkv_prep", _I, [ctypes.POINTER(QkvPrepParams), _I, _I, _P], "attention")
 _l.register("ti_attn_paged", _I, [ctypes.POINTER(AttnParams), _I, _I, _P], "attention")
-_l.register("ti_attn_prefill", _I, [_P, _I, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _F, _P, _P],
-            "attention")
+_l.register("ti_attn_prefill", _I, [_P, _I, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _F,
+                                _I, _P, _P, _I, _I, _I, _F, _P, _P], "attention")
 _l.register("ti_rope_unit_params_size", _I, [], "attention")
 _l.register("ti_rope_unit", _I, [ctypes.POINTER(RopeUnitParams), _I, _P], "attention")
 _l.register("ti_attn_general_params_size", _I, [], "attention")
@@ -201,7 +210,7 @@ _l.register("ti_rmsnorm_f32", _I, [_P, _P, _P, _I, _I, _I, _F, _I, _P], "rows")
 _l.register("ti_latent_store", _I, [_P, _I, _I, _P, _P, _P, _LL, _I, _I, _I, _F, _I, _P], "latent")
 _l.register("ti_latent_gather", _I, [_P, _P, _LL, _P, _I, _I, _I, _P], "latent")
 _l.register("ti_head_product", _I, [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P], "latent")
-_l.register("ti_gemm_f32", _I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P, _P, _I, _P], "rows")
+_l.register("ti_gemm_f32", _I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P, _P, _I, _F, _P, _P], "rows")
 
 _PARAM_SIZES = {"base": (("ti_topk_params_size", TopkParams), ("ti_edit_params_size", EditParams),
                          ("ti_sample_params_size", SampleParams), ("ti_gemm_epilogue_size", GemmEpilogue)),
@@ -580,16 +589,19 @@ def attn_paged(p: AttnParams, D: int, DV: int = None):
 
 
 def attn_prefill(q, kcache, vcache, num_blocks, block_tables, positions, tiles, gate_src, out, *, hq, hkv, D,
-                 max_blocks, ld, DV=None, scale=None, softcap=0.0, qk_max=0.0):
+                 max_blocks, ld, DV=None, scale=None, softcap=0.0, qk_max=0.0, window=0, slopes=None, head_gate=None, gcol=0, out_scale=1.0):
     """Causal GQA attention of prefill query tiles on the tcgen05 tensor cores (ops/csrc/attn_prefill.cu).
     `tiles`: int32 [3, n] = (sequence, first flat token, tokens <= 128) per tile, longest KV first.  DV: size of a value
     head (default D); softcap: scores become softcap * tanh(scale q.k / softcap); qk_max: a bound of |q.k| where there is
-    one (it selects a cheaper softmax); gate_src None: no output gate."""
+    one (it selects a cheaper softmax); gate_src None: no output gate.  window: keys seen (0: all); slopes: fp32 [hq], taken
+    off a score per token of distance; head_gate: rows whose column gcol + h gates head h; out_scale: factor of the output."""
     n = tiles.shape[1]
     scale = D ** -0.5 if scale is None else scale
     check(_l.lib().ti_attn_prefill(ptr(q), q.shape[0], ptr(kcache), ptr(vcache), num_blocks, ptr(block_tables), ptr(positions),
                               ptr(tiles[0]), ptr(tiles[1]), ptr(tiles[2]), n, ptr(gate_src), ptr(out), hq, hkv,
-                              max_blocks, ld, scale, D, D if DV is None else DV, softcap, qk_max, status_ptr(), stream()),
+                              max_blocks, ld, scale, D, D if DV is None else DV, softcap, qk_max, window, ptr(slopes), ptr(head_gate),
+                              0 if head_gate is None else head_gate.stride(0), gcol, out.stride(0) if out.dim() == 2 else 0, out_scale,
+                              status_ptr(), stream()),
           "ti_attn_prefill")
 
 
@@ -642,10 +654,11 @@ def topk_merge(p: TopkParams):
 GEPI_STORE, GEPI_SWIGLU, GEPI_ROWPAR, GEPI_F32, GEPI_RESID32, GEPI_SPLIT_GLU = 0, 1, 2, 3, 4, 5
 
 
-def gemm_epilogue(*, resid32=None, out2=None, n_split=0, scale=1.0, glu=(math.inf, 1.0, 0.0)) -> GemmEpilogue:
+def gemm_epilogue(*, resid32=None, out2=None, n_split=0, scale=1.0, glu=(math.inf, 1.0, 0.0), softcap=0.0, bias=None) -> GemmEpilogue:
     """Operands of the extended epilogues: an fp32 residual (GEPI_RESID32), the second output and the constants
-    (limit, alpha, bias) of the clamped gated unit (GEPI_SPLIT_GLU), a factor of the stored fp32 values (GEPI_F32)."""
-    return GemmEpilogue(ptr(resid32), ptr(out2), 0 if out2 is None else out2.stride(0), n_split, scale, *glu)
+    (limit, alpha, bias) of the clamped gated unit (GEPI_SPLIT_GLU), a factor and a cap of the stored fp32 values (GEPI_F32), and an fp32 vector [N]
+    added to the product first (any of them)."""
+    return GemmEpilogue(ptr(resid32), ptr(out2), 0 if out2 is None else out2.stride(0), n_split, scale, *glu, softcap, ptr(bias))
 
 
 class Limbs:
@@ -792,11 +805,11 @@ def gemm_f32(w, x, *, out, epi=GEPI_F32, ex=None, groups=None):
     check(_l.lib().ti_gemm_f32(ptr(w), ptr(x), e.resid32, ptr(out), e.out2, x.shape[0], N, K, x.stride(0), 0 if out is None else out.stride(0), e.ldo2,
                                e.n_split, epi, e.scale, e.glu_limit, e.glu_alpha, e.glu_bias,
                                *((0, 0, 0) if groups is None else (ptr(groups.tiles), ptr(groups.num_tiles), groups.tiles.shape[1])),
-                               stream()), "ti_gemm_f32")
+                               e.softcap, e.bias, stream()), "ti_gemm_f32")
 
 
 def resid_norm(y, x, w_out, h, w_next, W, eps, routed=None):
-    """x += rmsnorm(y) * w_out (fp32 rows), then h = rmsnorm(x) * w_next unless w_next is None.  With `routed` (a
+    """x += rmsnorm(y) * w_out (fp32 rows; w_out None: x += y), then h = rmsnorm(x) * w_next unless w_next is None.  With `routed` (a
     TokenGroups after `moe_permute`) y holds the experts' rows and h the input of the identity experts."""
     p = _resid_params(y, x, w_out, h, w_next, W, eps, routed)
     check(_l.lib().ti_resid_norm(ctypes.byref(p), x.shape[0], _f32(y), stream()), "ti_resid_norm")
@@ -807,7 +820,7 @@ def _resid_params(y, x, w_out, h, w_next, W, eps, routed=None) -> ResidNormParam
     p.y, p.x, p.w_out, p.w_next, p.h = ptr(y), ptr(x), ptr(w_out), ptr(w_next), ptr(h)
     if routed is not None:
         p.slot, p.weight, p.h_in, p.top = ptr(routed.slot), ptr(routed.weight), ptr(h), routed.top
-    p.W, p.P, p.ldy, p.eps = W, x.stride(0), y.stride(0), eps
+    p.W, p.P, p.ldy, p.eps = W, x.stride(0), 0 if y is None else y.stride(0), eps
     return p
 
 
@@ -904,7 +917,8 @@ def moe_counters(max_experts: int, device):
 
 
 def moe_route(g: TokenGroups, logits, correction, groups: int, keep: int, valid=None):
-    """Chooses the experts of every row of `logits` [T, >= choices] (fp32) and lays out the token tiles."""
+    """Chooses the experts of every row of `logits` [T, >= choices] (fp32) and lays out the token tiles.  correction None:
+    no corrections, and the weights are a softmax over the chosen logits alone."""
     p = _route_params(g, correction, groups, keep, valid)
     p.logits, p.ldl = ptr(logits), logits.stride(0)
     check(_l.lib().ti_moe_route(ctypes.byref(p), stream()), "ti_moe_route")
@@ -915,7 +929,7 @@ NORM_ROUTE_MAX_WIDTH = 8192      # columns of a row that `moe_norm_route` takes
 
 def moe_norm_route(y, x, w_out, h, w_next, W, eps, g: TokenGroups, router, correction, groups: int, keep: int, xs, valid=None):
     """`resid_norm` and, for the rows h it makes, the router product, `moe_route` and `moe_permute` (into xs) in one kernel,
-    for few tokens and fixed rows.  router: [choices, P] in the type of h."""
+    for few tokens and fixed rows (y None: x is complete, nothing is added).  router: [choices, P] in the type of h."""
     r, p = _resid_params(y, x, w_out, h, w_next, W, eps), _route_params(g, correction, groups, keep, valid)
     assert router.shape == (g.choices, x.stride(0)) and router.dtype == h.dtype and xs.shape[0] == g.rows and g.row_stride == g.T
     check(_l.lib().ti_moe_norm_route(ctypes.byref(r), ctypes.byref(p), ptr(router), ptr(g.slot), ptr(xs), _f32(h), stream()), "ti_moe_norm_route")
