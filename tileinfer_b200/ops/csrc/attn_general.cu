@@ -1,4 +1,5 @@
-// Around the paged attention kernels: the preparation of rotated, root-mean-square normalised heads, and a plain attention
+// Around the paged attention kernels: the preparation of rotated heads that are root-mean-square normalised one by one, or
+// all together before they are split, and a plain attention
 // kernel for what the tensor-core kernels do not take (32-bit mode, heads wider than 256).
 //
 // Cache layout as in attn_paged.cu, in bf16 or float: K pages [block][kv_head][16 tokens][dp], V pages transposed
@@ -75,6 +76,71 @@ __global__ void __launch_bounds__(128) rope_unit_kernel(const __grid_constant__ 
     const int c = lane + 32 * i;
     if (c < p.dp) dst[c] = from_f<T>(buf[c] * rr);
   }
+}
+
+struct NormRopeParams {
+  const void* proj;              // [T, ld]: H query heads at q_col, G key heads at k_col (dp each), G value heads at v_col (vp)
+  const float* q_w;              // [H * dp] weights of the norm over all query heads together (0 in the padding)
+  const float* k_w;              // [G * dp]
+  const float* inv_freq;         // [half] angle per position of dimensions 2i, 2i + 1
+  const int* positions;          // [T]
+  const long long* slot_mapping; // [T] flat slot = block * 16 + offset; outside the cache: not stored
+  void* q_out;                   // [T, H, dp]
+  void* kcache;
+  void* vcache;
+  int T, ld, q_col, k_col, v_col, H, G, dim, dp, vp, half, num_blocks;
+  float eps;
+};
+
+// A block per token: x / sqrt(mean over all heads of x^2 + eps) * w for the queries and for the keys, then the rotation of
+// neighbouring dimensions; values are only stored.
+template <typename T>
+__global__ void __launch_bounds__(256) norm_rope_kernel(const __grid_constant__ NormRopeParams p) {
+  extern __shared__ float cs[];                            // [half] cosines, [half] sines
+  __shared__ float red[2][8];
+  const int tid = threadIdx.x, t = blockIdx.x, nq = p.H * p.dp, nk = p.G * p.dp;
+  pdl_trigger();
+  pdl_wait();
+  const T* row = static_cast<const T*>(p.proj) + (size_t)t * p.ld;
+  const float pos = (float)p.positions[t];
+  for (int i = tid; i < p.half; i += 256) sincosf(pos * p.inv_freq[i], &cs[p.half + i], &cs[i]);
+  float sq = 0.f, sk = 0.f;
+  for (int c = tid * 8; c < nq + nk; c += 2048) {
+    float v[8], s = 0.f;
+    load8(c < nq ? row + p.q_col + c : row + p.k_col + c - nq, v);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) s += v[i] * v[i];
+    if (c < nq) sq += s;
+    else sk += s;
+  }
+  const float rq = rsqrtf(block_sum32(sq, red[0]) / (float)(p.H * p.dim) + p.eps);
+  const float rk = rsqrtf(block_sum32(sk, red[1]) / (float)(p.G * p.dim) + p.eps);
+  const long long slot = p.slot_mapping[t], blk = slot >> 4;
+  const int off = (int)(slot & 15);
+  const bool stored = slot >= 0 && blk < p.num_blocks;
+  for (int c = tid * 8; c < nq + (stored ? nk : 0); c += 2048) {
+    const bool is_q = c < nq;
+    const int e = is_q ? c : c - nq, d = e % p.dp;
+    float v[8], w[8];
+    load8(row + (is_q ? p.q_col : p.k_col) + e, v);
+    load8((is_q ? p.q_w : p.k_w) + e, w);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] *= (is_q ? rq : rk) * w[i];
+#pragma unroll
+    for (int i = 0; i < 8; i += 2) {
+      const int f = (d + i) >> 1;
+      if (f < p.half) {
+        const float a = v[i], b = v[i + 1], co = cs[f], si = cs[p.half + f];
+        v[i] = a * co - b * si;
+        v[i + 1] = b * co + a * si;
+      }
+    }
+    store8(is_q ? static_cast<T*>(p.q_out) + (size_t)t * nq + e
+                : static_cast<T*>(p.kcache) + (((size_t)blk * p.G + e / p.dp) * 16 + off) * p.dp + d, v);
+  }
+  if (!stored) return;
+  T* dst = static_cast<T*>(p.vcache) + (size_t)blk * p.G * p.vp * 16 + off;
+  for (int c = tid; c < p.G * p.vp; c += 256) dst[(size_t)c * 16] = row[p.v_col + c];
 }
 
 struct AttnGeneralParams {
@@ -207,6 +273,18 @@ static int launch_general(const AttnGeneralParams& p, cudaStream_t st) {
 extern "C" {
 
 int ti_rope_unit_params_size() { return (int)sizeof(ti::RopeUnitParams); }
+int ti_norm_rope_params_size() { return (int)sizeof(ti::NormRopeParams); }
+
+int ti_norm_rope(const ti::NormRopeParams* p, int f32, void* stream) {
+  if (p->T <= 0) return 0;
+  if (p->dp % 8 || p->vp % 8 || p->dim > p->dp || 2 * p->half > p->dim || p->num_blocks < 1 || p->ld % 8 || p->q_col % 8 || p->k_col % 8 ||
+      (((uintptr_t)p->proj | (uintptr_t)p->q_out | (uintptr_t)p->kcache | (uintptr_t)p->q_w | (uintptr_t)p->k_w) & 15))
+    return -2;
+  ti::launch_kernel(f32 ? ti::norm_rope_kernel<float> : ti::norm_rope_kernel<ti::bf16>, dim3(p->T), dim3(256), (size_t)p->half * 8,
+                    (cudaStream_t)stream, true, *p);
+  return (int)cudaGetLastError();
+}
+
 int ti_attn_general_params_size() { return (int)sizeof(ti::AttnGeneralParams); }
 
 int ti_rope_unit(const ti::RopeUnitParams* p, int f32, void* stream) {

@@ -1,14 +1,15 @@
 // Latent attention over a paged cache of latents, for decode tokens and short portions of prompts.
 //
 // With W_uk absorbed into the query (q~ = W_uk^T q, one row of R per head) every head attends to the SAME row c of the
-// cache, once as key and once as value:  s = scale * q~.c,  o~ = sum p c  (W_uv follows on o~, see latent_ops.cu).  One
+// cache, once as key and once as value:  s = scale * q~.c,  o~ = sum p c  (W_uv follows on o~, see latent_ops.cu).  A row
+// may carry columns behind the latent that only take part as key (a rotated part that all heads share).  One
 // cache row of R values per token serves all heads, so a block takes 16 or 32 heads as the rows of its MMAs and reads
 // each latent once from memory.
 //
 // A layer's mask is a parameter (window = 0: all earlier tokens; otherwise itself and the window - 1 tokens before it),
 // and so is the sink: one number per head that joins the denominator without key, value or scale (null: none).
 //
-// latent_decode.cu (bf16, padded R of 256, 384, 512): the tcgen05 form for the sizes of large models.
+// latent_decode.cu (bf16, padded R of 256, 384, 512, 576): the tcgen05 form for the sizes of large models.
 // latent_decode_kernel (bf16, other R up to 448): per (query token, head group, split) tiles of 64 keys, two tiles in flight by
 // cp.async; S = q~ c^T by mma.sync with the eight warps over (head tile, keys), softmax state in registers of the row's
 // threads, O += P c with the eight warps over column slices, the value fragments read from the SAME shared-memory tile
@@ -218,10 +219,10 @@ __global__ void __launch_bounds__(256) latent_decode_kernel(const __grid_constan
         const float sk = p.sink == nullptr ? kNeg : p.sink[head] * kLog2e;
         const float M = fmaxf(m_s[r], sk), w = exp2f(m_s[r] - M);
         const float inv = w / (l_s[r] * w + (p.sink == nullptr ? 0.f : exp2f(sk - M)));
-        bf16* dst = static_cast<bf16*>(p.out) + ((size_t)tok * p.H + head) * Rp + col0;
+        bf16* dst = static_cast<bf16*>(p.out) + ((size_t)tok * p.H + head) * p.Ro + col0;
 #pragma unroll
         for (int n = 0; n < RT; ++n)
-          *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16(o[a][n][2 * h] * inv, o[a][n][2 * h + 1] * inv);
+          if (col0 + n * 8 < p.Ro) *reinterpret_cast<uint32_t*>(dst + n * 8) = pack_bf16(o[a][n][2 * h] * inv, o[a][n][2 * h + 1] * inv);
       }
     return;
   }
@@ -266,8 +267,8 @@ __global__ void __launch_bounds__(128) latent_merge_kernel(const __grid_constant
   }
   __syncthreads();
   const float inv = 1.f / L;
-  bf16* dst = static_cast<bf16*>(p.out) + ((size_t)tok * p.H + head) * p.Rp;
-  for (int c = tid * 2; c < p.Rp; c += 256) {
+  bf16* dst = static_cast<bf16*>(p.out) + ((size_t)tok * p.H + head) * p.Ro;
+  for (int c = tid * 2; c < p.Ro; c += 256) {
     float a0 = 0.f, a1 = 0.f;
 #pragma unroll 4
     for (int s = 0; s < nact; ++s) {
@@ -341,14 +342,14 @@ __global__ void __launch_bounds__(128) latent_any_kernel(const __grid_constant__
       const T* c = cache + ((size_t)blk * 16 + (key & 15)) * p.Rp;
 #pragma unroll
       for (int e = 0; e < kAnyCols; ++e)
-        if (tid + 128 * e < p.Rp) o[e] = fmaf(w, as_float<T>(c[tid + 128 * e]), o[e]);
+        if (tid + 128 * e < p.Ro) o[e] = fmaf(w, as_float<T>(c[tid + 128 * e]), o[e]);
     }
     __syncthreads();
   }
-  T* dst = static_cast<T*>(p.out) + ((size_t)tok * p.H + head) * p.Rp;
+  T* dst = static_cast<T*>(p.out) + ((size_t)tok * p.H + head) * p.Ro;
 #pragma unroll
   for (int e = 0; e < kAnyCols; ++e)
-    if (tid + 128 * e < p.Rp) put(dst + tid + 128 * e, o[e] / l);
+    if (tid + 128 * e < p.Ro) put(dst + tid + 128 * e, o[e] / l);
 }
 
 void launch_latent_merge(const LatentAttnParams& p, int rows, int tile, cudaStream_t st) {
@@ -376,15 +377,18 @@ extern "C" {
 
 int ti_latent_attn_params_size() { return (int)sizeof(ti::LatentAttnParams); }
 
-// Largest padded latent size the split kernel takes; larger ones (and fp32) run on the general kernel, unsplit.
-int ti_latent_attn_max_split_rank() { return 512; }
+// Whether a split kernel takes rows of Rp columns of which Ro are values; others (and fp32) run on the general kernel, unsplit.
+int ti_latent_attn_splits(int Rp, int Ro) { return Rp <= 512 || (Rp == 576 && Ro <= 512); }
 
 int ti_latent_attn(const ti::LatentAttnParams* pp, int f32, void* stream) {
   const ti::LatentAttnParams& p = *pp;
   if (p.num_qg <= 0) return 0;
-  if (p.Rp % 64 || p.Rp > 128 * ti::kAnyCols || p.H < 1 || p.nsplit < 1 || p.nsplit > ti::kMaxLatentSplit || p.window < 0) return -2;
+  if (p.Rp % 64 || p.Rp > 128 * ti::kAnyCols || p.H < 1 || p.nsplit < 1 || p.nsplit > ti::kMaxLatentSplit || p.window < 0 ||
+      p.Ro < 64 || p.Ro > p.Rp || p.Ro % 64)
+    return -2;
   cudaStream_t st = (cudaStream_t)stream;
-  if (f32 || p.Rp > 512) {
+  if (f32 || !ti_latent_attn_splits(p.Rp, p.Ro)) {
+    if (p.nsplit != 1) return -2;
     const size_t smem = (p.Rp + 64) * sizeof(float);
     ti::launch_kernel(f32 ? ti::latent_any_kernel<float> : ti::latent_any_kernel<ti::bf16>, dim3(p.num_qg, p.H), dim3(128), smem,
                       st, true, p);

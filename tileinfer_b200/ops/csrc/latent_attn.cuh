@@ -17,10 +17,11 @@ struct LatentAttnParams {
   const float* sink;             // [H] or null
   float* o_part;                 // [num_qg * head groups * nsplit][rows][Rp]
   float* ml_part;                // [num_qg * head groups * nsplit][rows][2]
-  void* out;                     // [T][H][Rp]
+  void* out;                     // [T][H][Ro]
   unsigned* status;
   int H, R, Rp, max_blocks, nsplit, num_qg, window, num_blocks;
   float scale;
+  int Ro;                        // leading columns of a cache row that are value as well as key (the others are key alone)
 };
 
 constexpr float kNeg = -1e30f;
@@ -43,7 +44,7 @@ TI_DEVICE KeyRange key_range(const LatentAttnParams& p, int tok, int tile) {
 
 // Splits -> output (latent_attn.cu); `rows` heads per block and `tile` keys per tile of the kernel that made the splits.
 void launch_latent_merge(const LatentAttnParams& p, int rows, int tile, cudaStream_t st);
-// The tcgen05 form (latent_decode.cu): bf16, Rp 256, 384 or 512.  Returns a cudaError_t or a negative code.
+// The tcgen05 form (latent_decode.cu): bf16, Rp 256, 384, 512 or 576 (the last with Ro of at most 512).  Returns a cudaError_t or a negative code.
 int launch_latent_decode_tc(const LatentAttnParams& p, cudaStream_t st);
 
 }  // namespace ti

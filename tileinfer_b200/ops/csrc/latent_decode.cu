@@ -1,18 +1,18 @@
-// Latent attention of decode tokens on the 5th-generation tensor cores (bf16, padded latent size 256, 384 or 512).
+// Latent attention of decode tokens on the 5th-generation tensor cores (bf16, rows of 256, 384, 512 or 576 columns).
 //
 // All heads of a token attend to the same latents, so the latents are the wide operand and the heads the narrow one:
 // per tile of 64 keys   S^T [keys x heads] = C q~^T   and   O^T [R x heads] += C^T P^T,   where C [64 x R] is ONE copy
 // of the latents in shared memory: the K-major A operand of the first product, the MN-major A operand of the second.
 // N = 16 or 32 heads per block; tensor-core time follows the bytes of C, not the heads that a 128-row tile would waste.
 //
-//   warp 0     TMA producer: slots of 64 keys x 256 columns (384 at R = 384), one 4-D copy per 16-key page, through the
+//   warp 0     TMA producer: slots of 64 keys x 256 columns (whole rows at R = 384 and 576), one 4-D copy per 16-key page, through the
 //              block table
 //   warp 1     MMA issuer: S^T of the next tile (two buffers) while the softmax works on this one, then O^T slot by slot,
 //              each slot released as soon as it was read
 //   warps 2-9  softmax over the keys of a tile (lanes = keys in TMEM; the scores change hands through shared memory so that
 //              a thread owns one head and a share of the keys), lazy rescaling of O^T, P^T written as the bf16 B operand
 //
-// The ring holds two and a half tiles at R = 512 and more below.  Every wait is bounded; on expiry the status word is set, the roles leave and TMEM is freed.
+// The ring holds two tiles at R = 576, two and a half at 512 and more below.  At R = 576 the last 64 columns are key alone.  Every wait is bounded; on expiry the status word is set, the roles leave and TMEM is freed.
 #include "latent_attn.cuh"
 #include "tensor_map.cuh"
 
@@ -335,11 +335,12 @@ __global__ void __launch_bounds__(kDkThreads, 1) latent_decode_tc_kernel(const _
         float o[N];
         tmem_ld_n<N>(lane_base + o_col + b * N, o);
         const int r = b * 128 + quarter * 32 + lane;
+        if (r >= p.Ro) continue;
         if (p.nsplit == 1) {
-          bf16* dst = static_cast<bf16*>(p.out) + ((size_t)tok * p.H + hg * N) * Rp + r;
+          bf16* dst = static_cast<bf16*>(p.out) + ((size_t)tok * p.H + hg * N) * p.Ro + r;
 #pragma unroll
           for (int i = 0; i < N; ++i)
-            if (i < nh) dst[(size_t)i * Rp] = __float2bfloat16_rn(o[i] * ml_x[i]);
+            if (i < nh) dst[(size_t)i * p.Ro] = __float2bfloat16_rn(o[i] * ml_x[i]);
         } else {
           float* dst = p.o_part + item * N * Rp + r;
 #pragma unroll
@@ -377,14 +378,15 @@ static int launch_dk(LatentDecodeTcParams& p, cudaStream_t st) {
 }
 
 int launch_latent_decode_tc(const LatentAttnParams& a, cudaStream_t st) {
-  if ((a.Rp != 256 && a.Rp != 384 && a.Rp != 512) || a.num_blocks < 1) return -2;
+  if ((a.Rp != 256 && a.Rp != 384 && a.Rp != 512 && a.Rp != 576) || (a.Rp == 576 && a.Ro > 512) || a.num_blocks < 1) return -2;
   LatentDecodeTcParams p = {};
   p.a = a;
-  const int slabs = a.Rp % 256 == 0 ? 4 : 6;
+  const int slabs = a.Rp % 256 == 0 ? 4 : a.Rp / 64;
   const int rc = bf16_map_groups(&p.map_c, a.cache, a.Rp, (long long)a.num_blocks * 16, slabs, 2);
   if (rc) return rc;
   if (slabs == 4) return a.H > 16 ? launch_dk<32, 4>(p, st) : launch_dk<16, 4>(p, st);
-  return a.H > 16 ? launch_dk<32, 6>(p, st) : launch_dk<16, 6>(p, st);
+  if (slabs == 6) return a.H > 16 ? launch_dk<32, 6>(p, st) : launch_dk<16, 6>(p, st);
+  return a.H > 16 ? launch_dk<32, 9>(p, st) : launch_dk<16, 9>(p, st);
 }
 
 }  // namespace ti

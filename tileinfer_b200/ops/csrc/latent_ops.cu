@@ -1,5 +1,5 @@
-// Row operations and small products around latent attention: the latent's norm and its store into cache pages, and the
-// per-head products that absorb W_uk into the query and W_uv into the output.
+// Row operations and small products around latent attention: the latent's norm and its store into cache pages (beside a
+// rotated key part, with the rotation of the queries), and the per-head products that absorb W_uk into the query and W_uv into the output.
 //
 // Every kernel is templated on the activation type (bf16, or float in 32-bit mode).  Row pitches are padded to
 // multiples of 64 elements and the pad columns hold zeros (zero weight rows, zero norm weights), so that rows are read
@@ -38,6 +38,58 @@ __global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__
 #pragma unroll
     for (int i = 0; i < 8; ++i) v[i] *= rr * g[i];
     store8(dst + c, v);
+  }
+}
+
+// The same with a rotated part: a warp per (token, item), item 0 the cache row [rmsnorm(latent) * w | turned key part | 0],
+// item 1 + h the trailing part of query head h, turned in place.  Dimension i of a part turns with dimension i + half.
+struct LatentRopeParams {
+  void* proj;                    // [M, ld]: query heads at h * dp (dim plain, then 2 * half turned), latent and key part at col0
+  const float* w;                // [R]
+  const float* inv_freq;         // [half]
+  const int* positions;          // [M]
+  const long long* slots;        // [M]
+  void* cache;                   // [num_slots][Rp]
+  long long num_slots;
+  int ld, H, dp, dim, col0, half, M, R, Rp;
+  float eps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_rope_kernel(const __grid_constant__ LatentRopeParams p) {
+  const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31, m = (int)(item / (p.H + 1)), h = (int)(item - (long long)m * (p.H + 1)) - 1;
+  pdl_trigger();
+  pdl_wait();
+  if (m >= p.M) return;
+  T* row = static_cast<T*>(p.proj) + (size_t)m * p.ld;
+  const float pos = (float)p.positions[m];
+  const T* src;
+  T* dst;
+  if (h >= 0) {
+    src = dst = row + (size_t)h * p.dp + p.dim;
+  } else {
+    const long long slot = p.slots[m];
+    if (slot < 0 || slot >= p.num_slots) return;
+    src = row + p.col0;
+    dst = static_cast<T*>(p.cache) + (size_t)slot * p.Rp;
+    float ss = 0.f;
+    for (int c = lane; c < p.R; c += 32) {
+      const float v = to_f<T>(src[c]);
+      ss += v * v;
+    }
+    const float rr = rsqrtf(warp_sum(ss) / (float)p.R + p.eps);
+    for (int c = lane; c < p.R; c += 32) dst[c] = from_f<T>(to_f<T>(src[c]) * rr * p.w[c]);
+    for (int c = p.R + 2 * p.half + lane; c < p.Rp; c += 32) dst[c] = from_f<T>(0.f);
+    src += p.R;
+    dst += p.R;
+  }
+  for (int i = lane; i < p.half; i += 32) {
+    float sn, cs;
+    sincosf(pos * p.inv_freq[i], &sn, &cs);
+    const float u = to_f<T>(src[i]), v = to_f<T>(src[i + p.half]);
+    dst[i] = from_f<T>(u * cs - v * sn);
+    dst[i + p.half] = from_f<T>(v * cs + u * sn);
   }
 }
 
@@ -154,6 +206,17 @@ int ti_latent_store(const void* proj, int ld, int col0, const void* w, const voi
   else
     ti::launch_kernel(ti::latent_store_kernel<ti::bf16>, grid, dim3(128), 0, st, true, (const ti::bf16*)proj, ld, col0, (const float*)w,
                       (const long long*)slots, (ti::bf16*)cache, num_slots, M, R, Rp, eps);
+  return (int)cudaGetLastError();
+}
+
+int ti_latent_rope(void* proj, int ld, int H, int dp, int dim, int col0, const void* w, const void* inv_freq, int half, const void* positions,
+                   const void* slots, void* cache, long long num_slots, int M, int R, int Rp, float eps, int f32, void* stream) {
+  if (M <= 0) return 0;
+  if (dim + 2 * half > dp || R + 2 * half > Rp || half < 0 || H < 0) return -2;
+  const ti::LatentRopeParams p = {proj, (const float*)w, (const float*)inv_freq, (const int*)positions, (const long long*)slots, cache,
+                                  num_slots, ld, H, dp, dim, col0, half, M, R, Rp, eps};
+  const dim3 grid((unsigned)(((long long)M * (H + 1) + 3) / 4));
+  ti::launch_kernel(f32 ? ti::latent_rope_kernel<float> : ti::latent_rope_kernel<ti::bf16>, grid, dim3(128), 0, (cudaStream_t)stream, true, p);
   return (int)cudaGetLastError();
 }
 

@@ -76,7 +76,7 @@ class LatentAttnParams(ctypes.Structure):
     _fields_ = [("q", _P), ("cache", _P), ("block_tables", _P), ("positions", _P), ("qg_seq", _P), ("qg_tok0", _P),
                 ("qg_ntok", _P), ("sink", _P), ("o_part", _P), ("ml_part", _P), ("out", _P), ("status", _P),
                 ("H", _I), ("R", _I), ("Rp", _I), ("max_blocks", _I), ("nsplit", _I), ("num_qg", _I), ("window", _I),
-                ("num_blocks", _I), ("scale", _F)]
+                ("num_blocks", _I), ("scale", _F), ("Ro", _I)]
 
 
 class RopeUnitParams(ctypes.Structure):
@@ -202,12 +202,13 @@ _l.register("ti_gemm_epilogue_size", _I, [])
 _l.register("ti_gemm_bf16", _I, [_P, _I, _I, _I, _P, _I, _P, _P, _I, _I, _P, _P, ctypes.c_size_t, _P, _I, _P, _P])
 _l.register("ti_gemm_w8a16", _I, [_P, _P, _I, _I, _I, _P, _P, _P, _I, _P, _P, _I, _I, _P, _P, ctypes.c_size_t, _P, _I, _P, _P])
 _l.register("ti_latent_attn_params_size", _I, [], "latent")
-_l.register("ti_latent_attn_max_split_rank", _I, [], "latent")
+_l.register("ti_latent_attn_splits", _I, [_I, _I], "latent")
 _l.register("ti_latent_attn", _I, [ctypes.POINTER(LatentAttnParams), _I, _P], "latent")
 _l.register("ti_latent_prefill", _I, [_P, _I, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P], "latent")
 _l.register("ti_embed_pos", _I, [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P, _I, _P], "rows")
 _l.register("ti_rmsnorm_f32", _I, [_P, _P, _P, _I, _I, _I, _F, _I, _P], "rows")
 _l.register("ti_latent_store", _I, [_P, _I, _I, _P, _P, _P, _LL, _I, _I, _I, _F, _I, _P], "latent")
+_l.register("ti_latent_rope", _I, [_P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _LL, _I, _I, _I, _F, _I, _P], "latent")
 _l.register("ti_latent_gather", _I, [_P, _P, _LL, _P, _I, _I, _I, _P], "latent")
 _l.register("ti_head_product", _I, [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P], "latent")
 _l.register("ti_gemm_f32", _I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _F, _F, _F, _P, _P, _I, _F, _P, _P], "rows")
@@ -743,6 +744,16 @@ def rmsnorm_f32(x, norm_w, y, W, eps):
     check(_l.lib().ti_rmsnorm_f32(ptr(x), ptr(norm_w), ptr(y), x.shape[0], W, x.stride(0), eps, _f32(y), stream()), "ti_rmsnorm_f32")
 
 
+def latent_rope(proj, H, dp, dim, col0, norm_w, inv_freq, positions, slots, cache, R, eps):
+    """Turns dimensions dim .. dim + 2 * inv_freq.numel() of the H query heads (proj columns h * dp, in place), and stores
+    [normalised latent of R columns | turned key part] of proj[:, col0:] in the slots of `cache` [blocks, 16, Rp]."""
+    Rp = cache.shape[-1]
+    assert norm_w.numel() >= R and cache.dtype == proj.dtype
+    check(_l.lib().ti_latent_rope(ptr(proj), proj.stride(0), H, dp, dim, col0, ptr(norm_w), ptr(inv_freq), inv_freq.numel(), ptr(positions),
+                                  ptr(slots), ptr(cache), cache.numel() // Rp, proj.shape[0], R, Rp, eps, _f32(proj), stream()),
+          "ti_latent_rope")
+
+
 def latent_store(proj, col0, norm_w, slots, cache, R, eps):
     """Normalised latents proj[:, col0 : col0 + R] into their slots of `cache` [blocks, 16, Rp]."""
     Rp = cache.shape[-1]
@@ -783,9 +794,16 @@ def latent_part_floats(num_qg: int, H: int, Rp: int, nsplit: int) -> int:
     return num_qg * -(-H // latent_rows(H)) * nsplit * latent_rows(H) * Rp
 
 
+def latent_attn_splits(Rp: int, Ro: int) -> bool:
+    """Whether a kernel with splits takes cache rows of Rp columns of which the first Ro are values (bf16)."""
+    return bool(_l.lib().ti_latent_attn_splits(Rp, Ro))
+
+
 def latent_attn(p: LatentAttnParams, f32: bool):
+    """p.Ro 0: every column of a cache row is key and value."""
     if not p.status:
         p.status = status_ptr()
+    p.Ro = p.Ro or p.Rp
     check(_l.lib().ti_latent_attn(ctypes.byref(p), int(f32), stream()), "ti_latent_attn")
 
 
