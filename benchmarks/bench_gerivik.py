@@ -121,7 +121,7 @@ def kernel_rows(cfg, tag, lens, ctxs, prompt, ctx):
     logits = x.logits[:T * n].view(T, n)
     xs, act = x.xs[:g.rows * m.Wp].view(g.rows, m.Wp), x.act[:g.rows * L.ff].view(g.rows, L.ff)
     if g.row_stride:
-        row("norm + residual + next norm + router + routing + rows to experts", small(lambda: m._norm_and_route(L, x)),
+        row("norm + residual + next norm + router + routing + rows to experts", small(lambda: m._norm_and_route(L, x, x.y, L.norm1b)),
             nbytes=12 * W * T + 2 * W * (f.choices + T * f.top), like="rmsnorm")
     else:
         row("router product", small(lambda: L.router(x.h, logits, F.GEPI_F32)), **gemm(f.choices, W, 4))

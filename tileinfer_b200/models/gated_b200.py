@@ -20,10 +20,11 @@ from ..ops import functional as F
 from ..ops.functional import AttnGeneralParams, AttnParams, GlaParams, RopeUnitParams, ptr
 from ..utils.trace import nvtx_end, nvtx_mark
 from .gerivik import GLU_ALPHA, GLU_BIAS, GerivikConfig
-from .products_b200 import GroupedProduct, Product, pad64, pad_to
+from .experts_b200 import ExpertLayers
+from .paged_state_b200 import PAGE, PagedState
+from .products_b200 import Product, pad64, pad_to
 from .runtime_b200 import DeviceRuntime, StepCtx
 
-PAGE = 16
 LOG2E = 1.4426950408889634
 
 
@@ -40,7 +41,7 @@ class _Weights:
     """Tensors of one layer in kernel layout (shared by the layers that reuse them)."""
 
 
-class B200GatedModel(DeviceRuntime):
+class B200GatedModel(PagedState, ExpertLayers, DeviceRuntime):
     def __init__(self, cfg: GerivikConfig, src, *, quant="bf16", tp=1, rank=0, comm=None, config=None):
         assert torch.cuda.is_available(), "B200GatedModel needs a CUDA device"
         cfg.validate_tp(tp)
@@ -118,22 +119,8 @@ class B200GatedModel(DeviceRuntime):
         L.w_o = Product(pad_to(get(q + "o").view(-1, H, m.vdim), Wp, H, L.vp).reshape(Wp, L.n_mix), self.quant, dev)
         L.moe = None
         if spec.mlp is not None:
-            f, L.ff = spec.mlp, pad64(spec.mlp.ff)
-            if f.choices > 1024:
-                raise ValueError(f"the router takes at most 1024 experts, got {f.choices}")
-            L.moe = f
             L.norm2, L.norm2b = self._norm(get(p + "norm2"), Wp), self._norm(get(p + "norm2b"), Wp)
-            router = pad_to(get(p + "mlp.router"), f.choices, Wp)
-            L.router, L.router_rows = Product(router, "fp32" if self.f32 else "bf16", dev), router.to(self.dtype).contiguous()
-            L.correction = get(p + "mlp.correction").float().contiguous()
-            up, down = [], []
-            for e in range(f.experts):
-                g, u = (pad_to(get(f"{p}mlp.e{e}.{n}"), L.ff, Wp) for n in ("gate", "up"))
-                up.append(torch.stack([g, u], dim=1).reshape(2 * L.ff, Wp).to(torch.float32 if self.quant != "bf16" else torch.bfloat16))
-                down.append(pad_to(get(f"{p}mlp.e{e}.down"), Wp, L.ff).to(up[-1].dtype))
-            L.w_up = GroupedProduct(up, self.quant, dev)
-            del up
-            L.w_down = GroupedProduct(down, self.quant, dev)
+            self._build_experts(L, spec.mlp, p + "mlp.", get, (spec.mlp.limit, GLU_ALPHA, GLU_BIAS), get(p + "mlp.correction").float().contiguous())
         return L
 
     def weight_bytes(self, tokens: int = 1) -> int:
@@ -142,26 +129,15 @@ class B200GatedModel(DeviceRuntime):
         for L in self.layers:
             n += L.w_in.nbytes() + L.w_o.nbytes()
             if L.moe is not None:
-                share = min(1.0, tokens * L.moe.top / L.moe.choices)
-                n += L.router.nbytes() + int((L.w_up.nbytes() + L.w_down.nbytes()) * share)
+                n += self._expert_bytes(L, tokens)
         return n
 
     # ------------------------------------------------------------------ cache pages and state slots
     def _bytes_per_block(self) -> int:
         return sum(PAGE * L.G * (L.dp + L.vp) for L in (self.layers[i] for i in self.cfg.attn_layers)) * (4 if self.f32 else 2)
 
-    cache_bytes_per_block = _bytes_per_block
-
     def _state_bytes_per_slot(self) -> int:
         return sum(L.heads * L.dp * L.vp * 4 for L in (self.layers[i] for i in self.cfg.gla_layers))
-
-    def auto_num_blocks(self, util, block_size, num_slots, max_num_seqs, max_model_len) -> int:
-        free, total = torch.cuda.mem_get_info()
-        budget = free - (1.0 - util) * total - num_slots * self._state_bytes_per_slot() - (6 << 30)        # room for the activations of a long step
-        n = min(int(budget // max(1, self._bytes_per_block())), max_num_seqs * (max_model_len // block_size + 2) + 64)
-        if n < max_model_len // block_size + 2:
-            raise RuntimeError(f"not enough GPU memory for one sequence of {max_model_len} tokens ({n} cache blocks)")
-        return n
 
     def alloc_cache(self, num_blocks: int, block_size: int, num_slots: int):
         assert block_size == PAGE
@@ -173,52 +149,6 @@ class B200GatedModel(DeviceRuntime):
         for i in self.cfg.gla_layers:
             L = self.layers[i]
             self.state[i] = new(torch.float32, num_slots, L.heads, L.dp, L.vp)
-
-    def zero_state(self, slot: int):
-        for s in self.state.values():
-            s[slot].zero_()
-
-    def _to_host(self, parts):
-        """One pinned host copy of the tensors, asynchronous and ordered by the stream (see `_pinned`)."""
-        if not parts:
-            return None
-        dev = torch.cat(parts)
-        host = self._pinned(dev.shape, dev.dtype)
-        host.copy_(dev, non_blocking=True)
-        return host
-
-    def _done_with(self, data):
-        if data.device.type == "cpu" and data.is_pinned():
-            self._unpin(data)                          # later writers of the buffer are ordered after the copy from it
-
-    def state_out(self, slot: int):
-        return self._to_host([s[slot].flatten() for s in self.state.values()])
-
-    def state_in(self, slot: int, st):
-        """From a swapped-out state (pinned host memory) or a prefix snapshot (on the device, owned by the cache)."""
-        if st is None:
-            return
-        dev, at = st.to(self.dev, non_blocking=True), 0
-        for s in self.state.values():
-            n = s[slot].numel()
-            s[slot].copy_(dev[at:at + n].view(s[slot].shape))
-            at += n
-        self._done_with(st)
-
-    def blocks_out(self, block_ids: list):
-        idx = torch.tensor(block_ids, dtype=torch.long, device=self.dev)
-        return self._to_host([t[idx].flatten() for kv in self.cache.values() for t in kv])
-
-    def blocks_in(self, block_ids: list, data):
-        if data is None:
-            return
-        idx, at = torch.tensor(block_ids, dtype=torch.long, device=self.dev), 0
-        dev = data.to(self.dev, non_blocking=True)
-        for t in (t for kv in self.cache.values() for t in kv):
-            n = len(block_ids) * t[0].numel()
-            t[idx] = dev[at:at + n].view(-1, *t.shape[1:])
-            at += n
-        self._done_with(data)
 
     # ------------------------------------------------------------------ step
     def _alloc_ctx(self, T: int, S: int, max_blocks: int, num_qg: int, nsplit: int) -> StepCtx:
@@ -238,51 +168,13 @@ class B200GatedModel(DeviceRuntime):
                 x.ml_part = torch.empty(items // 64 * 32, dtype=torch.float32, device=dev)
         if gla:
             x.o = new(T * max(L.n_mix for L in gla), dtype=torch.float32, device=dev)
-        x.groups, moe = {}, [L for L in Ls if L.moe is not None]
-        if moe:
-            few = T <= self.FEW_TOKENS and self.Wp <= F.NORM_ROUTE_MAX_WIDTH
-            for L in moe:
-                key = (L.moe.experts, L.moe.choices, L.moe.top)
-                if key not in x.groups:
-                    fixed = few and L.moe.experts * T * self.Wp <= 1 << 26
-                    x.groups[key] = F.TokenGroups(T, *key, self.counters, self.f32, dev, fixed)
-            rows = max(g.rows for g in x.groups.values())
-            x.logits = new(T * max(-(-L.moe.choices // 8) * 8 for L in moe), dtype=torch.float32, device=dev)
-            x.xs = new(rows * self.Wp, dtype=dt, device=dev)          # token rows by expert, then the experts' outputs
-            x.act = new(rows * max(L.ff for L in moe), dtype=dt, device=dev)
+        self._alloc_experts(x, T, [L for L in Ls if L.moe is not None], new)
         x.snaps, x.chunks, x.short = [], {}, None          # chunks: chunk size -> (table, ranges); short: the other sequences
         return x
 
     def _prepare_step(self, x: StepCtx, batch):
-        """State snapshots wanted in this step, and which sequences run the recurrence in chunks."""
-        S = batch.num_seqs
-        if not self.cfg.gla_layers:
-            return
-        points = batch.snapshot_at if batch.snapshot_at and any(batch.snapshot_at) else [[]] * S
-        ns = max(len(p) for p in points)
-        rel, idx = torch.zeros(S, max(ns, 1), dtype=torch.int32), torch.zeros(S, max(ns, 1), dtype=torch.int32)
-        for s, pts in enumerate(points):
-            start = batch.context_lens[s] - (batch.cu_seqlens[s + 1] - batch.cu_seqlens[s])
-            for j, a in enumerate(pts):
-                rel[s, j], idx[s, j] = a - start, len(x.snaps)
-                x.snaps.append((s, a))
-        if x.snaps:
-            x.snap_rel, x.snap_idx, x.num_snap = rel.to(self.dev), idx.to(self.dev), ns
-            x.snap_state = {i: torch.empty(len(x.snaps), *self.state[i].shape[1:], dtype=torch.float32, device=self.dev)
-                            for i in self.cfg.gla_layers}
-        lens = [b - a for a, b in zip(batch.cu_seqlens[:-1], batch.cu_seqlens[1:])]
-        longs = [s for s in range(S) if lens[s] >= self.gla_chunk_min_tokens]
-        if longs:
-            up = lambda v: torch.tensor(v, dtype=torch.int32).to(self.dev, non_blocking=True)
-            x.short, x.longs = up([s for s in range(S) if lens[s] < self.gla_chunk_min_tokens]), up(longs)
-            entries = [{int(r): int(e) for r, e in zip(rel[s, :len(points[s])], idx[s])} for s in range(S)]
-            for n in {F.gla_chunk_size(self.layers[i].dp) for i in self.cfg.gla_layers}:
-                ck, rng = F.gla_chunk_table(batch.cu_seqlens, longs, n, entries)
-                x.chunks[n] = (ck.to(self.dev, non_blocking=True), rng.to(self.dev, non_blocking=True))
-
-    def _finish_step(self, x: StepCtx):
-        for k, key in enumerate(x.snaps):                  # snapshots stay on the device
-            self.snapshots[key] = torch.cat([t[k].flatten() for t in x.snap_state.values()])
+        if self.cfg.gla_layers:
+            self._prepare_recurrence(x, batch, [F.gla_chunk_size(self.layers[i].dp) for i in self.cfg.gla_layers], self.gla_chunk_min_tokens)
 
     def _rotate_and_store(self, i: int, L, x: StepCtx, proj):
         """Rotated unit heads of the queries (returned) and of the keys, and the values, into the cache pages."""
@@ -350,32 +242,6 @@ class B200GatedModel(DeviceRuntime):
         F.gla_finish(p, x.T, L.vp, self.f32)
         self._launches += 1 + bool(num)
 
-    FEW_TOKENS = 128                 # up to this many tokens the norm kernel routes the rows it makes
-
-    def _norm_and_route(self, L, x: StepCtx):
-        """The mixer's output into the residual, the experts' input x.h, its routing and its rows by expert."""
-        f, T, c, Wp = L.moe, x.T, self.cfg, self.Wp
-        g = x.groups[(f.experts, f.choices, f.top)]
-        xs = x.xs[:g.rows * Wp].view(g.rows, Wp)
-        if g.row_stride:
-            F.moe_norm_route(x.y, x.x, L.norm1b, x.h, L.norm2, self.W, c.rms_eps, g, L.router_rows, L.correction, f.groups, f.keep, xs,
-                             valid=x.slot_mapping)
-            self._launches += 1
-        else:
-            F.resid_norm(x.y, x.x, L.norm1b, x.h, L.norm2, self.W, c.rms_eps)
-            n = -(-f.choices // 8) * 8
-            logits = x.logits[:T * n].view(T, n)
-            self._launches += 3 + L.router(x.h, logits, F.GEPI_F32)
-            F.moe_route(g, logits, L.correction, f.groups, f.keep, valid=x.slot_mapping)
-            F.moe_permute(g, x.h, xs)
-        return g, xs
-
-    def _experts(self, L, x: StepCtx, g, xs):
-        """The experts' outputs, in the place of their rows."""
-        f, act = L.moe, x.act[:g.rows * L.ff].view(g.rows, L.ff)
-        ex = F.gemm_epilogue(out2=act, n_split=0, glu=(f.limit, GLU_ALPHA, GLU_BIAS))
-        self._launches += L.w_up(xs, g, None, F.GEPI_SPLIT_GLU, ex) + L.w_down(act, g, xs, F.GEPI_STORE)
-
     def _run_layers(self, x: StepCtx):
         c, T = self.cfg, x.T
         F.embed_pos(x.ids, x.positions, self.embed, None, None, x.x, self.W, c.rms_eps, scale=c.embedding_scale)
@@ -393,7 +259,7 @@ class B200GatedModel(DeviceRuntime):
                 F.resid_norm(x.y, x.x, L.norm1b, x.h, after, self.W, c.rms_eps)
                 self._launches += 1
             else:
-                g, rows = self._norm_and_route(L, x)
+                g, rows = self._norm_and_route(L, x, x.y, L.norm1b)
                 self._experts(L, x, g, rows)
                 F.resid_norm(rows, x.x, L.norm2b, x.h, after, self.W, c.rms_eps, routed=g)
                 self._launches += 1
@@ -407,6 +273,3 @@ class B200GatedModel(DeviceRuntime):
 
     def _status_ptr(self) -> int:
         return self.status
-
-    def peer_status(self) -> int:
-        return int(F._STATUS[0].item())

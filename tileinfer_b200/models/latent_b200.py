@@ -30,7 +30,89 @@ class _Layer:
     pass
 
 
-class B200LatentModel(DeviceRuntime):
+class LatentLayers:
+    """Launches of attention over paged latents, for executors with such layers.  A layer has heads, dp and vp (padded query
+    and value heads), Rp (padded cache row), Ro (its leading columns that are values), window, scale, uk_t [H, Rp, dp],
+    uv [H, vp, Ro], w_ukv (keys of all heads, then values; 16 bits) and, or None, sink and g_col (gate column)."""
+
+    def _latent_rows(self, L):
+        """The pages a layer attends to, [blocks, 16, Rp]."""
+        raise NotImplementedError
+
+    def _latent_nsplit(self, L, num_qg: int) -> int:
+        return F.latent_nsplit(num_qg, L.heads, L.Rp, L.window) if not self.f32 and F.latent_attn_splits(L.Rp, L.Ro) else 1
+
+    def _alloc_latent(self, x: StepCtx, T: int, num_qg: int, layers: list, new):
+        x.short_rows = (0, T)               # rows [a, b) that hold every token of the split attention
+        x.reach, x.latents = {}, {}         # window -> (cache slots in reach, query tiles) of the long portions
+        if not (num_qg and layers):
+            return
+        x.q_abs = new(T * max(L.heads * L.Rp for L in layers), dtype=self.dtype, device=self.dev)
+        x.o_lat = new(T * max(L.heads * L.Ro for L in layers), dtype=self.dtype, device=self.dev)
+        part = max((F.latent_part_floats(num_qg, L.heads, L.Rp, ns) for L in layers if (ns := self._latent_nsplit(L, num_qg)) > 1), default=0)
+        if part:
+            x.lat_part = torch.empty(part, dtype=torch.float32, device=self.dev)
+            x.lat_ml = torch.empty(part // 64 * 2, dtype=torch.float32, device=self.dev)
+
+    def _attn_latent_short(self, L, x: StepCtx, proj, cat):
+        """Decode tokens and short portions: absorbed queries against the paged latents."""
+        a, b = x.short_rows
+        T, H = x.T, L.heads
+        q_abs, o_lat = x.q_abs[:T * H * L.Rp].view(T, H * L.Rp), x.o_lat[:T * H * L.Ro].view(T, H * L.Ro)
+        F.head_product(proj[a:b], L.uk_t, q_abs[a:b])
+        p = LatentAttnParams()
+        p.q, p.cache, p.out, p.sink = ptr(q_abs), ptr(self._latent_rows(L)), ptr(o_lat), ptr(L.sink)
+        p.block_tables, p.positions = ptr(x.block_tables), ptr(x.positions)
+        p.qg_seq, p.qg_tok0, p.qg_ntok = ptr(x.qg[0]), ptr(x.qg[1]), ptr(x.qg[2])
+        p.nsplit = self._latent_nsplit(L, x.num_qg)
+        if p.nsplit > 1:
+            p.o_part, p.ml_part = ptr(x.lat_part), ptr(x.lat_ml)
+        p.H, p.R, p.Rp, p.Ro, p.max_blocks, p.num_qg = H, L.R, L.Rp, L.Ro, x.max_blocks, x.num_qg
+        p.window, p.num_blocks, p.scale, p.status = L.window, self.num_blocks, L.scale, self.status
+        F.latent_attn(p, self.f32)
+        F.head_product(o_lat[a:b], L.uv, cat[a:b], gate=None if L.g_col is None else proj[a:b], gcol=L.g_col or 0)
+        self._launches += 3 + (p.nsplit > 1)
+
+    def _prepare_latent(self, x: StepCtx, batch, layers: list):
+        """Which rows the split attention covers, and per window the cached rows in reach of the long portions of the step
+        with their query tiles (see `latent_prefill`)."""
+        bs, short, longs = self.block_size, [], []
+        for s in range(batch.num_seqs):
+            t0, t1 = batch.cu_seqlens[s], batch.cu_seqlens[s + 1]
+            (longs if t1 - t0 >= self.PREFILL_ATTN_MIN_TOKENS else short).append((s, t0, t1))
+        x.short_rows = (short[0][1], short[-1][2]) if short else (0, 0)
+        for window in {L.window for L in layers} if longs else ():
+            slots, tiles, base = [], [], 0
+            for s, t0, t1 in longs:
+                end = batch.context_lens[s]
+                start = end - (t1 - t0)
+                lo = max(0, start - window + 1)
+                pos = torch.arange(lo, end)
+                slots.append(torch.tensor(batch.block_tables[s], dtype=torch.long)[pos // bs] * bs + pos % bs)
+                for a in range(t0, t1, 128):
+                    p0, n = start + a - t0, min(128, t1 - a)
+                    tiles.append((p0 + n - max(0, p0 - window + 1), a, n, p0, base, lo))
+                base += end - lo
+            tiles.sort(key=lambda t: -t[0])                    # most keys first
+            x.reach[window] = (torch.cat(slots).to(self.dev, non_blocking=True),
+                               torch.tensor([t[1:] for t in tiles], dtype=torch.int32).t().contiguous().to(self.dev, non_blocking=True))
+
+    def _attn_latent_long(self, L, x: StepCtx, proj, cat):
+        """Long portions of prompts: keys and values of every cached latent in reach, then windowed query tiles."""
+        slots, tiles = x.reach[L.window]
+        n, key = slots.numel(), (self._latent_rows(L).data_ptr(), L.window)
+        if key not in x.latents:                               # layers that share latents share the gathered rows
+            x.latents[key] = torch.empty(n, L.Rp, dtype=self.dtype, device=self.dev)
+            F.latent_gather(self._latent_rows(L), slots, x.latents[key])
+            self._launches += 1
+        kv = torch.empty(n, L.w_ukv.N, dtype=self.dtype, device=self.dev)
+        F.gemm_bf16(L.w_ukv, x.latents[key], out=kv)
+        F.latent_prefill(proj, kv, tiles, cat, H=L.heads, dp=L.dp, vp=L.vp, window=L.window, scale=L.scale, sink=L.sink,
+                         gate=None if L.g_col is None else proj, gcol=L.g_col or 0, status=self.status)
+        self._launches += 2
+
+
+class B200LatentModel(LatentLayers, DeviceRuntime):
     def __init__(self, cfg: KabadraConfig, src, *, quant="bf16", tp=1, rank=0, comm=None, config=None):
         assert torch.cuda.is_available(), "B200LatentModel needs a CUDA device"
         cfg.validate_tp(tp)
@@ -68,7 +150,7 @@ class B200LatentModel(DeviceRuntime):
             L.heads, L.dim, L.vdim, L.R = m.heads, m.dim, m.vdim, m.kv_rank
             L.dp, L.vp, L.Rp = pad64(m.dim), pad64(m.vdim), pad64(m.kv_rank)
             L.window, L.scale = m.window, m.scale
-            L.owner, L.stores = c.latent_layer(i), m.kv_from is None
+            L.Ro, L.owner, L.stores = L.Rp, c.latent_layer(i), m.kv_from is None
             L.norm1 = self._norm(get(p + "norm1"), Wp)
             H = m.heads
             q = pad_to(get(p + "mix.q").view(H, m.dim, -1), H, L.dp, Wp).reshape(H * L.dp, Wp)
@@ -153,9 +235,6 @@ class B200LatentModel(DeviceRuntime):
             self._unpin(data)
 
     # ------------------------------------------------------------------ step
-    def _nsplit(self, L, num_qg: int) -> int:
-        return 1 if self.f32 or L.Rp > 512 else F.latent_nsplit(num_qg, L.heads, L.Rp, L.window)
-
     def _alloc_ctx(self, T: int, S: int, max_blocks: int, num_qg: int, nsplit: int) -> StepCtx:
         x, dev, dt = self._alloc_inputs(T, S, max_blocks, num_qg, nsplit), self.dev, self.dtype
         # rows of padding sequences in a captured step are never written: zeros, so that they stay finite
@@ -164,75 +243,14 @@ class B200LatentModel(DeviceRuntime):
         x.h = new(T, self.Wp, dtype=dt, device=dev)
         x.proj = new(T * max(L.n_proj for L in self.layers), dtype=dt, device=dev)
         x.cat = new(T * max(L.n_mix + L.ff for L in self.layers), dtype=dt, device=dev)
-        if num_qg:
-            x.q_abs = new(T * max(L.heads * L.Rp for L in self.layers), dtype=dt, device=dev)
-            x.o_lat = new(T * max(L.heads * L.Rp for L in self.layers), dtype=dt, device=dev)
-            part = max((F.latent_part_floats(num_qg, L.heads, L.Rp, ns) for L in self.layers if (ns := self._nsplit(L, num_qg)) > 1),
-                       default=0)
-            if part:
-                x.o_part = torch.empty(part, dtype=torch.float32, device=dev)
-                x.ml_part = torch.empty(part // 64 * 2, dtype=torch.float32, device=dev)
-        x.short = (0, T)                    # rows [a, b) that hold every token of the split attention
-        x.reach = {}                        # window -> (cache slots in reach, query tiles) of the long portions
+        self._alloc_latent(x, T, num_qg, self.layers, new)
         return x
 
-    def _attn_short(self, L, x: StepCtx, proj, cat):
-        """Decode tokens and short portions: absorbed queries against the paged latents."""
-        a, b = x.short
-        T, H = x.T, L.heads
-        q_abs, o_lat = x.q_abs[:T * H * L.Rp].view(T, H * L.Rp), x.o_lat[:T * H * L.Rp].view(T, H * L.Rp)
-        F.head_product(proj[a:b], L.uk_t, q_abs[a:b])
-        p = LatentAttnParams()
-        p.q, p.cache, p.out, p.sink = ptr(q_abs), ptr(self.cache[L.owner]), ptr(o_lat), ptr(L.sink)
-        p.block_tables, p.positions = ptr(x.block_tables), ptr(x.positions)
-        p.qg_seq, p.qg_tok0, p.qg_ntok = ptr(x.qg[0]), ptr(x.qg[1]), ptr(x.qg[2])
-        p.nsplit = self._nsplit(L, x.num_qg)
-        if p.nsplit > 1:
-            p.o_part, p.ml_part = ptr(x.o_part), ptr(x.ml_part)
-        p.H, p.R, p.Rp, p.max_blocks, p.num_qg = H, L.R, L.Rp, x.max_blocks, x.num_qg
-        p.window, p.num_blocks, p.scale, p.status = L.window, self.num_blocks, L.scale, self.status
-        F.latent_attn(p, self.f32)
-        F.head_product(o_lat[a:b], L.uv, cat[a:b], gate=proj[a:b], gcol=L.g_col)
-        self._launches += 3 + (p.nsplit > 1)
+    def _latent_rows(self, L):
+        return self.cache[L.owner]
 
     def _prepare_step(self, x: StepCtx, batch):
-        """Which rows the split attention covers, and per window the cached rows in reach of the long portions of the step
-        with their query tiles (see `latent_prefill`)."""
-        bs, short, longs = self.block_size, [], []
-        for s in range(batch.num_seqs):
-            t0, t1 = batch.cu_seqlens[s], batch.cu_seqlens[s + 1]
-            (longs if t1 - t0 >= self.PREFILL_ATTN_MIN_TOKENS else short).append((s, t0, t1))
-        x.short = (short[0][1], short[-1][2]) if short else (0, 0)
-        x.reach, x.latents = {}, {}
-        for window in {L.window for L in self.layers} if longs else ():
-            slots, tiles, base = [], [], 0
-            for s, t0, t1 in longs:
-                end = batch.context_lens[s]
-                start = end - (t1 - t0)
-                lo = max(0, start - window + 1)
-                pos = torch.arange(lo, end)
-                slots.append(torch.tensor(batch.block_tables[s], dtype=torch.long)[pos // bs] * bs + pos % bs)
-                for a in range(t0, t1, 128):
-                    p0, n = start + a - t0, min(128, t1 - a)
-                    tiles.append((p0 + n - max(0, p0 - window + 1), a, n, p0, base, lo))
-                base += end - lo
-            tiles.sort(key=lambda t: -t[0])                    # most keys first
-            x.reach[window] = (torch.cat(slots).to(self.dev, non_blocking=True),
-                               torch.tensor([t[1:] for t in tiles], dtype=torch.int32).t().contiguous().to(self.dev, non_blocking=True))
-
-    def _attn_long(self, L, x: StepCtx, proj, cat):
-        """Long portions of prompts: keys and values of every cached latent in reach, then windowed query tiles."""
-        slots, tiles = x.reach[L.window]
-        n, key = slots.numel(), (L.owner, L.window)
-        if key not in x.latents:                               # layers that share latents share the gathered rows
-            x.latents[key] = torch.empty(n, L.Rp, dtype=self.dtype, device=self.dev)
-            F.latent_gather(self.cache[L.owner], slots, x.latents[key])
-            self._launches += 1
-        kv = torch.empty(n, L.w_ukv.N, dtype=self.dtype, device=self.dev)
-        F.gemm_bf16(L.w_ukv, x.latents[key], out=kv)
-        F.latent_prefill(proj, kv, tiles, cat, H=L.heads, dp=L.dp, vp=L.vp, window=L.window, scale=L.scale, sink=L.sink,
-                         gate=proj, gcol=L.g_col, status=self.status)
-        self._launches += 2
+        self._prepare_latent(x, batch, self.layers)
 
     def _run_layers(self, x: StepCtx):
         c, T = self.cfg, x.T
@@ -252,9 +270,9 @@ class B200LatentModel(DeviceRuntime):
                 F.latent_store(proj, L.kv_col, L.kv_norm, x.slot_mapping, self.cache[i], L.R, c.rms_eps)
                 n += 1
             if x.num_qg:
-                self._attn_short(L, x, proj, cat)
+                self._attn_latent_short(L, x, proj, cat)
             if x.reach:
-                self._attn_long(L, x, proj, cat)               # after the split attention, whose row range may span these
+                self._attn_latent_long(L, x, proj, cat)        # after the split attention, whose row range may span these
             n += L.w_out(cat, x.x, F.GEPI_RESID32, F.gemm_epilogue(resid32=x.x))
             self._launches += n + 1
         nvtx_end()

@@ -26,6 +26,8 @@ GROUPS = {
     "hybrid": ("fused_ar.cu", "gdn.cu", "gdn_chunk.cu", "gemv_w8a16.cu"),
     "latent": ("latent_ops.cu", "latent_attn.cu", "latent_decode.cu", "latent_prefill.cu"),
     "gla": ("gla.cu", "gla_chunk.cu"),
+    "conv": ("conv.cu",),
+    "ssd": ("ssd.cu", "ssd_chunk.cu"),
     "moe": ("moe_route.cu", "gemm_grouped.cu"),
 }
 

@@ -105,6 +105,29 @@ class GlaParams(ctypes.Structure):
                 ("s_ws", _P), ("nc", _I), ("num_long", _I)]
 
 
+class NormRopeParams(ctypes.Structure):
+    _fields_ = [("proj", _P), ("q_w", _P), ("k_w", _P), ("inv_freq", _P), ("positions", _P), ("slot_mapping", _P), ("q_out", _P),
+                ("kcache", _P), ("vcache", _P), ("T", _I), ("ld", _I), ("q_col", _I), ("k_col", _I), ("v_col", _I), ("H", _I), ("G", _I),
+                ("dim", _I), ("dp", _I), ("vp", _I), ("half", _I), ("num_blocks", _I), ("eps", _F)]
+
+
+class ConvParams(ctypes.Structure):
+    _fields_ = [("proj", _P), ("w", _P), ("bias", _P), ("state", _P), ("slots", _P), ("cu", _P), ("tiles", _P), ("out", _P),
+                ("positions", _P), ("slot_mapping", _P), ("q_out", _P), ("kcache", _P), ("vcache", _P), ("snap_rel", _P), ("snap_idx", _P),
+                ("snap", _P), ("T", _I), ("S", _I), ("ld", _I), ("col", _I), ("C", _I), ("taps", _I), ("num_tiles", _I), ("ldo", _I),
+                ("silu", _I), ("H", _I), ("G", _I), ("dp", _I), ("vp", _I), ("num_blocks", _I), ("temp_every", _I), ("num_snap", _I),
+                ("temp_coef", _F)]
+
+
+class SsdParams(ctypes.Structure):
+    _fields_ = [("xbc", _P), ("proj", _P), ("dt_bias", _P), ("neg_a", _P), ("D", _P), ("norm", _P), ("state", _P), ("slots", _P),
+                ("cu", _P), ("seqs", _P), ("y", _P), ("out", _P), ("snap_rel", _P), ("snap_idx", _P), ("snap", _P),
+                ("ldx", _I), ("ld", _I), ("ldo", _I), ("x_col", _I), ("b_col", _I), ("c_col", _I), ("z_col", _I), ("dt_col", _I),
+                ("H", _I), ("G", _I), ("V", _I), ("vp", _I), ("num_snap", _I), ("norm_groups", _I), ("eps", _F),
+                ("ck_seq", _P), ("ck_tok0", _P), ("ck_ntok", _P), ("ck_snap", _P), ("long_seq", _P), ("long_ck", _P), ("g_ws", _P),
+                ("s_ws", _P), ("nc", _I), ("num_long", _I)]
+
+
 class MoeRouteParams(ctypes.Structure):
     _fields_ = [("logits", _P), ("correction", _P), ("valid", _P), ("ids", _P), ("weight", _P), ("pos", _P), ("counts", _P),
                 ("ticket", _P), ("first", _P), ("tiles", _P), ("num_tiles", _P), ("M", _I), ("E", _I), ("identity", _I), ("top", _I),
@@ -177,6 +200,15 @@ _l.register("ti_gla_step", _I, [ctypes.POINTER(GlaParams), _I, _I, _I, _I, _P], 
 _l.register("ti_gla_chunk_size", _I, [_I], "gla")
 _l.register("ti_gla_chunked", _I, [ctypes.POINTER(GlaParams), _I, _I, _P], "gla")
 _l.register("ti_gla_finish", _I, [ctypes.POINTER(GlaParams), _I, _I, _I, _P], "gla")
+_l.register("ti_norm_rope_params_size", _I, [], "attention")
+_l.register("ti_norm_rope", _I, [ctypes.POINTER(NormRopeParams), _I, _P], "attention")
+_l.register("ti_conv_params_size", _I, [], "conv")
+_l.register("ti_conv", _I, [ctypes.POINTER(ConvParams), _I, _P], "conv")
+_l.register("ti_ssd_params_size", _I, [], "ssd")
+_l.register("ti_ssd_step", _I, [ctypes.POINTER(SsdParams), _I, _I, _I, _P], "ssd")
+_l.register("ti_ssd_finish", _I, [ctypes.POINTER(SsdParams), _I, _I, _P], "ssd")
+_l.register("ti_ssd_chunk_size", _I, [_I], "ssd")
+_l.register("ti_ssd_chunked", _I, [ctypes.POINTER(SsdParams), _I, _P], "ssd")
 _l.register("ti_moe_route_params_size", _I, [], "moe")
 _l.register("ti_moe_route", _I, [ctypes.POINTER(MoeRouteParams), _P], "moe")
 _l.register("ti_moe_norm_route", _I, [ctypes.POINTER(ResidNormParams), ctypes.POINTER(MoeRouteParams), _P, _P, _P, _I, _P], "moe")
@@ -218,7 +250,10 @@ _PARAM_SIZES = {"base": (("ti_topk_params_size", TopkParams), ("ti_edit_params_s
                 "latent": (("ti_latent_attn_params_size", LatentAttnParams),),
                 "rows": (("ti_resid_norm_params_size", ResidNormParams),),
                 "attention": (("ti_qkv_prep_params_size", QkvPrepParams), ("ti_attn_params_size", AttnParams),
-                              ("ti_rope_unit_params_size", RopeUnitParams), ("ti_attn_general_params_size", AttnGeneralParams)),
+                              ("ti_rope_unit_params_size", RopeUnitParams), ("ti_attn_general_params_size", AttnGeneralParams),
+                              ("ti_norm_rope_params_size", NormRopeParams)),
+                "conv": (("ti_conv_params_size", ConvParams),),
+                "ssd": (("ti_ssd_params_size", SsdParams),),
                 "gla": (("ti_gla_params_size", GlaParams),),
                 "moe": (("ti_moe_route_params_size", MoeRouteParams),),
                 "hybrid": (("ti_gdn_params_size", GdnParams), ("ti_gdn_chunk_params_size", GdnChunkParams),
@@ -849,6 +884,11 @@ def rope_unit(p: RopeUnitParams, f32: bool):
     check(_l.lib().ti_rope_unit(ctypes.byref(p), int(f32), stream()), "ti_rope_unit")
 
 
+def norm_rope(p: NormRopeParams, f32: bool):
+    """Queries and keys normed over all their heads together, turned in neighbouring pairs; keys and values into the cache."""
+    check(_l.lib().ti_norm_rope(ctypes.byref(p), int(f32), stream()), "ti_norm_rope")
+
+
 def attn_general(p: AttnGeneralParams, f32: bool):
     if not p.status:
         p.status = status_ptr()
@@ -907,6 +947,59 @@ def gla_chunked(p: GlaParams, dk: int, dv: int):
 
 def gla_finish(p: GlaParams, T: int, dv: int, f32: bool):
     check(_l.lib().ti_gla_finish(ctypes.byref(p), T, dv, int(f32), stream()), "ti_gla_finish")
+
+
+# ------------------------------------------------------------------------------------ short convolutions
+CONV_TILE = 16          # tokens a block of the convolution walks
+
+
+def conv_tiles(cu_seqlens) -> torch.Tensor:
+    """int32 [3, n] = sequence | first flat token | tokens: the sequences of a step cut into tiles."""
+    rows = [(s, a, min(CONV_TILE, t1 - a)) for s, (t0, t1) in enumerate(zip(cu_seqlens[:-1], cu_seqlens[1:])) for a in range(t0, t1, CONV_TILE)]
+    return torch.tensor(rows, dtype=torch.int32).view(-1, 3).t().contiguous()
+
+
+def conv(p: ConvParams, f32: bool):
+    """Causal convolution of a step's tokens (two kernels when p.cu is set, else one)."""
+    check(_l.lib().ti_conv(ctypes.byref(p), int(f32), stream()), "ti_conv")
+
+
+# ------------------------------------------------------------------------------------ state-space mixer
+SSD_STATE_SIZES = (64, 128, 256, 512)     # state sizes the kernels are built for
+
+
+def ssd_chunk_size(Np: int) -> int:
+    """Tokens of a chunk for this state size (0: no chunked form)."""
+    return _l.lib().ti_ssd_chunk_size(Np)
+
+
+class SsdWorkspace:
+    """Running decays, step sizes and chunk states of the chunked form; grows on demand."""
+
+    def __init__(self, device):
+        self.device, self.g, self.s = device, None, None
+
+    def get(self, nc: int, H: int, Np: int, vp: int):
+        ng, ns = nc * H * 2 * ssd_chunk_size(Np), nc * H * Np * vp
+        if self.g is None or self.g.numel() < ng:
+            self.g = torch.empty(ng, dtype=torch.float32, device=self.device)
+        if self.s is None or self.s.numel() < ns:
+            self.s = torch.empty(ns, dtype=torch.float32, device=self.device)
+        return self.g, self.s
+
+
+def ssd_step(p: SsdParams, num_seqs: int, Np: int, f32: bool):
+    check(_l.lib().ti_ssd_step(ctypes.byref(p), num_seqs, Np, int(f32), stream()), "ti_ssd_step")
+
+
+def ssd_chunked(p: SsdParams, Np: int):
+    """Outputs and states of the sequences with chunks (bf16 inputs); three kernels."""
+    check(_l.lib().ti_ssd_chunked(ctypes.byref(p), Np, stream()), "ti_ssd_chunked")
+
+
+def ssd_finish(p: SsdParams, T: int, f32: bool):
+    """silu(z) gate and the norm of equal parts."""
+    check(_l.lib().ti_ssd_finish(ctypes.byref(p), T, int(f32), stream()), "ti_ssd_finish")
 
 
 # ------------------------------------------------------------------------------------ experts
