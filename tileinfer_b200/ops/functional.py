@@ -865,7 +865,7 @@ def resid_norm(y, x, w_out, h, w_next, W, eps, routed=None):
     """x += rmsnorm(y) * w_out (fp32 rows; w_out None: x += y), then h = rmsnorm(x) * w_next unless w_next is None.  With `routed` (a
     TokenGroups after `moe_permute`) y holds the experts' rows and h the input of the identity experts."""
     p = _resid_params(y, x, w_out, h, w_next, W, eps, routed)
-    check(_l.lib().ti_resid_norm(ctypes.byref(p), x.shape[0], _f32(y), stream()), "ti_resid_norm")
+    check(_l.lib().ti_resid_norm(ctypes.byref(p), x.shape[0], _f32(h), stream()), "ti_resid_norm")
 
 
 def _resid_params(y, x, w_out, h, w_next, W, eps, routed=None) -> ResidNormParams:
