@@ -192,3 +192,78 @@ def forward(cfg, w, tokens, dtype=torch.float32):
         stream.append(x)
     cap = cfg["logit_softcap"]
     return cap * torch.tanh(norm(x, w["final.norm"], eps) @ w["head"].T / cap), torch.stack(stream)
+
+
+# ---------------------------------------------------------------------------------------------- small models for tests
+def tensor_shapes(cfg):
+    """name -> shape of every tensor of a configuration."""
+    W, V = cfg["width"], cfg["vocab"]
+    s = {"embed": (V, W), "final.norm": (W,), "head": (V, W)}
+    for i, layer in enumerate(cfg["layers"]):
+        m, f, p = layer["mixer"], layer["mlp"], f"l{i}."
+        s[p + "norm1"] = (W,)
+        if f is not None:
+            s[p + "norm2"] = (W,)
+            ff = f["ff"] if f["kind"] == "dense" else f["expert"]["ff"]
+            units = [""] if f["kind"] == "dense" else [f"e{e}." for e in range(f["router"]["experts"])]
+            for u in units:
+                for n, shape in (("gate", (ff, W)), ("up", (ff, W)), ("down", (W, ff))):
+                    s[f"{p}mlp.{u}{n}"] = shape
+                    if u == "":
+                        s[f"{p}mlp.{n}.b"] = shape[:1]
+            if f["kind"] == "moe":
+                s[p + "mlp.router"] = (f["router"]["experts"], W)
+        p += "mix."
+        if layer["type"] == "latent_attention":
+            H, D, R, P, E = m["heads"], m["dim"], m["kv_rank"], m["rot_dim"], m["vdim"]
+            s[p + "q"], s[p + "dkv"], s[p + "dkv.norm"] = (H * (D + P), W), (R + P, W), (R,)
+            s[p + "uk"], s[p + "uv"], s[p + "o"] = (H * D, R), (H * E, R), (W, H * E)
+            continue
+        a, q = (m["left"], p + "left.") if layer["type"] == "parallel" else (m, p)
+        for n, rows in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])):
+            s[q + n] = (rows, W)
+            if layer["type"] == "attention":
+                s[f"{q}{n}.conv"] = (rows, m["conv"])
+            else:
+                s[f"{q}{n}.b"] = (rows,)
+                if n != "v":
+                    s[f"{q}{n}.norm"] = (rows,)
+        s[q + "o"] = (W, a["heads"] * a["vdim"])
+        if layer["type"] == "attention":
+            s[p + "g"] = (m["heads"], W)
+            continue
+        r, q = m["right"], p + "right."
+        inner, bc = r["heads"] * r["vdim"], r["groups"] * r["state"]
+        s[q + "in"], s[q + "o"], s[q + "norm"] = (2 * inner + 2 * bc + r["heads"], W), (W, inner), (inner,)
+        s[q + "conv"], s[q + "conv.b"] = (inner + 2 * bc, r["conv"]), (inner + 2 * bc,)
+        s[q + "dt_bias"] = s[q + "A_log"] = s[q + "D"] = (r["heads"],)
+    return s
+
+
+def random_weights(cfg, seed=0, decisive=False):
+    """bfloat16 weights at which every mechanism leaves a mark: scores of a few units, decays between a token and tens of
+    tokens, norms away from their neutral value, biases.  `decisive`: one channel of the residual is a constant that no layer
+    touches, and the routers see it with weights so far apart that every token chooses the same experts, whatever the
+    precision of its scores."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in tensor_shapes(cfg).items():
+        t, last = torch.randn(shape, generator=g), name.rsplit(".", 1)[-1]
+        if "norm" in last:
+            t = (1.0 if ".mix." in name else 0.0) + 0.2 * t
+        elif last == "b" or last in ("dt_bias", "A_log"):
+            t = 0.4 * t
+        elif last not in ("embed", "D"):
+            t = t * (1.7 if last == "router" else 1.0) / math.sqrt(shape[-1])
+        if decisive:
+            if name == "embed":
+                t[:, 0] = 4.0
+            elif last in ("o", "down") or name.endswith("down.b"):
+                t[0] = 0.0
+            elif last == "router":
+                t = 0.1 * t
+                t[:, 0] = 1.5 * torch.randperm(shape[0], generator=g)
+            elif name.endswith("norm2"):
+                t[0] = 0.0
+        out[name] = t.to(torch.bfloat16)
+    return out

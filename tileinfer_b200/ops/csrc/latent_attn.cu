@@ -388,7 +388,6 @@ int ti_latent_attn(const ti::LatentAttnParams* pp, int f32, void* stream) {
     return -2;
   cudaStream_t st = (cudaStream_t)stream;
   if (f32 || !ti_latent_attn_splits(p.Rp, p.Ro)) {
-    if (p.nsplit != 1) return -2;
     const size_t smem = (p.Rp + 64) * sizeof(float);
     ti::launch_kernel(f32 ? ti::latent_any_kernel<float> : ti::latent_any_kernel<ti::bf16>, dim3(p.num_qg, p.H), dim3(128), smem,
                       st, true, p);
