@@ -249,7 +249,7 @@ def _conv_setup(dtype, C, taps, lens, seed=0):
     proj = rnd(T, C + 24)
     state = rnd(S + 2, taps - 1, C)
     cu = [sum(lens[:i]) for i in range(S + 1)]
-    slots = torch.tensor([(3 * s + 1) % (S + 2) for s in range(S)], dtype=torch.int32).cuda()
+    slots = torch.tensor([S - s for s in range(S)], dtype=torch.int32).cuda()
     return proj, state, cu, slots, rnd(C, taps).float(), rnd(C).float()
 
 
@@ -337,7 +337,7 @@ class Ssm:
         self.H, self.V, self.N, self.G, self.vp, self.Np = H, V, N, G, pad64(V), next(s for s in F.SSD_STATE_SIZES if s >= N)
         x, B, C, z, dt = (t.to(dtype).float() for t in (rnd(T, H, V), rnd(T, G, N), rnd(T, G, N), rnd(T, H, V), rnd(T, H)))
         self.A, self.D, bias, norm = rnd(H) * 0.5 + decay, rnd(H), rnd(H) * 0.5, torch.rand(H * V, generator=g) + 0.5
-        self.slots = torch.tensor([(3 * s + 1) % (len(lens) + 2) for s in range(len(lens))], dtype=torch.int32)
+        self.slots = torch.tensor([len(lens) - s for s in range(len(lens))], dtype=torch.int32)
         S0 = rnd(len(lens) + 2, H, N, V)
         self.y, self.states, self.snaps = torch.zeros(T, H, V), S0.clone(), {}
         step = torch.nn.functional.softplus(dt + bias, threshold=1e9)

@@ -338,18 +338,21 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
                            head_gate=None if L.g_col is None else proj, gcol=L.g_col or 0, out_scale=L.out_scale)
             self._launches += 1
 
-    def _state_space(self, L, x: StepCtx, proj, mix):
-        T, xbc = x.T, x.xbc[:x.T * L.C].view(x.T, L.C)
-        cp = self._conv_params(L, x, proj)
-        cp.out, cp.ldo, cp.silu = ptr(xbc), L.C, 1
-        F.conv(cp, self.f32)
+    def _conv_inputs(self, L, x: StepCtx, proj):
+        """x, B and C of a state-space layer after convolution and silu."""
+        xbc = x.xbc[:x.T * L.C].view(x.T, L.C)
+        p = self._conv_params(L, x, proj)
+        p.out, p.ldo, p.silu = ptr(xbc), L.C, 1
+        F.conv(p, self.f32)
         self._launches += 1 + (x.cu is not None and L.taps > 1)
-        p = SsdParams()
+        return xbc
+
+    def _ssd_params(self, L, x: StepCtx, xbc, proj, mix) -> SsdParams:
+        p, wide = SsdParams(), L.SH * L.sv
         p.xbc, p.proj, p.dt_bias, p.neg_a, p.D, p.norm = ptr(xbc), ptr(proj), ptr(L.dt_bias), ptr(L.neg_a), ptr(L.D), ptr(L.s_norm)
         p.state, p.slots, p.cu, p.y, p.out = ptr(self.state[L.index, "ssm"]), ptr(x.slots), ptr(x.cu), ptr(x.y), ptr(mix[:, L.n_left:])
         if x.snaps:
             p.snap_rel, p.snap_idx, p.snap, p.num_snap = ptr(x.snap_rel), ptr(x.snap_idx), ptr(x.snap_state[L.index, "ssm"]), x.num_snap
-        wide = L.SH * L.sv
         p.ldx, p.ld, p.ldo, p.x_col, p.b_col, p.c_col = L.C, proj.stride(0), mix.stride(0), 0, wide, wide + L.SG * L.Np
         p.z_col, p.dt_col, p.H, p.G, p.V, p.vp, p.norm_groups, p.eps = L.z_col, L.dt_col, L.SH, L.SG, L.SV, L.sv, L.norm_groups, self.cfg.rms_eps
         if x.short is not None:
@@ -357,13 +360,18 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
             p.ck_seq, p.ck_tok0, p.ck_ntok, p.ck_snap = (ptr(r) for r in ck)
             p.long_seq, p.long_ck, p.nc, p.num_long = ptr(x.longs), ptr(rng), ck.shape[1], x.longs.numel()
             p.g_ws, p.s_ws = (ptr(w) for w in self.ssd_ws.get(p.nc, L.SH, L.Np, L.sv))
-            F.ssd_chunked(p, L.Np)
             p.seqs = ptr(x.short)
+        return p
+
+    def _state_space(self, L, x: StepCtx, proj, mix):
+        p = self._ssd_params(L, x, self._conv_inputs(L, x, proj), proj, mix)
+        if x.short is not None:
+            F.ssd_chunked(p, L.Np)
             self._launches += 3
         num = x.S if x.short is None else x.short.numel()
         if num:
             F.ssd_step(p, num, L.Np, self.f32)
-        F.ssd_finish(p, T, self.f32)
+        F.ssd_finish(p, x.T, self.f32)
         self._launches += 1 + bool(num)
 
     def _mixer(self, L, x: StepCtx, proj, mix):
