@@ -11,13 +11,13 @@
 //           of one k = 16 step of P V, 32-byte swizzle); pages are addressed through the block table;
 //   warp 1  MMA issuer: S = Q K^T (tcgen05.mma kind::f16, M = N = 128, accumulator in TMEM, two S buffers so the
 //           next tile's S is computed while the softmax works on this one), then O += P V (N = D);
-//   warps 2-5  softmax: one thread per query row (= TMEM lane): scale, causal mask, running maximum in the exp2
-//           domain with lazy rescaling (O in TMEM is only touched when the maximum grew by more than 2^8),
+//   warps 2-5  softmax: one thread per query row (= TMEM lane) with the 128 scores of a tile in registers: scale, mask,
+//           running maximum in the exp2 domain with lazy rescaling (O in TMEM is only touched when the maximum grew by more than 2^8),
 //           P written to shared memory as the bf16 A operand of the second product; at the end O / l times the
 //           sigmoid output gate goes to [T, hq*D].
 //
 // TMEM: S0 | S1 | O = 128 + 128 + D columns (512 allocated).  Shared memory at D = 256: Q 64 KB, K 64 KB,
-// V 64 KB, P 32 KB.  Causal alignment is by absolute position (bottom-right): a chunk that continues a cached
+// V 64 KB, P 32 KB; where heads are smaller K and V have two buffers each.  Causal alignment is by absolute position (bottom-right): a chunk that continues a cached
 // prefix sees all of it.  Values may be of another size than queries and keys; the gate may be absent, per dimension or per
 // head.  A window limits the keys (the walk starts at the page of the first one any row sees), and scores may lose a slope
 // per head times the distance of the key.  Scores may be
@@ -115,7 +115,7 @@ constexpr unsigned long long kAttnWaitNs = 500000000ull;
 constexpr int kAttnThreads = 224;        // warp 0: Q/K producer, 1: MMA issuer, 2..5: softmax, 6: V producer
 constexpr int kAttnProducerV = 6;
 constexpr float kMaskVal = -1e30f;
-constexpr float kFirstMax = -1e29f;      // a row may see no key of its first tile: exp2(kMaskVal - kFirstMax) is 0
+constexpr float kFirstMax = -1e29f;      // a row may see no key of its first tile: its scores are -inf, its weights 0
 constexpr float kRescaleGap = 8.f;       // log2 units the running maximum may lag behind before O is rescaled
 
 template <int D, int DV, int MODE> struct AttnPrefillGeom {
@@ -128,9 +128,10 @@ template <int D, int DV, int MODE> struct AttnPrefillGeom {
   static constexpr int kBarBytes = 128;
   static constexpr int kPTiles = MODE == SCORE_SERIES && kQBytes + kKBytes + kVBytes + 2 * kP + kBarBytes + 1024 + 1024 <= 227 * 1024 ? 2 : 1;
   static constexpr int kPBytes = kPTiles * kP;
+  static constexpr int kStages = kQBytes + 2 * (kKBytes + kVBytes) + kPBytes + kBarBytes + 1024 + 1024 <= 227 * 1024 ? 2 : 1;   // of K and of V
   static constexpr int kHalves = MODE == SCORE_SERIES ? 2 : 1;      // threads that share a query row
   static constexpr int kThreads = MODE == SCORE_SERIES ? 384 : kAttnThreads;
-  static constexpr size_t kNeeded = (size_t)kQBytes + kKBytes + kVBytes + kPBytes + kBarBytes + 1024;
+  static constexpr size_t kNeeded = (size_t)kQBytes + kStages * (kKBytes + kVBytes) + kPBytes + kBarBytes + 1024;
   // one CTA per SM (the kernel takes all 512 TMEM columns)
   static constexpr size_t kSmem = kNeeded > 120 * 1024 ? kNeeded : 120 * 1024;
 };
@@ -168,12 +169,13 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
   using G = AttnPrefillGeom<D, DV, MODE>;
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
-  const uint32_t q_s = smem_u32(smem), k_s = q_s + G::kQBytes, v_s = k_s + G::kKBytes, p_s = v_s + G::kVBytes;
+  const uint32_t q_s = smem_u32(smem), k_s = q_s + G::kQBytes, v_s = k_s + G::kStages * G::kKBytes, p_s = v_s + G::kStages * G::kVBytes;
   const uint32_t bars = p_s + G::kPBytes;
-  const uint32_t q_full = bars, k_full = bars + 8, k_empty = bars + 16, v_full = bars + 24, v_empty = bars + 32,
-                 s_full0 = bars + 40, p_full = bars + 56, p_empty = bars + 72, tmem_slot = bars + 88;    // p: one per P tile
-  uint32_t* tmem_slot_ptr = reinterpret_cast<uint32_t*>(smem + G::kQBytes + G::kKBytes + G::kVBytes + G::kPBytes + 88);
-  constexpr int NP = G::kPTiles;
+  // two each: k and v one per stage, p one per P tile
+  const uint32_t q_full = bars, k_full = bars + 8, k_empty = bars + 24, v_full = bars + 40, v_empty = bars + 56,
+                 s_full0 = bars + 72, p_full = bars + 88, p_empty = bars + 104, tmem_slot = bars + 120;
+  uint32_t* tmem_slot_ptr = reinterpret_cast<uint32_t*>(smem + (tmem_slot - q_s));
+  constexpr int NP = G::kPTiles, NS = G::kStages;
   __shared__ int s_abort;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -190,12 +192,7 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
   if (threadIdx.x == 0) {
     s_abort = 0;
     mbar_init(q_full, 1);
-    mbar_init(k_full, 1);
-    mbar_init(k_empty, 1);
-    mbar_init(v_full, 1);
-    mbar_init(v_empty, 1);
-    mbar_init(s_full0, 1);
-    mbar_init(s_full0 + 8, 1);
+    for (int i = 0; i < 10; ++i) mbar_init(k_full + 8 * i, 1);       // up to s_full
     for (int i = 0; i < NP; ++i) {
       mbar_init(p_full + 8 * i, 128 * G::kHalves);
       mbar_init(p_empty + 8 * i, 1);
@@ -226,21 +223,23 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
           int blk[8];
 #pragma unroll
           for (int g = 0; g < 8; ++g) blk[g] = bt[min(page0 + j * 8 + g, npages - 1)];   // pages past the end repeat the last one (masked)
-          if (j > 0 && !mbar_wait(k_empty, (uint32_t)((j - 1) & 1), kAttnWaitNs, p.status)) { *abort_flag = 1; break; }
-          mbar_expect_tx(k_full, G::kKBytes);
+          const int st = j % NS;
+          if (j >= NS && !mbar_wait(k_empty + 8 * st, (uint32_t)((j / NS - 1) & 1), kAttnWaitNs, p.status)) { *abort_flag = 1; break; }
+          mbar_expect_tx(k_full + 8 * st, G::kKBytes);
 #pragma unroll
           for (int g = 0; g < 8; ++g)
-            tma_load_4d(k_s + g * (G::kSlabs * 2048), &p.map_k, 0, 0, 0, (blk[g] * p.hkv + kh) * 2, k_full);
+            tma_load_4d(k_s + st * G::kKBytes + g * (G::kSlabs * 2048), &p.map_k, 0, 0, 0, (blk[g] * p.hkv + kh) * 2, k_full + 8 * st);
         }
       } else {
         for (int j = 0; j < ntiles && !*abort_flag; ++j) {
           int blk[8];
 #pragma unroll
           for (int g = 0; g < 8; ++g) blk[g] = bt[min(page0 + j * 8 + g, npages - 1)];
-          if (j > 0 && !mbar_wait(v_empty, (uint32_t)((j - 1) & 1), kAttnWaitNs, p.status)) { *abort_flag = 1; break; }
-          mbar_expect_tx(v_full, G::kVBytes);
+          const int st = j % NS;
+          if (j >= NS && !mbar_wait(v_empty + 8 * st, (uint32_t)((j / NS - 1) & 1), kAttnWaitNs, p.status)) { *abort_flag = 1; break; }
+          mbar_expect_tx(v_full + 8 * st, G::kVBytes);
 #pragma unroll
-          for (int g = 0; g < 8; ++g) tma_load_2d(v_s + g * G::kVPage, &p.map_v, 0, (blk[g] * p.hkv + kh) * DV, v_full);
+          for (int g = 0; g < 8; ++g) tma_load_2d(v_s + st * G::kVBytes + g * G::kVPage, &p.map_v, 0, (blk[g] * p.hkv + kh) * DV, v_full + 8 * st);
         }
       }
     }
@@ -249,14 +248,14 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
     if (elect_one()) {
       constexpr uint32_t idesc_s = idesc_f16_bf16(128, 128), idesc_o = idesc_f16_bf16(128, DV);
       auto issue_qk = [&](int j) {
-        const uint32_t d = tmem_base + (uint32_t)(j & 1) * 128u;
+        const uint32_t d = tmem_base + (uint32_t)(j & 1) * 128u, kb = k_s + (j % NS) * G::kKBytes;
 #pragma unroll
         for (int s = 0; s < G::kSlabs; ++s)
 #pragma unroll
           for (int ks = 0; ks < 4; ++ks)                     // K: per 8-key group the kSlabs 64-column slabs side by side
             umma_bf16(d, smem_desc_sw128(q_s + s * (128 * 128) + ks * 32),
-                      smem_desc_sw128_sbo(k_s + s * 1024 + ks * 32, G::kSlabs * 1024), idesc_s, (s | ks) ? 1u : 0u);
-        umma_commit(k_empty);
+                      smem_desc_sw128_sbo(kb + s * 1024 + ks * 32, G::kSlabs * 1024), idesc_s, (s | ks) ? 1u : 0u);
+        umma_commit(k_empty + 8 * (j % NS));
         umma_commit(s_full0 + 8 * (j & 1));
       };
       bool ok = mbar_wait(q_full, 0, kAttnWaitNs, p.status) && mbar_wait(k_full, 0, kAttnWaitNs, p.status);
@@ -266,19 +265,19 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
       }
       for (int j = 0; j < ntiles && ok && !*abort_flag; ++j) {
         if (j + 1 < ntiles) {
-          ok = mbar_wait(k_full, (uint32_t)((j + 1) & 1), kAttnWaitNs, p.status);
+          ok = mbar_wait(k_full + 8 * ((j + 1) % NS), (uint32_t)(((j + 1) / NS) & 1), kAttnWaitNs, p.status);
           if (!ok) break;
           tc_fence_after();
           issue_qk(j + 1);
         }
-        ok = mbar_wait(p_full + 8 * (j % NP), (uint32_t)((j / NP) & 1), kAttnWaitNs, p.status) && mbar_wait(v_full, (uint32_t)(j & 1), kAttnWaitNs, p.status);
+        ok = mbar_wait(p_full + 8 * (j % NP), (uint32_t)((j / NP) & 1), kAttnWaitNs, p.status) && mbar_wait(v_full + 8 * (j % NS), (uint32_t)((j / NS) & 1), kAttnWaitNs, p.status);
         if (!ok) break;
         tc_fence_after();
 #pragma unroll
         for (int g = 0; g < 8; ++g)
           umma_bf16(tmem_base + 256u, smem_desc_sw128(p_s + (j % NP) * G::kP + (g >> 2) * (128 * 128) + (g & 3) * 32),
-                    smem_desc_sw32(v_s + g * G::kVPage), idesc_o, (j | g) ? 1u : 0u);
-        umma_commit(v_empty);
+                    smem_desc_sw32(v_s + (j % NS) * G::kVBytes + g * G::kVPage), idesc_o, (j | g) ? 1u : 0u);
+        umma_commit(v_empty + 8 * (j % NS));
         umma_commit(p_empty + 8 * (j % NP));
       }
       if (!ok) *abort_flag = 1;
@@ -381,27 +380,38 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
       tc_fence_after();
       const uint32_t s_addr = lane_base + (uint32_t)(j & 1) * 128u;
       const int key0 = first + j * 128, from = lo - key0, to = pos - key0;       // the row sees keys from .. to of the tile
-      const bool need_mask = to < 127 || from > 0;
-      const float ahead = slope * (float)-to;
-      // ---- pass 1: row maximum
-      float mx = kMaskVal;
+      // ---- the row's scores (PLAIN: still to be scaled) and their maximum
+      uint32_t v[4][32];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        uint32_t v[32];
-        tmem_ld32(s_addr + c * 32, v);
-        tmem_ld_wait();
+      for (int c = 0; c < 4; ++c) tmem_ld32(s_addr + c * 32, v[c]);
+      tmem_ld_wait();
+      if (MODE != SCORE_PLAIN) {
+        const float ahead = slope * (float)-to;
 #pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          float s = prefill_score<MODE>(p, __uint_as_float(v[i]), fmaf(slope, (float)(c * 32 + i), ahead));
-          if (need_mask && (c * 32 + i > to || c * 32 + i < from)) s = kMaskVal;
-          mx = fmaxf(mx, s);
-        }
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            v[c][i] = __float_as_uint(prefill_score<MODE>(p, __uint_as_float(v[c][i]), fmaf(slope, (float)(c * 32 + i), ahead)));
       }
+      if (to < 127 || from > 0) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i > to || c * 32 + i < from) v[c][i] = 0xff800000u;
+      }
+      float mx = __uint_as_float(0xff800000u);
+#pragma unroll
+      for (int c = 0; c < 4; ++c)
+#pragma unroll
+        for (int i = 0; i < 32; ++i) mx = fmaxf(mx, __uint_as_float(v[c][i]));
+      const float factor = MODE == SCORE_PLAIN ? p.scale_log2e : 1.f;
+      mx *= factor;
       const float m_new = fmaxf(m_used, mx);
       const bool resc = m_new - m_used > kRescaleGap;
       float alpha = 1.f;
       if (resc) {
-        alpha = exp2f(m_used - m_new);
+        alpha = ex2_approx(m_used - m_new);
         l *= alpha;
         m_used = m_new;
       }
@@ -414,33 +424,24 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
         if (__any_sync(0xffffffffu, resc)) {
 #pragma unroll 1
           for (int c = 0; c < DV / 32; ++c) {
-            uint32_t v[32];
-            tmem_ld32(lane_base + 256u + c * 32, v);
+            uint32_t o[32];
+            tmem_ld32(lane_base + 256u + c * 32, o);
             tmem_ld_wait();
 #pragma unroll
-            for (int i = 0; i < 32; ++i) v[i] = __float_as_uint(__uint_as_float(v[i]) * alpha);
-            tmem_st32(lane_base + 256u + c * 32, v);
+            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+            tmem_st32(lane_base + 256u + c * 32, o);
           }
           tmem_st_wait();
         }
       }
-      // ---- pass 2: P = exp2(S - m), row sum, bf16 A operand in the 128-byte-swizzled K-major layout
+      // ---- P = exp2(S - m), row sum, bf16 A operand in the 128-byte-swizzled K-major layout
       float sum = 0.f;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        uint32_t v[32];
-        tmem_ld32(s_addr + c * 32, v);
-        tmem_ld_wait();
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          float s0 = prefill_score<MODE>(p, __uint_as_float(v[i]), fmaf(slope, (float)(c * 32 + i), ahead));
-          float s1 = prefill_score<MODE>(p, __uint_as_float(v[i + 1]), fmaf(slope, (float)(c * 32 + i + 1), ahead));
-          if (need_mask) {
-            if (c * 32 + i > to || c * 32 + i < from) s0 = kMaskVal;
-            if (c * 32 + i + 1 > to || c * 32 + i + 1 < from) s1 = kMaskVal;
-          }
-          const float p0 = exp2f(s0 - m_used), p1 = exp2f(s1 - m_used);
+          const float p0 = ex2_approx(fmaf(__uint_as_float(v[c][i]), factor, -m_used)), p1 = ex2_approx(fmaf(__uint_as_float(v[c][i + 1]), factor, -m_used));
           sum += p0 + p1;
           pk[i >> 1] = pack_bf16(p0, p1);
         }
