@@ -95,34 +95,66 @@ struct NormRopeParams {
 // A block per token: x / sqrt(mean over all heads of x^2 + eps) * w for the queries and for the keys, then the rotation of
 // neighbouring dimensions; values are only stored.
 template <typename T>
-__global__ void __launch_bounds__(256) norm_rope_kernel(const __grid_constant__ NormRopeParams p) {
+__global__ void __launch_bounds__(1024) norm_rope_kernel(const __grid_constant__ NormRopeParams p) {
   extern __shared__ float cs[];                            // [half] cosines, [half] sines
-  __shared__ float red[2][8];
-  const int tid = threadIdx.x, t = blockIdx.x, nq = p.H * p.dp, nk = p.G * p.dp;
+  __shared__ float red[2][32];
+  const int tid = threadIdx.x, nt = blockDim.x, t = blockIdx.x, nq = p.H * p.dp, nk = p.G * p.dp, nv = p.G * p.vp, step = nt * 8;
   pdl_trigger();
   pdl_wait();
   const T* row = static_cast<const T*>(p.proj) + (size_t)t * p.ld;
+  const long long slot = p.slot_mapping[t], blk = slot >> 4;
+  const int off = (int)(slot & 15);
+  const bool stored = slot >= 0 && blk < p.num_blocks;
+  auto source = [&](int c) { return c < nq ? row + p.q_col + c : row + p.k_col + c - nq; };
+  constexpr int KEEP = 1;                                  // vectors a thread keeps between the two passes
+  float keep[KEEP][8], sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j)
+    if (tid * 8 + j * step < nq + nk) load8(source(tid * 8 + j * step), keep[j]);
   const float pos = (float)p.positions[t];
-  for (int i = tid; i < p.half; i += 256) sincosf(pos * p.inv_freq[i], &cs[p.half + i], &cs[i]);
-  float sq = 0.f, sk = 0.f;
-  for (int c = tid * 8; c < nq + nk; c += 2048) {
-    float v[8], s = 0.f;
-    load8(c < nq ? row + p.q_col + c : row + p.k_col + c - nq, v);
+  for (int i = tid; i < p.half; i += nt) sincosf(pos * p.inv_freq[i], &cs[p.half + i], &cs[i]);
+  auto square = [&](int c, const float (&v)[8]) {
+    float s = 0.f;
 #pragma unroll
     for (int i = 0; i < 8; ++i) s += v[i] * v[i];
     if (c < nq) sq += s;
     else sk += s;
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j)
+    if (tid * 8 + j * step < nq + nk) square(tid * 8 + j * step, keep[j]);
+  for (int c = tid * 8 + KEEP * step; c < nq + nk; c += step) {
+    float v[8];
+    load8(source(c), v);
+    square(c, v);
   }
-  const float rq = rsqrtf(block_sum32(sq, red[0]) / (float)(p.H * p.dim) + p.eps);
-  const float rk = rsqrtf(block_sum32(sk, red[1]) / (float)(p.G * p.dim) + p.eps);
-  const long long slot = p.slot_mapping[t], blk = slot >> 4;
-  const int off = (int)(slot & 15);
-  const bool stored = slot >= 0 && blk < p.num_blocks;
-  for (int c = tid * 8; c < nq + (stored ? nk : 0); c += 2048) {
+  if (stored) {                                            // values while the sums meet
+    T* dst = static_cast<T*>(p.vcache) + (size_t)blk * nv * 16 + off;
+    for (int c = (nt - 1 - tid) * 8; c < nv; c += step) {
+      float v[8];
+      load8(row + p.v_col + c, v);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) dst[(size_t)(c + i) * 16] = from_f<T>(v[i]);
+    }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((tid & 31) == 0) {
+    red[0][tid >> 5] = sq;
+    red[1][tid >> 5] = sk;
+  }
+  __syncthreads();
+  sq = sk = 0.f;
+  for (int w = 0; w < nt >> 5; ++w) {
+    sq += red[0][w];
+    sk += red[1][w];
+  }
+  const float rq = rsqrtf(sq / (float)(p.H * p.dim) + p.eps), rk = rsqrtf(sk / (float)(p.G * p.dim) + p.eps);
+  auto put = [&](int c, float (&v)[8]) {
     const bool is_q = c < nq;
-    const int e = is_q ? c : c - nq, d = e % p.dp;
-    float v[8], w[8];
-    load8(row + (is_q ? p.q_col : p.k_col) + e, v);
+    if (!is_q && !stored) return;
+    const int e = is_q ? c : c - nq, g = e / p.dp, d = e - g * p.dp;
+    float w[8];
     load8((is_q ? p.q_w : p.k_w) + e, w);
 #pragma unroll
     for (int i = 0; i < 8; ++i) v[i] *= (is_q ? rq : rk) * w[i];
@@ -135,12 +167,16 @@ __global__ void __launch_bounds__(256) norm_rope_kernel(const __grid_constant__ 
         v[i + 1] = b * co + a * si;
       }
     }
-    store8(is_q ? static_cast<T*>(p.q_out) + (size_t)t * nq + e
-                : static_cast<T*>(p.kcache) + (((size_t)blk * p.G + e / p.dp) * 16 + off) * p.dp + d, v);
+    store8(is_q ? static_cast<T*>(p.q_out) + (size_t)t * nq + e : static_cast<T*>(p.kcache) + (((size_t)blk * p.G + g) * 16 + off) * p.dp + d, v);
+  };
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j)
+    if (tid * 8 + j * step < nq + nk) put(tid * 8 + j * step, keep[j]);
+  for (int c = tid * 8 + KEEP * step; c < nq + nk; c += step) {
+    float v[8];
+    load8(source(c), v);
+    put(c, v);
   }
-  if (!stored) return;
-  T* dst = static_cast<T*>(p.vcache) + (size_t)blk * p.G * p.vp * 16 + off;
-  for (int c = tid; c < p.G * p.vp; c += 256) dst[(size_t)c * 16] = row[p.v_col + c];
 }
 
 struct AttnGeneralParams {
@@ -277,10 +313,12 @@ int ti_norm_rope_params_size() { return (int)sizeof(ti::NormRopeParams); }
 
 int ti_norm_rope(const ti::NormRopeParams* p, int f32, void* stream) {
   if (p->T <= 0) return 0;
-  if (p->dp % 8 || p->vp % 8 || p->dim > p->dp || 2 * p->half > p->dim || p->num_blocks < 1 || p->ld % 8 || p->q_col % 8 || p->k_col % 8 ||
+  if (p->dp % 8 || p->vp % 8 || p->dim > p->dp || 2 * p->half > p->dim || p->num_blocks < 1 || p->ld % 8 || p->q_col % 8 || p->k_col % 8 || p->v_col % 8 ||
       (((uintptr_t)p->proj | (uintptr_t)p->q_out | (uintptr_t)p->kcache | (uintptr_t)p->q_w | (uintptr_t)p->k_w) & 15))
     return -2;
-  ti::launch_kernel(f32 ? ti::norm_rope_kernel<float> : ti::norm_rope_kernel<ti::bf16>, dim3(p->T), dim3(256), (size_t)p->half * 8,
+  // a row in one pass of the block where there are few tokens
+  const int vecs = ((p->H + p->G) * p->dp / 8 + 31) / 32 * 32, most = p->T <= 1024 ? 1024 : 256;
+  ti::launch_kernel(f32 ? ti::norm_rope_kernel<float> : ti::norm_rope_kernel<ti::bf16>, dim3(p->T), dim3(vecs < most ? vecs : most), (size_t)p->half * 8,
                     (cudaStream_t)stream, true, *p);
   return (int)cudaGetLastError();
 }

@@ -4,8 +4,9 @@
 // optionally through silu, or its channels are the query, key and value heads of an attention layer, which go to the query
 // rows (times a factor that grows with the logarithm of the position) and into the cache pages.
 //
-// A thread owns eight channels and walks the tokens of a tile with the window in registers.  In a decode step (one token per
-// sequence) it also moves the state on; in a step with longer portions several tiles read a sequence's state, so
+// A thread owns eight channels and walks the tokens of a tile with the window in registers, four inputs in flight.  In a
+// decode step (one token per sequence) it reads the state, which no kernel of the step writes before, ahead of the wait for
+// the projection, and moves it on; in a step with longer portions several tiles read a sequence's state, so
 // `conv_tail_kernel` does that afterwards, with the snapshots.
 #include "row_vec.cuh"
 
@@ -82,7 +83,6 @@ __global__ void __launch_bounds__(128) conv_kernel(const __grid_constant__ ConvP
     for (int j = 0; j < K; ++j) load8(p.w + (size_t)j * p.C + c, w[j]);
   }
   if (p.bias != nullptr) load8(p.bias + c, b);
-  pdl_wait();
   const bool single = p.cu == nullptr;
   const int s = single ? (int)blockIdx.y : p.tiles[blockIdx.y];
   const int t0 = single ? s : p.tiles[p.num_tiles + blockIdx.y], nt = single ? 1 : p.tiles[2 * p.num_tiles + blockIdx.y];
@@ -94,28 +94,42 @@ __global__ void __launch_bounds__(128) conv_kernel(const __grid_constant__ ConvP
     if (t >= begin) load8(proj + (size_t)t * p.ld, v);
     else load8(state + (size_t)(taps - 1 + t - begin) * p.C, v);
   };
+  constexpr int AHEAD = 4;
+  float u[K - 1 + AHEAD][8];
+  if (TAPS > 0 && single) {
+#pragma unroll
+    for (int j = 0; j < K - 1; ++j) load8(state + (size_t)j * p.C, u[j]);
+  }
+  pdl_wait();
   if (TAPS > 0) {
-    float u[K][8];
+    if (!single) {
 #pragma unroll
-    for (int j = 0; j < K - 1; ++j) input(t0 - (K - 1) + j, u[j]);
-    for (int t = t0; t < t0 + nt; ++t) {
-      load8(proj + (size_t)t * p.ld, u[K - 1]);
-      float y[8];
+      for (int j = 0; j < K - 1; ++j) input(t0 - (K - 1) + j, u[j]);
+    }
+    for (int a = 0; a < nt; a += AHEAD) {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        y[i] = b[i];
+      for (int k = 0; k < AHEAD; ++k)
+        if (a + k < nt) load8(proj + (size_t)(t0 + a + k) * p.ld, u[K - 1 + k]);
 #pragma unroll
-        for (int j = 0; j < K; ++j) y[i] = fmaf(w[j][i], u[j][i], y[i]);
+      for (int k = 0; k < AHEAD; ++k) {
+        if (a + k >= nt) break;
+        float y[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          y[i] = b[i];
+#pragma unroll
+          for (int j = 0; j < K; ++j) y[i] = fmaf(w[j][i], u[k + j][i], y[i]);
+        }
+        conv_emit<T>(p, t0 + a + k, c, y);
+      }
+      if (single) {
+#pragma unroll
+        for (int j = 0; j < K - 1; ++j) store8(state + (size_t)j * p.C, u[j + 1]);
       }
 #pragma unroll
       for (int j = 0; j < K - 1; ++j)
 #pragma unroll
-        for (int i = 0; i < 8; ++i) u[j][i] = u[j + 1][i];
-      conv_emit<T>(p, t, c, y);
-    }
-    if (single) {
-#pragma unroll
-      for (int j = 0; j < K - 1; ++j) store8(state + (size_t)j * p.C, u[j]);
+        for (int i = 0; i < 8; ++i) u[j][i] = u[AHEAD + j][i];
     }
   } else {
     for (int t = t0; t < t0 + nt; ++t) {

@@ -41,8 +41,8 @@ __global__ void __launch_bounds__(128) latent_store_kernel(const T* __restrict__
   }
 }
 
-// The same with a rotated part: a warp per (token, item), item 0 the cache row [rmsnorm(latent) * w | turned key part | 0],
-// item 1 + h the trailing part of query head h, turned in place.  Dimension i of a part turns with dimension i + half.
+// The same with a rotated part: a block per token.  Warp 0 writes the cache row [rmsnorm(latent) * w | turned key part | 0],
+// the others turn the trailing part of every query head in place.  Dimension i of a part turns with dimension i + half.
 struct LatentRopeParams {
   void* proj;                    // [M, ld]: query heads at h * dp (dim plain, then 2 * half turned), latent and key part at col0
   const float* w;                // [R]
@@ -56,41 +56,43 @@ struct LatentRopeParams {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(128) latent_rope_kernel(const __grid_constant__ LatentRopeParams p) {
-  const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31, m = (int)(item / (p.H + 1)), h = (int)(item - (long long)m * (p.H + 1)) - 1;
+__global__ void __launch_bounds__(256) latent_rope_kernel(const __grid_constant__ LatentRopeParams p) {
+  extern __shared__ float cs[];                            // [half] cosines, [half] sines
+  const int m = blockIdx.x, tid = threadIdx.x;
   pdl_trigger();
   pdl_wait();
-  if (m >= p.M) return;
   T* row = static_cast<T*>(p.proj) + (size_t)m * p.ld;
   const float pos = (float)p.positions[m];
-  const T* src;
-  T* dst;
-  if (h >= 0) {
-    src = dst = row + (size_t)h * p.dp + p.dim;
-  } else {
-    const long long slot = p.slots[m];
-    if (slot < 0 || slot >= p.num_slots) return;
-    src = row + p.col0;
-    dst = static_cast<T*>(p.cache) + (size_t)slot * p.Rp;
-    float ss = 0.f;
-    for (int c = lane; c < p.R; c += 32) {
-      const float v = to_f<T>(src[c]);
-      ss += v * v;
+  for (int i = tid; i < p.half; i += 256) sincosf(pos * p.inv_freq[i], &cs[p.half + i], &cs[i]);
+  __syncthreads();
+  auto turn = [&](const T* src, T* dst, int i) {
+    const float u = to_f<T>(src[i]), v = to_f<T>(src[i + p.half]), co = cs[i], si = cs[p.half + i];
+    dst[i] = from_f<T>(u * co - v * si);
+    dst[i + p.half] = from_f<T>(v * co + u * si);
+  };
+  if (tid >= 32) {
+    for (int k = tid - 32; k < p.H * p.half; k += 224) {
+      const int h = k / p.half;
+      T* part = row + (size_t)h * p.dp + p.dim;
+      turn(part, part, k - h * p.half);
     }
-    const float rr = rsqrtf(warp_sum(ss) / (float)p.R + p.eps);
-    for (int c = lane; c < p.R; c += 32) dst[c] = from_f<T>(to_f<T>(src[c]) * rr * p.w[c]);
-    for (int c = p.R + 2 * p.half + lane; c < p.Rp; c += 32) dst[c] = from_f<T>(0.f);
-    src += p.R;
-    dst += p.R;
+    return;
   }
-  for (int i = lane; i < p.half; i += 32) {
-    float sn, cs;
-    sincosf(pos * p.inv_freq[i], &sn, &cs);
-    const float u = to_f<T>(src[i]), v = to_f<T>(src[i + p.half]);
-    dst[i] = from_f<T>(u * cs - v * sn);
-    dst[i + p.half] = from_f<T>(v * cs + u * sn);
+  const long long slot = p.slots[m];
+  if (slot < 0 || slot >= p.num_slots) return;
+  const T* src = row + p.col0;
+  T* dst = static_cast<T*>(p.cache) + (size_t)slot * p.Rp;
+  float ss = 0.f;
+#pragma unroll 4
+  for (int c = tid; c < p.R; c += 32) {
+    const float v = to_f<T>(src[c]);
+    ss += v * v;
   }
+  const float rr = rsqrtf(warp_sum(ss) / (float)p.R + p.eps);
+#pragma unroll 4
+  for (int c = tid; c < p.R; c += 32) dst[c] = from_f<T>(to_f<T>(src[c]) * rr * p.w[c]);
+  for (int c = p.R + 2 * p.half + tid; c < p.Rp; c += 32) dst[c] = from_f<T>(0.f);
+  for (int i = tid; i < p.half; i += 32) turn(src + p.R, dst + p.R, i);
 }
 
 // Latent rows of listed cache slots -> dense rows (keys of a prefill step).  Negative or out-of-range slots give zeros.
@@ -212,11 +214,11 @@ int ti_latent_store(const void* proj, int ld, int col0, const void* w, const voi
 int ti_latent_rope(void* proj, int ld, int H, int dp, int dim, int col0, const void* w, const void* inv_freq, int half, const void* positions,
                    const void* slots, void* cache, long long num_slots, int M, int R, int Rp, float eps, int f32, void* stream) {
   if (M <= 0) return 0;
-  if (dim + 2 * half > dp || R + 2 * half > Rp || half < 0 || H < 0) return -2;
+  if (dim + 2 * half > dp || R + 2 * half > Rp || half < 0 || half > 4096 || H < 0) return -2;
   const ti::LatentRopeParams p = {proj, (const float*)w, (const float*)inv_freq, (const int*)positions, (const long long*)slots, cache,
                                   num_slots, ld, H, dp, dim, col0, half, M, R, Rp, eps};
-  const dim3 grid((unsigned)(((long long)M * (H + 1) + 3) / 4));
-  ti::launch_kernel(f32 ? ti::latent_rope_kernel<float> : ti::latent_rope_kernel<ti::bf16>, grid, dim3(128), 0, (cudaStream_t)stream, true, p);
+  ti::launch_kernel(f32 ? ti::latent_rope_kernel<float> : ti::latent_rope_kernel<ti::bf16>, dim3(M), dim3(256), (size_t)half * 8,
+                    (cudaStream_t)stream, true, p);
   return (int)cudaGetLastError();
 }
 
