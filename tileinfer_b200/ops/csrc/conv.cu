@@ -4,7 +4,7 @@
 // optionally through silu, or its channels are the query, key and value heads of an attention layer, which go to the query
 // rows (times a factor that grows with the logarithm of the position) and into the cache pages.
 //
-// A thread owns eight channels and walks the tokens of a tile with the window in registers, four inputs in flight.  In a
+// A thread owns eight channels of four neighbouring tokens, with all their inputs in flight at once.  In a
 // decode step (one token per sequence) it reads the state, which no kernel of the step writes before, ahead of the wait for
 // the projection, and moves it on; in a step with longer portions several tiles read a sequence's state, so
 // `conv_tail_kernel` does that afterwards, with the snapshots.
@@ -19,7 +19,7 @@ struct ConvParams {
   void* state;                   // [slots][taps - 1][C]
   const int* slots;              // [S]
   const int* cu;                 // [S + 1] token offsets, or null: one token per sequence
-  const int* tiles;              // [3][num_tiles] sequence, first flat token, tokens; unused without cu
+  const int* tiles;              // [3][num_tiles] sequence, first flat token, tokens (at most 16); unused without cu
   void* out;                     // [T, ldo], or null: heads
   const int* positions;          // heads: [T]
   const long long* slot_mapping; // heads: [T] flat cache slot = block * 16 + offset; outside the cache: not stored
@@ -66,6 +66,8 @@ TI_DEVICE void conv_emit(const ConvParams& p, int t, int c, float (&y)[8]) {
   for (int i = 0; i < 8; ++i) v[(size_t)i * 16] = from_f<T>(y[i]);
 }
 
+constexpr int kConvTile = 16, kConvTokens = 4;             // tokens of a tile, and of a thread
+
 // TAPS 0: any number of taps, the window read again for every token
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) conv_kernel(const __grid_constant__ ConvParams p) {
@@ -85,7 +87,8 @@ __global__ void __launch_bounds__(128) conv_kernel(const __grid_constant__ ConvP
   if (p.bias != nullptr) load8(p.bias + c, b);
   const bool single = p.cu == nullptr;
   const int s = single ? (int)blockIdx.y : p.tiles[blockIdx.y];
-  const int t0 = single ? s : p.tiles[p.num_tiles + blockIdx.y], nt = single ? 1 : p.tiles[2 * p.num_tiles + blockIdx.y];
+  const int t0 = single ? s : p.tiles[p.num_tiles + blockIdx.y] + (int)blockIdx.z * kConvTokens;
+  const int nt = single ? 1 : min(kConvTokens, p.tiles[2 * p.num_tiles + blockIdx.y] - (int)blockIdx.z * kConvTokens);
   const int begin = single ? s : p.cu[s];
   T* state = static_cast<T*>(p.state) + (size_t)p.slots[s] * (taps - 1) * p.C + c;
   const T* proj = static_cast<const T*>(p.proj) + p.col + c;
@@ -94,42 +97,36 @@ __global__ void __launch_bounds__(128) conv_kernel(const __grid_constant__ ConvP
     if (t >= begin) load8(proj + (size_t)t * p.ld, v);
     else load8(state + (size_t)(taps - 1 + t - begin) * p.C, v);
   };
-  constexpr int AHEAD = 4;
-  float u[K - 1 + AHEAD][8];
+  float u[K - 1 + kConvTokens][8];
   if (TAPS > 0 && single) {
 #pragma unroll
     for (int j = 0; j < K - 1; ++j) load8(state + (size_t)j * p.C, u[j]);
   }
   pdl_wait();
   if (TAPS > 0) {
+    if (nt <= 0) return;
     if (!single) {
 #pragma unroll
       for (int j = 0; j < K - 1; ++j) input(t0 - (K - 1) + j, u[j]);
     }
-    for (int a = 0; a < nt; a += AHEAD) {
 #pragma unroll
-      for (int k = 0; k < AHEAD; ++k)
-        if (a + k < nt) load8(proj + (size_t)(t0 + a + k) * p.ld, u[K - 1 + k]);
+    for (int k = 0; k < kConvTokens; ++k)
+      if (k < nt) load8(proj + (size_t)(t0 + k) * p.ld, u[K - 1 + k]);
 #pragma unroll
-      for (int k = 0; k < AHEAD; ++k) {
-        if (a + k >= nt) break;
-        float y[8];
+    for (int k = 0; k < kConvTokens; ++k) {
+      if (k >= nt) break;
+      float y[8];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-          y[i] = b[i];
+      for (int i = 0; i < 8; ++i) {
+        y[i] = b[i];
 #pragma unroll
-          for (int j = 0; j < K; ++j) y[i] = fmaf(w[j][i], u[k + j][i], y[i]);
-        }
-        conv_emit<T>(p, t0 + a + k, c, y);
+        for (int j = 0; j < K; ++j) y[i] = fmaf(w[j][i], u[k + j][i], y[i]);
       }
-      if (single) {
+      conv_emit<T>(p, t0 + k, c, y);
+    }
+    if (single) {
 #pragma unroll
-        for (int j = 0; j < K - 1; ++j) store8(state + (size_t)j * p.C, u[j + 1]);
-      }
-#pragma unroll
-      for (int j = 0; j < K - 1; ++j)
-#pragma unroll
-        for (int i = 0; i < 8; ++i) u[j][i] = u[AHEAD + j][i];
+      for (int j = 0; j < K - 1; ++j) store8(state + (size_t)j * p.C, u[j + 1]);
     }
   } else {
     for (int t = t0; t < t0 + nt; ++t) {
@@ -184,7 +181,7 @@ __global__ void __launch_bounds__(128) conv_tail_kernel(const __grid_constant__ 
 
 template <typename T>
 static int launch_conv(const ConvParams& p, cudaStream_t st) {
-  const dim3 grid((p.C / 8 + 127) / 128, p.cu == nullptr ? p.S : p.num_tiles);
+  const dim3 grid((p.C / 8 + 127) / 128, p.cu == nullptr ? p.S : p.num_tiles, p.cu == nullptr ? 1 : kConvTile / kConvTokens);
   switch (p.taps) {
     case 2: launch_kernel(conv_kernel<T, 2>, grid, dim3(128), 0, st, true, p); break;
     case 3: launch_kernel(conv_kernel<T, 3>, grid, dim3(128), 0, st, true, p); break;

@@ -950,7 +950,7 @@ def gla_finish(p: GlaParams, T: int, dv: int, f32: bool):
 
 
 # ------------------------------------------------------------------------------------ short convolutions
-CONV_TILE = 16          # tokens a block of the convolution walks
+CONV_TILE = 16          # tokens of a tile of the convolution (kConvTile in conv.cu)
 
 
 def conv_tiles(cu_seqlens) -> torch.Tensor:
