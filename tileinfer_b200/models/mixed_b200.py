@@ -24,8 +24,10 @@ import math
 import torch
 
 from ..ops import functional as F
-from ..ops.functional import AttnGeneralParams, AttnParams, ConvParams, LinearW, NormRopeParams, SsdParams, ptr
+from ..ops.functional import LinearW, NormRopeParams, SsdParams, ptr
 from ..utils.trace import nvtx_end, nvtx_mark
+from .attention_b200 import AttentionLayers, head_rows, pad8, pad_up
+from .conv_b200 import ConvLayers
 from .experts_b200 import ExpertLayers
 from .latent_b200 import LatentLayers
 from .nogidra import ConvAttention, DenseGlu, NogidraConfig, ParallelMixer, RotaryLatent
@@ -33,21 +35,7 @@ from .paged_state_b200 import PAGE, PagedState
 from .products_b200 import Product, pad64, pad_to
 from .runtime_b200 import DeviceRuntime, StepCtx
 
-LOG2E = 1.4426950408889634
 SILU_UNIT = (math.inf, 1.0, 0.0)        # g sigmoid(g) u: limit, alpha, bias
-
-
-def _pad_up(n: int, sizes) -> int:
-    return next((s for s in sizes if s >= n), pad64(n))
-
-
-def _pad8(n: int) -> int:
-    return -(-n // 8) * 8
-
-
-def _heads(w: torch.Tensor, H: int, n: int, np_: int) -> torch.Tensor:
-    """[H * n, ...] rows of H heads -> [H * np_, ...], each head padded with zero rows."""
-    return pad_to(w.reshape(H, n, -1), H, np_, w.numel() // (H * n)).reshape(H * np_, *w.shape[1:])
 
 
 class _Layer:
@@ -56,7 +44,7 @@ class _Layer:
     moe, ff = None, 0
 
 
-class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
+class B200MixedModel(PagedState, AttentionLayers, ConvLayers, ExpertLayers, LatentLayers, DeviceRuntime):
     def __init__(self, cfg: NogidraConfig, src, *, quant="bf16", tp=1, rank=0, comm=None, config=None):
         assert torch.cuda.is_available(), "B200MixedModel needs a CUDA device"
         cfg.validate_tp(tp)
@@ -127,27 +115,10 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
         L.w_up, L.up_bias = Product(pair(g, u), self.quant, self.dev), pair(self._vec(get(p + "gate.b"), L.ff), self._vec(get(p + "up.b"), L.ff)).contiguous()
         L.w_down, L.down_bias = Product(pad_to(get(p + "down"), self.Wp, L.ff), self.quant, self.dev), self._vec(get(p + "down.b"), self.Wp)
 
-    def _attention_sizes(self, L, m):
-        sizes = (64, 128, 256) if not self.f32 and max(m.dim, m.vdim) <= 256 else ()
-        L.attn, L.heads, L.G, L.dp, L.vp = True, m.heads, m.kv_heads, _pad_up(m.dim, sizes), _pad_up(m.vdim, sizes)
-        if max(L.dp, L.vp) > 1024:
-            raise ValueError(f"attention takes heads of at most 1024, got {max(m.dim, m.vdim)}")
-        G = m.heads // m.kv_heads                            # query heads of a block: at most 16
-        L.rep = G // max(d for d in range(1, 17) if G % d == 0)
-        L.k_col, L.v_col = L.heads * L.dp, (L.heads + L.G) * L.dp
-        L.window, L.scale, L.slopes, L.g_col, L.out_scale = m.window, m.scale, None, None, 1.0
-
     def _qkv(self, L, m, get, suffix=""):
         """The tensors q, k and v with their heads padded, one below the other."""
-        return torch.cat([_heads(get(f"q{suffix}"), m.heads, m.dim, L.dp), _heads(get(f"k{suffix}"), m.kv_heads, m.dim, L.dp),
-                          _heads(get(f"v{suffix}"), m.kv_heads, m.vdim, L.vp)])
-
-    def _out(self, w, H: int, n: int, np_: int):
-        """Columns of an output matrix for padded heads."""
-        return pad_to(w.view(-1, H, n), w.shape[0], H, np_).reshape(w.shape[0], H * np_)
-
-    def _angles(self, base: float, dims: int) -> torch.Tensor:
-        return torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64).float().to(self.dev)
+        return torch.cat([head_rows(get(f"q{suffix}"), m.heads, m.dim, L.dp), head_rows(get(f"k{suffix}"), m.kv_heads, m.dim, L.dp),
+                          head_rows(get(f"v{suffix}"), m.kv_heads, m.vdim, L.vp)])
 
     def _build_conv_attention(self, L, m: ConvAttention, p: str, get):
         self._attention_sizes(L, m)
@@ -156,8 +127,8 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
         L.conv_w, L.conv_b = self._qkv(L, m, q, ".conv").t().float().contiguous(), None
         L.g_col, L.slopes = L.C, torch.tensor(m.slopes(), dtype=torch.float32, device=self.dev)
         gate = q("g")
-        rows = torch.cat([self._qkv(L, m, q), pad_to(gate, _pad8(m.heads), gate.shape[1])])
-        return rows, self._out(q("o"), m.heads, m.vdim, L.vp), None
+        rows = torch.cat([self._qkv(L, m, q), pad_to(gate, pad8(m.heads), gate.shape[1])])
+        return rows, self._out_columns(q("o"), m.heads, m.vdim, L.vp), None
 
     def _build_latent(self, L, m: RotaryLatent, p: str, get):
         H, R, P, dev = m.heads, m.kv_rank, m.rot_dim, self.dev
@@ -169,7 +140,7 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
         L.inv_freq, L.kv_norm = self._angles(m.rot_base, P), self._vec(get(p + "dkv.norm"), R)
         q, dkv = get(p + "q"), get(p + "dkv")
         L.kv_col = H * L.dp
-        rows = torch.cat([_heads(q, H, m.dim + P, L.dp), pad_to(dkv, pad64(R + P), dkv.shape[1])])
+        rows = torch.cat([head_rows(q, H, m.dim + P, L.dp), pad_to(dkv, pad64(R + P), dkv.shape[1])])
         # a query head [plain | turned] meets a cache row [latent | turned key part]: W_uk for the first, an identity for the second
         uk = pad_to(get(p + "uk").float().view(H, m.dim, R), H, L.dp, L.Rp)
         uk[:, m.dim:m.dim + P, R:R + P] = torch.eye(P, device=dev)
@@ -178,18 +149,18 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
         L.uv = uv[..., :L.Ro].to(self.dtype).contiguous()                        # [H, vp, Ro]
         if not self.f32:                                                         # rows [K of all heads | V of all heads]
             L.w_ukv = LinearW(torch.cat([uk.reshape(H * L.dp, L.Rp), uv.reshape(H * L.vp, L.Rp)]), False, dev)
-        return rows, self._out(get(p + "o"), H, m.vdim, L.vp), None
+        return rows, self._out_columns(get(p + "o"), H, m.vdim, L.vp), None
 
     def _build_parallel(self, L, m: ParallelMixer, p: str, get):
         a, r, dev = m.left, m.right, self.dev
         self._attention_sizes(L, a)
         left, right = (lambda n: get(p + "left." + n)), (lambda n: get(p + "right." + n))
         L.dim, L.half, L.inv_freq, L.out_scale = a.dim, a.rot_dims // 2, self._angles(a.rot_base, a.rot_dims), m.left_scale
-        L.q_w = _heads(left("q.norm").float(), a.heads, a.dim, L.dp).contiguous()
-        L.k_w = _heads(left("k.norm").float(), a.kv_heads, a.dim, L.dp).contiguous()
+        L.q_w = head_rows(left("q.norm").float(), a.heads, a.dim, L.dp).contiguous()
+        L.k_w = head_rows(left("k.norm").float(), a.kv_heads, a.dim, L.dp).contiguous()
         # state-space half: z | x | B | C | step sizes
         L.ssm, L.SH, L.SV, L.SG, L.norm_groups = True, r.heads, r.vdim, r.groups, r.norm_groups
-        L.sv, L.Np = pad64(r.vdim), _pad_up(r.state, F.SSD_STATE_SIZES)
+        L.sv, L.Np = pad64(r.vdim), pad_up(r.state, F.SSD_STATE_SIZES)
         if L.Np not in F.SSD_STATE_SIZES:
             raise ValueError(f"the state-space mixer takes states of at most {F.SSD_STATE_SIZES[-1]} per head, got {r.state}")
         bc, wide = r.groups * r.state, L.SH * L.sv
@@ -200,15 +171,15 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
         def channels(t):
             """x, B and C with their heads and groups padded."""
             x, B, C = t.split([r.inner, bc, bc])
-            return torch.cat([_heads(x, r.heads, r.vdim, L.sv), _heads(B, r.groups, r.state, L.Np), _heads(C, r.groups, r.state, L.Np)])
+            return torch.cat([head_rows(x, r.heads, r.vdim, L.sv), head_rows(B, r.groups, r.state, L.Np), head_rows(C, r.groups, r.state, L.Np)])
         L.conv_w, L.conv_b = channels(right("conv")).t().float().contiguous(), channels(right("conv.b")).float().contiguous()
         L.dt_bias, L.D = right("dt_bias").float().contiguous(), right("D").float().contiguous()
         L.neg_a = -torch.exp(right("A_log").float()).contiguous()
-        L.s_norm = _heads(right("norm").float(), r.heads, r.vdim, L.sv).mul(m.right_scale).contiguous()
+        L.s_norm = head_rows(right("norm").float(), r.heads, r.vdim, L.sv).mul(m.right_scale).contiguous()
         z, xbc, dt = right("in").split([r.inner, r.conv_channels, r.heads])
-        rows = torch.cat([self._qkv(L, a, left), _heads(z, r.heads, r.vdim, L.sv), channels(xbc), pad_to(dt, _pad8(r.heads), dt.shape[1])])
+        rows = torch.cat([self._qkv(L, a, left), head_rows(z, r.heads, r.vdim, L.sv), channels(xbc), pad_to(dt, pad8(r.heads), dt.shape[1])])
         L.n_left = L.heads * L.vp
-        out = torch.cat([self._out(left("o"), a.heads, a.vdim, L.vp), self._out(right("o"), r.heads, r.vdim, L.sv)], 1)
+        out = torch.cat([self._out_columns(left("o"), a.heads, a.vdim, L.vp), self._out_columns(right("o"), r.heads, r.vdim, L.sv)], 1)
         return rows, out, self._qkv(L, a, left, ".b")
 
     def weight_bytes(self, tokens: int = 1) -> int:
@@ -256,12 +227,7 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
         dense = max((L.ff for L in Ls if L.moe is None), default=0)
         if dense:
             x.ff = new(T * dense, dtype=dt, device=dev)
-        if self.attn_layers:
-            x.q = new(T * max(L.heads * L.dp for L in self.attn_layers), dtype=dt, device=dev)
-            if num_qg and not self.f32:
-                items = max(num_qg * L.G * L.rep * nsplit * (L.vp if L.vp <= 256 else 0) for L in self.attn_layers)
-                x.o_part = torch.empty(items * 16, dtype=torch.float32, device=dev)
-                x.ml_part = torch.empty(items // 64 * 32, dtype=torch.float32, device=dev)
+        self._alloc_attention(x, T, num_qg, nsplit, self.attn_layers, new)
         if self.ssm_layers:
             x.xbc = new(T * max(L.C for L in self.ssm_layers), dtype=dt, device=dev)
             x.y = new(T * max(L.SH * L.sv for L in self.ssm_layers), dtype=torch.float32, device=dev)
@@ -278,16 +244,6 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
 
     def _latent_rows(self, L):
         return self.cache[L.index][0]
-
-    def _conv_params(self, L, x: StepCtx, proj) -> ConvParams:
-        p = ConvParams()
-        p.proj, p.w, p.bias, p.state, p.slots = ptr(proj), ptr(L.conv_w), ptr(L.conv_b), ptr(self.state[L.index, "conv"]), ptr(x.slots)
-        p.T, p.S, p.ld, p.col, p.C, p.taps = x.T, x.S, proj.stride(0), L.conv_col, L.C, L.taps
-        if x.cu is not None:
-            p.cu, p.tiles, p.num_tiles = ptr(x.cu), ptr(x.conv_tiles), x.conv_tiles.shape[1]
-        if x.snaps:
-            p.snap_rel, p.snap_idx, p.snap, p.num_snap = ptr(x.snap_rel), ptr(x.snap_idx), ptr(x.snap_state[L.index, "conv"]), x.num_snap
-        return p
 
     def _conv_heads(self, L, x: StepCtx, proj):
         """Queries (returned), keys and values after their convolutions; keys and values into the cache pages."""
@@ -310,42 +266,6 @@ class B200MixedModel(PagedState, ExpertLayers, LatentLayers, DeviceRuntime):
         F.norm_rope(r, self.f32)
         self._launches += 1
         return q
-
-    def _attention(self, L, x: StepCtx, q, proj, mix):
-        """Windowed attention of the step's tokens over the cache pages into the leading columns of mix."""
-        kc, vc = self.cache[L.index]
-        if x.num_qg:
-            general = self.f32 or max(L.dp, L.vp) > 256
-            a = AttnGeneralParams() if general else AttnParams()
-            a.q, a.kcache, a.vcache, a.block_tables, a.positions = ptr(q), ptr(kc), ptr(vc), ptr(x.block_tables), ptr(x.positions)
-            a.qg_seq, a.qg_tok0, a.qg_ntok, a.out, a.status = ptr(x.qg[0]), ptr(x.qg[1]), ptr(x.qg[2]), ptr(mix), self.status
-            a.max_blocks, a.num_qg, a.num_blocks, a.ldo = x.max_blocks, x.num_qg, self.num_blocks, mix.stride(0)
-            a.window, a.slopes, a.out_scale = L.window, ptr(L.slopes), L.out_scale
-            if L.g_col is not None:
-                a.head_gate, a.ldg, a.gcol = ptr(proj), proj.stride(0), L.g_col
-            if general:
-                a.H, a.G, a.dp, a.vp, a.scale = L.heads, L.G, L.dp, L.vp, L.scale
-                F.attn_general(a, self.f32)
-            else:
-                a.o_part, a.ml_part, a.scale_log2e = ptr(x.o_part), ptr(x.ml_part), L.scale * LOG2E
-                # a split takes a page per warp at least
-                a.hq, a.hkv, a.rep, a.nsplit = L.heads, L.G, L.rep, max(1, min(x.nsplit, (L.window // PAGE + 2) // 4))
-                F.attn_paged(a, L.dp, L.vp)
-            self._launches += 1 + (not general)
-        if x.tiles is not None:
-            F.attn_prefill(q, kc, vc, self.num_blocks, x.block_tables, x.positions, x.tiles, None, mix, hq=L.heads, hkv=L.G, D=L.dp, DV=L.vp,
-                           max_blocks=x.max_blocks, ld=0, scale=L.scale, window=L.window, slopes=L.slopes,
-                           head_gate=None if L.g_col is None else proj, gcol=L.g_col or 0, out_scale=L.out_scale)
-            self._launches += 1
-
-    def _conv_inputs(self, L, x: StepCtx, proj):
-        """x, B and C of a state-space layer after convolution and silu."""
-        xbc = x.xbc[:x.T * L.C].view(x.T, L.C)
-        p = self._conv_params(L, x, proj)
-        p.out, p.ldo, p.silu = ptr(xbc), L.C, 1
-        F.conv(p, self.f32)
-        self._launches += 1 + (x.cu is not None and L.taps > 1)
-        return xbc
 
     def _ssd_params(self, L, x: StepCtx, xbc, proj, mix) -> SsdParams:
         p, wide = SsdParams(), L.SH * L.sv

@@ -12,7 +12,7 @@ from .reference_cpu import Batch, rmsnorm, rope_partial
 from .weights import fake_quant
 
 
-def _turn_pairs(x, positions, dims, base):
+def turn_pairs(x, positions, dims, base):
     """Neighbouring dimensions (2i, 2i + 1) of x [T, heads, dim] turn together."""
     inv = base ** (-torch.arange(0, dims, 2, dtype=torch.float64) / dims)
     a = positions[:, None, None].float() * inv.float()
@@ -170,7 +170,7 @@ class TorchMixedModel:
 
     def _normed(self, i: int, m, p: str, h, batch: Batch):
         T, eps = h.shape[0], self.cfg.rms_eps
-        part = lambda n, heads: _turn_pairs(rmsnorm(self._linear(h, p + n).float(), self.w[f"{p}{n}.norm"], eps, one_plus=False)
+        part = lambda n, heads: turn_pairs(rmsnorm(self._linear(h, p + n).float(), self.w[f"{p}{n}.norm"], eps, one_plus=False)
                                             .view(T, heads, m.dim), batch.positions, m.rot_dims, m.rot_base)
         self._store(self.pages[i][0], part("k", m.kv_heads), batch)
         self._store(self.pages[i][1], self._linear(h, p + "v").view(T, m.kv_heads, m.vdim), batch)

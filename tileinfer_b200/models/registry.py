@@ -79,7 +79,20 @@ def _nogidra() -> Family:
     return Family("nogidra", lambda: n.PRESETS, n.ARCHITECTURE, n.load_config, n.make_weights, executor, ("w8a16", "bf16", "fp32"))
 
 
-_MAKERS = {"hybrid": _hybrid, "kabadra": _kabadra, "gerivik": _gerivik, "nogidra": _nogidra}
+def _luvapel() -> Family:
+    from . import luvapel as v
+
+    def executor(device):
+        if device == "cuda":
+            from .delta_b200 import B200DeltaModel
+            return B200DeltaModel
+        from .delta_cpu import TorchDeltaModel
+        return TorchDeltaModel
+
+    return Family("luvapel", lambda: v.PRESETS, v.ARCHITECTURE, v.load_config, v.make_weights, executor, ("w8a16", "bf16", "fp32"))
+
+
+_MAKERS = {"hybrid": _hybrid, "kabadra": _kabadra, "gerivik": _gerivik, "nogidra": _nogidra, "luvapel": _luvapel}
 
 
 def family(name: str) -> Family:

@@ -27,6 +27,7 @@ GROUPS = {
     "latent": ("latent_ops.cu", "latent_attn.cu", "latent_decode.cu", "latent_prefill.cu"),
     "gla": ("gla.cu", "gla_chunk.cu"),
     "conv": ("conv.cu",),
+    "delta": ("delta.cu", "delta_chunk.cu"),
     "ssd": ("ssd.cu", "ssd_chunk.cu"),
     "moe": ("moe_route.cu", "gemm_grouped.cu"),
 }

@@ -10,7 +10,7 @@ namespace ti {
 
 struct RopeUnitParams {
   const void* proj;              // [T, ld]: H query heads at q_col, G key heads at k_col (dp each), G value heads at v_col (vp)
-  const float* inv_freq;         // [half] angle per position of pair i, i + half
+  const float* inv_freq;         // [half] angle per position of pair i, i + half (pairs: 2i, 2i + 1)
   const int* positions;          // [T]
   const long long* slot_mapping; // [T] flat slot = block * 16 + offset; outside the cache: not stored
   void* q_out;                   // [T, H, dp]
@@ -19,10 +19,13 @@ struct RopeUnitParams {
   unsigned* status;
   int T, ld, q_col, k_col, v_col, H, G, dim, dp, vp, half, num_blocks;
   float eps;
+  int pairs;                     // neighbouring dimensions turn together
+  const float* q_w;              // null, or [H * dp]: factors of the normed head, ahead of the rotation (0 in the padding)
+  const float* k_w;              // [G * dp]
 };
 
-// A warp per (token, head): rotation of the first 2 * half dimensions, then x / sqrt(mean(x^2) + eps); values are only
-// stored.  Everything up to the store is fp32.
+// A warp per (token, head): x / sqrt(mean(x^2) + eps), optionally times a weight, and the rotation of the first 2 * half
+// dimensions; values (which may be the columns of the keys) are only stored.  Everything up to the store is fp32.
 template <typename T, int E>
 __global__ void __launch_bounds__(128) rope_unit_kernel(const __grid_constant__ RopeUnitParams p) {
   extern __shared__ float sh[];
@@ -47,6 +50,7 @@ __global__ void __launch_bounds__(128) rope_unit_kernel(const __grid_constant__ 
   const bool is_q = head < p.H;
   if (!is_q && !stored) return;
   const T* src = row + (is_q ? p.q_col + (size_t)head * p.dp : p.k_col + (size_t)(head - p.H) * p.dp);
+  const float* w = p.q_w == nullptr ? nullptr : is_q ? p.q_w + (size_t)head * p.dp : p.k_w + (size_t)(head - p.H) * p.dp;
   float* buf = sh + (size_t)warp * p.dp;
   float ss = 0.f;
 #pragma unroll
@@ -54,7 +58,7 @@ __global__ void __launch_bounds__(128) rope_unit_kernel(const __grid_constant__ 
     const int c = lane + 32 * i;
     if (c < p.dp) {
       const float v = to_f<T>(src[c]);
-      buf[c] = v;
+      buf[c] = w == nullptr ? v : v * w[c];
       ss += v * v;                                         // a rotation keeps the sum of squares
     }
   }
@@ -64,9 +68,10 @@ __global__ void __launch_bounds__(128) rope_unit_kernel(const __grid_constant__ 
   for (int i = lane; i < p.half; i += 32) {
     float sn, cs;
     sincosf(pos * p.inv_freq[i], &sn, &cs);
-    const float u = buf[i], v = buf[i + p.half];
-    buf[i] = u * cs - v * sn;
-    buf[i + p.half] = v * cs + u * sn;
+    const int a = p.pairs ? 2 * i : i, b = p.pairs ? 2 * i + 1 : i + p.half;
+    const float u = buf[a], v = buf[b];
+    buf[a] = u * cs - v * sn;
+    buf[b] = v * cs + u * sn;
   }
   __syncwarp();
   T* dst = is_q ? static_cast<T*>(p.q_out) + ((size_t)t * p.H + head) * p.dp
@@ -197,6 +202,7 @@ struct AttnGeneralParams {
   const void* head_gate;   // null, or [T, ldg]: the sigmoid of column gcol + h scales head h
   int ldg, gcol;
   float out_scale;         // factor of the output
+  const void* gate;        // null, or [T, ldg]: the sigmoid of column gcol + h * vp + d scales dimension d of head h
 };
 
 // One query token and head per block; the four warps take the pages in turn and keep running maxima, sums and outputs.
@@ -275,6 +281,7 @@ __global__ void __launch_bounds__(128) attn_general_kernel(const __grid_constant
     float o = 0.f;
 #pragma unroll
     for (int i = 0; i < 4; ++i) o = fmaf(w[i], acc_s[i * p.vp + c], o);
+    if (p.gate != nullptr) o *= sigmoid_exact(to_f<T>(static_cast<const T*>(p.gate)[(size_t)tok * p.ldg + p.gcol + (size_t)h * p.vp + c]));
     out[c] = from_f<T>(o * f);
   }
 }

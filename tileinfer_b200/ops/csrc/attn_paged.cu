@@ -113,7 +113,7 @@ struct AttnParams {
   const int* qg_ntok;            // [num_qg] tokens in the group (1 or 2; 0 = padding group)
   float* o_part;                 // [num_qg * hkv * nsplit, 16, D]
   float* ml_part;                // [num_qg * hkv * nsplit, 16, 2]
-  const __nv_bfloat16* gate_src; // merge: proj [T, ld] (gate of q head h at h*2D + D)
+  const __nv_bfloat16* gate_src; // merge: null, or [T, ld]: gates of head h at column gate_col + h * gate_stride (stride 0: h*2D + D)
   __nv_bfloat16* out;            // merge: [T, hq*D]
   int hq, hkv, max_blocks, nsplit, ld, num_qg;
   float scale_log2e;
@@ -126,6 +126,7 @@ struct AttnParams {
   const __nv_bfloat16* head_gate;// merge: null, or [T, ldg]: gate of head h at column gcol + h
   int ldg, gcol, ldo;            // ldo: row pitch of `out` (0: hq*D)
   float out_scale;               // merge: factor of the output
+  int gate_col, gate_stride;
 };
 
 TI_DEVICE float attn_score(const AttnParams& p, float qk) {
@@ -526,7 +527,7 @@ __global__ void __launch_bounds__(D / 2) attn_merge_kernel(const __grid_constant
   if (p.head_gate != nullptr) inv *= sigmoid_f(__bfloat162float(p.head_gate[(size_t)tok * p.ldg + p.gcol + head]));
   float g0 = 1.f, g1 = 1.f;
   if (p.gate_src != nullptr) {
-    const uint32_t gw = *reinterpret_cast<const uint32_t*>(p.gate_src + (size_t)tok * p.ld + (size_t)head * 2 * D + D + d);
+    const uint32_t gw = *reinterpret_cast<const uint32_t*>(p.gate_src + (size_t)tok * p.ld + p.gate_col + (size_t)head * p.gate_stride + d);
     g0 = sigmoid_f(bf16lo(gw));
     g1 = sigmoid_f(bf16hi(gw));
   }
@@ -573,9 +574,13 @@ int ti_attn_paged(const ti::AttnParams* p, int D, int DV, void* stream) {
   if (p->num_qg <= 0) return 0;
   const int rep = p->rep < 1 ? 1 : p->rep;
   if (p->hq % (p->hkv * rep) || p->hq / (p->hkv * rep) > 16 || p->nsplit < 1 || p->nsplit > ti::kMaxSplit) return -2;
-  if (p->window < 0 || p->ldo % 2 || (p->gate_src != nullptr && D != DV)) return -2;
+  if (p->window < 0 || p->ldo % 2 || p->gate_col % 2 || p->gate_stride % 2 || (p->gate_src != nullptr && D != DV)) return -2;
   ti::AttnParams a = *p;
   a.rep = rep;
+  if (a.gate_stride == 0) {
+    a.gate_stride = 2 * D;
+    a.gate_col = D;
+  }
   dim3 grid(p->num_qg, p->hkv * rep, p->nsplit), mgrid(p->num_qg, p->hkv * rep, 16);
   cudaStream_t st = (cudaStream_t)stream;
   static const int pipe_mode = [] {

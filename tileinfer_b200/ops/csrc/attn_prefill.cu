@@ -39,7 +39,7 @@ struct AttnPrefillParams {
   const int* qt_seq;               // [num_tiles] sequence of the query tile
   const int* qt_tok0;              // [num_tiles] first flat token
   const int* qt_ntok;              // [num_tiles] tokens in the tile (1..128; 0 = padding tile)
-  const __nv_bfloat16* gate_src;   // proj [T, ld]: gate of q head h at h*2D + D
+  const __nv_bfloat16* gate_src;   // null, or [T, ld]: gates of head h at column gate_col + h * gate_stride
   __nv_bfloat16* out;              // [T, hq*D]
   unsigned* status;
   int hq, hkv, max_blocks, ld;
@@ -50,6 +50,7 @@ struct AttnPrefillParams {
   const __nv_bfloat16* head_gate;  // null, or [T, ldg]: gate of head h at column gcol + h
   int ldg, gcol, ldo;              // ldo: row pitch of `out`
   float out_scale;
+  int gate_col, gate_stride;
 };
 
 // How a score follows from q.k: scaled; capped with the series, reference 0 instead of a running maximum; capped; scaled,
@@ -350,7 +351,7 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
         tc_fence_after();
         const size_t tok = (size_t)tok0 + (valid ? r : 0);
         const float inv = head_factor(p, tok, head) / (l_s[r] + l_s[128 + r]);
-        const __nv_bfloat16* gate = p.gate_src + tok * p.ld + (size_t)head * 2 * D + D;
+        const __nv_bfloat16* gate = p.gate_src + tok * p.ld + p.gate_col + (size_t)head * p.gate_stride;
         __nv_bfloat16* dst = p.out + tok * (size_t)p.ldo + (size_t)head * DV;
 #pragma unroll 1
         for (int c = half * (DV / 64); c < (half + 1) * (DV / 64); ++c) {
@@ -468,7 +469,7 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
       tc_fence_after();
       const size_t tok = (size_t)tok0 + (valid ? r : 0);
       const float inv = head_factor(p, tok, head) / l;
-      const __nv_bfloat16* gate = p.gate_src + tok * p.ld + (size_t)head * 2 * D + D;
+      const __nv_bfloat16* gate = p.gate_src + tok * p.ld + p.gate_col + (size_t)head * p.gate_stride;
       __nv_bfloat16* dst = p.out + tok * (size_t)p.ldo + (size_t)head * DV;
 #pragma unroll 1
       for (int c = 0; c < DV / 32; ++c) {
@@ -518,7 +519,8 @@ extern "C" {
 // out[tok, head*DV + d] = softmax(score(q k^T), causal by position) v * sigmoid(gate) for the tokens of the listed query
 // tiles (up to 128 consecutive tokens of one sequence each; longest first gives the best balance).
 // q: bf16 [T, hq, D] (normalised, rotated); kcache / vcache: the paged cache of this layer, `num_blocks` pages;
-// positions: absolute position of every flat token; gate_src: the projection rows [T, ld] holding the gates, or null.
+// positions: absolute position of every flat token; gate_src: null, or rows [T, ld] with the gates of head h at column
+// gate_col + h * gate_stride (stride 0: h*2D + D).
 // score(x) = scale x, or with softcap > 0 softcap * tanh(scale x / softcap).  `qk_max`: a bound of |q.k|, or <= 0.  With
 // `slopes` [hq] a score loses slopes[h] per token of distance; `window`, `head_gate` [T, ldg], `ldo` (row pitch of out) and
 // `out_scale` as in AttnPrefillParams.
@@ -526,11 +528,11 @@ int ti_attn_prefill(const void* q, int T, const void* kcache, const void* vcache
                     const void* positions, const void* qt_seq, const void* qt_tok0, const void* qt_ntok, int num_tiles,
                     const void* gate_src, void* out, int hq, int hkv, int max_blocks, int ld, float scale, int D, int DV,
                     float softcap, float qk_max, int window, const void* slopes, const void* head_gate, int ldg, int gcol, int ldo,
-                    float out_scale, void* status, void* stream) {
+                    float out_scale, int gate_col, int gate_stride, void* status, void* stream) {
   if (num_tiles <= 0) return 0;
   if (hq % hkv || T < 1 || num_blocks < 1 || (gate_src != nullptr && D != DV)) return -2;
   // the gate and the output are read / written 16 bytes at a time: refuse layouts that would make those accesses misaligned
-  if ((ld & 7) || (ldo & 7) || (reinterpret_cast<uintptr_t>(gate_src) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return -4;
+  if ((ld & 7) || (ldo & 7) || (gate_col & 7) || (gate_stride & 7) || (reinterpret_cast<uintptr_t>(gate_src) & 15) || (reinterpret_cast<uintptr_t>(out) & 15)) return -4;
   if (window < 0 || (softcap > 0.f && (window > 0 || slopes != nullptr))) return -2;     // caps come without windows and slopes
   if ((D != 64 && D != 128 && D != 256) || (DV != 64 && DV != 128 && DV != 256)) return -3;
   constexpr float kLog2e = 1.4426950408889634f;
@@ -568,6 +570,8 @@ int ti_attn_prefill(const void* q, int T, const void* kcache, const void* vcache
   p.gcol = gcol;
   p.ldo = ldo > 0 ? ldo : hq * DV;
   p.out_scale = out_scale;
+  p.gate_stride = gate_stride > 0 ? gate_stride : 2 * D;
+  p.gate_col = gate_stride > 0 ? gate_col : D;
   cudaStream_t st = (cudaStream_t)stream;
 #define TI_AP(A, B) if (D == A && DV == B) return ti::launch_attn_prefill<A, B>(p, num_tiles, mode, st)
   TI_AP(64, 64); TI_AP(64, 128); TI_AP(64, 256);

@@ -65,8 +65,8 @@ constexpr unsigned long long kGemmWaitNs = 2000000000ull;
 // Operands of the epilogues for designs with an fp32 residual stream, a clamped gated unit, biases, scaled or capped logits.
 struct GemmEpilogue {
   const float* resid32;            // RESID32: [M, ldo] fp32
-  __nv_bfloat16* out2;             // SPLIT_GLU: [M, ldo2], column (n - n_split) / 2 of the (gate, up) row pairs
-  int ldo2, n_split;               // SPLIT_GLU: rows below n_split are stored as they are, the others are pairs
+  __nv_bfloat16* out2;             // SPLIT_GLU: [M, ldo2], column (n - n_split) / 2 of the (gate, up) row pairs; SPLIT_RELU2: column n - n_split
+  int ldo2, n_split;               // SPLIT_GLU, SPLIT_RELU2: rows below n_split are stored as they are
   float scale;                     // F32: factor of the stored values
   float glu_limit, glu_alpha, glu_bias;   // g = min(g, limit), u = clamp(u, +-limit): g sigmoid(alpha g) (u + bias)
   float softcap;                   // F32: > 0 stores softcap * tanh(value / softcap)
@@ -105,13 +105,19 @@ template <int BN> TI_DEVICE constexpr uint32_t idesc_bf16() {
 }
 
 // RESID32: fp32 out = fp32 residual + product.  SPLIT_GLU: the first n_split rows are stored (bf16), the interleaved
-// (gate, up) rows after them go through the clamped gated unit into a second output.
-enum { GEPI_STORE = 0, GEPI_SWIGLU = 1, GEPI_ROWPAR = 2, GEPI_F32 = 3, GEPI_RESID32 = 4, GEPI_SPLIT_GLU = 5 };
+// (gate, up) rows after them go through the clamped gated unit into a second output.  SPLIT_RELU2: the first n_split rows
+// are stored, the square of the positive part of the others goes to the second output.
+enum { GEPI_STORE = 0, GEPI_SWIGLU = 1, GEPI_ROWPAR = 2, GEPI_F32 = 3, GEPI_RESID32 = 4, GEPI_SPLIT_GLU = 5, GEPI_SPLIT_RELU2 = 6 };
 
 TI_DEVICE float clamped_glu(const GemmEpilogue& e, float g, float u) {
   g = fminf(g, e.glu_limit);
   u = fminf(fmaxf(u, -e.glu_limit), e.glu_limit);
   return g * sigmoid_f(e.glu_alpha * g) * (u + e.glu_bias);
+}
+
+TI_DEVICE float relu2(float v) {
+  v = fmaxf(v, 0.f);
+  return v * v;
 }
 
 TI_DEVICE float f32_value(const GemmEpilogue& e, float v) {
@@ -133,6 +139,11 @@ TI_DEVICE void gemm_epilogue4(const GemmParams& p, int m, int n, float4 v, uint2
   if (p.epi == GEPI_SPLIT_GLU && n >= p.ex.n_split) {
     *reinterpret_cast<uint32_t*>(p.ex.out2 + (size_t)m * p.ex.ldo2 + ((n - p.ex.n_split) >> 1)) =
         pack_bf16(clamped_glu(p.ex, v.x, v.y), clamped_glu(p.ex, v.z, v.w));
+    return;
+  }
+  if (p.epi == GEPI_SPLIT_RELU2 && n >= p.ex.n_split) {
+    *reinterpret_cast<uint2*>(p.ex.out2 + (size_t)m * p.ex.ldo2 + (n - p.ex.n_split)) =
+        make_uint2(pack_bf16(relu2(v.x), relu2(v.y)), pack_bf16(relu2(v.z), relu2(v.w)));
     return;
   }
   if (p.epi == GEPI_SWIGLU) {
@@ -213,6 +224,12 @@ TI_DEVICE void gemm_store8(const GemmParams& p, int m, int n, float4 a, float4 b
     *reinterpret_cast<uint2*>(p.ex.out2 + (size_t)m * p.ex.ldo2 + ((n - p.ex.n_split) >> 1)) =
         make_uint2(pack_bf16(clamped_glu(p.ex, v[0], v[1]), clamped_glu(p.ex, v[2], v[3])),
                    pack_bf16(clamped_glu(p.ex, v[4], v[5]), clamped_glu(p.ex, v[6], v[7])));
+    return;
+  }
+  if (p.epi == GEPI_SPLIT_RELU2 && n >= p.ex.n_split) {
+    *reinterpret_cast<uint4*>(p.ex.out2 + (size_t)m * p.ex.ldo2 + (n - p.ex.n_split)) =
+        make_uint4(pack_bf16(relu2(v[0]), relu2(v[1])), pack_bf16(relu2(v[2]), relu2(v[3])), pack_bf16(relu2(v[4]), relu2(v[5])),
+                   pack_bf16(relu2(v[6]), relu2(v[7])));
     return;
   }
   float r[8];
@@ -596,6 +613,7 @@ static int set_epilogue(GemmParams& p, const GemmEpilogue* ex) {
   if (p.epi == GEPI_RESID32 && (p.ex.resid32 == nullptr || p.N % 8 || p.ldo % 8 || ((uintptr_t)p.out | (uintptr_t)p.ex.resid32) % 16)) return -2;
   if (p.ex.bias != nullptr && (p.N % 8 || (uintptr_t)p.ex.bias % 16)) return -2;
   if (p.epi == GEPI_SPLIT_GLU && (p.ex.out2 == nullptr || p.N % 8 || p.ex.n_split % 8 || p.ex.ldo2 % 4 || (uintptr_t)p.ex.out2 % 8)) return -2;
+  if (p.epi == GEPI_SPLIT_RELU2 && (p.ex.out2 == nullptr || p.N % 8 || p.ex.n_split % 8 || p.ex.ldo2 % 8 || (uintptr_t)p.ex.out2 % 16)) return -2;
   return 0;
 }
 

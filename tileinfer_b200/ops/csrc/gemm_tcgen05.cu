@@ -175,7 +175,7 @@ int ti_gemm_w8a16(const void* w, const void* wscale, int n_tiles, int N, int K, 
                   const void* xscale, int M, const void* resid, void* out, int ldo, int epi, void* status, void* part,
                   size_t part_bytes, void* tile_count, int n_count, const ti::GemmEpilogue* ex, void* stream) {
   if (M <= 0) return 0;
-  if (K % 64 || N < 1 || epi < 0 || epi > 5) return -2;
+  if (K % 64 || N < 1 || epi < 0 || epi > 6) return -2;
   ti::GemmParams p = {};
   const int KB = K / 64, KS = (KB + ti::kKS - 1) / ti::kKS;      // 64-byte slabs of the weight layout; 128-byte stages
   const int BN = M <= 32 ? 32 : (M <= 64 ? 64 : 128);
@@ -217,7 +217,7 @@ int ti_gemm_bf16(const void* w, int n_tiles, int N, int K, const void* x, int M,
                  int epi, void* status, void* part, size_t part_bytes, void* tile_count, int n_count, const ti::GemmEpilogue* ex,
                  void* stream) {
   if (M <= 0) return 0;
-  if (K % 32 || N < 1 || epi < 0 || epi > 5) return -2;
+  if (K % 32 || N < 1 || epi < 0 || epi > 6) return -2;
   ti::GemmParams p = {};
   const int KB = K / 32, KS = (KB + ti::kKS - 1) / ti::kKS;    // 64-byte slabs; 128-byte stages
   // a single weight tile (a router): smaller token tiles, so that there are enough of them for all SMs

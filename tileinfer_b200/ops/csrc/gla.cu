@@ -3,8 +3,9 @@
 //     a_t = sigmoid(W_a2 x_t + b)^(1/tau)      S <- diag(a_t) S + k_t v_t^T      o_t = S^T q_t / sqrt(dim)
 // with x_t the narrow inner product of the decay.  Decode steps and short portions run here; long portions run in chunks
 // (gla_chunk.cu).  A block owns 64 columns of one head's state of one sequence in registers while it walks the sequence's
-// tokens; everything but the projections is fp32.  `gla_finish_kernel` applies the head's RMSNorm and the silu gate.
+// tokens; everything but the projections is fp32.  `head_norm_kernel` applies the head's RMSNorm and the silu gate.
 #include "gla.cuh"
+#include "head_norm.cuh"
 
 namespace ti {
 
@@ -69,36 +70,6 @@ __global__ void __launch_bounds__(256) gla_step_kernel(const __grid_constant__ G
   for (int i = 0; i < NR; ++i) *reinterpret_cast<float4*>(state + (size_t)(rg + 16 * i) * dv) = S[i];
 }
 
-// out[t, h] = rmsnorm(o[t, h]) * norm * silu(gate[t, h]); a warp per (token, head)
-template <typename T>
-__global__ void __launch_bounds__(256) gla_finish_kernel(const __grid_constant__ GlaParams p, int items, int dv) {
-  const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  pdl_trigger();
-  pdl_wait();
-  if (item >= items) return;
-  const int t = item / p.H, h = item - t * p.H;
-  const float* o = p.o + (size_t)t * p.H * dv + h * dv;
-  const T* g = static_cast<const T*>(p.proj) + (size_t)t * p.ld + p.g_col + h * dv;
-  T* out = static_cast<T*>(p.out) + (size_t)t * p.ldo + h * dv;
-  float ss = 0.f;
-  for (int c = lane * 8; c < dv; c += 256) {
-    float v[8];
-    load8(o + c, v);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) ss += v[i] * v[i];
-  }
-  const float rr = rsqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
-  for (int c = lane * 8; c < dv; c += 256) {
-    float v[8], w[8], z[8];
-    load8(o + c, v);
-    load8(p.norm + c, w);
-    load8(g + c, z);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] *= rr * w[i] * z[i] * sigmoid_exact(z[i]);
-    store8(out + c, v);
-  }
-}
-
 template <typename T>
 static int launch_step(const GlaParams& p, int S, int DK, int dv, cudaStream_t st) {
   const dim3 grid(dv / 64, p.H, S);
@@ -132,13 +103,8 @@ int ti_gla_step(const ti::GlaParams* p, int S, int dk, int dv, int f32, void* st
 
 // out[t, h] = rmsnorm(o[t, h]) * norm * silu(gate)
 int ti_gla_finish(const ti::GlaParams* p, int T, int dv, int f32, void* stream) {
-  if (T <= 0) return 0;
-  if (dv % 64 || !gla_aligned(p)) return -2;
-  const int items = T * p->H;
-  const dim3 grid((items + 7) / 8);
-  if (f32) ti::launch_kernel(ti::gla_finish_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, true, *p, items, dv);
-  else ti::launch_kernel(ti::gla_finish_kernel<ti::bf16>, grid, dim3(256), 0, (cudaStream_t)stream, true, *p, items, dv);
-  return (int)cudaGetLastError();
+  const ti::HeadNormParams n = {p->o, p->proj, p->norm, p->out, p->ld, p->ldo, p->g_col, p->H, dv, p->vdim, 0, 1, p->eps};
+  return ti::launch_head_norm(n, T, f32, (cudaStream_t)stream);
 }
 
 }  // extern "C"

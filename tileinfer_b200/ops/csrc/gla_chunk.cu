@@ -17,29 +17,11 @@
 // Decays, scores and states are fp32.  Where they enter a tensor-core product they are split into two bf16 terms
 // (x = hi + lo, about 16 bits); q, k and v are the bf16 projections, exact.
 #include "gla.cuh"
+#include "mma_split.cuh"
 
 namespace ti {
 
-constexpr float kLog2e = 1.4426950408889634f;
 constexpr float kMaxSpan = 80.f;        // log2 of the decay inside a block of 16 tokens that the products take
-
-TI_DEVICE float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
-  return y;
-}
-TI_DEVICE void ldsm4(uint32_t (&r)[4], const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-TI_DEVICE void ldsm4t(uint32_t (&r)[4], const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];\n" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
-}
-// (a, b) -> packed hi parts and packed lo parts
-TI_DEVICE void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16(a, b);
-  lo = pack_bf16(a - bf16lo(hi), b - bf16hi(hi));
-}
-TI_DEVICE void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) { mma_bf16_16816(d, a[0], a[1], a[2], a[3], b0, b1); }
 
 // shared-memory pitches: rows of the ldmatrix operands start 16 bytes apart modulo 128
 template <int DK> struct GlaGeom {

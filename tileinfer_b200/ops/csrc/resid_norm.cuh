@@ -115,4 +115,80 @@ TI_DEVICE void resid_norm_row(const ResidNormParams& p, int m, float (&y)[KEEP][
   }
 }
 
+// x[m] += rmsnorm(sigmoid(gate[m]) * Y) * w_out and h[m] = x[m], with Y = y[m], or of two branches
+// scale * (rmsnorm(y[m]) * w_y + rmsnorm(y2[m]) * w_y2).  `gate` holds logits.
+struct GatedNormParams {
+  const void* y;           // [M][ldy]
+  const void* y2;          // [M][ldy] or null
+  const void* gate;        // [M][ldg]
+  const float* w_y;        // [P], with y2
+  const float* w_y2;       // [P], with y2
+  const float* w_out;      // [P]
+  float* x;                // [M][P]
+  void* h;                 // [M][P] or null
+  int W, P, ldy, ldg;
+  float eps, scale;
+};
+
+// KEEP x 8 columns per thread; `red`: 96 floats of shared memory
+template <typename T, int KEEP>
+TI_DEVICE void gated_norm_row(const GatedNormParams& p, int m, float* red) {
+  const int step = blockDim.x * 8;
+  const bool two = p.y2 != nullptr;                        // uniform over the grid
+  float y[KEEP][8], z[KEEP][8], g[KEEP][8], s1 = 0.f, s2 = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * 8 + j * step;
+    if (c >= p.P) continue;
+    load8(static_cast<const T*>(p.y) + (size_t)m * p.ldy + c, y[j]);
+    load8(static_cast<const T*>(p.gate) + (size_t)m * p.ldg + c, g[j]);
+    if (two) load8(static_cast<const T*>(p.y2) + (size_t)m * p.ldy + c, z[j]);
+  }
+  if (two) {
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+      if (threadIdx.x * 8 + j * step >= p.P) continue;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        s1 = fmaf(y[j][i], y[j][i], s1);
+        s2 = fmaf(z[j][i], z[j][i], s2);
+      }
+    }
+    const float r1 = p.scale * rsqrtf(block_sum32(s1, red) / (float)p.W + p.eps), r2 = p.scale * rsqrtf(block_sum32(s2, red + 32) / (float)p.W + p.eps);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+      const int c = threadIdx.x * 8 + j * step;
+      if (c >= p.P) continue;
+      float a[8], b[8];
+      load8(p.w_y + c, a);
+      load8(p.w_y2 + c, b);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[j][i] = y[j][i] * r1 * a[i] + z[j][i] * r2 * b[i];
+    }
+  }
+  s1 = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    if (threadIdx.x * 8 + j * step >= p.P) continue;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      y[j][i] *= sigmoid_exact(g[j][i]);
+      s1 = fmaf(y[j][i], y[j][i], s1);
+    }
+  }
+  const float rr = rsqrtf(block_sum32(s1, red + 64) / (float)p.W + p.eps);
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = threadIdx.x * 8 + j * step;
+    if (c >= p.P) continue;
+    float x[8], w[8];
+    load8(p.x + (size_t)m * p.P + c, x);
+    load8(p.w_out + c, w);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) x[i] = fmaf(y[j][i] * rr, w[i], x[i]);
+    store8(p.x + (size_t)m * p.P + c, x);
+    if (p.h != nullptr) store8(static_cast<T*>(p.h) + (size_t)m * p.P + c, x);
+  }
+}
+
 }  // namespace ti

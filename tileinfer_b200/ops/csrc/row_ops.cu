@@ -9,13 +9,13 @@
 namespace ti {
 
 // ---------------------------------------------------------------- embedding
-// x[m, :] = rmsnorm(embed[ids[m]] + pos[positions[m]]) * w * scale in fp32.  Either of `pos` and `w` may be null (no w: no norm).  Block 0 also
-// advances the device step counter.
+// x[m, :] = rmsnorm(embed[ids[m]] + pos[positions[m]]) * w * scale in fp32.  Either of `pos` and `w` may be null (no w: no norm).  With `h`
+// the row is stored as T as well.  Block 0 also advances the device step counter.
 template <typename T>
 __global__ void __launch_bounds__(256) embed_pos_kernel(const long long* __restrict__ ids, const int* __restrict__ positions,
                                                         const T* __restrict__ embed, const T* __restrict__ pos,
                                                         const float* __restrict__ w, float* __restrict__ x, int W, int P,
-                                                        int vocab, int max_pos, float eps, float scale, unsigned* step) {
+                                                        int vocab, int max_pos, float eps, float scale, unsigned* step, T* __restrict__ h) {
   __shared__ float red[8];
   pdl_trigger();
   pdl_wait();
@@ -42,6 +42,7 @@ __global__ void __launch_bounds__(256) embed_pos_kernel(const long long* __restr
 #pragma unroll
     for (int i = 0; i < 8; ++i) a[i] = (a[i] + b[i]) * rr * g[i];
     store8(x + (size_t)m * P + c, a);
+    if (h != nullptr) store8(h + (size_t)m * P + c, a);
   }
   if (step != nullptr && m == 0 && threadIdx.x == 0) *step = *step + 1u;
 }
@@ -107,6 +108,14 @@ __global__ void __launch_bounds__(256) resid_norm_kernel(const __grid_constant__
   resid_norm_row<T, KEEP, ROUTED, FEW>(p, blockIdx.x, y, red);
 }
 
+template <typename T, int KEEP>
+__global__ void __launch_bounds__(256) gated_norm_kernel(const __grid_constant__ GatedNormParams p) {
+  __shared__ float red[96];
+  pdl_trigger();
+  pdl_wait();
+  gated_norm_row<T, KEEP>(p, blockIdx.x, red);
+}
+
 // ---------------------------------------------------------------- fp32 matrix product (32-bit mode)
 // y[M, N] = x[M, K] W[N, K]^T in plain fp32 FMAs, 64 x 64 tiles, with the epilogues of the tcgen05 product that an fp32
 // residual stream uses.  K a multiple of 16.
@@ -115,7 +124,7 @@ struct GemmF32Params {
   const float* x;       // [M][ldx]
   const float* resid;   // epi 4: [M][ldo]
   float* out;           // [M][ldo]
-  float* out2;          // epi 5: [M][ldo2], column (n - n_split) / 2 for the pairs of rows from n_split on
+  float* out2;          // epi 5: [M][ldo2], column (n - n_split) / 2 for the pairs of rows from n_split on; epi 6: column n - n_split, squared positive part
   int M, N, K, ldx, ldo, ldo2, n_split, epi;
   float scale, glu_limit, glu_alpha, glu_bias;
   // several weight matrices side by side: [3][max_tiles] weight matrix, first row of x, rows (at most 64) of a row tile
@@ -177,6 +186,14 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ G
         p.out2[(size_t)m * p.ldo2 + ((n - p.n_split) >> 1)] = g * sigmoid_exact(p.glu_alpha * g) * (u + p.glu_bias);
         continue;
       }
+      if (p.epi == 6 && n >= p.n_split) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float v = fmaxf(acc[i][j + e], 0.f);
+          if (n + e < p.N) p.out2[(size_t)m * p.ldo2 + n + e - p.n_split] = v * v;
+        }
+        continue;
+      }
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         if (n + e >= p.N) continue;
@@ -198,16 +215,16 @@ extern "C" {
 
 // f32 selects the activation / table type: 0 bf16, 1 float.  P: row pitch (a multiple of 8), W: true width.
 int ti_embed_pos(const void* ids, const void* positions, const void* embed, const void* pos, const void* w, void* x, int M,
-                 int W, int P, int vocab, int max_pos, float eps, float scale, void* step, int f32, void* stream) {
+                 int W, int P, int vocab, int max_pos, float eps, float scale, void* step, void* h, int f32, void* stream) {
   if (M <= 0) return 0;
   if (P % 8 || W > P || vocab < 1 || (pos != nullptr && max_pos < 1)) return -2;
   cudaStream_t st = (cudaStream_t)stream;
   if (f32)
     ti::launch_kernel(ti::embed_pos_kernel<float>, dim3(M), dim3(256), 0, st, true, (const long long*)ids, (const int*)positions,
-                      (const float*)embed, (const float*)pos, (const float*)w, (float*)x, W, P, vocab, max_pos, eps, scale, (unsigned*)step);
+                      (const float*)embed, (const float*)pos, (const float*)w, (float*)x, W, P, vocab, max_pos, eps, scale, (unsigned*)step, (float*)h);
   else
     ti::launch_kernel(ti::embed_pos_kernel<ti::bf16>, dim3(M), dim3(256), 0, st, true, (const long long*)ids, (const int*)positions,
-                      (const ti::bf16*)embed, (const ti::bf16*)pos, (const float*)w, (float*)x, W, P, vocab, max_pos, eps, scale, (unsigned*)step);
+                      (const ti::bf16*)embed, (const ti::bf16*)pos, (const float*)w, (float*)x, W, P, vocab, max_pos, eps, scale, (unsigned*)step, (ti::bf16*)h);
   return (int)cudaGetLastError();
 }
 
@@ -245,11 +262,30 @@ int ti_resid_norm(const ti::ResidNormParams* p, int M, int f32, void* stream) {
   return (int)cudaGetLastError();
 }
 
+int ti_gated_norm_params_size() { return (int)sizeof(ti::GatedNormParams); }
+
+int ti_gated_norm(const ti::GatedNormParams* p, int M, int f32, void* stream) {
+  if (M <= 0) return 0;
+  if (p->P % 8 || p->ldy % 8 || p->ldg % 8 || p->W > p->P || p->P > 256 * 8 * 8 || (p->y2 != nullptr && (p->w_y == nullptr || p->w_y2 == nullptr)) ||
+      (((uintptr_t)p->y | (uintptr_t)p->y2 | (uintptr_t)p->gate | (uintptr_t)p->x | (uintptr_t)p->h) & 15))
+    return -2;
+  cudaStream_t st = (cudaStream_t)stream;
+  const int threads = p->P >= 2048 ? 256 : (p->P / 8 + 31) / 32 * 32, keep = (p->P / 8 + threads - 1) / threads;
+#define TI_GN(T, K) ti::launch_kernel(ti::gated_norm_kernel<T, K>, dim3(M), dim3(threads), 0, st, true, *p)
+  if (f32) {
+    if (keep <= 1) TI_GN(float, 1); else if (keep <= 2) TI_GN(float, 2); else if (keep <= 4) TI_GN(float, 4); else TI_GN(float, 8);
+  } else {
+    if (keep <= 1) TI_GN(ti::bf16, 1); else if (keep <= 2) TI_GN(ti::bf16, 2); else if (keep <= 4) TI_GN(ti::bf16, 4); else TI_GN(ti::bf16, 8);
+  }
+#undef TI_GN
+  return (int)cudaGetLastError();
+}
+
 int ti_gemm_f32(const void* w, const void* x, const void* resid, void* out, void* out2, int M, int N, int K, int ldx, int ldo,
                 int ldo2, int n_split, int epi, float scale, float glu_limit, float glu_alpha, float glu_bias, const void* tiles,
                 const void* num_tiles, int max_tiles, float softcap, const void* bias, void* stream) {
   if (M <= 0) return 0;
-  if (K % 16 || ldx % 4 || n_split % 2 || (epi != 3 && epi != 4 && epi != 5)) return -2;
+  if (K % 16 || ldx % 4 || n_split % 2 || epi < 3 || epi > 6) return -2;
   ti::GemmF32Params p = {(const float*)w, (const float*)x, (const float*)resid, (float*)out, (float*)out2, M, N, K, ldx, ldo,
                          ldo2, n_split, epi, scale, glu_limit, glu_alpha, glu_bias, (const int*)tiles, (const int*)num_tiles, max_tiles, softcap, (const float*)bias};
   ti::launch_kernel(ti::gemm_f32_kernel, dim3((N + 63) / 64, tiles != nullptr ? max_tiles : (M + 63) / 64), dim3(256), 0, (cudaStream_t)stream, true, p);

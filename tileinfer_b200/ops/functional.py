@@ -65,7 +65,7 @@ class AttnParams(ctypes.Structure):
                 ("qg_seq", _P), ("qg_tok0", _P), ("qg_ntok", _P), ("o_part", _P), ("ml_part", _P),
                 ("gate_src", _P), ("out", _P), ("hq", _I), ("hkv", _I), ("max_blocks", _I), ("nsplit", _I),
                 ("ld", _I), ("num_qg", _I), ("scale_log2e", _F), ("num_blocks", _I), ("status", _P), ("cap_in", _F), ("cap_out", _F),
-                ("rep", _I), ("window", _I), ("slopes", _P), ("head_gate", _P), ("ldg", _I), ("gcol", _I), ("ldo", _I), ("out_scale", _F)]
+                ("rep", _I), ("window", _I), ("slopes", _P), ("head_gate", _P), ("ldg", _I), ("gcol", _I), ("ldo", _I), ("out_scale", _F), ("gate_col", _I), ("gate_stride", _I)]
 
     def __init__(self, *args, **kw):
         super().__init__(*args, **kw)
@@ -82,14 +82,14 @@ class LatentAttnParams(ctypes.Structure):
 class RopeUnitParams(ctypes.Structure):
     _fields_ = [("proj", _P), ("inv_freq", _P), ("positions", _P), ("slot_mapping", _P), ("q_out", _P), ("kcache", _P), ("vcache", _P),
                 ("status", _P), ("T", _I), ("ld", _I), ("q_col", _I), ("k_col", _I), ("v_col", _I), ("H", _I), ("G", _I), ("dim", _I),
-                ("dp", _I), ("vp", _I), ("half", _I), ("num_blocks", _I), ("eps", _F)]
+                ("dp", _I), ("vp", _I), ("half", _I), ("num_blocks", _I), ("eps", _F), ("pairs", _I), ("q_w", _P), ("k_w", _P)]
 
 
 class AttnGeneralParams(ctypes.Structure):
     _fields_ = [("q", _P), ("kcache", _P), ("vcache", _P), ("block_tables", _P), ("positions", _P), ("qg_seq", _P), ("qg_tok0", _P),
                 ("qg_ntok", _P), ("out", _P), ("status", _P), ("H", _I), ("G", _I), ("dp", _I), ("vp", _I), ("max_blocks", _I),
                 ("num_qg", _I), ("num_blocks", _I), ("ldo", _I), ("scale", _F), ("softcap", _F), ("window", _I), ("slopes", _P),
-                ("head_gate", _P), ("ldg", _I), ("gcol", _I), ("out_scale", _F)]
+                ("head_gate", _P), ("ldg", _I), ("gcol", _I), ("out_scale", _F), ("gate", _P)]
 
     def __init__(self, *args, **kw):
         super().__init__(*args, **kw)
@@ -126,6 +126,25 @@ class SsdParams(ctypes.Structure):
                 ("H", _I), ("G", _I), ("V", _I), ("vp", _I), ("num_snap", _I), ("norm_groups", _I), ("eps", _F),
                 ("ck_seq", _P), ("ck_tok0", _P), ("ck_ntok", _P), ("ck_snap", _P), ("long_seq", _P), ("long_ck", _P), ("g_ws", _P),
                 ("s_ws", _P), ("nc", _I), ("num_long", _I)]
+
+
+class DeltaParams(ctypes.Structure):
+    _fields_ = [("src", _P), ("proj", _P), ("bias", _P), ("neg_a", _P), ("w2", _P), ("w0", _P), ("state", _P), ("slots", _P), ("cu", _P),
+                ("seqs", _P), ("o", _P), ("snap_rel", _P), ("snap_idx", _P), ("snap", _P),
+                ("lds", _I), ("ld", _I), ("H", _I), ("rep", _I), ("R", _I), ("q_col", _I), ("k_col", _I), ("v_col", _I), ("b_col", _I),
+                ("a_col", _I), ("num_snap", _I), ("q_scale", _F), ("decay_scale", _F),
+                ("ck_seq", _P), ("ck_tok0", _P), ("ck_ntok", _P), ("ck_snap", _P), ("long_seq", _P), ("long_ck", _P), ("t_ws", _P),
+                ("q_ws", _P), ("s_ws", _P), ("f_ws", _P), ("nc", _I), ("num_long", _I)]
+
+
+class HeadNormParams(ctypes.Structure):
+    _fields_ = [("o", _P), ("gate", _P), ("norm", _P), ("out", _P), ("ld", _I), ("ldo", _I), ("g_col", _I), ("H", _I), ("dv", _I),
+                ("vdim", _I), ("norm_stride", _I), ("silu", _I), ("eps", _F)]
+
+
+class GatedNormParams(ctypes.Structure):
+    _fields_ = [("y", _P), ("y2", _P), ("gate", _P), ("w_y", _P), ("w_y2", _P), ("w_out", _P), ("x", _P), ("h", _P),
+                ("W", _I), ("P", _I), ("ldy", _I), ("ldg", _I), ("eps", _F), ("scale", _F)]
 
 
 class MoeRouteParams(ctypes.Structure):
@@ -190,7 +209,7 @@ _l.register("ti_attn_params_size", _I, [], "attention")
 _l.register("ti_qkv_prep", _I, [ctypes.POINTER(QkvPrepParams), _I, _I, _P], "attention")
 _l.register("ti_attn_paged", _I, [ctypes.POINTER(AttnParams), _I, _I, _P], "attention")
 _l.register("ti_attn_prefill", _I, [_P, _I, _P, _P, _I, _P, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _F, _I, _I, _F, _F,
-                                _I, _P, _P, _I, _I, _I, _F, _P, _P], "attention")
+                                _I, _P, _P, _I, _I, _I, _F, _I, _I, _P, _P], "attention")
 _l.register("ti_rope_unit_params_size", _I, [], "attention")
 _l.register("ti_rope_unit", _I, [ctypes.POINTER(RopeUnitParams), _I, _P], "attention")
 _l.register("ti_attn_general_params_size", _I, [], "attention")
@@ -209,6 +228,14 @@ _l.register("ti_ssd_step", _I, [ctypes.POINTER(SsdParams), _I, _I, _I, _P], "ssd
 _l.register("ti_ssd_finish", _I, [ctypes.POINTER(SsdParams), _I, _I, _P], "ssd")
 _l.register("ti_ssd_chunk_size", _I, [_I], "ssd")
 _l.register("ti_ssd_chunked", _I, [ctypes.POINTER(SsdParams), _I, _P], "ssd")
+_l.register("ti_delta_params_size", _I, [], "delta")
+_l.register("ti_head_norm_params_size", _I, [], "delta")
+_l.register("ti_delta_step", _I, [ctypes.POINTER(DeltaParams), _I, _I, _I, _I, _I, _P], "delta")
+_l.register("ti_delta_chunk_size", _I, [_I], "delta")
+_l.register("ti_delta_chunked", _I, [ctypes.POINTER(DeltaParams), _I, _I, _I, _P], "delta")
+_l.register("ti_head_norm", _I, [ctypes.POINTER(HeadNormParams), _I, _I, _P], "delta")
+_l.register("ti_gated_norm_params_size", _I, [], "rows")
+_l.register("ti_gated_norm", _I, [ctypes.POINTER(GatedNormParams), _I, _I, _P], "rows")
 _l.register("ti_moe_route_params_size", _I, [], "moe")
 _l.register("ti_moe_route", _I, [ctypes.POINTER(MoeRouteParams), _P], "moe")
 _l.register("ti_moe_norm_route", _I, [ctypes.POINTER(ResidNormParams), ctypes.POINTER(MoeRouteParams), _P, _P, _P, _I, _P], "moe")
@@ -237,7 +264,7 @@ _l.register("ti_latent_attn_params_size", _I, [], "latent")
 _l.register("ti_latent_attn_splits", _I, [_I, _I], "latent")
 _l.register("ti_latent_attn", _I, [ctypes.POINTER(LatentAttnParams), _I, _P], "latent")
 _l.register("ti_latent_prefill", _I, [_P, _I, _I, _P, _I, _I, _P, _I, _P, _P, _I, _I, _P, _I, _I, _I, _I, _I, _I, _F, _P, _P], "latent")
-_l.register("ti_embed_pos", _I, [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P, _I, _P], "rows")
+_l.register("ti_embed_pos", _I, [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _F, _F, _P, _P, _I, _P], "rows")
 _l.register("ti_rmsnorm_f32", _I, [_P, _P, _P, _I, _I, _I, _F, _I, _P], "rows")
 _l.register("ti_latent_store", _I, [_P, _I, _I, _P, _P, _P, _LL, _I, _I, _I, _F, _I, _P], "latent")
 _l.register("ti_latent_rope", _I, [_P, _I, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _LL, _I, _I, _I, _F, _I, _P], "latent")
@@ -248,12 +275,13 @@ _l.register("ti_gemm_f32", _I, [_P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, 
 _PARAM_SIZES = {"base": (("ti_topk_params_size", TopkParams), ("ti_edit_params_size", EditParams),
                          ("ti_sample_params_size", SampleParams), ("ti_gemm_epilogue_size", GemmEpilogue)),
                 "latent": (("ti_latent_attn_params_size", LatentAttnParams),),
-                "rows": (("ti_resid_norm_params_size", ResidNormParams),),
+                "rows": (("ti_resid_norm_params_size", ResidNormParams), ("ti_gated_norm_params_size", GatedNormParams)),
                 "attention": (("ti_qkv_prep_params_size", QkvPrepParams), ("ti_attn_params_size", AttnParams),
                               ("ti_rope_unit_params_size", RopeUnitParams), ("ti_attn_general_params_size", AttnGeneralParams),
                               ("ti_norm_rope_params_size", NormRopeParams)),
                 "conv": (("ti_conv_params_size", ConvParams),),
                 "ssd": (("ti_ssd_params_size", SsdParams),),
+                "delta": (("ti_delta_params_size", DeltaParams), ("ti_head_norm_params_size", HeadNormParams)),
                 "gla": (("ti_gla_params_size", GlaParams),),
                 "moe": (("ti_moe_route_params_size", MoeRouteParams),),
                 "hybrid": (("ti_gdn_params_size", GdnParams), ("ti_gdn_chunk_params_size", GdnChunkParams),
@@ -625,18 +653,20 @@ def attn_paged(p: AttnParams, D: int, DV: int = None):
 
 
 def attn_prefill(q, kcache, vcache, num_blocks, block_tables, positions, tiles, gate_src, out, *, hq, hkv, D,
-                 max_blocks, ld, DV=None, scale=None, softcap=0.0, qk_max=0.0, window=0, slopes=None, head_gate=None, gcol=0, out_scale=1.0):
+                 max_blocks, ld, DV=None, scale=None, softcap=0.0, qk_max=0.0, window=0, slopes=None, head_gate=None, gcol=0, out_scale=1.0,
+                 gate_col=0, gate_stride=0):
     """Causal GQA attention of prefill query tiles on the tcgen05 tensor cores (ops/csrc/attn_prefill.cu).
     `tiles`: int32 [3, n] = (sequence, first flat token, tokens <= 128) per tile, longest KV first.  DV: size of a value
     head (default D); softcap: scores become softcap * tanh(scale q.k / softcap); qk_max: a bound of |q.k| where there is
-    one (it selects a cheaper softmax); gate_src None: no output gate.  window: keys seen (0: all); slopes: fp32 [hq], taken
+    one (it selects a cheaper softmax); gate_src None: no output gate, else rows of pitch `ld` with the gates of head h at column
+    gate_col + h * gate_stride (stride 0: h * 2 D + D).  window: keys seen (0: all); slopes: fp32 [hq], taken
     off a score per token of distance; head_gate: rows whose column gcol + h gates head h; out_scale: factor of the output."""
     n = tiles.shape[1]
     scale = D ** -0.5 if scale is None else scale
     check(_l.lib().ti_attn_prefill(ptr(q), q.shape[0], ptr(kcache), ptr(vcache), num_blocks, ptr(block_tables), ptr(positions),
                               ptr(tiles[0]), ptr(tiles[1]), ptr(tiles[2]), n, ptr(gate_src), ptr(out), hq, hkv,
                               max_blocks, ld, scale, D, D if DV is None else DV, softcap, qk_max, window, ptr(slopes), ptr(head_gate),
-                              0 if head_gate is None else head_gate.stride(0), gcol, out.stride(0) if out.dim() == 2 else 0, out_scale,
+                              0 if head_gate is None else head_gate.stride(0), gcol, out.stride(0) if out.dim() == 2 else 0, out_scale, gate_col, gate_stride,
                               status_ptr(), stream()),
           "ti_attn_prefill")
 
@@ -687,12 +717,12 @@ def topk_merge(p: TopkParams):
 
 
 # ------------------------------------------------------------------------------------ prefill GEMM (tcgen05)
-GEPI_STORE, GEPI_SWIGLU, GEPI_ROWPAR, GEPI_F32, GEPI_RESID32, GEPI_SPLIT_GLU = 0, 1, 2, 3, 4, 5
+GEPI_STORE, GEPI_SWIGLU, GEPI_ROWPAR, GEPI_F32, GEPI_RESID32, GEPI_SPLIT_GLU, GEPI_SPLIT_RELU2 = 0, 1, 2, 3, 4, 5, 6
 
 
 def gemm_epilogue(*, resid32=None, out2=None, n_split=0, scale=1.0, glu=(math.inf, 1.0, 0.0), softcap=0.0, bias=None) -> GemmEpilogue:
     """Operands of the extended epilogues: an fp32 residual (GEPI_RESID32), the second output and the constants
-    (limit, alpha, bias) of the clamped gated unit (GEPI_SPLIT_GLU), a factor and a cap of the stored fp32 values (GEPI_F32), and an fp32 vector [N]
+    (limit, alpha, bias) of the clamped gated unit (GEPI_SPLIT_GLU; GEPI_SPLIT_RELU2 squares the positive part instead), a factor and a cap of the stored fp32 values (GEPI_F32), and an fp32 vector [N]
     added to the product first (any of them)."""
     return GemmEpilogue(ptr(resid32), ptr(out2), 0 if out2 is None else out2.stride(0), n_split, scale, *glu, softcap, ptr(bias))
 
@@ -767,10 +797,11 @@ def _f32(t) -> int:
     return int(t.dtype == torch.float32)
 
 
-def embed_pos(ids, positions, embed, pos, norm_w, x, W, eps, step_ptr=0, scale=1.0):
-    """x[m] (fp32) = rmsnorm(embed[ids[m]] + pos[positions[m]]) * norm_w * scale; `pos` and `norm_w` (no norm) may be None."""
+def embed_pos(ids, positions, embed, pos, norm_w, x, W, eps, step_ptr=0, scale=1.0, h=None):
+    """x[m] (fp32) = rmsnorm(embed[ids[m]] + pos[positions[m]]) * norm_w * scale; `pos` and `norm_w` (no norm) may be None.  h: the
+    row once more, in the activations' type."""
     check(_l.lib().ti_embed_pos(ptr(ids), ptr(positions), ptr(embed), ptr(pos), ptr(norm_w), ptr(x), x.shape[0], W, x.stride(0),
-                                embed.shape[0], 0 if pos is None else pos.shape[0], eps, scale, step_ptr, _f32(embed), stream()), "ti_embed_pos")
+                                embed.shape[0], 0 if pos is None else pos.shape[0], eps, scale, step_ptr, ptr(h), _f32(embed), stream()), "ti_embed_pos")
 
 
 def rmsnorm_f32(x, norm_w, y, W, eps):
@@ -851,7 +882,7 @@ def latent_prefill(q, kv, tiles, out, *, H, dp, vp, window, scale, sink=None, ga
 
 
 def gemm_f32(w, x, *, out, epi=GEPI_F32, ex=None, groups=None):
-    """y = x W^T in fp32 FMAs (w [N, K] row-major) with the GEPI_F32 / GEPI_RESID32 / GEPI_SPLIT_GLU epilogues.  With
+    """y = x W^T in fp32 FMAs (w [N, K] row-major) with the GEPI_F32 / GEPI_RESID32 / GEPI_SPLIT_GLU / GEPI_SPLIT_RELU2 epilogues.  With
     `groups` w is [E, N, K] and the rows of x meet the matrices of the token tiles (of at most 64 rows)."""
     e = ex if ex is not None else gemm_epilogue()
     N, K = w.shape[-2:]
@@ -859,6 +890,14 @@ def gemm_f32(w, x, *, out, epi=GEPI_F32, ex=None, groups=None):
                                e.n_split, epi, e.scale, e.glu_limit, e.glu_alpha, e.glu_bias,
                                *((0, 0, 0) if groups is None else (ptr(groups.tiles), ptr(groups.num_tiles), groups.tiles.shape[1])),
                                e.softcap, e.bias, stream()), "ti_gemm_f32")
+
+
+def gated_norm(y, gate, x, w_out, h, W, eps, y2=None, w_y=None, w_y2=None, scale=1.0):
+    """x += rmsnorm(sigmoid(gate) * Y) * w_out (fp32 rows) and h = x, with Y = y, or scale * (rmsnorm(y) * w_y + rmsnorm(y2) * w_y2)."""
+    p = GatedNormParams()
+    p.y, p.y2, p.gate, p.w_y, p.w_y2, p.w_out, p.x, p.h = (ptr(t) for t in (y, y2, gate, w_y, w_y2, w_out, x, h))
+    p.W, p.P, p.ldy, p.ldg, p.eps, p.scale = W, x.stride(0), y.stride(0), gate.stride(0), eps, scale
+    check(_l.lib().ti_gated_norm(ctypes.byref(p), x.shape[0], _f32(y), stream()), "ti_gated_norm")
 
 
 def resid_norm(y, x, w_out, h, w_next, W, eps, routed=None):
@@ -962,6 +1001,45 @@ def conv_tiles(cu_seqlens) -> torch.Tensor:
 def conv(p: ConvParams, f32: bool):
     """Causal convolution of a step's tokens (two kernels when p.cu is set, else one)."""
     check(_l.lib().ti_conv(ctypes.byref(p), int(f32), stream()), "ti_conv")
+
+
+# ------------------------------------------------------------------------------------ delta rules
+def delta_chunk_size(dk: int) -> int:
+    """Tokens of a chunk for this key size (0: no chunked form)."""
+    return _l.lib().ti_delta_chunk_size(dk)
+
+
+class DeltaWorkspace:
+    """The matrices of the chunks (ops/csrc/delta_chunk.cu); grows on demand."""
+
+    def __init__(self, device):
+        self.device, self.w = device, [None] * 4
+
+    def get(self, nc: int, H: int, dk: int, dv: int):
+        sizes = (nc * H * dk * dk, nc * H * delta_chunk_size(dk) * dk, nc * H * dk * dv, nc * H * dk)
+        for i, n in enumerate(sizes):
+            if self.w[i] is None or self.w[i].numel() < n:
+                self.w[i] = torch.empty(n, dtype=torch.float32, device=self.device)
+        return self.w
+
+
+def delta_step(p: DeltaParams, num_seqs: int, dk: int, dv: int, general: bool, f32: bool):
+    check(_l.lib().ti_delta_step(ctypes.byref(p), num_seqs, dk, dv, int(general), int(f32), stream()), "ti_delta_step")
+
+
+def delta_chunked(p: DeltaParams, dk: int, dv: int, general: bool):
+    """Outputs and states of the sequences with chunks (bf16 inputs); three kernels."""
+    check(_l.lib().ti_delta_chunked(ctypes.byref(p), dk, dv, int(general), stream()), "ti_delta_chunked")
+
+
+def head_norm(o, gate, g_col, norm, out, vdim, eps, silu: bool):
+    """out[t, h] = rmsnorm(o[t, h]) * norm * (silu or sigmoid)(gate): o [T, H, dv] fp32, gate rows with the heads at column g_col,
+    norm [dv] or [H, dv], out rows with head h at column h * dv."""
+    p = HeadNormParams()
+    p.o, p.gate, p.norm, p.out = ptr(o), ptr(gate), ptr(norm), ptr(out)
+    p.ld, p.ldo, p.g_col, p.H, p.dv = gate.stride(0), out.stride(0), g_col, o.shape[1], o.shape[2]
+    p.vdim, p.norm_stride, p.silu, p.eps = vdim, 0 if norm.dim() == 1 else o.shape[2], int(silu), eps
+    check(_l.lib().ti_head_norm(ctypes.byref(p), o.shape[0], _f32(gate), stream()), "ti_head_norm")
 
 
 # ------------------------------------------------------------------------------------ state-space mixer
