@@ -10,7 +10,7 @@ replays whose inputs advance on the device), max over ranks.  `e2e` is the same 
 `LLM.generate_token_ids`, every step including the pinned-host -> device copy of its inputs and the
 device -> host read of the sampled token; like the reference's own harness
 (tests/bench_multi_gpu.py:57-115) it subtracts a max_tokens=1 call from a full call.
-`--workload kabadra` / `gerivik` / `nogidra` measure that model beside the closest model of equal size instead (one GPU).
+`--workload kabadra` / `gerivik` / `nogidra` / `luvapel` measure that model beside the closest model of equal size instead (one GPU).
 `--impl reference` runs the unmodified reference package from baseline/_ref instead.
 """
 from __future__ import annotations
@@ -224,7 +224,7 @@ def main():
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--model", default="preset:qwen3.6-27b")
-    ap.add_argument("--workload", default="decode", choices=["decode", "kabadra", "gerivik", "nogidra"])
+    ap.add_argument("--workload", default="decode", choices=["decode", "kabadra", "gerivik", "nogidra", "luvapel"])
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     if args.workload != "decode":

@@ -419,16 +419,20 @@ def test_slow_states_carry_the_first_token(tmp_path, kind):
         for n in ("l0.mix.a", "l0.mix.w2"):
             w[n] = (0.02 * w[n].float()).to(BF16)
     else:
+        # steps are small wherever channel 0 of the embedding is one, which is everywhere but at the first token
         w["l0.mix.right.A_log"], w["l0.mix.left.out"] = torch.full_like(w["l0.mix.right.A_log"], -7.0), torch.zeros_like(w["l0.mix.left.out"])
+        w["embed"][:, 0], w["embed"][:2, 0], w["l0.mix.right.b"][:, 0] = 1.0, -1.0, -0.4
+    w["embed"][:2] *= 8                                     # the first token writes more than the others
     folder = oracle.write_model(str(tmp_path / "m"), cfg, w)
-    t = lc.tokens(cfg, 400)
-    u = [(t[0] + 1) % cfg["vocab"]] + t[1:]
+    t = [0] + [max(2, x) for x in lc.tokens(cfg, 399)]
+    u = [1] + t[1:]
     change = _want(cfg, w, u) - _want(cfg, w, t)
-    for quant, tol in (("fp32", 2e-2), ("bf16", 0.6)):
+    assert change[300:].abs().max() > 0.1
+    for quant, tol in (("fp32", 2e-2), ("bf16", 0.5)):
         eng = lc.engine(folder, quant, "cuda")
         for sizes in ([400], [350, 1], [70]):
             d = lc.replay(eng, lc.cut("a", 400, sizes), {"a": u})["a"] - lc.replay(eng, lc.cut("a", 400, sizes), {"a": t})["a"]
-            assert change[300:].abs().max() > 1e-2 and rel(d[300:], change[300:]) < tol
+            assert rel(d[300:], change[300:]) < tol
 
 
 def test_long_decoding(tmp_path):
