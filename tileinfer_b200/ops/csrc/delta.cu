@@ -10,11 +10,13 @@
 
 namespace ti {
 
-// thread = (row group of 16, four columns): rows rg + 16 i, i < NR
+// Threads own the state as (row group of 16, four columns): rows rg + 16 i, i < NR.  For the second product of a general decay
+// they are (key channel, part of the ranks) and keep their part of the matrix, up to 32 ranks of it, in registers.
 template <typename T, int NR, bool GENERAL>
 __global__ void __launch_bounds__(256) delta_step_kernel(const __grid_constant__ DeltaParams p) {
-  constexpr int DK = NR * 16;
+  constexpr int DK = NR * 16, PARTS = DK >= 256 ? 1 : 256 / DK, CH = DK > 256 ? DK / 256 : 1, KEEP = GENERAL && DK <= 256 ? 32 : 1;
   __shared__ float w_s[2][GENERAL ? DK : 1], p_s[2][GENERAL ? DK : 1], u_s[2][DK], c_s[2][GENERAL ? DK : 1], q_s[2][DK];
+  __shared__ float z_s[GENERAL ? PARTS : 1][GENERAL ? DK : 1], x_s[GENERAL ? 256 : 1];
   __shared__ __align__(16) float red[2][8][128];
   __shared__ float dots[2][8][2];
   const int tid = threadIdx.x, rg = tid >> 4, cq = (tid & 15) * 4, warp = tid >> 5, lane = tid & 31;
@@ -24,6 +26,13 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const __grid_constant__
   float4 S[NR];
 #pragma unroll
   for (int i = 0; i < NR; ++i) S[i] = *reinterpret_cast<const float4*>(state + (size_t)(rg + 16 * i) * dv);
+  // ranks of this thread: r0 + PARTS i
+  const int ch = PARTS > 1 ? tid % DK : tid, r0 = PARTS > 1 ? tid / DK : 0, cols = p.H * DK;
+  float keep[KEEP];
+  if (GENERAL && KEEP > 1) {
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) keep[i] = r0 + PARTS * i < p.R ? __ldg(p.w2 + (size_t)(r0 + PARTS * i) * cols + h * DK + ch) : 0.f;
+  }
   pdl_trigger();
   pdl_wait();                                              // the inputs come from the kernels before
   const int t0 = p.cu == nullptr ? s : p.cu[s], t1 = p.cu == nullptr ? s + 1 : p.cu[s + 1];
@@ -32,8 +41,38 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const __grid_constant__
     const T* src = static_cast<const T*>(p.src) + (size_t)t * p.lds;
     const T* row = static_cast<const T*>(p.proj) + (size_t)t * p.ld;
     const T *kp = src + p.k_col + kh * DK, *qp = src + p.q_col + kh * DK;
+    float z[CH];
+    if (GENERAL) {
+      // z = W_2 tanh(x) + w_0, 256 ranks at a time
+#pragma unroll
+      for (int j = 0; j < CH; ++j) z[j] = 0.f;
+      for (int rb = 0; rb < p.R; rb += 256) {
+        if (rb) __syncthreads();
+        if (rb + tid < p.R) x_s[tid] = tanhf(to_f<T>(row[p.a_col + rb + tid]));
+        __syncthreads();
+        const int rn = min(256, p.R - rb);
+        if (KEEP > 1 && rb == 0) {
+#pragma unroll
+          for (int i = 0; i < KEEP; ++i)
+            if (r0 + PARTS * i < rn) z[0] = fmaf(keep[i], x_s[r0 + PARTS * i], z[0]);
+        }
+        for (int r = r0 + (KEEP > 1 && rb == 0 ? PARTS * KEEP : 0); r < rn; r += PARTS)
+#pragma unroll
+          for (int j = 0; j < CH; ++j) z[j] = fmaf(__ldg(p.w2 + (size_t)(rb + r) * cols + h * DK + ch + 256 * j), x_s[r], z[j]);
+      }
+      if (PARTS > 1) {
+        z_s[r0][ch] = z[0];
+        __syncthreads();
+        z[0] = 0.f;
+        if (tid < DK) {
+#pragma unroll
+          for (int i = 0; i < PARTS; ++i) z[0] += z_s[i][ch];
+        }
+      }
+    }
     // every warp takes the lengths by itself
     float kk = 0.f, qq = 0.f;
+#pragma unroll
     for (int d = lane; d < DK; d += 32) {
       const float k = to_f<T>(kp[d]), q = to_f<T>(qp[d]);
       kk = fmaf(k, k, kk);
@@ -46,29 +85,18 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const __grid_constant__
       g = expf(p.neg_a[h] * softplus_exact(to_f<T>(row[p.a_col + h]) + p.bias[h]));
       beta = sigmoid_exact(to_f<T>(row[p.b_col + h]));
     }
-    for (int d0 = 0; d0 < DK; d0 += 256) {
-      const int d = d0 + tid;
+#pragma unroll
+    for (int j = 0; j < CH; ++j) {
+      const int d = tid + 256 * j;
+      if (d >= DK) continue;
+      const float k = to_f<T>(kp[d]), u = k * rk;
+      u_s[b][d] = u;
+      q_s[b][d] = to_f<T>(qp[d]) * qf;
       if (GENERAL) {
-        // the inner product's values pass from lane to lane
-        const int col = h * DK + min(d, DK - 1);
-        float z = p.w0[col];
-        for (int r0 = 0; r0 < p.R; r0 += 32) {
-          const float x = r0 + lane < p.R ? tanhf(to_f<T>(row[p.a_col + r0 + lane])) : 0.f;
-          const int n = min(32, p.R - r0);
-#pragma unroll 4
-          for (int r = 0; r < n; ++r) z = fmaf(__shfl_sync(0xffffffffu, x, r), __ldg(p.w2 + (size_t)(r0 + r) * p.H * DK + col), z);
-        }
-        if (d < DK) {
-          const float k = to_f<T>(kp[d]), u = k * rk;
-          w_s[b][d] = expf(-p.decay_scale * sigmoid_exact(z));
-          p_s[b][d] = sigmoid_exact(to_f<T>(row[p.b_col + col]) + p.bias[col]) * u;
-          u_s[b][d] = u;
-          c_s[b][d] = k;
-          q_s[b][d] = to_f<T>(qp[d]);
-        }
-      } else if (d < DK) {
-        u_s[b][d] = to_f<T>(kp[d]) * rk;
-        q_s[b][d] = to_f<T>(qp[d]) * qf;
+        const int col = h * DK + d;
+        w_s[b][d] = expf(-p.decay_scale * sigmoid_exact(z[j] + p.w0[col]));
+        p_s[b][d] = sigmoid_exact(to_f<T>(row[p.b_col + col]) + p.bias[col]) * u;
+        c_s[b][d] = k;
       }
     }
     const T* vp = src + p.v_col + h * dv + col0;

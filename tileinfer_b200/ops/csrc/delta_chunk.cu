@@ -86,8 +86,10 @@ TI_DEVICE void mma3(float (&acc)[2][4], const uint32_t (&ah)[4], const uint32_t 
 }
 
 // ------------------------------------------------------------------------------------------------ the matrices of a chunk
+constexpr int kPrepWarps = 16, kPrepThreads = 32 * kPrepWarps;
+
 template <int DK, bool GENERAL>
-__global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_constant__ DeltaParams p, int dv) {
+__global__ void __launch_bounds__(kPrepThreads) delta_chunk_prepare_kernel(const __grid_constant__ DeltaParams p, int dv) {
   using M = DeltaGeom<DK>;
   constexpr int C = M::C, MT = M::MT, KT = M::KT, KP = M::KP, AP = M::AP, VP = M::VP, GP = M::GP, FP = M::FP;
   extern __shared__ __align__(16) uint8_t smem[];
@@ -113,31 +115,52 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
   pdl_wait();
   const bf16 *src = static_cast<const bf16*>(p.src) + (size_t)tok0 * p.lds, *proj = static_cast<const bf16*>(p.proj) + (size_t)tok0 * p.ld;
 
+  // ---- the first value columns, requested now and used last
+  const int vj = tid >> 3, vc = (tid & 7) * 8;                     // row and column of a thread's 16 bytes (C 32: half of the threads)
+  const bool has_v = vj < n && vj < C;
+  const bf16* vsrc = src + (size_t)(has_v ? vj : 0) * p.lds + p.v_col + h * dv + vc;
+  uint4 vnext = make_uint4(0u, 0u, 0u, 0u);
+  if (has_v) vnext = *reinterpret_cast<const uint4*>(vsrc);
   // ---- lengths, decays and rates of the tokens
-  for (int j = warp; j < C; j += 8) {
-    float kk = 0.f, qq = 0.f;
-    if (j < n)
+  {
+    constexpr int NT = C / kPrepWarps;
+    float kk[NT], qq[NT], ga[NT], gb[NT];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const int j = warp + kPrepWarps * i;
+      kk[i] = qq[i] = ga[i] = gb[i] = 0.f;
+      if (j >= n) continue;
+#pragma unroll
       for (int d = lane * 2; d < DK; d += 64) {
         const uint32_t k = *reinterpret_cast<const uint32_t*>(src + (size_t)j * p.lds + p.k_col + kh * DK + d);
-        kk += bf16lo(k) * bf16lo(k) + bf16hi(k) * bf16hi(k);
+        kk[i] += bf16lo(k) * bf16lo(k) + bf16hi(k) * bf16hi(k);
         if (GENERAL) continue;
         const uint32_t q = *reinterpret_cast<const uint32_t*>(src + (size_t)j * p.lds + p.q_col + kh * DK + d);
-        qq += bf16lo(q) * bf16lo(q) + bf16hi(q) * bf16hi(q);
+        qq[i] += bf16lo(q) * bf16lo(q) + bf16hi(q) * bf16hi(q);
       }
-    kk = warp_sum(kk);
-    if (!GENERAL) qq = warp_sum(qq);
-    if (lane == 0) {
-      rk[j] = rsqrtf(kk + kUnitEps);
-      rq[j] = rsqrtf(qq + kUnitEps) * p.q_scale;
       if (!GENERAL) {
-        cg[j] = j < n ? p.neg_a[h] * softplus_exact(__bfloat162float(proj[(size_t)j * p.ld + p.a_col + h]) + p.bias[h]) * kLog2e : 0.f;
-        bt[j] = j < n ? sigmoid_exact(__bfloat162float(proj[(size_t)j * p.ld + p.b_col + h])) : 0.f;
+        ga[i] = __bfloat162float(proj[(size_t)j * p.ld + p.a_col + h]);
+        gb[i] = __bfloat162float(proj[(size_t)j * p.ld + p.b_col + h]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const int j = warp + kPrepWarps * i;
+      kk[i] = warp_sum(kk[i]);
+      if (!GENERAL) qq[i] = warp_sum(qq[i]);
+      if (lane == 0) {
+        rk[j] = rsqrtf(kk[i] + kUnitEps);
+        rq[j] = rsqrtf(qq[i] + kUnitEps) * p.q_scale;
+        if (!GENERAL) {
+          cg[j] = j < n ? p.neg_a[h] * softplus_exact(ga[i] + p.bias[h]) * kLog2e : 0.f;
+          bt[j] = j < n ? sigmoid_exact(gb[i]) : 0.f;
+        }
       }
     }
   }
   if (GENERAL) {
     // log2 decays of (channel, segment of SEG tokens), their running sums
-    constexpr int NS = 256 / DK, SEG = C / NS, RC = 32;
+    constexpr int NS = kPrepThreads / DK, SEG = C / NS, RC = 32;
     float* xin = reinterpret_cast<float*>(UH);             // [C][RC]
     const int d = tid % DK, seg = tid / DK, col = h * DK + d, cols = p.H * DK;
     float z[SEG];
@@ -147,15 +170,21 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
     for (int r0 = 0; r0 < p.R; r0 += RC) {
       const int rn = min(RC, p.R - r0);
       __syncthreads();
-      for (int i = tid; i < C * RC; i += 256) {
+      for (int i = tid; i < C * RC; i += kPrepThreads) {
         const int j = i / RC, r = i - j * RC;
         xin[i] = j < n && r < rn ? tanhf(__bfloat162float(proj[(size_t)j * p.ld + p.a_col + r0 + r])) : 0.f;
       }
       __syncthreads();
-      for (int r = 0; r < rn; ++r) {
-        const float a = __ldg(p.w2 + (size_t)(r0 + r) * cols + col);
+#pragma unroll 2
+      for (int r = 0; r < rn; r += 4) {                    // ranks past the last meet zeros
+        float a[4];
 #pragma unroll
-        for (int j = 0; j < SEG; ++j) z[j] = fmaf(a, xin[(seg * SEG + j) * RC + r], z[j]);
+        for (int e = 0; e < 4; ++e) a[e] = __ldg(p.w2 + (size_t)min(r0 + r + e, p.R - 1) * cols + col);
+#pragma unroll
+        for (int j = 0; j < SEG; ++j) {
+          const float4 x = *reinterpret_cast<const float4*>(xin + (seg * SEG + j) * RC + r);
+          z[j] = fmaf(a[0], x.x, fmaf(a[1], x.y, fmaf(a[2], x.z, fmaf(a[3], x.w, z[j]))));
+        }
       }
     }
     float run = 0.f;
@@ -194,14 +223,15 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
       }
     }
     __syncthreads();
-    for (int d = tid; d < DK; d += 256) {
+    for (int d = tid; d < DK; d += kPrepThreads) {
       sc[d] = 1.f;
       p.f_ws[ch * DK + d] = ex2(cg[C - 1]);
     }
   }
   // ---- the scaled operands
-  for (int i = tid; i < C * DK / 8; i += 256) {
-    const int j = i / (DK / 8), d = (i - j * (DK / 8)) * 8;
+#pragma unroll
+  for (int it = 0; it < C * DK / 8 / kPrepThreads; ++it) {
+    const int i = tid + it * kPrepThreads, j = i / (DK / 8), d = (i - j * (DK / 8)) * 8;
     float k[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, q[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, a[8], u[8], e[8], f[8];
     uint4 kr = make_uint4(0u, 0u, 0u, 0u), qr = kr;
     if (j < n) {
@@ -248,52 +278,54 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
   }
   __syncthreads();
 
-  // ---- the C x C products, blocks on and below the diagonal: a warp takes u~ or q~ against p^ or k^ for blocks I and MT-1-I
+  // ---- the C x C products, blocks of 16 x 16 on and below the diagonal (LB of them): u~ and q~ against p^ and k^, each by
+  //      four warps (gated: keys and queries against the keys, each by eight)
+  constexpr int LB = MT * (MT + 1) / 2;
+  constexpr int kLI[10] = {0, 1, 1, 2, 2, 2, 3, 3, 3, 3}, kLJ[10] = {0, 0, 1, 0, 1, 2, 0, 1, 2, 3};
+  for (int i = tid; i < C * C; i += kPrepThreads)          // A is read above its diagonal too
+    if (((i % C) >> 4) > (i / C) >> 4) F[(i / C) * FP + i % C] = 0.f;
   {
-    const bool with_q = warp & 1, with_k = warp & 2;
-#pragma unroll
-    for (int part = 0; part < MT / 2; ++part) {
-      // GENERAL: two warps share the row blocks of a product; gated: four share them (the keys meet queries and keys only)
-      const int I = GENERAL ? (part == 0 ? (warp >> 2) : MT - 1 - (warp >> 2)) : (warp >> 1);
-      if ((GENERAL && MT == 2 && part > 0) || (!GENERAL && (part > 0 || I >= MT))) continue;
-      float acc[MT][2][4] = {};
+    constexpr int SHARE = GENERAL ? 4 : 8, NB = (LB + SHARE - 1) / SHARE;
+    const bool with_q = warp & 1, with_k = GENERAL && (warp & 2);
+    const int first = GENERAL ? warp >> 2 : warp >> 1;
+    float acc[NB][2][4] = {};
 #pragma unroll 2
-      for (int kt = 0; kt < KT; ++kt) {
+    for (int kt = 0; kt < KT; ++kt) {
+#pragma unroll
+      for (int b = 0; b < NB; ++b) {
+        const int at = first + SHARE * b;
+        if (at >= LB) continue;
+        const int I = kLI[at], J = kLJ[at];
         uint32_t ah[4], al[4], bh[4], bl[4];
         if (GENERAL) {
           frag_a(ah, with_q ? QH : UH, KP, 16 * I, 16 * kt, lane);
           frag_a(al, with_q ? QL : UL, KP, 16 * I, 16 * kt, lane);
+          frag_bt(bh, with_k ? KH : PH, KP, 16 * kt, 16 * J, lane);
+          frag_bt(bl, with_k ? KL : PL, KP, 16 * kt, 16 * J, lane);
+          mma3(acc[b], ah, al, bh, bl);
         } else {
           frag_a(ah, with_q ? KL : KH, KP, 16 * I, 16 * kt, lane);
-        }
-#pragma unroll
-        for (int J = 0; J < MT; ++J) {
-          if (J > I) continue;
-          if (GENERAL) {
-            frag_bt(bh, with_k ? KH : PH, KP, 16 * kt, 16 * J, lane);
-            frag_bt(bl, with_k ? KL : PL, KP, 16 * kt, 16 * J, lane);
-            mma3(acc[J], ah, al, bh, bl);
-          } else {
-            frag_bt(bh, KH, KP, 16 * kt, 16 * J, lane);
-            mma(acc[J][0], ah, bh[0], bh[1]);
-            mma(acc[J][1], ah, bh[2], bh[3]);
-          }
+          frag_bt(bh, KH, KP, 16 * kt, 16 * J, lane);
+          mma(acc[b][0], ah, bh[0], bh[1]);
+          mma(acc[b][1], ah, bh[2], bh[3]);
         }
       }
+    }
 #pragma unroll
-      for (int J = 0; J < MT; ++J) {                       // blocks above the diagonal are zero; only A is read there
-        if (J > I && (with_q || (GENERAL && with_k))) continue;
+    for (int b = 0; b < NB; ++b) {
+      const int at = first + SHARE * b;
+      if (at >= LB) continue;
+      const int I = kLI[at], J = kLJ[at];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const int i = 16 * I + g + ((e >> 1) & 1) * 8, j = 16 * J + (e >> 2) * 8 + 2 * t + (e & 1);
-          float& v = acc[J][e >> 2][e & 3];
-          if (!GENERAL) v = i >= j ? v * (with_q ? rq[i] : bt[i] * rk[i]) * rk[j] * ex2(cg[i] - cg[j]) : 0.f;
-          if (with_q ? j > i : j >= i) v = 0.f;
-          if (!with_q && (!GENERAL || !with_k)) F[i * FP + j] = v;
-        }
-        if (with_q) store_tile(acc[J], GENERAL && with_k ? WH : AH, GENERAL && with_k ? WL : AL, AP, 16 * I, 16 * J, g, t);
-        else if (GENERAL && with_k) store_tile(acc[J], NH, NL, AP, 16 * I, 16 * J, g, t);
+      for (int e = 0; e < 8; ++e) {
+        const int i = 16 * I + g + ((e >> 1) & 1) * 8, j = 16 * J + (e >> 2) * 8 + 2 * t + (e & 1);
+        float& v = acc[b][e >> 2][e & 3];
+        if (!GENERAL) v = i >= j ? v * (with_q ? rq[i] : bt[i] * rk[i]) * rk[j] * ex2(cg[i] - cg[j]) : 0.f;
+        if (with_q ? j > i : j >= i) v = 0.f;
+        if (!with_q && !with_k) F[i * FP + j] = v;
       }
+      if (with_q) store_tile(acc[b], with_k ? WH : AH, with_k ? WL : AL, AP, 16 * I, 16 * J, g, t);
+      else if (with_k) store_tile(acc[b], NH, NL, AP, 16 * I, 16 * J, g, t);
     }
   }
   __syncthreads();
@@ -320,37 +352,37 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
     __syncthreads();
 #pragma unroll
     for (int s = 16; s < C; s *= 2) {                      // [M11 0; -M22 A21 M11, M22]
-      const int quads = s * s / 4, pairs = C / (2 * s);
+      const int duos = s * s / 2, pairs = C / (2 * s);
       for (int pass = 0; pass < 2; ++pass) {
-        for (int e = tid; e < quads * pairs; e += 256) {
-          const int pr = e / quads, r = (e - pr * quads) / (s / 4), c0 = ((e - pr * quads) % (s / 4)) * 4, o = pr * 2 * s;
-          float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int e = tid; e < duos * pairs; e += kPrepThreads) {
+          const int pr = e / duos, r = (e - pr * duos) / (s / 2), c0 = ((e - pr * duos) % (s / 2)) * 2, o = pr * 2 * s;
+          float2 sum = make_float2(0.f, 0.f);
           const float *a = F + (o + s + r) * FP + (pass == 0 ? o : o + s), *m = pass == 0 ? F + o * FP + o + c0 : tmp + pr * s * s + c0;
           const int mp = pass == 0 ? FP : s;
 #pragma unroll 8
           for (int k = 0; k < s; ++k) {
-            const float4 v = *reinterpret_cast<const float4*>(m + k * mp);
+            const float2 v = *reinterpret_cast<const float2*>(m + k * mp);
             const float f = a[k];
-            sum.x = fmaf(f, v.x, sum.x); sum.y = fmaf(f, v.y, sum.y);
-            sum.z = fmaf(f, v.z, sum.z); sum.w = fmaf(f, v.w, sum.w);
+            sum.x = fmaf(f, v.x, sum.x);
+            sum.y = fmaf(f, v.y, sum.y);
           }
-          if (pass == 0) *reinterpret_cast<float4*>(tmp + pr * s * s + r * s + c0) = sum;
-          else *reinterpret_cast<float4*>(F + (o + s + r) * FP + o + c0) = make_float4(-sum.x, -sum.y, -sum.z, -sum.w);
+          if (pass == 0) *reinterpret_cast<float2*>(tmp + pr * s * s + r * s + c0) = sum;
+          else *reinterpret_cast<float2*>(F + (o + s + r) * FP + o + c0) = make_float2(-sum.x, -sum.y);
         }
         __syncthreads();
       }
     }
-    constexpr int NE = C * C / 512;                        // pairs of columns per thread
+    constexpr int NE = C * C / 2 / kPrepThreads;           // pairs of columns per thread
     float2 m[NE];
 #pragma unroll
     for (int e = 0; e < NE; ++e) {
-      const int at = (tid + e * 256) * 2, i = at / C, j = at % C;
+      const int at = (tid + e * kPrepThreads) * 2, i = at / C, j = at % C;
       m[e] = make_float2(j <= i ? F[i * FP + j] : 0.f, j + 1 <= i ? F[i * FP + j + 1] : 0.f);
     }
     __syncthreads();
 #pragma unroll
     for (int e = 0; e < NE; ++e) {
-      const int at = (tid + e * 256) * 2, i = at / C, j = at % C;
+      const int at = (tid + e * kPrepThreads) * 2, i = at / C, j = at % C;
       uint32_t hi, lo;
       split2(m[e].x, m[e].y, hi, lo);
       *reinterpret_cast<uint32_t*>(MH + i * AP + j) = hi;
@@ -364,20 +396,17 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
     __syncthreads();
   }
 
-  // items of a C x DK product: tiles of 16 x 16, column tile varies first
-  constexpr int NI = MT * KT / 8;
-  // blocks on and below the diagonal of a C x C matrix, two rounds of eight warps
-  constexpr int kI4[2][8] = {{3, 2, 3, 1, 2, 3, 3, 0}, {-1, -1, -1, -1, 1, 2, -1, -1}}, kJ4[2][8] = {{0, 0, 1, 0, 1, 2, 3, 0}, {0, 0, 0, 0, 1, 2, 0, 0}};
-  constexpr int kI2[8] = {0, 1, 1, -1, -1, -1, -1, -1}, kJ2[8] = {0, 0, 1, 0, 0, 0, 0, 0};
-  auto low_i = [&](int r) { return MT == 4 ? kI4[r][warp] : (r == 0 ? kI2[warp] : -1); };
-  auto low_j = [&](int r) { return MT == 4 ? kJ4[r][warp] : kJ2[warp]; };
+  // tiles of a C x DK product, column tile varies first; blocks on and below the diagonal of a C x C matrix, one per warp
+  constexpr int NI = MT * KT / kPrepWarps;
+  const bool has_low = warp < LB;
+  const int lowI = has_low ? kLI[warp] : 0, lowJ = has_low ? kLJ[warp] : 0;
 
   // ---- D = M u~, N = M (u~ k^T)
   {
-    float acc[NI][2][4] = {}, nn[2][2][4] = {};
+    float acc[NI][2][4] = {}, nn[2][4] = {};
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      const int id = warp + 8 * i, c0 = (id % KT) * 16, I = id / KT;
+      const int id = warp + kPrepWarps * i, c0 = (id % KT) * 16, I = id / KT;
 #pragma unroll
       for (int kt = 0; kt < MT; ++kt) {
         if (kt > I) continue;
@@ -389,39 +418,30 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
         mma3(acc[i], ah, al, bh, bl);
       }
     }
-    if (GENERAL) {
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int I = low_i(r), J = low_j(r);
-        if (I < 0) continue;
-        for (int kt = J; kt <= I; ++kt) {
-          uint32_t ah[4], al[4], bh[4], bl[4];
-          frag_a(ah, MH, AP, 16 * I, 16 * kt, lane);
-          frag_a(al, ML, AP, 16 * I, 16 * kt, lane);
-          frag_b(bh, NH, AP, 16 * kt, 16 * J, lane);
-          frag_b(bl, NL, AP, 16 * kt, 16 * J, lane);
-          mma3(nn[r], ah, al, bh, bl);
-        }
+    if (GENERAL && has_low) {
+      for (int kt = lowJ; kt <= lowI; ++kt) {
+        uint32_t ah[4], al[4], bh[4], bl[4];
+        frag_a(ah, MH, AP, 16 * lowI, 16 * kt, lane);
+        frag_a(al, ML, AP, 16 * lowI, 16 * kt, lane);
+        frag_b(bh, NH, AP, 16 * kt, 16 * lowJ, lane);
+        frag_b(bl, NL, AP, 16 * kt, 16 * lowJ, lane);
+        mma3(nn, ah, al, bh, bl);
       }
     }
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
-      const int id = warp + 8 * i;
+      const int id = warp + kPrepWarps * i;
       store_tile(acc[i], UH, UL, KP, (id / KT) * 16, (id % KT) * 16, g, t);
     }
-    if (GENERAL) {
-#pragma unroll
-      for (int r = 0; r < 2; ++r)
-        if (low_i(r) >= 0) store_tile(nn[r], NH, NL, AP, 16 * low_i(r), 16 * low_j(r), g, t);
-    }
+    if (GENERAL && has_low) store_tile(nn, NH, NL, AP, 16 * lowI, 16 * lowJ, g, t);
     __syncthreads();
   }
 
   // ---- Q = q~ - A D into the workspace; E = (k^ - N^T p^) exp(G_C) in the place of k^
 #pragma unroll
   for (int i = 0; i < NI; ++i) {
-    const int id = warp + 8 * i, ct = id % KT, c0 = ct * 16, I = id / KT;
+    const int id = warp + kPrepWarps * i, ct = id % KT, c0 = ct * 16, I = id / KT;
     float acc[2][4] = {}, ee[2][4] = {}, q[2][4];
 #pragma unroll
     for (int kt = 0; kt < MT; ++kt) {
@@ -458,72 +478,61 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
     store_tile(q, KH, KL, KP, 16 * I, c0, g, t);
   }
   // ---- W = (q~ k^T) - A N in the place of the first
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    const int I = low_i(r), J = low_j(r);
-    if (I < 0) continue;
+  if (has_low) {
     float acc[2][4] = {}, w[2][4] = {};
-    for (int kt = J; kt <= I; ++kt) {
+    for (int kt = lowJ; kt <= lowI; ++kt) {
       uint32_t ah[4], al[4], bh[4], bl[4];
-      frag_a(ah, AH, AP, 16 * I, 16 * kt, lane);
-      frag_a(al, AL, AP, 16 * I, 16 * kt, lane);
-      frag_b(bh, NH, AP, 16 * kt, 16 * J, lane);
-      frag_b(bl, NL, AP, 16 * kt, 16 * J, lane);
+      frag_a(ah, AH, AP, 16 * lowI, 16 * kt, lane);
+      frag_a(al, AL, AP, 16 * lowI, 16 * kt, lane);
+      frag_b(bh, NH, AP, 16 * kt, 16 * lowJ, lane);
+      frag_b(bl, NL, AP, 16 * kt, 16 * lowJ, lane);
       mma3(acc, ah, al, bh, bl);
     }
-    if (GENERAL) load_tile(w, WH, WL, AP, 16 * I, 16 * J, g, t);
+    if (GENERAL) load_tile(w, WH, WL, AP, 16 * lowI, 16 * lowJ, g, t);
 #pragma unroll
     for (int e = 0; e < 8; ++e) w[e >> 2][e & 3] -= acc[e >> 2][e & 3];
-    store_tile(w, WH, WL, AP, 16 * I, 16 * J, g, t);
+    store_tile(w, WH, WL, AP, 16 * lowI, 16 * lowJ, g, t);
   }
-  // ---- -R = -exp(G_C) p^T D into the workspace
+  // ---- -R = -exp(G_C) p^T D into the workspace: a warp takes RUN column tiles of one row tile
   {
-    constexpr int NR = KT * KT / 8;                        // tiles of a warp: row tile fixed for a run of column tiles
-    constexpr int RUN = KT < 8 ? NR : KT;
-#pragma unroll 1
-    for (int r0 = 0; r0 < NR; r0 += RUN) {
-      const int rt = KT < 8 ? warp % KT : warp + 8 * (r0 / RUN), first = KT < 8 ? (warp / KT) * RUN : 0;
-      uint32_t ah[MT][4], al[MT][4];
+    constexpr int RUN = KT * KT / kPrepWarps;
+    const int rt = warp % KT, first = (warp / KT) * RUN;
+    uint32_t ah[MT][4], al[MT][4];
+#pragma unroll
+    for (int kt = 0; kt < MT; ++kt) {
+      frag_at(ah[kt], PH, KP, 16 * rt, 16 * kt, lane);
+      frag_at(al[kt], PL, KP, 16 * rt, 16 * kt, lane);
+    }
+    const float s0 = -sc[16 * rt + g], s1 = -sc[16 * rt + g + 8];
+#pragma unroll 2
+    for (int ct = first; ct < first + RUN; ++ct) {
+      float acc[2][4] = {};
 #pragma unroll
       for (int kt = 0; kt < MT; ++kt) {
-        frag_at(ah[kt], PH, KP, 16 * rt, 16 * kt, lane);
-        frag_at(al[kt], PL, KP, 16 * rt, 16 * kt, lane);
+        uint32_t bh[4], bl[4];
+        frag_b(bh, UH, KP, 16 * kt, 16 * ct, lane);
+        frag_b(bl, UL, KP, 16 * kt, 16 * ct, lane);
+        mma3(acc, ah[kt], al[kt], bh, bl);
       }
-      const float s0 = -sc[16 * rt + g], s1 = -sc[16 * rt + g + 8];
-#pragma unroll 2
-      for (int ct = first; ct < first + RUN; ++ct) {
-        float acc[2][4] = {};
 #pragma unroll
-        for (int kt = 0; kt < MT; ++kt) {
-          uint32_t bh[4], bl[4];
-          frag_b(bh, UH, KP, 16 * kt, 16 * ct, lane);
-          frag_b(bl, UL, KP, 16 * kt, 16 * ct, lane);
-          mma3(acc, ah[kt], al[kt], bh, bl);
-        }
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e >> 2][e & 3] *= e & 2 ? s1 : s0;
-        uint4 hi, lo;
-        pack_tile(acc, hi, lo);
-        uint4* dst = p.t_ws + ((ch * KT + rt) * KT + ct) * 64 + lane;
-        dst[0] = hi;
-        dst[32] = lo;
-      }
+      for (int e = 0; e < 8; ++e) acc[e >> 2][e & 3] *= e & 2 ? s1 : s0;
+      uint4 hi, lo;
+      pack_tile(acc, hi, lo);
+      uint4* dst = p.t_ws + ((ch * KT + rt) * KT + ct) * 64 + lane;
+      dst[0] = hi;
+      dst[32] = lo;
     }
   }
   // ---- E^T V (transposed: rows are value columns) and W V, 64 value columns at a time
   for (int v0 = 0; v0 < dv; v0 += 64) {
     __syncthreads();
-    for (int i = tid; i < C * 8; i += 256) {
-      const int j = i >> 3, c = (i & 7) * 8;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (j < n) v = *reinterpret_cast<const uint4*>(src + (size_t)j * p.lds + p.v_col + h * dv + v0 + c);
-      *reinterpret_cast<uint4*>(V + j * VP + c) = v;
-    }
+    if (vj < C) *reinterpret_cast<uint4*>(V + vj * VP + vc) = vnext;
+    if (has_v && v0 + 64 < dv) vnext = *reinterpret_cast<const uint4*>(vsrc + v0 + 64);
     __syncthreads();
-    constexpr int NE = 4 * KT / 8;
+    constexpr int NE = 4 * KT / kPrepWarps;
 #pragma unroll
     for (int i = 0; i < NE; ++i) {
-      const int id = warp + 8 * i, ct = id % KT, vt = id / KT;
+      const int id = warp + kPrepWarps * i, ct = id % KT, vt = id / KT;
       float acc[2][4] = {};
 #pragma unroll
       for (int kt = 0; kt < MT; ++kt) {
@@ -541,9 +550,8 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
       dst[0] = make_float4(acc[0][0], acc[0][1], acc[0][2], acc[0][3]);
       dst[32] = make_float4(acc[1][0], acc[1][1], acc[1][2], acc[1][3]);
     }
-#pragma unroll
-    for (int i = 0; i < MT / 2; ++i) {
-      const int id = warp + 8 * i, I = MT == 4 ? (i == 0 ? id % 4 : 3 - id % 4) : id % 2, vt = id / MT;
+    if (warp < 4 * MT) {
+      const int vt = warp / MT, I = (warp + vt) % MT;      // neighbours share a scheduler: the long rows go to all of them
       float acc[2][4] = {};
       for (int kt = 0; kt <= I; ++kt) {
         uint32_t ah[4], al[4], b[4];
@@ -567,21 +575,22 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(const __grid_c
 }
 
 // ------------------------------------------------------------------------------------------------ scan over the chunks
-// A block owns 32 columns of a head's state (transposed: rows are value columns), a warp 16 key channels of it in fp32
-// accumulators.  Per chunk the state goes to shared memory as two bf16 terms, every warp multiplies all of it with its rows of
-// -R, and the decay and what the chunk adds come on top in fp32.
-template <int DK>
+// A block owns 16 NV columns of a head's state (transposed: rows are value columns), a warp 16 key channels of it in fp32
+// registers.  Per chunk the state goes to shared memory as two bf16 terms, every warp multiplies all of it with its rows of
+// -R, and the decay and what the chunk adds come on top in fp32.  The three products of the terms are summed apart, so that
+// no chain of products is longer than the keys have tiles.
+template <int DK, int NV>
 __global__ void __launch_bounds__(DK * 2) delta_chunk_scan_kernel(const __grid_constant__ DeltaParams p, int dv) {
   constexpr int KT = DK / 16, PF = KT == 8 ? 8 : 4;
   extern __shared__ __align__(16) uint8_t smem[];
-  uint4 (*sh)[KT][2][2][32] = reinterpret_cast<uint4 (*)[KT][2][2][32]>(smem);       // [buffer][key tile][term][16 columns][lane]
+  uint4 (*sh)[KT][2][NV][32] = reinterpret_cast<uint4 (*)[KT][2][NV][32]>(smem);     // [buffer][key tile][term][16 columns][lane]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-  const int vt0 = blockIdx.x * 2, h = blockIdx.y, s = p.long_seq[blockIdx.z], c0 = p.long_ck[blockIdx.z], c1 = p.long_ck[blockIdx.z + 1];
+  const int vt0 = blockIdx.x * NV, h = blockIdx.y, s = p.long_seq[blockIdx.z], c0 = p.long_ck[blockIdx.z], c1 = p.long_ck[blockIdx.z + 1];
   float* state = p.state + ((size_t)p.slots[s] * p.H + h) * DK * dv;
   const int key0 = warp * 16 + 2 * t, col0 = vt0 * 16 + g;
-  float S[2][2][4];                                        // [16 columns][8 keys]
+  float S[NV][2][4];                                       // [16 columns][8 keys]
 #pragma unroll
-  for (int v = 0; v < 2; ++v)
+  for (int v = 0; v < NV; ++v)
 #pragma unroll
     for (int e = 0; e < 8; ++e) S[v][e >> 2][e & 3] = state[(size_t)(key0 + (e >> 2) * 8 + (e & 1)) * dv + col0 + v * 16 + (e & 2) * 4];
   pdl_trigger();
@@ -591,11 +600,11 @@ __global__ void __launch_bounds__(DK * 2) delta_chunk_scan_kernel(const __grid_c
   float4* sp = p.s_ws + ((((size_t)c0 * p.H + h) * (dv / 16) + vt0) * KT + warp) * 64 + lane;
   const float* fp = p.f_ws + ((size_t)c0 * p.H + h) * DK + key0;
   uint4 bh[PF], bl[PF];
-  float4 add[2][2];
+  float4 add[NV][2];
   float2 f[2];
   auto fetch_small = [&]() {
 #pragma unroll
-    for (int v = 0; v < 2; ++v)
+    for (int v = 0; v < NV; ++v)
 #pragma unroll
       for (int e = 0; e < 2; ++e) add[v][e] = sp[v * KT * 64 + e * 32];
     f[0] = *reinterpret_cast<const float2*>(fp);
@@ -609,18 +618,23 @@ __global__ void __launch_bounds__(DK * 2) delta_chunk_scan_kernel(const __grid_c
   fetch_small();
   for (int c = c0; c < c1; ++c) {
     const int b = c & 1;
+    uint4 hi[NV], lo[NV];
 #pragma unroll
-    for (int v = 0; v < 2; ++v) {
-      uint4 hi, lo;
-      pack_tile(S[v], hi, lo);
-      sh[b][warp][0][v][lane] = hi;
-      sh[b][warp][1][v][lane] = lo;
-      uint4* dst = reinterpret_cast<uint4*>(sp + v * KT * 64);           // what the chunk added has been read
-      dst[0] = hi;
-      dst[32] = lo;
+    for (int v = 0; v < NV; ++v) {
+      pack_tile(S[v], hi[v], lo[v]);
+      sh[b][warp][0][v][lane] = hi[v];
+      sh[b][warp][1][v][lane] = lo[v];
     }
+    __syncthreads();
 #pragma unroll
-    for (int v = 0; v < 2; ++v)
+    for (int v = 0; v < NV; ++v) {
+      uint4* dst = reinterpret_cast<uint4*>(sp + v * KT * 64);           // what the chunk added has been read
+      dst[0] = hi[v];
+      dst[32] = lo[v];
+    }
+    float acc[NV][2][2][4] = {};                           // the two cross products
+#pragma unroll
+    for (int v = 0; v < NV; ++v)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         S[v][e][0] = fmaf(f[e].x, S[v][e][0], add[v][e].x);
@@ -632,31 +646,19 @@ __global__ void __launch_bounds__(DK * 2) delta_chunk_scan_kernel(const __grid_c
     sp += sstep;
     fp += (size_t)p.H * DK;
     if (more) fetch_small();
-    __syncthreads();
 #pragma unroll
     for (int k0 = 0; k0 < KT; k0 += PF) {
 #pragma unroll
       for (int k = 0; k < PF; ++k) {
-        uint4 a[2][2];
 #pragma unroll
-        for (int v = 0; v < 2; ++v) {
-          a[0][v] = sh[b][k0 + k][0][v][lane];
-          a[1][v] = sh[b][k0 + k][1][v][lane];
-        }
-#pragma unroll
-        for (int v = 0; v < 2; ++v) {
-          mma_bf16_16816(S[v][0], a[0][v].x, a[0][v].y, a[0][v].z, a[0][v].w, bh[k].x, bh[k].z);
-          mma_bf16_16816(S[v][1], a[0][v].x, a[0][v].y, a[0][v].z, a[0][v].w, bh[k].y, bh[k].w);
-        }
-#pragma unroll
-        for (int v = 0; v < 2; ++v) {
-          mma_bf16_16816(S[v][0], a[1][v].x, a[1][v].y, a[1][v].z, a[1][v].w, bh[k].x, bh[k].z);
-          mma_bf16_16816(S[v][1], a[1][v].x, a[1][v].y, a[1][v].z, a[1][v].w, bh[k].y, bh[k].w);
-        }
-#pragma unroll
-        for (int v = 0; v < 2; ++v) {
-          mma_bf16_16816(S[v][0], a[0][v].x, a[0][v].y, a[0][v].z, a[0][v].w, bl[k].x, bl[k].z);
-          mma_bf16_16816(S[v][1], a[0][v].x, a[0][v].y, a[0][v].z, a[0][v].w, bl[k].y, bl[k].w);
+        for (int v = 0; v < NV; ++v) {
+          const uint4 a = sh[b][k0 + k][0][v][lane], z = sh[b][k0 + k][1][v][lane];
+          mma_bf16_16816(S[v][0], a.x, a.y, a.z, a.w, bh[k].x, bh[k].z);
+          mma_bf16_16816(S[v][1], a.x, a.y, a.z, a.w, bh[k].y, bh[k].w);
+          mma_bf16_16816(acc[v][0][0], z.x, z.y, z.z, z.w, bh[k].x, bh[k].z);
+          mma_bf16_16816(acc[v][0][1], z.x, z.y, z.z, z.w, bh[k].y, bh[k].w);
+          mma_bf16_16816(acc[v][1][0], a.x, a.y, a.z, a.w, bl[k].x, bl[k].z);
+          mma_bf16_16816(acc[v][1][1], a.x, a.y, a.z, a.w, bl[k].y, bl[k].w);
         }
         // the word PF tiles ahead: of this chunk, or of the next
         if (k0 + PF < KT || more) {
@@ -666,18 +668,22 @@ __global__ void __launch_bounds__(DK * 2) delta_chunk_scan_kernel(const __grid_c
         }
       }
     }
+#pragma unroll
+    for (int v = 0; v < NV; ++v)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) S[v][e >> 2][e & 3] += acc[v][0][e >> 2][e & 3] + acc[v][1][e >> 2][e & 3];
     tp += tstep;
     const int snap = p.ck_snap[c];
     if (snap >= 0) {
       float* dst = p.snap + ((size_t)snap * p.H + h) * DK * dv;
 #pragma unroll
-      for (int v = 0; v < 2; ++v)
+      for (int v = 0; v < NV; ++v)
 #pragma unroll
         for (int e = 0; e < 8; ++e) dst[(size_t)(key0 + (e >> 2) * 8 + (e & 1)) * dv + col0 + v * 16 + (e & 2) * 4] = S[v][e >> 2][e & 3];
     }
   }
 #pragma unroll
-  for (int v = 0; v < 2; ++v)
+  for (int v = 0; v < NV; ++v)
 #pragma unroll
     for (int e = 0; e < 8; ++e) state[(size_t)(key0 + (e >> 2) * 8 + (e & 1)) * dv + col0 + v * 16 + (e & 2) * 4] = S[v][e >> 2][e & 3];
 }
@@ -731,17 +737,28 @@ __global__ void __launch_bounds__(256) delta_chunk_out_kernel(const __grid_const
   }
 }
 
+// TI_DELTA_SCAN: the number of blocks up to which the narrow form of the scan runs
+static int scan_blocks() {
+  static const int n = [] { const char* e = getenv("TI_DELTA_SCAN"); return e == nullptr ? 148 : atoi(e); }();
+  return n;
+}
+
 template <int DK, bool GENERAL>
 static int launch_delta_chunked(const DeltaParams& p, int dv, cudaStream_t st) {
   using M = DeltaGeom<DK>;
   static bool configured = false;
   if (!configured) {
     cudaFuncSetAttribute(delta_chunk_prepare_kernel<DK, GENERAL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)M::kSmem);
-    cudaFuncSetAttribute(delta_chunk_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)M::kScan);
+    cudaFuncSetAttribute(delta_chunk_scan_kernel<DK, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)M::kScan / 2);
+    cudaFuncSetAttribute(delta_chunk_scan_kernel<DK, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)M::kScan);
     configured = true;
   }
-  launch_kernel(delta_chunk_prepare_kernel<DK, GENERAL>, dim3(p.nc, p.H), dim3(256), M::kSmem, st, true, p, dv);
-  launch_kernel(delta_chunk_scan_kernel<DK>, dim3(dv / 32, p.H, p.num_long), dim3(DK * 2), M::kScan, st, true, p, dv);
+  launch_kernel(delta_chunk_prepare_kernel<DK, GENERAL>, dim3(p.nc, p.H), dim3(kPrepThreads), M::kSmem, st, true, p, dv);
+  // narrow blocks while they fit the SMs at once; wide ones read a chunk's matrix half as often
+  if ((long long)dv / 16 * p.H * p.num_long <= scan_blocks())
+    launch_kernel(delta_chunk_scan_kernel<DK, 1>, dim3(dv / 16, p.H, p.num_long), dim3(DK * 2), M::kScan / 2, st, true, p, dv);
+  else
+    launch_kernel(delta_chunk_scan_kernel<DK, 2>, dim3(dv / 32, p.H, p.num_long), dim3(DK * 2), M::kScan, st, true, p, dv);
   launch_kernel(delta_chunk_out_kernel<DK>, dim3(p.nc, p.H, (dv + 127) / 128), dim3(256), 0, st, true, p, dv);
   return (int)cudaGetLastError();
 }

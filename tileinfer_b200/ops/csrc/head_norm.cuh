@@ -14,31 +14,43 @@ struct HeadNormParams {
   float eps;
 };
 
-// a warp per (token, head)
-template <typename T>
+// LPI lanes per (token, head), eight columns each at a time
+template <typename T, int LPI>
 __global__ void __launch_bounds__(256) head_norm_kernel(const __grid_constant__ HeadNormParams p, int items) {
-  const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31, dv = p.dv;
+  const int item = (blockIdx.x * 256 + threadIdx.x) / LPI, lane = threadIdx.x & (LPI - 1), dv = p.dv;
   pdl_trigger();
   pdl_wait();
-  if (item >= items) return;
-  const int t = item / p.H, h = item - t * p.H;
+  const bool live = item < items;                          // the lanes of a warp meet in the shuffles
+  const int t = live ? item / p.H : 0, h = live ? item - t * p.H : 0;
   const float* o = p.o + (size_t)t * p.H * dv + h * dv;
   const float* norm = p.norm + (size_t)h * p.norm_stride;
   const T* g = static_cast<const T*>(p.gate) + (size_t)t * p.ld + p.g_col + h * dv;
   T* out = static_cast<T*>(p.out) + (size_t)t * p.ldo + h * dv;
-  float ss = 0.f;
-  for (int c = lane * 8; c < dv; c += 256) {
-    float v[8];
-    load8(o + c, v);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) ss += v[i] * v[i];
+  float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, z[8], ss = 0.f;
+  if (LPI < 32 || lane * 8 < dv) {
+    load8(o + lane * 8, v);
+    load8(g + lane * 8, z);
   }
-  const float rr = rsqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
-  for (int c = lane * 8; c < dv; c += 256) {
-    float v[8], w[8], z[8];
-    load8(o + c, v);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ss += v[i] * v[i];
+  if (LPI == 32)
+    for (int c = lane * 8 + 256; c < dv; c += 256) {
+      float u[8];
+      load8(o + c, u);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) ss += u[i] * u[i];
+    }
+#pragma unroll
+  for (int s = LPI / 2; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  if (!live) return;
+  const float rr = rsqrtf(ss / (float)p.vdim + p.eps);
+  for (int c = lane * 8; c < dv; c += LPI * 8) {
+    float w[8];
     load8(norm + c, w);
-    load8(g + c, z);
+    if (LPI == 32 && c >= 256) {
+      load8(o + c, v);
+      load8(g + c, z);
+    }
 #pragma unroll
     for (int i = 0; i < 8; ++i) v[i] *= rr * w[i] * sigmoid_exact(z[i]) * (p.silu ? z[i] : 1.f);
     store8(out + c, v);
@@ -49,7 +61,12 @@ inline int launch_head_norm(const HeadNormParams& p, int T, int f32, cudaStream_
   if (T <= 0) return 0;
   if (p.dv % 64 || p.ld % 8 || p.ldo % 8 || p.g_col % 8 || p.norm_stride % 4 || (((uintptr_t)p.gate | (uintptr_t)p.out | (uintptr_t)p.o | (uintptr_t)p.norm) & 15)) return -2;
   const int items = T * p.H;
-  launch_kernel(f32 ? head_norm_kernel<float> : head_norm_kernel<bf16>, dim3((items + 7) / 8), dim3(256), 0, st, true, p, items);
+#define TI_HN(L)                                                                                                           \
+  launch_kernel(f32 ? head_norm_kernel<float, L> : head_norm_kernel<bf16, L>, dim3((items + 256 / L - 1) / (256 / L)), dim3(256), 0, st, true, p, items)
+  if (p.dv == 64) TI_HN(8);
+  else if (p.dv == 128) TI_HN(16);
+  else TI_HN(32);
+#undef TI_HN
   return (int)cudaGetLastError();
 }
 
