@@ -142,16 +142,27 @@ TI_DEVICE float head_factor(const AttnPrefillParams& p, size_t tok, int head) {
   return p.head_gate == nullptr ? p.out_scale : p.out_scale * sigmoid_f(__bfloat162float(p.head_gate[tok * p.ldg + p.gcol + head]));
 }
 
+// Gates of 32 output columns of a row, and the request for a whole row of them ahead of its use: the rows of a tile lie far
+// apart, and reading them only at the end would cost a memory round trip per 32 columns.
+TI_DEVICE void load_gates(const AttnPrefillParams& p, const __nv_bfloat16* gate, int c, uint4 (&g)[4]) {
+  if (p.gate_src == nullptr) return;
+#pragma unroll
+  for (int q = 0; q < 4; ++q) g[q] = *reinterpret_cast<const uint4*>(gate + c * 32 + q * 8);
+}
+TI_DEVICE void prefetch_gates(const AttnPrefillParams& p, const __nv_bfloat16* gate, int columns) {
+  if (p.gate_src == nullptr) return;
+  for (int c = 0; c < columns; c += 64) asm volatile("prefetch.global.L2 [%0];\n" ::"l"(gate + c));
+}
+
 // 32 output columns of a row: times 1 / l and the sigmoid gate, as bf16
-TI_DEVICE void store_rows32(const AttnPrefillParams& p, const uint32_t (&v)[32], float inv, const __nv_bfloat16* gate, __nv_bfloat16* dst, int c) {
+TI_DEVICE void store_rows32(const AttnPrefillParams& p, const uint32_t (&v)[32], float inv, const uint4 (&gates)[4], __nv_bfloat16* dst, int c) {
 #pragma unroll
   for (int q4 = 0; q4 < 4; ++q4) {
     float f[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(v[q4 * 8 + e]) * inv;
     if (p.gate_src != nullptr) {
-      const uint4 gw = *reinterpret_cast<const uint4*>(gate + c * 32 + q4 * 8);
-      const uint32_t g4[4] = {gw.x, gw.y, gw.z, gw.w};
+      const uint32_t g4[4] = {gates[q4].x, gates[q4].y, gates[q4].z, gates[q4].w};
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         f[2 * e] *= sigmoid_f(bf16lo(g4[e]));
@@ -357,8 +368,10 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
         for (int c = half * (DV / 64); c < (half + 1) * (DV / 64); ++c) {
           uint32_t v[32];
           tmem_ld32(lane_base + 256u + c * 32, v);
+          uint4 gates[4];
+          load_gates(p, gate, c, gates);
           tmem_ld_wait();
-          if (valid) store_rows32(p, v, inv, gate, dst, c);
+          if (valid) store_rows32(p, v, inv, gates, dst, c);
         }
       }
       tc_fence_before();
@@ -372,6 +385,9 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
     const int lo = p.window > 0 ? pos - p.window + 1 : 0;
     const float slope = MODE == SCORE_BIASED ? p.slopes[head] * 1.4426950408889634f : 0.f;
     const uint32_t lane_base = tmem_base + ((uint32_t)(quarter * 32) << 16);
+    const size_t tok = (size_t)tok0 + (valid ? r : 0);
+    const __nv_bfloat16* gate = p.gate_src + tok * p.ld + p.gate_col + (size_t)head * p.gate_stride;
+    prefetch_gates(p, gate, DV);
     float m_used = kFirstMax, l = 0.f;
     bool ok = true;
     for (int j = 0; j < ntiles; ++j) {
@@ -461,24 +477,25 @@ __global__ void __launch_bounds__((AttnPrefillGeom<D, DV, MODE>::kThreads), 1) a
       asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(p_full) : "memory");
     }
     // ---- epilogue: O / l * sigmoid(gate) -> bf16
+    uint4 gates[4], next[4];
+    load_gates(p, gate, 0, gates);
     if (ok) {
       ok = mbar_wait(p_empty, (uint32_t)((ntiles - 1) & 1), kAttnWaitNs, p.status);
       ok = __all_sync(0xffffffffu, ok);
     }
     if (ok) {
       tc_fence_after();
-      const size_t tok = (size_t)tok0 + (valid ? r : 0);
       const float inv = head_factor(p, tok, head) / l;
-      const __nv_bfloat16* gate = p.gate_src + tok * p.ld + p.gate_col + (size_t)head * p.gate_stride;
       __nv_bfloat16* dst = p.out + tok * (size_t)p.ldo + (size_t)head * DV;
 #pragma unroll 1
       for (int c = 0; c < DV / 32; ++c) {
         uint32_t v[32];
         tmem_ld32(lane_base + 256u + c * 32, v);
+        if (c + 1 < DV / 32) load_gates(p, gate, c + 1, next);
         tmem_ld_wait();
-        if (valid) {
-          store_rows32(p, v, inv, gate, dst, c);
-        }
+        if (valid) store_rows32(p, v, inv, gates, dst, c);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) gates[q] = next[q];
       }
     } else {
       *abort_flag = 1;

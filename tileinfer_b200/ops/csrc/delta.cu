@@ -10,11 +10,18 @@
 
 namespace ti {
 
+constexpr int kW2Smem = 64 * 1024;       // the head's rows of a decay's second matrix go to shared memory if they fit
+
+TI_DEVICE void copy16_async(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(smem_u32(dst)), "l"(src));
+}
+
 // Threads own the state as (row group of 16, four columns): rows rg + 16 i, i < NR.  For the second product of a general decay
-// they are (key channel, part of the ranks) and keep their part of the matrix, up to 32 ranks of it, in registers.
+// they are (key channel, part of the ranks).
 template <typename T, int NR, bool GENERAL>
-__global__ void __launch_bounds__(256) delta_step_kernel(const __grid_constant__ DeltaParams p) {
-  constexpr int DK = NR * 16, PARTS = DK >= 256 ? 1 : 256 / DK, CH = DK > 256 ? DK / 256 : 1, KEEP = GENERAL && DK <= 256 ? 32 : 1;
+__global__ void __launch_bounds__(256, NR <= 4 ? 4 : NR <= 8 ? 3 : 1) delta_step_kernel(const __grid_constant__ DeltaParams p) {
+  constexpr int DK = NR * 16, PARTS = DK >= 256 ? 1 : 256 / DK, CH = DK > 256 ? DK / 256 : 1;
+  extern __shared__ __align__(16) uint8_t smem[];
   __shared__ float w_s[2][GENERAL ? DK : 1], p_s[2][GENERAL ? DK : 1], u_s[2][DK], c_s[2][GENERAL ? DK : 1], q_s[2][DK];
   __shared__ float z_s[GENERAL ? PARTS : 1][GENERAL ? DK : 1], x_s[GENERAL ? 256 : 1];
   __shared__ __align__(16) float red[2][8][128];
@@ -28,14 +35,18 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const __grid_constant__
   for (int i = 0; i < NR; ++i) S[i] = *reinterpret_cast<const float4*>(state + (size_t)(rg + 16 * i) * dv);
   // ranks of this thread: r0 + PARTS i
   const int ch = PARTS > 1 ? tid % DK : tid, r0 = PARTS > 1 ? tid / DK : 0, cols = p.H * DK;
-  float keep[KEEP];
-  if (GENERAL && KEEP > 1) {
-#pragma unroll
-    for (int i = 0; i < KEEP; ++i) keep[i] = r0 + PARTS * i < p.R ? __ldg(p.w2 + (size_t)(r0 + PARTS * i) * cols + h * DK + ch) : 0.f;
+  const float* w2 = GENERAL ? p.w2 + h * DK : nullptr;
+  int w2_ld = cols;
+  if (GENERAL && (size_t)p.R * DK * 4 <= kW2Smem) {
+    float* dst = reinterpret_cast<float*>(smem);           // [R][DK]
+    for (int i = tid * 4; i < p.R * DK; i += 1024) copy16_async(dst + i, w2 + (size_t)(i / DK) * cols + i % DK);
+    w2 = dst;
+    w2_ld = DK;
   }
   pdl_trigger();
   pdl_wait();                                              // the inputs come from the kernels before
   const int t0 = p.cu == nullptr ? s : p.cu[s], t1 = p.cu == nullptr ? s + 1 : p.cu[s + 1];
+  if (GENERAL) asm volatile("cp.async.wait_all;\n" ::: "memory");            // visible behind the first barrier
   for (int t = t0; t < t1; ++t) {
     const int b = t & 1;
     const T* src = static_cast<const T*>(p.src) + (size_t)t * p.lds;
@@ -51,14 +62,10 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const __grid_constant__
         if (rb + tid < p.R) x_s[tid] = tanhf(to_f<T>(row[p.a_col + rb + tid]));
         __syncthreads();
         const int rn = min(256, p.R - rb);
-        if (KEEP > 1 && rb == 0) {
+#pragma unroll 4
+        for (int r = r0; r < rn; r += PARTS)
 #pragma unroll
-          for (int i = 0; i < KEEP; ++i)
-            if (r0 + PARTS * i < rn) z[0] = fmaf(keep[i], x_s[r0 + PARTS * i], z[0]);
-        }
-        for (int r = r0 + (KEEP > 1 && rb == 0 ? PARTS * KEEP : 0); r < rn; r += PARTS)
-#pragma unroll
-          for (int j = 0; j < CH; ++j) z[j] = fmaf(__ldg(p.w2 + (size_t)(rb + r) * cols + h * DK + ch + 256 * j), x_s[r], z[j]);
+          for (int j = 0; j < CH; ++j) z[j] = fmaf(w2[(size_t)(rb + r) * w2_ld + ch + 256 * j], x_s[r], z[j]);
       }
       if (PARTS > 1) {
         z_s[r0][ch] = z[0];
@@ -168,14 +175,25 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const __grid_constant__
   for (int i = 0; i < NR; ++i) *reinterpret_cast<float4*>(state + (size_t)(rg + 16 * i) * dv) = S[i];
 }
 
+template <typename T, int NR, bool GENERAL>
+static void launch_delta_rows(const DeltaParams& p, dim3 grid, cudaStream_t st) {
+  static bool configured = false;
+  if (!configured) {
+    cudaFuncSetAttribute(delta_step_kernel<T, NR, GENERAL>, cudaFuncAttributeMaxDynamicSharedMemorySize, kW2Smem);
+    configured = true;
+  }
+  const size_t need = GENERAL ? (size_t)p.R * NR * 64 : 0;
+  launch_kernel(delta_step_kernel<T, NR, GENERAL>, grid, dim3(256), need <= kW2Smem ? need : 0, st, true, p);
+}
+
 template <typename T, bool GENERAL>
 static int launch_delta(const DeltaParams& p, int S, int DK, int dv, cudaStream_t st) {
   const dim3 grid(dv / 64, p.H, S);
   switch (DK) {
-    case 64: launch_kernel(delta_step_kernel<T, 4, GENERAL>, grid, dim3(256), 0, st, true, p); break;
-    case 128: launch_kernel(delta_step_kernel<T, 8, GENERAL>, grid, dim3(256), 0, st, true, p); break;
-    case 256: launch_kernel(delta_step_kernel<T, 16, GENERAL>, grid, dim3(256), 0, st, true, p); break;
-    case 512: launch_kernel(delta_step_kernel<T, 32, GENERAL>, grid, dim3(256), 0, st, true, p); break;
+    case 64: launch_delta_rows<T, 4, GENERAL>(p, grid, st); break;
+    case 128: launch_delta_rows<T, 8, GENERAL>(p, grid, st); break;
+    case 256: launch_delta_rows<T, 16, GENERAL>(p, grid, st); break;
+    case 512: launch_delta_rows<T, 32, GENERAL>(p, grid, st); break;
     default: return -3;
   }
   return (int)cudaGetLastError();
@@ -191,7 +209,7 @@ int ti_head_norm_params_size() { return (int)sizeof(ti::HeadNormParams); }
 // o[t, h] and the states for the tokens cu[s] .. cu[s+1] of the S sequences (all, or those of `seqs`; cu null: one token each)
 int ti_delta_step(const ti::DeltaParams* p, int S, int dk, int dv, int general, int f32, void* stream) {
   if (S <= 0) return 0;
-  if (dv % 64 || p->rep < 1 || p->H % p->rep || (general && (p->R < 1 || p->rep != 1)) || ((uintptr_t)p->state & 15)) return -2;
+  if (dv % 64 || p->rep < 1 || p->H % p->rep || (general && (p->R < 1 || p->rep != 1 || ((uintptr_t)p->w2 & 15))) || ((uintptr_t)p->state & 15)) return -2;
   cudaStream_t st = (cudaStream_t)stream;
   if (general) return f32 ? ti::launch_delta<float, true>(*p, S, dk, dv, st) : ti::launch_delta<ti::bf16, true>(*p, S, dk, dv, st);
   return f32 ? ti::launch_delta<float, false>(*p, S, dk, dv, st) : ti::launch_delta<ti::bf16, false>(*p, S, dk, dv, st);
